@@ -10,11 +10,12 @@
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
 import sys
-from typing import List
+from typing import List, Optional
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
@@ -44,26 +45,57 @@ def _run(cmd: List[str]) -> None:
         raise RuntimeError("command failed: " + " ".join(cmd) + "\n" + r.stdout)
 
 
-def build_kernels(verbose: bool = False, ptxas_v: bool = False) -> str:
+# translation units every library holds, and those of the mixers, residual forms and activation types
+_UNITS_BASE = ("runtime",)
+_UNITS_BF16 = ("gemm", "elementwise", "attention")
+_UNITS_F32 = ("attention_f32",)
+_UNITS_STREAMS = ("streams", "recurrent")
+
+
+def units_for(cfg) -> Optional[List[str]]:
+    """Translation units (``csrc/<unit>.cu``) that a model given by ``cfg`` calls outside of sampling, or None for all of
+    them.  Known for models that list their layers."""
+    if not cfg.layer_specs or cfg.quant.method != "none":
+        return None
+    return sorted(_UNITS_BASE + (_UNITS_F32 if cfg.dtype == "float32" else _UNITS_BF16) + _UNITS_STREAMS)
+
+
+def _sources() -> List[str]:
+    return sorted(f[:-3] for f in os.listdir(CSRC) if f.endswith(".cu"))
+
+
+def _headers() -> List[str]:
+    return [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
+
+
+def kernels_current() -> bool:
+    """The full kernel library exists and is newer than its sources."""
+    headers = _headers()
+    return not any(_newer(os.path.join(CSRC, u + ".cu"), KERNEL_LIB, headers) for u in _sources())
+
+
+def build_kernels(verbose: bool = False, ptxas_v: bool = False, units: Optional[List[str]] = None) -> str:
+    """Compile what is out of date and link it: the full library, or one of the given translation units only."""
     os.makedirs(OUT, exist_ok=True)
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    cus = sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
-    objs, jobs = [], []
-    for f in cus:
-        src = os.path.join(CSRC, f)
-        obj = os.path.join(OUT, f[:-3] + ".o")
-        objs.append(obj)
-        if _newer(src, obj, headers):
-            cmd = [_nvcc()] + NVCC_FLAGS + (["-Xptxas", "-v"] if ptxas_v else []) + ["-I", CSRC, "-c", src, "-o", obj]
-            jobs.append(cmd)
-    if jobs:
-        if verbose:
-            print(f"[atlas_b200.build] compiling {len(jobs)} CUDA file(s) for sm_100a", file=sys.stderr)
-        with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
-            list(ex.map(_run, jobs))
-    if jobs or not os.path.exists(KERNEL_LIB):
-        _run([_nvcc(), "-shared", "-o", KERNEL_LIB] + objs + ["-lcudart"])
-    return KERNEL_LIB
+    lib = KERNEL_LIB if units is None else os.path.join(OUT, "libatlas_b200_kernels_" + "_".join(units) + ".so")
+    with open(os.path.join(OUT, ".lock"), "w") as lock:          # two processes of a fresh checkout build one after the other
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        headers = _headers()
+        objs, jobs = [], []
+        for u in (_sources() if units is None else units):
+            src, obj = os.path.join(CSRC, u + ".cu"), os.path.join(OUT, u + ".o")
+            objs.append(obj)
+            if _newer(src, obj, headers):
+                jobs.append([_nvcc()] + NVCC_FLAGS + (["-Xptxas", "-v"] if ptxas_v else []) + ["-I", CSRC, "-c", src, "-o", obj])
+        if jobs:
+            if verbose:
+                print(f"[atlas_b200.build] compiling {len(jobs)} CUDA file(s) for sm_100a", file=sys.stderr)
+            with cf.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
+                list(ex.map(_run, jobs))
+        if jobs or any(_newer(o, lib, []) for o in objs):
+            _run([_nvcc(), "-shared", "-o", lib + ".part"] + objs + ["-lcudart"])
+            os.replace(lib + ".part", lib)
+    return lib
 
 
 def build_runtime(verbose: bool = False) -> str:

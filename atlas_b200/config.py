@@ -13,6 +13,7 @@ from __future__ import annotations
 
 import dataclasses
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
@@ -26,7 +27,28 @@ _FAMILY_ALIASES = {
     "holo3_1_moe": "hybrid",
     "nemotron_h": "hybrid", "nemotron_h_puzzle": "hybrid",
     "deepseek_v2": "moe", "deepseek_v3": "moe", "deepseek_v32": "moe", "kimi_k2": "moe",
+    "papidra": "hybrid",
 }
+
+# widths the attention kernels are instantiated for; heads of any other size are zero-padded to the next one
+ATTENTION_WIDTHS = (64, 128, 256)
+
+
+def padded_head_width(*dims: int) -> int:
+    """Cache width of heads whose query / key / value sizes are ``dims``."""
+    for w in ATTENTION_WIDTHS:
+        if max(dims) <= w:
+            return w
+    raise ValueError(f"attention heads of {max(dims)} channels are not supported (at most {ATTENTION_WIDTHS[-1]})")
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a model whose layers differ in kind or size: the mixer's kind, whether a feed-forward sublayer
+    follows, and the :class:`ModelConfig` fields that hold for this layer only."""
+    kind: str                              # a mixer kind of ``layers.MIXERS``
+    has_mlp: bool = True
+    overrides: Dict[str, Any] = field(default_factory=dict)
 
 
 @dataclass
@@ -126,13 +148,29 @@ class ModelConfig:
     linear_conv_kernel_dim: int = 4
     # single-module blocks (Nemotron-H): per layer "mamba" | "attention" | "mlp"; empty for the other families
     block_types: List[str] = field(default_factory=list)
+    # layers of different kinds and sizes, each with its own values of the fields of this class
+    layer_specs: List[LayerSpec] = field(default_factory=list)
+    # hyper-connections: number of residual streams (0 = one plain residual stream in the activations' dtype)
+    residual_streams: int = 0
     mamba_num_heads: int = 0
     mamba_head_dim: int = 64
     ssm_state_size: int = 128
     mamba_n_groups: int = 8
     mamba_conv_kernel: int = 4
     mamba_dt_min: float = 0.0
-    mlp_activation: str = "silu_glu"  # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down)
+    mamba_norm_groups: int = 0        # parts of the gated output norm (0 = one per B / C group)
+    # WKV recurrence (RWKV-style time mixing)
+    wkv_num_heads: int = 0
+    wkv_head_dim: int = 0
+    mlp_activation: str = "silu_glu"  # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down) | clamped_glu
+    glu_limit: float = 0.0            # clamped_glu: bound on the gate (above) and on the up branch (both sides)
+    glu_alpha: float = 1.702          # clamped_glu: slope inside the gate's sigmoid
+    # attention variants: chunked visibility (a token sees its own chunk only), a learned per-head sink in the softmax
+    # denominator, the number of rotated dimensions when it is not a fraction of head_dim
+    attn_chunk: int = 0
+    attn_sinks: bool = False
+    rotary_dims: Optional[int] = None
+    attn_cache_width: int = 0         # padded width of cached heads (0 = head_dim)
     # multi-head latent attention (DeepSeek): 0 = plain GQA.  head_dim is then the padded cache width
     kv_lora_rank: int = 0
     q_lora_rank: int = 0
@@ -171,10 +209,20 @@ class ModelConfig:
 
     @property
     def rotary_dim(self) -> int:
+        if self.rotary_dims is not None:
+            return self.rotary_dims
         return int(self.head_dim * self.partial_rotary_factor)
 
+    def for_layer(self, i: int) -> "ModelConfig":
+        """The configuration as layer ``i`` sees it (its own sizes in place of the model's)."""
+        if not self.layer_specs:
+            return self
+        return dataclasses.replace(self, layer_specs=[], **self.layer_specs[i].overrides)
+
     def layer_kind(self, i: int) -> str:
-        """Mixer kind of layer ``i``: ``attention``, ``gdn``, ``mamba2`` or ``none`` (an FFN-only block)."""
+        """Mixer kind of layer ``i``: ``attention``, ``gdn``, ``mamba2``, ``wkv``, ``parallel`` or ``none`` (an FFN-only block)."""
+        if self.layer_specs:
+            return self.layer_specs[i].kind
         if self.block_types:
             return {"mamba": "mamba2", "attention": "attention"}.get(self.block_types[i], "none")
         if self.family != "hybrid":
@@ -207,6 +255,8 @@ class ModelConfig:
     def param_count(self) -> int:
         h, L = self.hidden_size, self.num_hidden_layers
         n = self.vocab_size * h * (1 if self.tie_word_embeddings else 2)
+        if self.layer_specs:
+            return n + sum(self.for_layer(i)._spec_layer_params(s) for i, s in enumerate(self.layer_specs))
         for i in range(L):
             if self.layer_kind(i) == "attention":
                 qmul = 2 if self.attn_output_gate else 1
@@ -229,10 +279,29 @@ class ModelConfig:
                 n += 3 * h * self.intermediate_size
         return n
 
+    def _spec_layer_params(self, spec: LayerSpec) -> int:
+        """Projection weights of one layer described by a :class:`LayerSpec` (``self`` is the layer's own view)."""
+        h = self.hidden_size
+        n = 3 * h * self.intermediate_size if spec.has_mlp else 0
+        if spec.kind in ("attention", "parallel"):
+            dv = self.v_head_dim or self.head_dim
+            n += h * (self.q_size + self.kv_size + self.num_key_value_heads * dv) + self.num_attention_heads * dv * h
+        if spec.kind in ("mamba2", "parallel"):
+            di = self.mamba_num_heads * self.mamba_head_dim
+            n += h * (2 * di + 2 * self.mamba_n_groups * self.ssm_state_size + self.mamba_num_heads) + di * h
+        if spec.kind == "wkv":
+            n += 5 * h * self.wkv_num_heads * self.wkv_head_dim
+        return n
+
     # ------------------------------------------------------------------ parsing
     @staticmethod
     def from_hf(cfg: Dict[str, Any]) -> "ModelConfig":
         outer = cfg
+        native = _NATIVE_ARCHITECTURES.get(str(cfg.get("architecture", "")).lower())
+        if native is not None:
+            c = native(cfg)
+            c.validate()
+            return c
         if "text_config" in cfg and isinstance(cfg["text_config"], dict):
             merged = dict(cfg["text_config"])
             for k in ("quantization_config", "torch_dtype"):
@@ -373,11 +442,76 @@ class ModelConfig:
             raise ValueError("num_attention_heads must be a multiple of num_key_value_heads")
         if self.num_experts and not self.num_experts_per_tok:
             raise ValueError("MoE config needs num_experts_per_tok")
-        if self.family == "hybrid" and not self.linear_num_value_heads and not self.block_types:
+        if self.family == "hybrid" and not self.linear_num_value_heads and not (self.block_types or self.layer_specs):
             raise ValueError("hybrid config needs linear_num_value_heads")
 
     def to_dict(self) -> Dict[str, Any]:
         return dataclasses.asdict(self)
+
+
+# ---------------------------------------------------------------------------- configurations that list their layers
+def _rotary_overrides(rot: Optional[Dict[str, Any]]) -> Dict[str, Any]:
+    """``{dims, base, scaling}`` -> rotary fields; ``scaling`` is YaRN's ``{factor, original, fast, slow}``."""
+    if not rot:
+        return {"rotary_dims": 0}
+    sc = rot.get("scaling")
+    return {"rotary_dims": int(rot["dims"]), "rope_theta": float(rot["base"]),
+            "rope_scaling": None if not sc else {
+                "rope_type": "yarn", "factor": float(sc["factor"]), "original_max_position_embeddings": float(sc["original"]),
+                "beta_fast": float(sc["fast"]), "beta_slow": float(sc["slow"]),
+                "attention_factor": 0.1 * math.log(float(sc["factor"])) + 1.0}}
+
+
+def _attention_overrides(m: Dict[str, Any]) -> Dict[str, Any]:
+    d, dv = int(m["dim"]), int(m.get("vdim", m["dim"]))
+    return {"num_attention_heads": int(m["heads"]), "num_key_value_heads": int(m["kv_heads"]), "head_dim": d, "v_head_dim": dv,
+            "attn_cache_width": padded_head_width(d, dv), "attn_scale": float(m["scale"]), "attn_sinks": True,
+            "attn_chunk": int((m.get("mask") or {}).get("size", 0)), **_rotary_overrides(m.get("rot"))}
+
+
+def _mamba2_overrides(m: Dict[str, Any]) -> Dict[str, Any]:
+    return {"mamba_num_heads": int(m["heads"]), "mamba_head_dim": int(m["vdim"]), "ssm_state_size": int(m["state"]),
+            "mamba_n_groups": int(m["groups"]), "mamba_norm_groups": int(m["norm_groups"]), "mamba_conv_kernel": int(m["conv"]),
+            "mamba_dt_min": 0.0}
+
+
+def _papidra_layer(lc: Dict[str, Any]) -> LayerSpec:
+    kind, m, mlp = str(lc["type"]), lc["mixer"], lc.get("mlp")
+    over: Dict[str, Any] = {}
+    if kind == "wkv":
+        over.update(wkv_num_heads=int(m["heads"]), wkv_head_dim=int(m["dim"]))
+    elif kind == "parallel":
+        over.update(_attention_overrides(m["left"]))
+        over.update(_mamba2_overrides(m["right"]))
+    else:
+        raise ValueError(f"unsupported Papidra layer type '{kind}'")
+    if mlp is not None:
+        if mlp.get("kind", "dense") != "dense":
+            raise ValueError(f"unsupported Papidra feed-forward '{mlp['kind']}'")
+        over.update(intermediate_size=int(mlp["ff"]), glu_limit=float(mlp["limit"]), mlp_activation="clamped_glu")
+    return LayerSpec(kind, mlp is not None, over)
+
+
+def papidra_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """Papidra: WKV layers and layers with attention and Mamba-2 side by side, on hyper-connected residual streams."""
+    specs = [_papidra_layer(lc) for lc in cfg["layers"]]
+    c = ModelConfig(model_type="papidra", family="hybrid", vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                    intermediate_size=max([s.overrides.get("intermediate_size", 0) for s in specs] + [1]),
+                    num_hidden_layers=len(specs), num_attention_heads=1, num_key_value_heads=1, head_dim=64,
+                    rms_norm_eps=float(cfg["norm"]["eps"]), embed_scale=float(cfg["embedding"]["scale"]),
+                    residual_streams=int(cfg["streams"]), tie_word_embeddings=True, layer_specs=specs,
+                    mlp_activation="clamped_glu", dtype=str(cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))),
+                    quant=QuantConfig(kv_cache_dtype="bf16"), bos_token_id=cfg.get("bos_token_id"), eos_token_id=cfg.get("eos_token_id"))
+    for s in specs:
+        if "num_attention_heads" in s.overrides:            # the model-wide view sizes buffers by the widest heads
+            for k in ("num_attention_heads", "num_key_value_heads", "head_dim"):
+                setattr(c, k, s.overrides[k])
+            break
+    return c
+
+
+# ``architecture`` of a config.json that lists its layers one by one -> its reader
+_NATIVE_ARCHITECTURES = {"papidra": papidra_config}
 
 
 # ---------------------------------------------------------------------------- presets
@@ -469,6 +603,33 @@ def tiny_deepseek(dtype: str = "float32") -> ModelConfig:
                        max_position_embeddings=4096, dtype=dtype)
 
 
+def _papidra(vocab: int, width: int, ff: int, pattern: str, streams: int, wkv: tuple, attn: tuple, mamba: tuple, chunk: int,
+             dtype: str) -> ModelConfig:
+    """``pattern``: ``w`` = WKV layer without feed-forward, ``p`` = parallel layer with one; ``wkv`` (heads, dim), ``attn``
+    (heads, kv heads, dim), ``mamba`` (heads, channels, state, groups)."""
+    left = {"heads": attn[0], "kv_heads": attn[1], "dim": attn[2], "vdim": attn[2], "scale": attn[2] ** -0.5, "mask": {"size": chunk},
+            "rot": {"base": 5e5, "dims": attn[2], "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": mamba[0], "vdim": mamba[1], "state": mamba[2], "groups": mamba[3], "norm_groups": mamba[3], "conv": 4}
+    layers = [{"type": "wkv", "mixer": {"heads": wkv[0], "dim": wkv[1]}, "mlp": None} if ch == "w" else
+              {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}}
+              for ch in pattern]
+    return papidra_config({"vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+                           "streams": streams, "layers": layers, "dtype": dtype})
+
+
+def tiny_papidra(dtype: str = "float32") -> ModelConfig:
+    c = _papidra(1024, 256, 384, "wpwp", 2, (4, 64), (4, 2, 64), (8, 32, 32, 2), 48, dtype)
+    c.max_position_embeddings = 4096
+    return c
+
+
+def papidra_8b(quant: str = "none") -> ModelConfig:
+    """Layers of the size of an 8B decoder: width 4096, 32 heads of 128 (8 kv), 128 Mamba-2 heads of 64, 64 WKV heads of 64."""
+    c = _papidra(131072, 4096, 14336, "wp" * 16, 4, (64, 64), (32, 8, 128), (128, 64, 128, 8), 4096, "bfloat16")
+    c.quant = QuantConfig(method=quant, kv_cache_dtype="bf16")
+    return c
+
+
 def nemotron_h_8b(quant: str = "none") -> ModelConfig:
     pattern = "M-M-M-MM-M-M-M*-M-M-M*-M-M-M-M*-M-M-M-M*-M-MM-M-M-M-M-M-"
     blocks = [{"M": "mamba", "*": "attention", "-": "mlp"}[ch] for ch in pattern]
@@ -484,6 +645,7 @@ PRESETS = {
     "llama3-8b": llama3_8b, "llama3-70b": llama3_70b,
     "qwen3-30b-a3b": qwen3_30b_a3b, "qwen3-next-80b": qwen3_next_80b,
     "tiny-nemotron-h": tiny_nemotron_h, "nemotron-h-8b": nemotron_h_8b, "tiny-deepseek": tiny_deepseek,
+    "tiny-papidra": tiny_papidra, "papidra-8b": papidra_8b,
 }
 
 

@@ -33,6 +33,8 @@ struct AttnParams {
   float qk_scale_log2;                          // softmax scale * k_scale * log2(e)
   float v_scale;
   int Hq, Hkv, block_size, window;
+  int chunk;                                    // > 0: a row sees keys of its own chunk-token block of the sequence only
+  const float* sinks;                           // [Hq] or null: exp(sink) joins the softmax denominator
   // decode
   int num_splits;
   float* part_o;                                // [B, Hq, splits, D]
@@ -84,6 +86,21 @@ ATLAS_DEVICE uint32_t hmul2_u32(uint32_t a, uint32_t b) {
   asm("mul.rn.f16x2 %0, %1, %2;\n" : "=r"(r) : "r"(a), "r"(b));
   return r;
 }
+// first position a row at `pos` can see
+ATLAS_DEVICE int first_visible(const AttnParams& p, int pos) {
+  int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  if (p.chunk > 0) lo = max(lo, pos - pos % p.chunk);
+  return lo;
+}
+// A sink joins the denominator of a row with running maximum m (log2 units) and sum l.  Returns the factor on what was
+// accumulated so far.
+ATLAS_DEVICE float add_sink(float sink, float& m, float& l) {
+  const float s = sink * 1.4426950408889634f, top = fmaxf(m, s);
+  const float f = m == -INFINITY ? 0.f : exp2f(m - top);
+  l = l * f + exp2f(s - top);
+  m = top;
+  return f;
+}
 template <int D, bool PREFILL, bool KV16 = false, bool KV4 = false>
 __global__ void __launch_bounds__(128)
 paged_attn_kernel(const AttnParams p) {
@@ -96,6 +113,7 @@ paged_attn_kernel(const AttnParams p) {
   const int G = p.Hq / p.Hkv;
 
   int b, kvh, q_row0, q_len, L, qhead = 0, tile_q0 = 0, split = 0;
+  int g0 = 0, gn = G;                   // decode: the query heads [g0, g0 + gn) of the group are this CTA's tile rows
   if (PREFILL) {
     const int tile = blockIdx.x * 4 + warp;
     if (tile >= p.num_tiles) return;
@@ -105,12 +123,17 @@ paged_attn_kernel(const AttnParams p) {
     kvh = qhead / G;
   } else {
     b = p.seq_base + blockIdx.z;
-    kvh = blockIdx.x;
+    const int gt = (G + 15) >> 4;
+    kvh = blockIdx.x / gt;
+    g0 = (blockIdx.x % gt) << 4;
+    gn = min(16, G - g0);
     split = blockIdx.y;
   }
   L = p.seq_lens[b];
   q_row0 = p.query_start_loc[b];
   q_len = p.query_start_loc[b + 1] - q_row0;
+  // a bf16 cache keeps the query as it is and scales the fp32 scores instead
+  const float q_scale = KV16 ? 1.f : p.qk_scale_log2, s_scale = KV16 ? p.qk_scale_log2 : 1.f;
 
   // ---- query fragments (scaled, f16)
   uint32_t qf[KS][4];
@@ -122,7 +145,7 @@ paged_attn_kernel(const AttnParams p) {
       if (PREFILL) {
         if (tile_q0 + r < q_len) qrow[h] = p.q + (long long)(q_row0 + tile_q0 + r) * p.ldq + qhead * D;
       } else {
-        if (r < G) qrow[h] = p.q + (long long)q_row0 * p.ldq + (kvh * G + r) * D;
+        if (r < gn) qrow[h] = p.q + (long long)q_row0 * p.ldq + (kvh * G + g0 + r) * D;
       }
     }
 #pragma unroll
@@ -134,8 +157,8 @@ paged_attn_kernel(const AttnParams p) {
           const uint2 raw = *reinterpret_cast<const uint2*>(qrow[h] + c * DQ + ks * 4);
           const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x);
           const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
-          v[0] = __low2float(lo) * p.qk_scale_log2; v[1] = __high2float(lo) * p.qk_scale_log2;
-          v[2] = __low2float(hi) * p.qk_scale_log2; v[3] = __high2float(hi) * p.qk_scale_log2;
+          v[0] = __low2float(lo) * q_scale; v[1] = __high2float(lo) * q_scale;
+          v[2] = __low2float(hi) * q_scale; v[3] = __high2float(hi) * q_scale;
         }
         qf[ks][h] = KV16 ? pack_bf16x2(v[0], v[1]) : pack_f16x2(v[0], v[1]);         // a0 / a1 : k = c*2 + {0,1}
         qf[ks][2 + h] = KV16 ? pack_bf16x2(v[2], v[3]) : pack_f16x2(v[2], v[3]);     // a2 / a3 : k = c*2 + 8 + {0,1}
@@ -152,19 +175,18 @@ paged_attn_kernel(const AttnParams p) {
     qpos[0] = first_pos + rq;
     qpos[1] = first_pos + rq + 8;
     const int last_pos = min(L - 1, first_pos + 15);
-    pg_begin = 0;
-    if (p.window > 0) pg_begin = max(0, first_pos - p.window + 1) >> 4;
+    pg_begin = first_visible(p, first_pos) >> 4;
     pg_end = (last_pos >> 4) + 1;
     pg_step = 1;
   } else {
     qpos[0] = qpos[1] = L - 1;
-    const int per_split = (n_pages + p.num_splits - 1) / p.num_splits;
-    int lo = split * per_split;
-    if (p.window > 0) lo = max(lo, max(0, L - p.window) >> 4);
-    pg_begin = lo + warp;
-    pg_end = min(n_pages, (split + 1) * per_split);
+    const int pg_lo = first_visible(p, L - 1) >> 4;              // the splits share the visible pages
+    const int per_split = (n_pages - pg_lo + p.num_splits - 1) / p.num_splits;
+    pg_begin = pg_lo + split * per_split + warp;
+    pg_end = min(n_pages, pg_lo + (split + 1) * per_split);
     pg_step = 4;
   }
+  const int lo_pos[2] = {first_visible(p, qpos[0]), first_visible(p, qpos[1])};
 
   float o[NT][4];
 #pragma unroll
@@ -237,10 +259,9 @@ paged_attn_kernel(const AttnParams p) {
         const int tok = tok0 + c * 4 + 2 * i + j;
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
-          bool ok = tok <= qpos[h] && tok < L;
-          if (p.window > 0) ok = ok && tok > qpos[h] - p.window;
+          const bool ok = tok <= qpos[h] && tok < L && tok >= lo_pos[h];
           float& sv = s[i][2 * h + j];
-          sv = ok ? sv : -INFINITY;
+          sv = ok ? sv * s_scale : -INFINITY;
           mx[h] = fmaxf(mx[h], sv);
         }
       }
@@ -339,7 +360,8 @@ paged_attn_kernel(const AttnParams p) {
     for (int h = 0; h < 2; ++h) {
       const int r = rq + 8 * h;
       if (tile_q0 + r >= q_len) continue;
-      const float inv = l_run[h] > 0.f ? p.v_scale / l_run[h] : 0.f;
+      const float f = p.sinks ? add_sink(p.sinks[qhead], m_run[h], l_run[h]) : 1.f;
+      const float inv = l_run[h] > 0.f ? p.v_scale * f / l_run[h] : 0.f;
       __nv_bfloat16* orow = p.out + (long long)(q_row0 + tile_q0 + r) * p.ldo + qhead * D;
 #pragma unroll
       for (int j = 0; j < NT; ++j)
@@ -363,7 +385,7 @@ paged_attn_kernel(const AttnParams p) {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
       const int r = rq + 8 * h;
-      if (r < G) {
+      if (r < gn) {
         float* dst = sm_o + ((warp * 16 + r) * D);
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
@@ -373,7 +395,7 @@ paged_attn_kernel(const AttnParams p) {
       }
     }
     __syncthreads();
-    for (int idx = threadIdx.x; idx < G * D; idx += 128) {
+    for (int idx = threadIdx.x; idx < gn * D; idx += 128) {
       const int r = idx / D, d = idx % D;
       float m = -INFINITY;
 #pragma unroll
@@ -386,8 +408,9 @@ paged_attn_kernel(const AttnParams p) {
         acc += f * sm_o[(w * 16 + r) * D + d];
         l += f * sm_l[w * 16 + r];
       }
-      const int head = kvh * G + r;
+      const int head = kvh * G + g0 + r;
       if (p.num_splits == 1) {
+        if (p.sinks) acc *= add_sink(p.sinks[head], m, l);
         const float inv = l > 0.f ? p.v_scale / l : 0.f;
         p.out[(long long)q_row0 * p.ldo + head * D + d] = __float2bfloat16_rn(acc * inv);
       } else {
@@ -1278,7 +1301,7 @@ attn_decode_f8_kernel(const AttnParams p, int stages, status_t* status) {
 __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                   __nv_bfloat16* out, long long ldo, const int* query_start_loc, int seq_base, int Hq,
                                   int D, int splits, float v_scale, uint8_t* q_out, long long ldqo, float* s_out,
-                                  long long s_ld) {
+                                  long long s_ld, const float* sinks) {
   __shared__ float wmax[8];
   const int head = blockIdx.x, bi = blockIdx.y, d = threadIdx.x;
   const long long base = ((long long)bi * Hq + head) * splits;
@@ -1293,6 +1316,7 @@ __global__ void attn_merge_kernel(const float* __restrict__ part_o, const float*
     acc += f * part_o[(base + s) * D + d];
     l += f * part_ml[(base + s) * 2 + 1];
   }
+  if (sinks) acc *= add_sink(sinks[head], m, l);
   const float inv = l > 0.f ? v_scale / l : 0.f;
   const int row = query_start_loc[seq_base + bi];
   if (q_out == nullptr) {
@@ -1350,7 +1374,7 @@ static int launch_decode_bs(const AttnParams& p, int B, status_t* status, cudaSt
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     if (launch_chain(attn_merge_kernel, g2, dim3(D), 0, st, p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base,
-                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld) != cudaSuccess)
+                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld, p.sinks) != cudaSuccess)
       return -22;
   }
   return 0;
@@ -1370,7 +1394,7 @@ static int launch_decode_f8(const AttnParams& p, int B, status_t* status, cudaSt
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     if (launch_chain(attn_merge_kernel, g2, dim3(D), 0, st, p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base,
-                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld) != cudaSuccess)
+                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld, p.sinks) != cudaSuccess)
       return -22;
   }
   return 0;
@@ -1400,7 +1424,7 @@ static int launch_decode_cp(const AttnParams& p, int B, cudaStream_t st) {
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     if (launch_chain(attn_merge_kernel, g2, dim3(D), 0, st, p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base,
-                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld) != cudaSuccess)
+                     p.Hq, D, p.num_splits, p.v_scale, p.q_out, p.ldqo, p.s_out, p.s_ld, p.sinks) != cudaSuccess)
       return -22;
   }
   return 0;
@@ -1452,6 +1476,7 @@ static int fill_common(AttnParams& p, const void* q, long long ldq, void* out, l
   p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.window = window;
   p.num_splits = 1; p.part_o = nullptr; p.part_ml = nullptr; p.tile_seq = nullptr; p.tile_q0 = nullptr; p.num_tiles = 0;
   p.q_out = nullptr; p.ldqo = 0; p.s_out = nullptr; p.s_ld = 0;
+  p.chunk = 0; p.sinks = nullptr;
   return 0;
 }
 
@@ -1534,13 +1559,13 @@ static int launch_kv16(const AttnParams& p, int B, bool prefill, cudaStream_t st
   }
   const int smem = (128 + 4 * 16 * D) * (int)sizeof(float);
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_kernel<D, false, true>), smem) != cudaSuccess) return -20;
-  dim3 grid(p.Hkv, p.num_splits, B);
+  dim3 grid(p.Hkv * ((p.Hq / p.Hkv + 15) / 16), p.num_splits, B);
   paged_attn_kernel<D, false, true><<<grid, 128, smem, st>>>(p);
   if (cudaGetLastError() != cudaSuccess) return -21;
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     attn_merge_kernel<<<g2, D, 0, st>>>(p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base, p.Hq, D, p.num_splits,
-                                       p.v_scale, nullptr, 0, nullptr, 0);
+                                       p.v_scale, nullptr, 0, nullptr, 0, p.sinks);
     if (cudaGetLastError() != cudaSuccess) return -22;
   }
   return 0;
@@ -1567,7 +1592,7 @@ static int launch_kv4(const AttnParams& p, int B, bool prefill, cudaStream_t st)
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     attn_merge_kernel<<<g2, D, 0, st>>>(p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base, p.Hq, D, p.num_splits,
-                                       p.v_scale, nullptr, 0, nullptr, 0);
+                                       p.v_scale, nullptr, 0, nullptr, 0, nullptr);
     if (cudaGetLastError() != cudaSuccess) return -22;
   }
   return 0;
@@ -1612,17 +1637,19 @@ extern "C" int atlas_attn_prefill_kv4(const void* q, long long ldq, void* out, l
   return launch_kv4<256>(p, 0, true, st);
 }
 
-// Same contracts as atlas_attn_decode / atlas_attn_prefill with a bf16 cache (K [nb, Hkv, bs, D], V [nb, Hkv, D, bs]).
+// Same contracts as atlas_attn_decode / atlas_attn_prefill with a bf16 cache (K [nb, Hkv, bs, D], V [nb, Hkv, D, bs]), any
+// number of query heads per kv head, and optional chunked visibility (`chunk` > 0) and softmax sinks (fp32 [Hq]).
 extern "C" int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache,
                                       const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                       const int* query_start_loc, int seq_base, int B, float scale, int Hq, int Hkv, int D,
-                                      int block_size, int window, int num_splits, float* part_o, float* part_ml, void* stream) {
+                                      int block_size, int window, int num_splits, float* part_o, float* part_ml, void* stream,
+                                      int chunk, const float* sinks) {
   if (B <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, seq_base, scale,
                        1.f, 1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
-  if (Hq / Hkv > 16) return -5;
+  p.chunk = chunk; p.sinks = sinks;
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   if (p.num_splits > 1 && (!part_o || !part_ml)) return -3;
   p.part_o = part_o; p.part_ml = part_ml;
@@ -1635,12 +1662,14 @@ extern "C" int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, l
 extern "C" int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache,
                                        const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                        const int* query_start_loc, const int* tile_seq, const int* tile_q0, int num_tiles,
-                                       float scale, int Hq, int Hkv, int D, int block_size, int window, void* stream) {
+                                       float scale, int Hq, int Hkv, int D, int block_size, int window, void* stream, int chunk,
+                                       const float* sinks) {
   if (num_tiles <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, 0, scale, 1.f,
                        1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
+  p.chunk = chunk; p.sinks = sinks;
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.num_tiles = num_tiles;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (D == 64) return launch_kv16<64>(p, 0, true, st);

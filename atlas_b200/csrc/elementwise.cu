@@ -633,6 +633,33 @@ shared_expert_blend_kernel(__nv_bfloat16* y, long long ldy, const __nv_bfloat16*
   }
 }
 
+// y = relu(x)^2, eight bf16 per thread
+__global__ void __launch_bounds__(256)
+relu2_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* y, long long ldy, int cols) {
+  const long long t = blockIdx.x;
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < cols; c += gridDim.y * blockDim.x * 8) {
+    if (c + 8 <= cols) {
+      const uint4 v = *reinterpret_cast<const uint4*>(x + t * ldx + c);
+      const __nv_bfloat162* hv = reinterpret_cast<const __nv_bfloat162*>(&v);
+      uint4 o;
+      __nv_bfloat162* ho = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        float2 f = __bfloat1622float2(hv[i]);
+        f.x = f.x > 0.f ? f.x * f.x : 0.f;
+        f.y = f.y > 0.f ? f.y * f.y : 0.f;
+        ho[i] = __floats2bfloat162_rn(f.x, f.y);
+      }
+      *reinterpret_cast<uint4*>(y + t * ldy + c) = o;
+    } else {
+      for (int i = c; i < cols; ++i) {
+        const float f = __bfloat162float(x[t * ldx + i]);
+        y[t * ldy + i] = __float2bfloat16_rn(f > 0.f ? f * f : 0.f);
+      }
+    }
+  }
+}
+
 }  // namespace atlas
 
 using namespace atlas;
@@ -789,5 +816,14 @@ extern "C" int atlas_shared_expert_blend(void* y, long long ldy, const void* s, 
   shared_expert_blend_kernel<<<T, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
       reinterpret_cast<__nv_bfloat16*>(y), ldy, reinterpret_cast<const __nv_bfloat16*>(s), lds,
       reinterpret_cast<const __nv_bfloat16*>(x), ldx, reinterpret_cast<const __nv_bfloat16*>(wg), H);
+  return cudaGetLastError() == cudaSuccess ? 0 : -20;
+}
+
+extern "C" int atlas_relu2(const void* x, long long ldx, void* y, long long ldy, int T, int cols, void* stream) {
+  if (T <= 0 || cols <= 0) return 0;
+  if ((ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(y) & 15)) return -1;
+  dim3 grid(T, min(8, (cols / 8 + 255) / 256 > 0 ? (cols / 8 + 255) / 256 : 1));
+  relu2_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx,
+                                                                          reinterpret_cast<__nv_bfloat16*>(y), ldy, cols);
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }

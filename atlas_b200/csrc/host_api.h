@@ -131,6 +131,51 @@ int atlas_attn_prefill(const void* q, long long ldq, void* out, long long ldo, c
                        const int* query_start_loc, const int* tile_seq, const int* tile_q0, int num_tiles, float scale,
                        float k_scale, float v_scale, int Hq, int Hkv, int D, int block_size, int window, void* stream);
 
+int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
+                           const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int seq_base, int B,
+                           float scale, int Hq, int Hkv, int D, int block_size, int window, int num_splits, float* part_o,
+                           float* part_ml, void* stream, int chunk, const float* sinks);
+int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
+                            const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
+                            const int* tile_q0, int num_tiles, float scale, int Hq, int Hkv, int D, int block_size, int window,
+                            void* stream, int chunk, const float* sinks);
+
+// ---- 32-bit attention (attention_f32.cu)
+int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const int* positions,
+                            const float* rope, float* k_cache, float* v_cache, const int* slot_mapping, int T, int Hq, int Hkv, int D,
+                            int rotary, int block_size, void* stream);
+int atlas_attn_f32(const float* q, long long ldq, float* out, long long ldo, const float* k_cache, const float* v_cache,
+                   const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int B, int T, float scale, int Hq,
+                   int Hkv, int D, int block_size, int window, int chunk, const float* sinks, void* stream);
+
+// ---- residual streams, token shift, clamped gated unit (streams.cu); f32 = activations are fp32 instead of bf16
+int atlas_hyper_norm(float* x, int rows, int S, int W, const void* y, long long ldy, const void* y2, long long ldy2, const float* w1,
+                     const float* w2, const float* mix, const float* write, const float* read, const float* norm_w, void* out,
+                     long long ldo, int init, int store, float scale, float eps, int f32, void* stream);
+int atlas_token_shift_mix(const void* x, long long ldx, const float* mu, const void* shift, const int* seq_of_token, const int* qsl,
+                          const int* slots, const unsigned char* has, void* out, int rows, int W, int f32, void* stream);
+int atlas_clamped_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha, int f32,
+                      void* stream);
+int atlas_tanh(void* x, long long n, int f32, void* stream);
+
+// ---- linear recurrences (recurrent.cu)
+int atlas_mamba2_scan(const void* y, long long ldy, const void* dt, long long lddt, const float* A_log, const float* D,
+                      const float* dt_bias, float dt_min, float* h, void* out, long long ldo, const int* qsl, const int* slots,
+                      const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B, int H,
+                      int P, int N, int G, int commit, int one_row, int f32, void* stream);
+int atlas_wkv_scan(const void* r, long long ldr, const void* k, long long ldk, const void* v, long long ldv, const void* raw, long long ldw,
+                   const float* w0, const float* u, float* h, void* out, long long ldo, const void* x, long long ldx, void* shift, int W,
+                   const int* qsl, const int* slots, const unsigned char* has, const int* limit, const int* snap_rows,
+                   const int* snap_slots, int snaps, int B, int H, int D, int commit, int one_row, int f32, void* stream);
+int atlas_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
+                          int groups, int gsize, float eps, int gate_first, int f32, void* stream);
+int atlas_conv1d_bias_silu(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
+                           const int* seq_of_token, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
+                           int rows, int f32, void* stream);
+int atlas_conv1d_state(const void* x, long long ldx, int C, int W, void* state, const int* qsl, const int* slots,
+                       const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B, int f32,
+                       void* stream);
+
 // ---- sampling (sampling.cu)
 int atlas_argmax(const void* logits, long long ld, int B, int V, int is_bf16, long long* out, float* out_val,
                  void* stream);

@@ -1,0 +1,312 @@
+// Hyper-connected residual streams (fp32), the token-shift mixes of WKV layers and the clamped gated unit.
+//
+//   hyper_norm_kernel       one CTA per token: rewrites the S streams with the last sublayer's connection and output
+//                             x'[t] = sum_s mix[s, t] * x[s] + write[t] * y
+//                           reads the next sublayer's input u = sum_s read[s] * x'[s] and writes rmsnorm(u) * w.  The write
+//                           of one sublayer and the read + norm of the next one share a single pass over the streams.
+//                           With a second output y2 (two mixers side by side) y is half the sum of both after an RMS norm
+//                           each; at the start of the model the streams are set to the scaled embedding instead.
+//   token_shift_mix_kernel  out[s] = x + (x_prev - x) * mu[s] for S mixes, x_prev = the previous token's row (from the
+//                           sequence's state slot for the first row of a chunk, zeros at the start of a sequence)
+//   clamped_glu_kernel      g = min(gate, limit), u = clamp(up, +-limit):  g * sigmoid(alpha g) * (u + 1)
+//
+// Every kernel exists for bf16 and fp32 activations (template parameter T).
+#include "common.cuh"
+#include "host_api.h"
+#include "vec_io.cuh"
+
+namespace atlas {
+
+template <typename T>
+struct HyperParams {
+  float* x;                                    // [T, S, W]
+  const T* y; long long ldy;
+  const T* y2; long long ldy2;
+  const float* w1; const float* w2;            // [W] norm weights of y / y2
+  const float* mix; const float* write; const float* read;
+  const float* norm_w;
+  T* out; long long ldo;
+  int S, W, init, store;
+  float scale, eps;
+};
+
+constexpr int kMaxStreams = 8;
+
+ATLAS_DEVICE float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();                             // red may still be read from an earlier reduction
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) s += red[i];
+  return s;
+}
+
+// kS: number of streams known at compile time (0 = p.S, at most kMaxStreams)
+template <typename T, int kS, int V>
+__global__ void __launch_bounds__(512)
+hyper_norm_kernel(const HyperParams<T> p) {
+  constexpr int kN = kS > 0 ? kS : kMaxStreams;
+  extern __shared__ float su[];                // [W] the read mix
+  __shared__ float red[16];
+  __shared__ float cf[kMaxStreams * (kMaxStreams + 2)];
+  chain_trigger();
+  const int S = kS > 0 ? kS : p.S;
+  const long long t = blockIdx.x;
+  for (int i = threadIdx.x; i < S * S; i += blockDim.x) cf[i] = p.init ? 0.f : p.mix[i];
+  for (int i = threadIdx.x; i < S; i += blockDim.x) {
+    cf[S * S + i] = p.init ? p.scale : p.write[i];
+    cf[S * S + S + i] = p.read[i];
+  }
+  chain_wait();
+  const T* y = p.y + t * p.ldy;
+  const T* y2 = p.y2 ? p.y2 + t * p.ldy2 : nullptr;
+  float r1 = 1.f, r2 = 0.f;
+  if (y2) {
+    float a = 0.f, b = 0.f;
+    for (int e = threadIdx.x * V; e < p.W; e += blockDim.x * V) {
+      float f[V], g[V];
+      load_vec<V>(y + e, f);
+      load_vec<V>(y2 + e, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) { a += f[i] * f[i]; b += g[i] * g[i]; }
+    }
+    r1 = 0.5f / sqrtf(block_sum(a, red) / (float)p.W + p.eps);
+    r2 = 0.5f / sqrtf(block_sum(b, red) / (float)p.W + p.eps);
+  }
+  __syncthreads();
+  float wr[kN], rd[kN];
+#pragma unroll
+  for (int s = 0; s < kN; ++s)
+    if (s < S) { wr[s] = cf[S * S + s]; rd[s] = cf[S * S + S + s]; }
+  float* x = p.x + t * (long long)S * p.W;
+  float ss = 0.f;
+  for (int e = threadIdx.x * V; e < p.W; e += blockDim.x * V) {
+    float yv[V];
+    load_vec<V>(y + e, yv);
+    if (y2) {
+      float g[V], a[V], b[V];
+      load_vec<V>(y2 + e, g);
+      load_vec<V>(p.w1 + e, a);
+      load_vec<V>(p.w2 + e, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) yv[i] = yv[i] * r1 * a[i] + g[i] * r2 * b[i];
+    }
+    float old[kN][V];
+    if (!p.init) {
+#pragma unroll
+      for (int s = 0; s < kN; ++s)
+        if (s < S) load_vec<V>(x + (long long)s * p.W + e, old[s]);
+    }
+    float u[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) u[i] = 0.f;
+#pragma unroll
+    for (int q = 0; q < kN; ++q) {
+      if (q >= S) break;
+      float n[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) n[i] = wr[q] * yv[i];
+      if (!p.init) {
+#pragma unroll
+        for (int s = 0; s < kN; ++s) {
+          if (s >= S) break;
+          const float m = cf[s * S + q];
+#pragma unroll
+          for (int i = 0; i < V; ++i) n[i] = fmaf(m, old[s][i], n[i]);
+        }
+      }
+      if (p.store) store_vec<V>(x + (long long)q * p.W + e, n);
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[i] = fmaf(rd[q], n[i], u[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) { su[e + i] = u[i]; ss += u[i] * u[i]; }
+  }
+  const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps);
+  for (int e = threadIdx.x * V; e < p.W; e += blockDim.x * V) {
+    float w[V], o[V];
+    load_vec<V>(p.norm_w + e, w);
+#pragma unroll
+    for (int i = 0; i < V; ++i) o[i] = su[e + i] * rstd * w[i];
+    store_vec<V>(p.out + t * p.ldo + e, o);
+  }
+}
+
+template <typename T, int V>
+static int launch_hyper(const HyperParams<T>& p, int rows, cudaStream_t st) {
+  const int smem = p.W * (int)sizeof(float);
+  int threads = 128;
+  while (threads < 512 && threads * V < p.W) threads *= 2;
+  void (*k)(const HyperParams<T>) = nullptr;
+  switch (p.S) {
+    case 1: k = hyper_norm_kernel<T, 1, V>; break;
+    case 2: k = hyper_norm_kernel<T, 2, V>; break;
+    case 3: k = hyper_norm_kernel<T, 3, V>; break;
+    case 4: k = hyper_norm_kernel<T, 4, V>; break;
+    default: k = hyper_norm_kernel<T, 0, V>; break;
+  }
+  if (smem > 40 * 1024 && ensure_dynamic_smem(reinterpret_cast<const void*>(k), smem) != cudaSuccess) return -20;
+  launch_chain_if(rows <= 256, k, dim3(rows), dim3(threads), smem, st, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+template <typename T>
+static int hyper_norm(float* x, int rows, int S, int W, const void* y, long long ldy, const void* y2, long long ldy2,
+                      const float* w1, const float* w2, const float* mix, const float* write, const float* read,
+                      const float* norm_w, void* out, long long ldo, int init, int store, float scale, float eps, cudaStream_t st) {
+  HyperParams<T> p;
+  p.x = x; p.y = reinterpret_cast<const T*>(y); p.ldy = ldy; p.y2 = reinterpret_cast<const T*>(y2); p.ldy2 = ldy2;
+  p.w1 = w1; p.w2 = w2; p.mix = mix; p.write = write; p.read = read; p.norm_w = norm_w;
+  p.out = reinterpret_cast<T*>(out); p.ldo = ldo; p.S = S; p.W = W; p.init = init; p.store = store; p.scale = scale; p.eps = eps;
+  const bool vec = W % 4 == 0 && vec_ok<T, 4>(y, ldy) && vec_ok<T, 4>(y2, ldy2) && vec_ok<T, 4>(out, ldo) &&
+                   vec_ok<float, 4>(x, 0) && vec_ok<float, 4>(norm_w, 0) && vec_ok<float, 4>(w1, 0) && vec_ok<float, 4>(w2, 0);
+  return vec ? launch_hyper<T, 4>(p, rows, st) : launch_hyper<T, 1>(p, rows, st);
+}
+
+// ----------------------------------------------------------------------------- token shift
+constexpr int kShiftRows = 8;                  // consecutive rows of one thread: mu stays in registers, the previous row too
+
+template <typename T, int S, int V>
+__global__ void __launch_bounds__(256)
+token_shift_mix_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ mu, const T* __restrict__ shift,
+                       const int* __restrict__ seq_of_token, const int* __restrict__ query_start_loc,
+                       const int* __restrict__ state_slots, const unsigned char* __restrict__ has_state, T* out, int rows, int W) {
+  chain_trigger();
+  chain_wait();
+  const int e = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (e >= W) return;
+  float m[S][V];
+#pragma unroll
+  for (int s = 0; s < S; ++s) load_vec<V>(mu + (long long)s * W + e, m[s]);
+  const int t0 = blockIdx.x * kShiftRows, t1 = min(rows, t0 + kShiftRows);
+  float prev[V];
+  for (int t = t0; t < t1; ++t) {
+    const int b = seq_of_token[t];
+    if (t == query_start_loc[b]) {
+      if (has_state[b]) {
+        load_vec<V>(shift + (long long)state_slots[b] * W + e, prev);
+      } else {
+#pragma unroll
+        for (int i = 0; i < V; ++i) prev[i] = 0.f;
+      }
+    } else if (t == t0) {
+      load_vec<V>(x + (long long)(t - 1) * ldx + e, prev);
+    }
+    float c[V];
+    load_vec<V>(x + (long long)t * ldx + e, c);
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+      float o[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) o[i] = fmaf(prev[i] - c[i], m[s][i], c[i]);
+      store_vec<V>(out + ((long long)s * rows + t) * W + e, o);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) prev[i] = c[i];
+  }
+}
+
+template <typename T, int V>
+static int launch_shift(const void* x, long long ldx, const float* mu, const void* shift, const int* seq, const int* qsl,
+                        const int* slots, const unsigned char* has, void* out, int rows, int W, cudaStream_t st) {
+  dim3 grid((rows + kShiftRows - 1) / kShiftRows, (W + 256 * V - 1) / (256 * V));
+  launch_chain_if(rows <= 256, token_shift_mix_kernel<T, 5, V>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(x), ldx, mu,
+                  reinterpret_cast<const T*>(shift), seq, qsl, slots, has, reinterpret_cast<T*>(out), rows, W);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+// ----------------------------------------------------------------------------- clamped gated unit, tanh
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+clamped_glu_kernel(const T* __restrict__ gu, long long ld, int I, T* y, long long ldy, float limit, float alpha) {
+  chain_trigger();
+  chain_wait();
+  const long long t = blockIdx.x;
+  const int e = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (e >= I) return;
+  float g[V], u[V], o[V];
+  load_vec<V>(gu + t * ld + e, g);
+  load_vec<V>(gu + t * ld + I + e, u);
+#pragma unroll
+  for (int i = 0; i < V; ++i) {
+    const float a = fminf(g[i], limit), b = fminf(fmaxf(u[i], -limit), limit);
+    o[i] = a / (1.f + expf(-alpha * a)) * (b + 1.f);
+  }
+  store_vec<V>(y + t * ldy + e, o);
+}
+
+template <typename T, int V>
+static int launch_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha, cudaStream_t st) {
+  dim3 grid(rows, (I + 256 * V - 1) / (256 * V));
+  launch_chain_if(rows <= 256, clamped_glu_kernel<T, V>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(gu), ld, I,
+                  reinterpret_cast<T*>(y), ldy, limit, alpha);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+tanh_kernel(T* x, long long n) {
+  chain_trigger();
+  chain_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = from_f32<T>(tanhf(to_f32(x[i])));
+}
+
+}  // namespace atlas
+
+using namespace atlas;
+
+// x [rows, S, W] fp32; y / y2 / out in bf16 (f32 = 0) or fp32 (f32 = 1)
+extern "C" int atlas_hyper_norm(float* x, int rows, int S, int W, const void* y, long long ldy, const void* y2, long long ldy2,
+                                const float* w1, const float* w2, const float* mix, const float* write, const float* read,
+                                const float* norm_w, void* out, long long ldo, int init, int store, float scale, float eps,
+                                int f32, void* stream) {
+  if (rows <= 0) return 0;
+  if (S < 1 || S > kMaxStreams || W < 1 || W > 50 * 1024) return -1;
+  if (y2 && (!w1 || !w2 || init)) return -2;
+  if (!init && (!mix || !write)) return -3;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return f32 ? hyper_norm<float>(x, rows, S, W, y, ldy, y2, ldy2, w1, w2, mix, write, read, norm_w, out, ldo, init, store, scale, eps, st)
+             : hyper_norm<__nv_bfloat16>(x, rows, S, W, y, ldy, y2, ldy2, w1, w2, mix, write, read, norm_w, out, ldo, init, store, scale,
+                                         eps, st);
+}
+
+// five mixes: mu [5, W] fp32, out [5, rows, W]; shift [slots, W] holds every sequence's previous row
+extern "C" int atlas_token_shift_mix(const void* x, long long ldx, const float* mu, const void* shift, const int* seq_of_token,
+                                     const int* qsl, const int* slots, const unsigned char* has, void* out, int rows, int W,
+                                     int f32, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) {
+    const bool vec = W % 4 == 0 && vec_ok<float, 4>(x, ldx) && vec_ok<float, 4>(mu, 0) && vec_ok<float, 4>(shift, W) && vec_ok<float, 4>(out, W);
+    return vec ? launch_shift<float, 4>(x, ldx, mu, shift, seq_of_token, qsl, slots, has, out, rows, W, st)
+               : launch_shift<float, 1>(x, ldx, mu, shift, seq_of_token, qsl, slots, has, out, rows, W, st);
+  }
+  using B = __nv_bfloat16;
+  const bool vec = W % 4 == 0 && vec_ok<B, 4>(x, ldx) && vec_ok<float, 4>(mu, 0) && vec_ok<B, 4>(shift, W) && vec_ok<B, 4>(out, W);
+  return vec ? launch_shift<B, 4>(x, ldx, mu, shift, seq_of_token, qsl, slots, has, out, rows, W, st)
+             : launch_shift<B, 1>(x, ldx, mu, shift, seq_of_token, qsl, slots, has, out, rows, W, st);
+}
+
+extern "C" int atlas_clamped_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha,
+                                 int f32, void* stream) {
+  if (rows <= 0 || I <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) {
+    const bool vec = I % 4 == 0 && vec_ok<float, 4>(gu, ld) && vec_ok<float, 4>(y, ldy);
+    return vec ? launch_glu<float, 4>(gu, ld, rows, I, y, ldy, limit, alpha, st) : launch_glu<float, 1>(gu, ld, rows, I, y, ldy, limit, alpha, st);
+  }
+  using B = __nv_bfloat16;
+  const bool vec = I % 8 == 0 && vec_ok<B, 8>(gu, ld) && vec_ok<B, 8>(y, ldy);
+  return vec ? launch_glu<B, 8>(gu, ld, rows, I, y, ldy, limit, alpha, st) : launch_glu<B, 1>(gu, ld, rows, I, y, ldy, limit, alpha, st);
+}
+
+extern "C" int atlas_tanh(void* x, long long n, int f32, void* stream) {
+  if (n <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid((unsigned)((n + 255) / 256));
+  if (f32) launch_chain_if(n <= 65536, tanh_kernel<float>, grid, dim3(256), 0, st, reinterpret_cast<float*>(x), n);
+  else launch_chain_if(n <= 65536, tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, reinterpret_cast<__nv_bfloat16*>(x), n);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}

@@ -81,7 +81,7 @@ class LLMEngine:
             from .layers import Attention
             self.selector = BlockSelector(num_blocks, self.cfg.block_size, self.cfg.sparse_attention_blocks)
             for l in model.layers:
-                if l.kind == "attention" and type(l.mixer) is Attention:
+                if l.kind == "attention" and type(l.mixer) is Attention and l.mixer.plain:
                     l.mixer.selector = self.selector
         self.scheduler = Scheduler(self.cfg, self.pool, self.radix, self.state_pool, self.hybrid, host_tier=self.host_tier)
         self.sampler = Sampler(self.mcfg.vocab_size, self.mcfg.eos_ids())
@@ -496,6 +496,50 @@ class LLMEngine:
                              seq.finish_reason.value if seq.finish_reason else None, len(seq.prompt_tokens),
                              seq.num_cached_tokens, ttft, dec, seq.logprobs if seq.logprobs else None,
                              seq.spec_accepted)
+
+    # ------------------------------------------------------------------ given tokens instead of sampled ones
+    @torch.inference_mode()
+    def feed(self, entries: Seq[tuple], end: Seq[str] = ()) -> List[torch.Tensor]:
+        """One step over given tokens (trace replay, scoring): nothing is sampled.
+
+        ``entries``: ``(request_id, tokens, want)`` with the request's next tokens and the places among them whose logits
+        are asked for; all entries run as one batch, on the pages, state slots and kernels that generation uses.  A
+        request is admitted at its first entry and those in ``end`` are released after the step.  Returns fp32 logits
+        ``[len(want), vocab]`` per entry, in the entries' order."""
+        sched = self.scheduler
+        seqs: List[Sequence] = []
+        for rid, tokens, _ in entries:
+            if not tokens or any(t < 0 or t >= self.mcfg.vocab_size for t in tokens):
+                raise RequestRejected(f"request {rid}: empty entry or token id out of range")
+            seq = self._seqs.get(rid)
+            if seq is None:
+                seq = Sequence(rid, [], SamplingParams())
+                sched.admit_now(seq)
+                self._seqs[rid] = seq
+            if seq.num_tokens + len(tokens) > self.cfg.max_seq_len:
+                raise RequestRejected(f"request {rid} exceeds max_seq_len {self.cfg.max_seq_len}")
+            seq.prompt_tokens.extend(int(t) for t in tokens)
+            seqs.append(seq)
+        result: List[torch.Tensor] = [torch.empty(0, self.mcfg.vocab_size)] * len(seqs)
+        if seqs:
+            out = sched.plan_fed(seqs)
+            batch = self.runner.build_batch(out, self.snapshot_base)
+            hidden = self.runner.forward(batch)
+            row0, first = 0, {}
+            for it in out.items:
+                first[it.seq.request_id] = row0
+                row0 += it.num_tokens
+            rows = [first[s.request_id] + w for s, e in zip(seqs, entries) for w in e[2]]
+            if rows:
+                logits = self.runner.logits(hidden, rows).float().cpu()
+                result = list(logits.split([len(e[2]) for e in entries]))
+            for it in out.items:
+                sched.on_chunk_computed(it)
+        for rid in end:
+            seq = self._seqs.pop(rid, None)
+            if seq is not None:
+                sched.finish(seq, FinishReason.STOP)
+        return result
 
     # ------------------------------------------------------------------ convenience
     def generate(self, prompts: Seq[Seq[int]], sampling: Optional[SamplingParams] = None,

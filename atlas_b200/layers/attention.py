@@ -28,9 +28,14 @@ class Attention:
         self.hq = cfg.num_attention_heads // tp
         self.hkv = max(1, cfg.num_key_value_heads // tp)
         self.kv_rep = max(1, tp // cfg.num_key_value_heads)     # ranks sharing one kv head
-        self.d = cfg.head_dim
+        # ``d`` is the width of a head in the cache and the kernels; query / key and value heads of other sizes are
+        # zero-padded to it by their projections, which leaves scores and outputs unchanged
+        self.dqk, self.dv = cfg.head_dim, cfg.v_head_dim or cfg.head_dim
+        self.d = cfg.attn_cache_width or cfg.head_dim
         self.gated = cfg.attn_output_gate
-        self.scale = cfg.attn_scale or self.d ** -0.5
+        self.scale = cfg.attn_scale or self.dqk ** -0.5
+        self.chunk = cfg.attn_chunk         # > 0: a token sees keys of its own ``chunk``-token block of the sequence only
+        self.sinks: Optional[torch.Tensor] = None       # [hq] fp32: extra term exp(sink) of the softmax denominator
         # models with per-layer attention kinds (Gemma): only "sliding_attention" layers use the window
         kinds = cfg.layer_types if (cfg.family != "hybrid" and cfg.layer_types) else None
         self.local = bool(kinds) and kinds[layer_idx] == "sliding_attention"
@@ -53,9 +58,15 @@ class Attention:
         return w[head * self.d:(head + self.hkv) * self.d]
 
     def load(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, o: torch.Tensor,
-             q_norm=None, k_norm=None, qkv_bias=None) -> None:
+             q_norm=None, k_norm=None, qkv_bias=None, sinks: Optional[torch.Tensor] = None) -> None:
         """Takes full (unsharded) HF-layout tensors; slices for this rank, fuses, quantizes."""
         cfg, tp, r = self.cfg, self.pctx.tp_size, self.pctx.tp_rank
+        if self.d != self.dqk or self.d != self.dv:
+            assert not self.gated and q_norm is None and qkv_bias is None, "padded heads: plain q / k / v projections only"
+            q, k, v = self._pad_rows(q, self.dqk), self._pad_rows(k, self.dqk), self._pad_rows(v, self.dv)
+            o = self._pad_rows(o.t(), self.dv).t()
+        if sinks is not None:
+            self.sinks = shard_rows(sinks.reshape(-1, 1), r, tp).reshape(-1).float().to(o.device).contiguous()
         if self.gated:   # HF q_proj rows are per head [q(D) | gate(D)]
             qg = q.view(cfg.num_attention_heads, 2, self.d, -1)
             q, gate = qg[:, 0].reshape(-1, q.shape[-1]), qg[:, 1].reshape(-1, q.shape[-1])
@@ -67,20 +78,34 @@ class Attention:
         self.o = make_weight(shard_cols(o, r, tp).contiguous(), self.quant_kind)
         self.q_norm, self.k_norm = q_norm, k_norm
 
+    def _pad_rows(self, w: torch.Tensor, d: int) -> torch.Tensor:
+        """``[heads * d, K]`` with every head's rows zero-padded to the cache width."""
+        if d == self.d:
+            return w
+        heads = w.reshape(-1, d, w.shape[-1])
+        return torch.nn.functional.pad(heads, (0, 0, 0, self.d - d)).reshape(-1, w.shape[-1])
+
     def init_random(self, gen, std, dtype, device) -> None:
         cfg = self.cfg
         h = cfg.hidden_size
         qmul = 2 if self.gated else 1
-        q = randn_weight(gen, cfg.num_attention_heads * self.d * qmul, h, std, dtype, device)
-        k = randn_weight(gen, cfg.num_key_value_heads * self.d, h, std, dtype, device)
-        v = randn_weight(gen, cfg.num_key_value_heads * self.d, h, std, dtype, device)
-        o = randn_weight(gen, h, cfg.num_attention_heads * self.d, std, dtype, device)
+        q = randn_weight(gen, cfg.num_attention_heads * self.dqk * qmul, h, std, dtype, device)
+        k = randn_weight(gen, cfg.num_key_value_heads * self.dqk, h, std, dtype, device)
+        v = randn_weight(gen, cfg.num_key_value_heads * self.dv, h, std, dtype, device)
+        o = randn_weight(gen, h, cfg.num_attention_heads * self.dv, std, dtype, device)
         qn = kn = None
         if cfg.qk_norm:
             base = 0.0 if cfg.norm_plus_one else 1.0
             qn = torch.full((self.d,), base, dtype=dtype, device=device)
             kn = torch.full((self.d,), base, dtype=dtype, device=device)
-        self.load(q, k, v, o, qn, kn)
+        sinks = torch.zeros(cfg.num_attention_heads, dtype=torch.float32, device=device) if cfg.attn_sinks else None
+        self.load(q, k, v, o, qn, kn, sinks=sinks)
+
+    @property
+    def plain(self) -> bool:
+        """No chunked visibility and no sink: every cache dtype and attention kernel applies.  Otherwise the layer keeps a
+        cache in the model's own dtype."""
+        return not self.chunk and not self.cfg.attn_sinks
 
     # ------------------------------------------------------------------ forward
     def forward(self, act: Act, batch, kv: Tuple[torch.Tensor, torch.Tensor, float, float],
@@ -123,11 +148,11 @@ class Attention:
                                   k_scale, v_scale, self.window)
         else:
             if (self.o.kind == "fp8_block" and not self.gated and self.o.bias is None and not self.kv_rotate
-                    and (self.lora is None or batch.adapter_rows is None)):
+                    and (self.lora is None or batch.adapter_rows is None) and self.plain):
                 a = ops.paged_attention_fp8_out(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window)
                 if a is not None:
                     return a                  # decode step: rows already quantised for the output projection
-            out = ops.paged_attention(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window)
+            out = ops.paged_attention(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window, self.chunk, self.sinks)
         if self.kv_rotate:
             out = ops.head_rotate(out)        # sum_j p_j (H v_j) = H o, and H is its own inverse
         out = out.reshape(T, nq)

@@ -46,14 +46,6 @@ def mamba2_scan_ref(x, dt, a_log, b, c, d_skip, dt_bias, dt_min, h):
     return torch.stack(ys).to(x.dtype), h
 
 
-def gated_group_rmsnorm_ref(y, z, w, group: int, eps: float):
-    """``rmsnorm_per_group(y * silu(z)) * w`` over the last dimension split into groups of ``group``."""
-    v = y.float() * F.silu(z.float())
-    g = v.view(*v.shape[:-1], -1, group)
-    g = g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)
-    return (g.view(v.shape) * w.float()).to(y.dtype)
-
-
 class Mamba2Mixer:
     def __init__(self, cfg: ModelConfig, layer_idx: int, pctx: ParallelCtx, quant_kind: str):
         self.cfg, self.layer_idx, self.pctx, self.quant_kind = cfg, layer_idx, pctx, quant_kind
@@ -61,6 +53,10 @@ class Mamba2Mixer:
         assert cfg.mamba_num_heads % tp == 0 and cfg.mamba_n_groups % tp == 0, "mamba heads and groups must divide by tp"
         self.h, self.p, self.n = cfg.mamba_num_heads // tp, cfg.mamba_head_dim, cfg.ssm_state_size
         self.g = cfg.mamba_n_groups // tp
+        # the output norm's parts: one per B / C group unless the model counts them separately
+        norm_groups = cfg.mamba_norm_groups or cfg.mamba_n_groups
+        assert norm_groups % tp == 0, "norm groups must divide by tp"
+        self.norm_groups = norm_groups // tp
         self.d_inner = self.h * self.p
         self.conv_dim = self.d_inner + 2 * self.g * self.n
         self.W = cfg.mamba_conv_kernel
@@ -119,11 +115,7 @@ class Mamba2Mixer:
         else:
             y = self._forward_ref(xbc, dt, batch.query_lens_host, batch.state_slots_host, batch.has_state_host, state,
                                   commit=not batch.spec_verify, snapshot_plan=batch.snapshot_plan)
-        group = self.d_inner // self.g
-        if ops.on_gpu(proj) and y.dtype == torch.bfloat16:
-            out = ops.cuda_ops().mamba2_gated_norm(y, z, self.norm_w, group, self.cfg.rms_norm_eps)
-        else:
-            out = gated_group_rmsnorm_ref(y, z, self.norm_w, group, self.cfg.rms_norm_eps)
+        out = ops.group_norm_gate(y, z, self.norm_w, self.d_inner // self.norm_groups, self.cfg.rms_norm_eps, gate_first=True)
         return self.pctx.row_parallel_linear(out, self.out_proj)
 
     def _forward_ref(self, xbc, dt, qlens: List[int], slots: List[int], has_state: List[bool], state: dict, commit: bool,

@@ -47,11 +47,16 @@ class DenseMLP:
 
     def hidden_act(self, act: Act) -> Act:
         """gate|up GEMM + SiLU * mul: the input of the down projection (no adapters)."""
-        if self.activation == "gelu_tanh_glu":
-            return ops.glu_act(ops.linear(act, self.gate_up), self.down.kind == "fp8_block", "gelu_tanh")
+        if self.activation in ("gelu_tanh_glu", "clamped_glu"):
+            return self._glu(ops.linear(act, self.gate_up), self.down.kind == "fp8_block")
         if self.down.kind == "fp8_block" and ops.swiglu_fusable(act, self.gate_up):
             return ops.linear_swiglu(act, self.gate_up)
         return ops.silu_mul_act(ops.linear(act, self.gate_up), want_fp8=self.down.kind == "fp8_block")
+
+    def _glu(self, gate_up: torch.Tensor, want_fp8: bool) -> Act:
+        if self.activation == "clamped_glu":
+            return ops.clamped_glu_act(gate_up, self.cfg.glu_limit, self.cfg.glu_alpha)
+        return ops.glu_act(gate_up, want_fp8, "gelu_tanh")
 
     def _relu2(self, act: Act, reduce: bool) -> torch.Tensor:
         u = ops.linear(act, self.gate_up)
@@ -62,7 +67,7 @@ class DenseMLP:
         if self.activation == "relu2":
             return self._relu2(act, reduce)
         use_lora = self.lora is not None and batch is not None and batch.adapter_rows is not None and self.lora_prefix
-        if self.activation == "gelu_tanh_glu" and not use_lora:
+        if self.activation in ("gelu_tanh_glu", "clamped_glu") and not use_lora:
             a = self.hidden_act(act)
             return self.pctx.row_parallel_linear(a, self.down) if (self.shard and reduce) else ops.linear(a, self.down)
         if not use_lora and self.down.kind == "fp8_block" and ops.swiglu_fusable(act, self.gate_up):
@@ -73,8 +78,8 @@ class DenseMLP:
             xin, half = act.plain(), gu.shape[1] // 2
             add_delta(gu, self.lora, self.lora_prefix + "gate_proj", xin, batch, 0, half)
             add_delta(gu, self.lora, self.lora_prefix + "up_proj", xin, batch, half, half)
-        if self.activation == "gelu_tanh_glu":
-            a = ops.glu_act(gu, False, "gelu_tanh")
+        if self.activation in ("gelu_tanh_glu", "clamped_glu"):
+            a = self._glu(gu, False)
         else:
             a = ops.silu_mul_act(gu, want_fp8=self.down.kind == "fp8_block" and not use_lora)
         if use_lora:

@@ -17,6 +17,7 @@ import torch
 from ..config import ModelConfig
 from ..layers import ParallelCtx
 from ..layers.moe import ExpertWeights
+from ..layers.wkv import MIXES
 from ..models import DecoderLM, build_model
 from ..models.decoder import quant_kinds
 from ..ops import LinearWeight
@@ -264,9 +265,39 @@ def _load_single_blocks(model: DecoderLM, ck: Checkpoint, dense_kind: str) -> No
     ck.close()
 
 
+def _load_papidra(model: DecoderLM, ck: Checkpoint) -> None:
+    """Papidra naming: ``embed``, ``l<i>.{norm1, norm2, mix.*, mlp.*, hc1.*, hc2.*}``, ``final.norm``; the embedding table is
+    the output projection."""
+    wt = lambda name: ck.get(name).to(device=model.device, dtype=model.dtype)
+    f32 = lambda name: ck.get(name).to(device=model.device, dtype=torch.float32).contiguous()
+    model.embed = wt("embed").contiguous()
+    for i, layer in enumerate(model.layers):
+        pre, mx = f"l{i}.", layer.mixer
+        layer.input_norm = f32(pre + "norm1")
+        layer.conn1.load(*(ck.get(f"{pre}hc1.{n}") for n in ("in", "out", "mix")), model.device)
+        if layer.kind == "wkv":
+            mx.load([ck.get(f"{pre}mix.mu.{s}") for s in MIXES], *(wt(f"{pre}mix.{n}") for n in ("r", "k", "v", "g", "w1", "w2")),
+                    *(ck.get(f"{pre}mix.{n}") for n in ("w0", "u", "norm")), wt(pre + "mix.o"), model.device)
+        else:
+            a, b = pre + "mix.left.", pre + "mix.right."
+            mx.left.load(*(wt(a + n) for n in "qkvo"), sinks=ck.get(a + "sink"))
+            mx.right.load(wt(b + "in"), wt(b + "conv"), wt(b + "conv.b"), f32(b + "A_log"), f32(b + "D"), f32(b + "dt_bias"),
+                          f32(b + "norm"), wt(b + "o"))
+            mx.left_norm, mx.right_norm = f32(a + "out"), f32(b + "out")
+        if layer.ffn is not None:
+            layer.post_norm = f32(pre + "norm2")
+            layer.conn2.load(*(ck.get(f"{pre}hc2.{n}") for n in ("in", "out", "mix")), model.device)
+            layer.ffn.load(*(wt(f"{pre}mlp.{n}") for n in ("gate", "up", "down")))
+    model.final_norm = f32("final.norm")
+    model.set_lm_head(model.embed)
+    ck.close()
+
+
 def load_weights(model: DecoderLM, ck: Checkpoint) -> None:
     cfg = model.cfg
     dense_kind, expert_kind = quant_kinds(cfg)
+    if cfg.model_type == "papidra":
+        return _load_papidra(model, ck)
     if cfg.block_types:
         if any(k.endswith((".weight_scale_inv", ".weight_scale", ".weight_packed")) for k in ck.keys()):
             dense_kind = "dense"

@@ -17,9 +17,10 @@ import torch
 
 from .. import ops
 from ..config import ModelConfig
-from ..layers import Attention, DenseMLP, GatedDeltaNet, Mamba2Mixer, MLAttention, MoE, ParallelCtx
+from ..layers import (MIXERS, Attention, DenseMLP, GatedDeltaNet, HyperConnection, Mamba2Mixer, MLAttention, MoE, ParallelCtx,
+                      ParallelMixer)
 from ..layers.common import make_weight, randn_weight, shard_rows
-from ..ops import Act, LinearWeight, reference as ref
+from ..ops import Act, LinearWeight, StreamDelta, reference as ref
 from .batch import ForwardBatch
 
 # tensor-parallel steps with at least this many rows run sequence-parallel (reduce-scatter / all-gather fused into the
@@ -51,7 +52,7 @@ def kv_element_bytes(dtype) -> float:
 def alloc_kv(num_blocks: int, block_size: int, hkv: int, d: int, dtype, device):
     """Paged K and V pools as logical ``[num_blocks, block_size, Hkv, D]`` tensors (the GPU pools are views
     of the kernels' physical layout)."""
-    if torch.device(device).type == "cuda" and (kv_dtype_is_quantised(dtype) or dtype == torch.bfloat16):
+    if torch.device(device).type == "cuda" and (kv_dtype_is_quantised(dtype) or dtype in (torch.bfloat16, torch.float32)):
         return ops.cuda_ops().alloc_kv_cache(num_blocks, block_size, hkv, d, dtype, device)
     if dtype == KV_NVFP4:
         raise ValueError("the NVFP4 KV cache exists on the GPU kernels only")
@@ -250,6 +251,68 @@ class SingleBlock:
         return h, residual
 
 
+class StreamLayer:
+    """A layer on hyper-connected residual streams (``layers/hyper.py``): a mixer of any kind and, where the model's layer
+    list says so, a feed-forward sublayer.  Same ``forward`` protocol as :class:`DecoderLayer`, with the pending
+    :class:`StreamDelta` in place of the previous layer's output and the streams in place of the residual."""
+
+    def __init__(self, cfg: ModelConfig, idx: int, pctx: ParallelCtx):
+        spec = cfg.layer_specs[idx]
+        self.cfg, self.idx = cfg.for_layer(idx), idx
+        dense_kind, _ = quant_kinds(cfg)
+        self.kind, self.is_moe = spec.kind, False
+        self.mixer = MIXERS[spec.kind](self.cfg, idx, pctx, dense_kind)
+        self.ffn = DenseMLP(self.cfg, pctx, dense_kind) if spec.has_mlp else None
+        self.conn1 = HyperConnection(cfg.residual_streams)
+        self.conn2 = HyperConnection(cfg.residual_streams) if spec.has_mlp else None
+        self.input_norm: Optional[torch.Tensor] = None         # fp32
+        self.post_norm: Optional[torch.Tensor] = None
+        self.rope_override: Optional[torch.Tensor] = None      # this layer's own rotary table
+
+    def init_random(self, gen, std, dtype, device):
+        ones = lambda: torch.ones(self.cfg.hidden_size, dtype=torch.float32, device=device)
+        self.mixer.init_random(gen, std, dtype, device)
+        self.conn1.init_random(gen, device)
+        self.input_norm = ones()
+        if self.ffn is not None:
+            self.ffn.init_random(gen, std, dtype, device)
+            self.conn2.init_random(gen, device)
+            self.post_norm = ones()
+
+    def accepts_prenormed(self) -> bool:
+        return False
+
+    def forward(self, x: StreamDelta, streams: Optional[torch.Tensor], batch: ForwardBatch, cache: CacheStore, rope_cache,
+                next_norm=None):
+        eps = self.cfg.rms_norm_eps
+        rope_cache = rope_cache if self.rope_override is None else self.rope_override
+        h, streams = ops.hyper_norm(streams, x, self.conn1.read, self.input_norm, eps)
+        act = Act(x=h)
+        if self.kind == "parallel":
+            a, b = self.mixer.forward(act, batch, cache.layer_kv(self.idx), rope_cache, cache.states[self.idx])
+            x = StreamDelta(a, self.conn1, y2=b, w1=self.mixer.left_norm, w2=self.mixer.right_norm)
+        elif self.kind == "attention":
+            x = StreamDelta(self.mixer.forward(act, batch, cache.layer_kv(self.idx), rope_cache), self.conn1)
+        else:
+            x = StreamDelta(self.mixer.forward(act, batch, cache.states[self.idx]), self.conn1)
+        if self.ffn is not None:
+            h, streams = ops.hyper_norm(streams, x, self.conn2.read, self.post_norm, eps)
+            x = StreamDelta(self.ffn.forward(Act(x=h), batch=batch), self.conn2)
+        return x, streams
+
+
+def attention_of(layer):
+    """The attention block of a layer (None without one): the owner of the layer's KV cache."""
+    if layer.kind == "parallel":
+        return layer.mixer.left
+    return layer.mixer if layer.kind == "attention" else None
+
+
+def recurrent_of(layer):
+    """The mixer of a layer that owns a recurrent state slot (None without one)."""
+    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel") else None
+
+
 class DecoderLM:
     def __init__(self, cfg: ModelConfig, pctx: Optional[ParallelCtx] = None, device="cpu", ep_mode: str = "auto",
                  with_mtp: Optional[bool] = None):
@@ -257,7 +320,11 @@ class DecoderLM:
         self.pctx = pctx or ParallelCtx()
         self.device = torch.device(device)
         self.dtype = torch_dtype(cfg.dtype)
-        if cfg.block_types:
+        if cfg.layer_specs:
+            if cfg.residual_streams < 1:
+                raise ValueError("a model given by a list of layers runs on hyper-connected residual streams")
+            self.layers = [StreamLayer(cfg, i, self.pctx) for i in range(cfg.num_hidden_layers)]
+        elif cfg.block_types:
             self.layers = [SingleBlock(cfg, i, self.pctx) for i in range(cfg.num_hidden_layers)]
         else:
             self.layers = [DecoderLayer(cfg, i, self.pctx, ep_mode) for i in range(cfg.num_hidden_layers)]
@@ -277,6 +344,8 @@ class DecoderLM:
         self.aux_hidden: List[torch.Tensor] = []
         self.dflash = None                   # models.dflash.BlockDiffusionDrafter
         self.vision = None                   # models.vision.VisionTower (multimodal checkpoints)
+        if self.dtype == torch.float32 and self.device.type == "cuda":
+            torch.backends.cuda.matmul.allow_tf32 = False      # a 32-bit model multiplies in full 32-bit
 
     # ------------------------------------------------------------------ weights
     def init_random(self, seed: int = 0, std: float = 0.02, max_pos: Optional[int] = None) -> "DecoderLM":
@@ -288,7 +357,7 @@ class DecoderLM:
         for layer in self.layers:
             layer.init_random(gen, std, dt, dev)
         base = 0.0 if cfg.norm_plus_one else 1.0
-        self.final_norm = torch.full((cfg.hidden_size,), base, dtype=dt, device=dev)
+        self.final_norm = torch.full((cfg.hidden_size,), base, dtype=torch.float32 if cfg.residual_streams else dt, device=dev)
         head = self.embed if cfg.tie_word_embeddings else randn_weight(gen, cfg.vocab_size, cfg.hidden_size, std, dt, dev)
         self.set_lm_head(head)
         if self.mtp is not None:
@@ -302,8 +371,10 @@ class DecoderLM:
         if getattr(self, "lora", None) is None:
             self.lora = LoraSet(max_slots)
             for l in self.layers:
-                if l.kind == "attention":
-                    l.mixer.lora = self.lora
+                if attention_of(l) is not None:
+                    attention_of(l).lora = self.lora
+                if l.ffn is None:
+                    continue
                 l.ffn.lora, l.ffn.lora_prefix = self.lora, f"layers.{l.idx}.mlp."
                 shared = getattr(l.ffn, "shared", None)
                 if shared is not None:
@@ -320,7 +391,7 @@ class DecoderLM:
         from ..layers.attention import Attention
         cfg = self.cfg
         d = cfg.head_dim
-        if cfg.kv_lora_rank > 0 or d & (d - 1):
+        if cfg.kv_lora_rank > 0 or cfg.layer_specs or d & (d - 1):
             return False
         if self.device.type == "cuda" and not (d == 128 and cfg.rotary_dim == 128):
             return False
@@ -349,16 +420,37 @@ class DecoderLM:
             for l in self.layers:
                 if l.kind == "attention" and getattr(l.mixer, "local", False):
                     l.rope_override = local
+        tables: Dict[str, torch.Tensor] = {}
+        for l in self.layers if cfg.layer_specs else ():
+            if attention_of(l) is not None:
+                key = (l.cfg.rotary_dim, l.cfg.rope_theta, l.cfg.rope_scaling)
+                if str(key) not in tables:
+                    tables[str(key)] = ref.build_rope_cache(key[0], mp, key[1], key[2], self.device)
+                l.rope_override = tables[str(key)]
 
     # ------------------------------------------------------------------ cache allocation
     def attention_layers(self) -> List[int]:
-        return [l.idx for l in self.layers if l.kind == "attention"]
+        return [l.idx for l in self.layers if attention_of(l) is not None]
 
     def gdn_layers(self) -> List[int]:
-        """Layers with a recurrent state slot (Gated DeltaNet or Mamba-2)."""
-        return [l.idx for l in self.layers if l.kind in ("gdn", "mamba2")]
+        """Layers with a recurrent state slot (Gated DeltaNet, Mamba-2, WKV, attention beside Mamba-2)."""
+        return [l.idx for l in self.layers if recurrent_of(l) is not None]
+
+    def _cache_dtype(self, layer, kv_dtype, high_precision) -> torch.dtype:
+        """Cache dtype of one layer: the engine's, 16 bits for layers that ask for high precision, the model's own for
+        attention variants (chunks, sinks) whose kernels read nothing else."""
+        a = attention_of(layer)
+        if not getattr(a, "plain", True):
+            return self.dtype
+        if layer.idx in high_precision and kv_dtype_is_quantised(kv_dtype):
+            return torch.bfloat16 if self.dtype == torch.bfloat16 else self.dtype
+        return kv_dtype
 
     def kv_bytes_per_block(self, block_size: int, kv_dtype: torch.dtype, high_precision_layers=()) -> int:
+        if self.cfg.layer_specs:
+            owners = [(l, attention_of(l)) for l in self.layers if attention_of(l) is not None]
+            return int(sum(2 * block_size * a.hkv * a.d * kv_element_bytes(self._cache_dtype(l, kv_dtype, set(high_precision_layers)))
+                           for l, a in owners))
         n_attn = len(self.attention_layers()) + (1 if self.mtp is not None else 0)
         hkv = self.layers[self.attention_layers()[0]].mixer.hkv if n_attn else 0
         n_hi = len([i for i in self.attention_layers() if i in set(high_precision_layers)])
@@ -372,11 +464,11 @@ class DecoderLM:
         store = CacheStore(block_size=block_size, num_blocks=num_blocks)
         hi = set(high_precision_layers)
         for l in self.layers:
-            if l.kind == "attention":
-                dt = (torch.bfloat16 if self.dtype == torch.bfloat16 else self.dtype) if (l.idx in hi and kv_dtype_is_quantised(kv_dtype)) else kv_dtype
-                store.kv[l.idx] = alloc_kv(num_blocks, block_size, l.mixer.hkv, self.cfg.head_dim, dt, self.device)
+            a = attention_of(l)
+            if a is not None:
+                store.kv[l.idx] = alloc_kv(num_blocks, block_size, a.hkv, a.d, self._cache_dtype(l, kv_dtype, hi), self.device)
                 store.kv_scales[l.idx] = (1.0, 1.0)
-            elif l.kind in ("gdn", "mamba2"):
+            if recurrent_of(l) is not None:
                 store.states[l.idx] = l.mixer.alloc_state(max(1, state_slots), self.device, self.dtype)
         if self.mtp is not None:
             self.mtp.alloc_cache(store, num_blocks, block_size, kv_dtype, self.device)
@@ -388,7 +480,7 @@ class DecoderLM:
         if checked.ENABLED:
             checked.index_range("input_ids", ids, 0, self.cfg.vocab_size)
         e = self.embed[ids.long()]
-        if self.cfg.embed_scale != 1.0:
+        if self.cfg.embed_scale != 1.0 and not self.cfg.residual_streams:
             e = e * torch.tensor(self.cfg.embed_scale, dtype=e.dtype)      # the factor is rounded to the weight dtype first
         return e
 
@@ -460,7 +552,9 @@ class DecoderLM:
         if sp is not None:
             return self._forward_seq_parallel(x, batch, cache, sp)
         residual = None
-        if batch.inputs_embeds is not None:
+        if self.cfg.residual_streams:
+            x = StreamDelta(x, scale=self.cfg.embed_scale)      # fp32 streams start from the scaled embedding
+        elif batch.inputs_embeds is not None:
             x = x.clone()                     # fused epilogues update the residual stream in place
         if layer_ids is not None:
             layers = [self.layers[i] for i in layer_ids]
@@ -468,20 +562,39 @@ class DecoderLM:
                 nxt = layers[k + 1] if k + 1 < len(layers) else None
                 next_norm = nxt.input_norm if (nxt is not None and nxt.accepts_prenormed()) else None
                 x, residual = layer.forward(x, residual, batch, cache, self.rope_cache, next_norm=next_norm)
-            y, _ = ops.rmsnorm(x, self.final_norm, self.cfg.rms_norm_eps, residual, self.cfg.norm_plus_one)
-            return y
+            return self._final_norm(x, residual)
         n = len(self.layers)
         self.aux_hidden = []
         for i, layer in enumerate(self.layers):
             nxt = self.layers[i + 1] if i + 1 < n else None
             next_norm = nxt.input_norm if (nxt is not None and nxt.accepts_prenormed()) else None
             x, residual = layer.forward(x, residual, batch, cache, self.rope_cache, next_norm=next_norm)
-            if i in self.capture_layers:
+            if i in self.capture_layers and isinstance(x, StreamDelta):
+                self.aux_hidden.append(self._stream_sum(x, residual))
+            elif i in self.capture_layers:
                 # the stream after layer i: already summed when the layer's epilogue handed over normalised activations
                 self.aux_hidden.append(residual.clone() if isinstance(x, Act) else (x + residual if residual is not None else x.clone()))
         self.last_prenorm = (x, residual)
+        return self._final_norm(x, residual)
+
+    def _final_norm(self, x, residual) -> torch.Tensor:
+        if isinstance(x, StreamDelta):
+            y, _ = ops.hyper_norm(residual, x, self._stream_ones, self.final_norm, self.cfg.rms_norm_eps, write=False)
+            return y
         y, _ = ops.rmsnorm(x, self.final_norm, self.cfg.rms_norm_eps, residual, self.cfg.norm_plus_one)
         return y
+
+    @property
+    def _stream_ones(self) -> torch.Tensor:
+        t = getattr(self, "_ones", None)
+        if t is None:
+            t = self._ones = torch.ones(self.cfg.residual_streams, dtype=torch.float32, device=self.device)
+        return t
+
+    def _stream_sum(self, x: StreamDelta, streams: torch.Tensor) -> torch.Tensor:
+        """Sum of the residual streams with a pending update applied (fp32)."""
+        _, after = ops.hyper_norm(streams.clone(), x, self._stream_ones, self.final_norm, self.cfg.rms_norm_eps)
+        return after.sum(1)
 
     @torch.inference_mode()
     def compute_logits(self, hidden: torch.Tensor, indices: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -567,7 +680,7 @@ class DecoderLM:
     def commit_spec(self, accepted_rows: List[int], cache: CacheStore) -> None:
         """After speculative verification: fold the accepted rows into every GDN layer's state."""
         for l in self.layers:
-            if l.kind in ("gdn", "mamba2"):
+            if recurrent_of(l) is not None:
                 l.mixer.commit(accepted_rows, cache.states[l.idx])
 
     # ------------------------------------------------------------------ oracle

@@ -112,6 +112,30 @@ class Act:
         return self.q, self.s
 
 
+@dataclass
+class StreamDelta:
+    """What the last sublayer leaves for the residual streams (``layers/hyper.py``).
+
+    Start of the model (``conn`` is None): every stream becomes ``y * scale``.  Otherwise the streams are rewritten with the
+    sublayer's connection ``conn`` and its output ``y``, or, with ``y2``, half the sum of ``y`` and ``y2`` after an RMS norm
+    each with the weights ``w1`` / ``w2``."""
+    y: torch.Tensor
+    conn: Optional[object] = None            # layers.hyper.HyperConnection
+    scale: float = 1.0
+    y2: Optional[torch.Tensor] = None
+    w1: Optional[torch.Tensor] = None
+    w2: Optional[torch.Tensor] = None
+
+
+def hyper_norm(streams: Optional[torch.Tensor], delta: StreamDelta, read: torch.Tensor, norm_w: torch.Tensor, eps: float,
+               write: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Apply ``delta`` to ``streams [T, S, W]`` (fp32, in place; None at the start), read ``u = sum_s read[s] * streams[s]``
+    and return ``(rmsnorm(u) * norm_w, streams)``.  ``write=False`` leaves the streams as they are (last read of a step)."""
+    if on_gpu(delta.y):
+        return cuda_ops().hyper_norm(streams, delta, read, norm_w, eps, write)
+    return ref.hyper_norm(streams, delta, read, norm_w, eps)
+
+
 # ----------------------------------------------------------------------------- elementwise / norm
 def quant_fp8(x: torch.Tensor, group: int = 128):
     if on_gpu(x):
@@ -157,6 +181,28 @@ def glu_act(gate_up: torch.Tensor, want_fp8=False, kind: str = "silu") -> Act:
             q, s = Q.per_token_group_quant_fp8(ref.gelu_tanh_mul(gate_up), 128)
         return Act(q=q, s=s, dtype=gate_up.dtype)
     return Act(x=cuda_ops().gelu_tanh_mul(gate_up) if gpu else ref.gelu_tanh_mul(gate_up))
+
+
+def clamped_glu_act(gate_up: torch.Tensor, limit: float, alpha: float) -> Act:
+    """``g * sigmoid(alpha * g) * (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``."""
+    if on_gpu(gate_up):
+        return Act(x=cuda_ops().clamped_glu(gate_up, limit, alpha))
+    return Act(x=ref.clamped_glu(gate_up, limit, alpha))
+
+
+def tanh_(x: torch.Tensor) -> torch.Tensor:
+    """``tanh`` in place."""
+    if on_gpu(x):
+        return cuda_ops().tanh_(x)
+    return x.tanh_()
+
+
+def group_norm_gate(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, group: int, eps: float, gate_first: bool) -> torch.Tensor:
+    """RMS norm over groups of ``group`` channels joined with a SiLU gate: ``norm(y * silu(z)) * w`` with ``gate_first``
+    (Mamba-2), ``norm(y) * w * silu(z)`` otherwise (WKV).  ``z`` may be a column slice."""
+    if on_gpu(y):
+        return cuda_ops().group_norm_gate(y, z, w, group, eps, gate_first)
+    return ref.group_norm_gate(y, z, w, group, eps, gate_first)
 
 
 def silu_mul_act(gate_up: torch.Tensor, want_fp8=False) -> Act:
@@ -274,12 +320,14 @@ def head_rotate(x: torch.Tensor) -> torch.Tensor:
     return ref.head_rotate(x)
 
 
-def paged_attention(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None) -> torch.Tensor:
-    """Attention of the step's query rows over the paged cache. ``batch`` is a ``ForwardBatch``."""
+def paged_attention(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None, chunk=0,
+                    sinks=None) -> torch.Tensor:
+    """Attention of the step's query rows over the paged cache. ``batch`` is a ``ForwardBatch``.  ``chunk`` > 0: a token sees
+    only keys of its own ``chunk``-token block of the sequence; ``sinks [Hq]``: ``exp(sink)`` joins the softmax denominator."""
     if on_gpu(q):
-        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window)
+        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk, sinks)
     return ref.paged_attention(q, k_cache, v_cache, batch.block_tables, batch.seq_lens, batch.query_start_loc,
-                               scale, k_scale, v_scale, sliding_window)
+                               scale, k_scale, v_scale, sliding_window, chunk, sinks)
 
 
 def paged_attention_fp8_out(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None) -> Optional[Act]:

@@ -36,13 +36,38 @@ class KernelError(RuntimeError):
     pass
 
 
+class _KernelLibrary(C.CDLL):
+    """The kernel library.  A library built for one model holds only the translation units that model calls
+    (``build.units_for``): an entry point outside of them raises when it is called, not when it is bound."""
+
+    def __getattr__(self, name):
+        try:
+            return super().__getattr__(name)
+        except AttributeError:
+            if not name.startswith("atlas_"):
+                raise
+
+            def absent(*_):
+                raise KernelError(f"{name} is not part of {self._name}: run `python -m atlas_b200.build`")
+            setattr(self, name, absent)
+            return absent
+
+
+def use_library(path: str) -> None:
+    """Load ``path`` instead of the full library (before the first kernel call of the process)."""
+    global LIB_PATH
+    if _LIB is not None and path != LIB_PATH:
+        raise KernelError(f"{LIB_PATH} is already loaded")
+    LIB_PATH = path
+
+
 def load() -> None:
     global _LIB
     if _LIB is not None:
         return
     if not os.path.exists(LIB_PATH):
         raise KernelError(f"{LIB_PATH} is missing: run `python -m atlas_b200.build` (the GPU path has no eager fallback)")
-    lib = C.CDLL(LIB_PATH)
+    lib = _KernelLibrary(LIB_PATH)
     lib.atlas_status_ptr.restype = C.c_void_p
     lib.atlas_read_status.restype = C.c_ulonglong
     lib.atlas_gemm.argtypes = [_i, _vp, _vp, _vp, _vp, _ll, _ll, _vp, _i, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
@@ -421,6 +446,9 @@ def gemm_fp8_fused(xq, xs, wq, ws, mode: int = 0, out=None, residual=None, norm_
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None) -> torch.Tensor:
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
+    if x.shape[1] % 8:                 # rows that TMA cannot address (16-byte strides): a vendor product
+        y = torch.nn.functional.linear(x, w)
+        return y if out is None else out.copy_(y)
     if x.stride(1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
     return _gemm(0, x, w, None, None, out)
@@ -473,8 +501,8 @@ def _kv_layout_ok(k_cache: torch.Tensor, v_cache: torch.Tensor) -> None:
     nb, bs, hkv, d = k_cache.shape
     if k_cache.stride() != (hkv * bs * d, d, bs * d, 1) or v_cache.stride() != (hkv * bs * d, 1, d * bs, bs):
         raise KernelError("KV cache is not in the kernel layout (allocate it with ops.cuda.alloc_kv_cache)")
-    if k_cache.dtype not in (FP8, torch.bfloat16, torch.uint8):
-        raise KernelError("the GPU attention kernels read an FP8 (e4m3), bf16 or NVFP4 KV cache")
+    if k_cache.dtype not in (FP8, torch.bfloat16, torch.uint8, torch.float32):
+        raise KernelError("the GPU attention kernels read an FP8 (e4m3), bf16, NVFP4 or fp32 KV cache")
 
 
 def wht_d128(x: torch.Tensor) -> torch.Tensor:
@@ -493,6 +521,13 @@ def qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v
     Hkv = k.shape[1]
     _dev(q)
     _kv_layout_ok(k_cache, v_cache)
+    if q.dtype == torch.float32:
+        if q_norm_w is not None or rotate:
+            raise KernelError("32-bit attention has neither head norms nor a rotated cache")
+        if checked.ENABLED:
+            checked.kv_write(slot_mapping, positions, k_cache.shape[0], k_cache.shape[1], rope_cache.shape[0] if rotary_dim else 0)
+        from . import cuda_recurrent
+        return cuda_recurrent.rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping)
     assert q.stride(2) == 1 and q.stride(1) == D and k.stride(1) == D and v.stride(1) == D
     assert positions.dtype == torch.int32 and slot_mapping.dtype == torch.int32 and rope_cache.dtype == torch.float32
     bs = k_cache.shape[1]
@@ -522,7 +557,7 @@ def decode_splits(B: int, hkv: int, max_seq_len: int, sms: int) -> int:
     return int(max(1, min((2 * sms + ctas - 1) // ctas, (pages + 7) // 8, 64)))
 
 
-def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window):
+def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk=0, sinks=None):
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     d = _dev(q)
@@ -534,8 +569,15 @@ def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding
     st = _stream()
     if checked.ENABLED:
         checked.paged_read(batch.block_tables, batch.seq_lens, k_cache.shape[0], k_cache.shape[1])
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != Hq or not sinks.is_contiguous()):
+        raise KernelError("attention sinks are one fp32 value per query head")
+    if k_cache.dtype == torch.float32:
+        from . import cuda_recurrent
+        return cuda_recurrent.attention_f32(q, k_cache, v_cache, batch, scale, window, int(chunk), sinks)
     if k_cache.dtype == torch.bfloat16:
-        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d)
+        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, chunk=int(chunk), sinks=sinks)
+    if chunk or sinks is not None:
+        raise KernelError("chunked attention and softmax sinks need a bf16 or fp32 KV cache")
     if is_nvfp4_kv(k_cache):
         return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=(float(k_scale), float(v_scale)))
     if nd > 0:
@@ -652,7 +694,7 @@ def _tc_tiles(q, batch, nd: int, tok: int):
     return tiles
 
 
-def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None):
+def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None, chunk=0, sinks=None):
     """bf16 KV cache (or, with ``scales = (k_scale, v_scale)``, an NVFP4 one): the general mma.sync kernel serves decode
     rows (split-K + merge) and prefill tiles."""
     T, Hq, D = q.shape
@@ -669,12 +711,13 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
         raise KernelError("the NVFP4 KV cache is implemented for head_dim 128")
     if not getattr(L, "_kv16_bound", False):
         L.atlas_attn_decode_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i,
-                                             _vp, _vp, _vp]
-        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp]
+                                             _vp, _vp, _vp, _i, _vp]
+        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp, _i, _vp]
         L._kv16_bound = True
     bt, st, nd = batch.block_tables, _stream(), batch.num_decodes
     if nd > 0:
-        splits = decode_splits(nd, Hkv, batch.max_seq_len, _num_sms[d])
+        visible = min(batch.max_seq_len, chunk or batch.max_seq_len, window or batch.max_seq_len)
+        splits = decode_splits(nd, Hkv * ((Hq // Hkv + 15) // 16), visible, _num_sms[d])
         po = pml = None
         if splits > 1:
             po = scratch("attn_part_o", nd * Hq * splits * D * 4, q.device)
@@ -687,8 +730,8 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
         else:
             _check(L.atlas_attn_decode_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                             bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
-                                            0, nd, float(scale), Hq, Hkv, D, bs, window, splits, _ptr(po), _ptr(pml), st),
-                   "attn_decode_kv16")
+                                            0, nd, float(scale), Hq, Hkv, D, bs, window, splits, _ptr(po), _ptr(pml), st, chunk,
+                                            _ptr(sinks)), "attn_decode_kv16")
     if batch.num_seqs > nd:
         tiles = getattr(batch, "_attn_tiles", None)
         if tiles is None:
@@ -709,8 +752,8 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
         else:
             _check(L.atlas_attn_prefill_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                              bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
-                                             tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, float(scale), Hq, Hkv, D, bs, window, st),
-                   "attn_prefill_kv16")
+                                             tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, float(scale), Hq, Hkv, D, bs, window, st, chunk,
+                                             _ptr(sinks)), "attn_prefill_kv16")
     return out
 
 
@@ -824,18 +867,48 @@ def gdn_commit(layer, mixed, a, b, qlens, slots, has_state, state, num_accepted_
 
 
 def mamba2_forward(layer, xbc, dt, batch, state, commit):
-    from . import cuda_gdn
-    return cuda_gdn.mamba2_forward(layer, xbc, dt, batch, state, commit)
+    from . import cuda_recurrent
+    return cuda_recurrent.mamba2_forward(layer, xbc, dt, batch, state, commit)
 
 
 def mamba2_commit(layer, xbc, dt, qlens, slots, has_state, state, num_accepted_rows):
-    from . import cuda_gdn
-    return cuda_gdn.mamba2_commit(layer, xbc, dt, qlens, slots, has_state, state, num_accepted_rows)
+    from . import cuda_recurrent
+    return cuda_recurrent.mamba2_commit(layer, xbc, dt, qlens, slots, has_state, state, num_accepted_rows)
 
 
-def mamba2_gated_norm(y, z, w, group, eps):
-    from . import cuda_gdn
-    return cuda_gdn.mamba2_gated_norm(y, z, w, group, eps)
+def wkv_forward(layer, x, r, k, v, raw, batch, state, commit):
+    from . import cuda_recurrent
+    return cuda_recurrent.wkv_forward(layer, x, r, k, v, raw, batch, state, commit)
+
+
+def wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted_rows):
+    from . import cuda_recurrent
+    return cuda_recurrent.wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted_rows)
+
+
+def group_norm_gate(y, z, w, group, eps, gate_first):
+    from . import cuda_recurrent
+    return cuda_recurrent.group_norm_gate(y, z, w, group, eps, gate_first)
+
+
+def hyper_norm(streams, delta, read, norm_w, eps, write):
+    from . import cuda_recurrent
+    return cuda_recurrent.hyper_norm(streams, delta, read, norm_w, eps, write)
+
+
+def token_shift_mix(x, mu, batch, shift):
+    from . import cuda_recurrent
+    return cuda_recurrent.token_shift_mix(x, mu, batch, shift)
+
+
+def clamped_glu(gate_up, limit, alpha):
+    from . import cuda_recurrent
+    return cuda_recurrent.clamped_glu(gate_up, limit, alpha)
+
+
+def tanh_(x):
+    from . import cuda_recurrent
+    return cuda_recurrent.tanh_(x)
 
 
 def relu_squared(x):

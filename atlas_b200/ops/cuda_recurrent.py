@@ -1,0 +1,213 @@
+"""Binding of the residual-stream, recurrence and 32-bit attention kernels (``csrc/streams.cu``, ``csrc/recurrent.cu``,
+``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
+from __future__ import annotations
+
+import ctypes as C
+from typing import List, Optional
+
+import torch
+
+from . import cuda as K
+from .cuda_gdn import _Meta
+
+_vp, _ll, _i, _f = C.c_void_p, C.c_longlong, C.c_int, C.c_float
+_bound = False
+
+
+def _lib():
+    global _bound
+    lib = K.lib()
+    if not _bound:
+        lib.atlas_hyper_norm.argtypes = [_vp, _i, _i, _i, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _f, _f, _i, _vp]
+        lib.atlas_token_shift_mix.argtypes = [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]
+        lib.atlas_clamped_glu.argtypes = [_vp, _ll, _i, _i, _vp, _ll, _f, _f, _i, _vp]
+        lib.atlas_tanh.argtypes = [_vp, _ll, _i, _vp]
+        lib.atlas_mamba2_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp] + [_i] * 9 + [_vp]
+        lib.atlas_wkv_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _vp, _vp, _vp,
+                                       _vp, _vp, _vp] + [_i] * 7 + [_vp]
+        lib.atlas_group_norm_gate.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _i, _i, _vp]
+        lib.atlas_conv1d_bias_silu.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _vp]
+        lib.atlas_conv1d_state.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]
+        lib.atlas_rope_kv_write_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp]
+        lib.atlas_attn_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp, _vp]
+        _bound = True
+    return lib
+
+
+def _f32(t: torch.Tensor) -> int:
+    if t.dtype not in (torch.bfloat16, torch.float32):
+        raise K.KernelError(f"activations must be bf16 or fp32, not {t.dtype}")
+    assert t.stride(-1) == 1
+    return 1 if t.dtype == torch.float32 else 0
+
+
+def step_meta(batch, device) -> _Meta:
+    """Device-side sequence metadata of the step, shared by all recurrent layers of one forward pass."""
+    meta = getattr(batch, "_gdn_meta", None)
+    if meta is None:
+        meta = _Meta(batch.query_lens_host, batch.state_slots_host, batch.has_state_host, device, batch.snapshot_plan)
+        batch._gdn_meta = meta
+    return meta
+
+
+# ----------------------------------------------------------------------------- residual streams
+def hyper_norm(streams: Optional[torch.Tensor], delta, read, norm_w, eps: float, write: bool):
+    y, y2, conn = delta.y, delta.y2, delta.conn
+    T, W = y.shape
+    S = read.shape[0]
+    K._dev(y)
+    f32 = _f32(y)
+    if conn is None:
+        streams = torch.empty(T, S, W, dtype=torch.float32, device=y.device)
+    assert streams.dtype == torch.float32 and streams.shape == (T, S, W) and streams.is_contiguous()
+    assert read.dtype == norm_w.dtype == torch.float32 and norm_w.numel() == W
+    if y2 is not None:
+        assert y2.dtype == y.dtype and y2.shape == y.shape and delta.w1.dtype == delta.w2.dtype == torch.float32
+    out = torch.empty(T, W, dtype=y.dtype, device=y.device)
+    K._check(_lib().atlas_hyper_norm(streams.data_ptr(), T, S, W, y.data_ptr(), y.stride(0), K._ptr(y2), y2.stride(0) if y2 is not None else 0,
+                                     K._ptr(delta.w1), K._ptr(delta.w2), K._ptr(conn.mix if conn else None),
+                                     K._ptr(conn.write if conn else None), read.data_ptr(), norm_w.data_ptr(), out.data_ptr(), W,
+                                     0 if conn else 1, 1 if write else 0, float(delta.scale), float(eps), f32, K._stream()), "hyper_norm")
+    return out, streams
+
+
+def token_shift_mix(x, mu, batch, shift):
+    T, W = x.shape
+    K._dev(x)
+    f32 = _f32(x)
+    assert mu.shape == (5, W) and mu.dtype == torch.float32 and shift.dtype == x.dtype and shift.is_contiguous()
+    meta = step_meta(batch, x.device)
+    out = torch.empty(5, T, W, dtype=x.dtype, device=x.device)
+    K._check(_lib().atlas_token_shift_mix(x.data_ptr(), x.stride(0), mu.data_ptr(), shift.data_ptr(), meta.seq_of.data_ptr(),
+                                          meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr(), out.data_ptr(), T, W, f32,
+                                          K._stream()), "token_shift_mix")
+    return out
+
+
+def clamped_glu(gate_up, limit: float, alpha: float):
+    T, I2 = gate_up.shape
+    K._dev(gate_up)
+    f32 = _f32(gate_up)
+    y = torch.empty(T, I2 // 2, dtype=gate_up.dtype, device=gate_up.device)
+    K._check(_lib().atlas_clamped_glu(gate_up.data_ptr(), gate_up.stride(0), T, I2 // 2, y.data_ptr(), y.stride(0), float(limit),
+                                      float(alpha), f32, K._stream()), "clamped_glu")
+    return y
+
+
+def tanh_(x):
+    K._dev(x)
+    assert x.is_contiguous()
+    K._check(_lib().atlas_tanh(x.data_ptr(), x.numel(), _f32(x), K._stream()), "tanh")
+    return x
+
+
+# ----------------------------------------------------------------------------- recurrences
+def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool):
+    T, n = y.shape
+    K._dev(y)
+    f32 = _f32(y)
+    assert z.dtype == y.dtype and z.shape == y.shape and z.stride(1) == 1 and n % group == 0
+    wf = w if w.dtype == torch.float32 else _float_cached(w)
+    out = torch.empty(T, n, dtype=y.dtype, device=y.device)
+    K._check(_lib().atlas_group_norm_gate(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), wf.data_ptr(), out.data_ptr(), n, T,
+                                          n // group, group, float(eps), 1 if gate_first else 0, f32, K._stream()), "group_norm_gate")
+    return out
+
+
+_float_cache: dict = {}
+
+
+def _float_cached(t: torch.Tensor) -> torch.Tensor:
+    hit = _float_cache.get(t.data_ptr())
+    if hit is None or hit[0] is not t:
+        hit = _float_cache[t.data_ptr()] = (t, t.float().contiguous())
+    return hit[1]
+
+
+def _mamba2_run(layer, xbc, dt, meta: _Meta, state, commit: bool):
+    lib, st = _lib(), K._stream()
+    K._dev(xbc)
+    f32 = _f32(xbc)
+    T, Cc = xbc.shape
+    conv, h = state["conv"], state["h"]
+    assert conv.dtype == xbc.dtype and h.dtype == torch.float32 and conv.is_contiguous() and h.is_contiguous()
+    assert dt.dtype == xbc.dtype and dt.stride(1) == 1 and layer.conv_w.dtype == xbc.dtype and layer.conv_w.is_contiguous()
+    assert layer.conv_b is None or layer.conv_b.dtype == xbc.dtype
+    y = torch.empty(T, Cc, dtype=xbc.dtype, device=xbc.device)
+    out = torch.empty(T, layer.d_inner, dtype=xbc.dtype, device=xbc.device)
+    K._check(lib.atlas_conv1d_bias_silu(xbc.data_ptr(), xbc.stride(0), layer.conv_w.data_ptr(), K._ptr(layer.conv_b), Cc, layer.W,
+                                        conv.data_ptr(), meta.seq_of.data_ptr(), meta.qsl.data_ptr(), meta.slots.data_ptr(),
+                                        meta.has.data_ptr(), y.data_ptr(), Cc, T, f32, st), "conv1d")
+    K._check(lib.atlas_mamba2_scan(y.data_ptr(), Cc, dt.data_ptr(), dt.stride(0), layer.A_log.data_ptr(), layer.D.data_ptr(),
+                                   layer.dt_bias.data_ptr(), float(layer.cfg.mamba_dt_min), h.data_ptr(), out.data_ptr(),
+                                   layer.d_inner, meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr(),
+                                   K._ptr(meta.limit), meta.snap_rows.data_ptr(), meta.snap_slots.data_ptr(), meta.snaps, meta.B,
+                                   layer.h, layer.p, layer.n, layer.g, 1 if commit else 0, meta.one_row, f32, st), "mamba2_scan")
+    if commit:
+        K._check(lib.atlas_conv1d_state(xbc.data_ptr(), xbc.stride(0), Cc, layer.W, conv.data_ptr(), meta.qsl.data_ptr(),
+                                        meta.slots.data_ptr(), meta.has.data_ptr(), K._ptr(meta.limit),
+                                        meta.snap_rows.data_ptr(), meta.snap_slots.data_ptr(), meta.snaps, meta.B, f32, st),
+                 "conv1d_state")
+    return out
+
+
+def mamba2_forward(layer, xbc, dt, batch, state, commit):
+    return _mamba2_run(layer, xbc, dt, step_meta(batch, xbc.device), state, commit)
+
+
+def mamba2_commit(layer, xbc, dt, qlens, slots, has_state, state, num_accepted_rows):
+    meta = _Meta(qlens, slots, has_state, xbc.device, None, limit=list(num_accepted_rows))
+    _mamba2_run(layer, xbc, dt, meta, state, True)
+
+
+def _wkv_run(layer, x, r, k, v, raw, meta: _Meta, state, commit: bool):
+    K._dev(x)
+    f32 = _f32(x)
+    shift, h = state["shift"], state["h"]
+    for t in (k, v, raw) + ((r,) if r is not None else ()):
+        assert t.dtype == x.dtype and t.stride(1) == 1
+    assert shift.dtype == x.dtype and h.dtype == torch.float32 and shift.is_contiguous() and h.is_contiguous()
+    out = torch.empty(x.shape[0], layer.inner, dtype=x.dtype, device=x.device) if r is not None else None
+    K._check(_lib().atlas_wkv_scan(K._ptr(r), r.stride(0) if r is not None else 0, k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
+                                   raw.data_ptr(), raw.stride(0), layer.w0.data_ptr(), layer.u.data_ptr(), h.data_ptr(), K._ptr(out),
+                                   layer.inner, x.data_ptr(), x.stride(0), shift.data_ptr(), x.shape[1], meta.qsl.data_ptr(),
+                                   meta.slots.data_ptr(), meta.has.data_ptr(), K._ptr(meta.limit), meta.snap_rows.data_ptr(),
+                                   meta.snap_slots.data_ptr(), meta.snaps, meta.B, layer.h, layer.d, 1 if commit else 0, meta.one_row,
+                                   f32, K._stream()), "wkv_scan")
+    return out
+
+
+def wkv_forward(layer, x, r, k, v, raw, batch, state, commit):
+    return _wkv_run(layer, x, r, k, v, raw, step_meta(batch, x.device), state, commit)
+
+
+def wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted_rows):
+    meta = _Meta(qlens, slots, has_state, x.device, None, limit=list(num_accepted_rows))
+    _wkv_run(layer, x, None, k, v, raw, meta, state, True)
+
+
+# ----------------------------------------------------------------------------- 32-bit attention
+def rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping):
+    T, Hq, D = q.shape
+    Hkv = k.shape[1]
+    K._dev(q)
+    assert q.stride(2) == 1 and q.stride(1) == k.stride(1) == v.stride(1) == D and k_cache.dtype == torch.float32
+    assert positions.dtype == slot_mapping.dtype == torch.int32 and rope_cache.dtype == torch.float32
+    K._check(_lib().atlas_rope_kv_write_f32(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
+                                            positions.data_ptr(), rope_cache.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
+                                            slot_mapping.data_ptr(), T, Hq, Hkv, D, rotary_dim, k_cache.shape[1], K._stream()),
+             "rope_kv_write_f32")
+    return q
+
+
+def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, sinks):
+    T, Hq, D = q.shape
+    K._dev(q)
+    assert k_cache.dtype == torch.float32 and q.stride(2) == 1 and q.stride(1) == D
+    out = torch.empty(T, Hq, D, dtype=q.dtype, device=q.device)
+    bt = batch.block_tables
+    K._check(_lib().atlas_attn_f32(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
+                                   bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
+                                   batch.num_seqs, T, float(scale), Hq, k_cache.shape[2], D, k_cache.shape[1], window, chunk,
+                                   K._ptr(sinks), K._stream()), "attn_f32")
+    return out

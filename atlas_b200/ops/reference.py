@@ -185,8 +185,12 @@ def qk_norm_rope_kv_write(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     block_tables: torch.Tensor, seq_lens: torch.Tensor, query_start_loc: torch.Tensor,
                     scale: float, k_scale: float = 1.0, v_scale: float = 1.0,
-                    sliding_window: Optional[int] = None) -> torch.Tensor:
+                    sliding_window: Optional[int] = None, chunk: int = 0,
+                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of new query rows over the paged cache (prefill chunks and decode alike).
+
+    ``chunk`` > 0 limits a row to keys of its own ``chunk``-token block (counted from the sequence's first token);
+    ``sinks [Hq]`` adds ``exp(sink)`` to every row's softmax denominator.
 
     Sequence ``b`` owns query rows ``query_start_loc[b]:query_start_loc[b+1]``; its last row sits
     at position ``seq_lens[b]-1``.  ``q [T,Hq,D]`` -> ``out [T,Hq,D]``.
@@ -213,14 +217,66 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         mask = kpos <= qpos
         if sliding_window:
             mask &= kpos > qpos - sliding_window
+        if chunk:
+            mask &= torch.div(kpos, chunk, rounding_mode="floor") == torch.div(qpos, chunk, rounding_mode="floor")
         s = s.masked_fill(~mask[None, None], float("-inf"))
-        p = torch.softmax(s, dim=-1)
+        if sinks is not None:
+            s = torch.cat([s, sinks.float().view(Hkv, G, 1, 1).expand(Hkv, G, ql, 1)], -1)
+        p = torch.softmax(s, dim=-1)[..., :L]
         o = torch.einsum("hgqk,khd->qhgd", p, vv).reshape(ql, Hq, D)
         out[q0:q1] = o.to(q.dtype)
     return out
 
 
+# ----------------------------------------------------------------------------- residual streams, WKV
+def hyper_norm(streams, delta, read, norm_w, eps):
+    """See ``ops.hyper_norm``; everything in fp32, the result in the dtype of ``delta.y``."""
+    y = delta.y.float()
+    if delta.conn is None:
+        x = (y * delta.scale)[:, None, :].expand(-1, read.shape[0], -1).clone()
+    else:
+        if delta.y2 is not None:
+            unit = lambda t: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps)
+            y = 0.5 * (unit(y) * delta.w1.float() + unit(delta.y2.float()) * delta.w2.float())
+        c = delta.conn
+        x = torch.einsum("st,nsw->ntw", c.mix, streams) + c.write[None, :, None] * y[:, None, :]
+    u = torch.einsum("s,nsw->nw", read.float(), x)
+    h = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    return h.to(delta.y.dtype), x
+
+
+def token_shift_mix(x: torch.Tensor, prev: torch.Tensor, mu: torch.Tensor) -> torch.Tensor:
+    """``x + (prev - x) * mu_s`` for every row of ``mu [S, W]``: ``[S, T, W]``."""
+    xf, pf = x.float(), prev.float()
+    return (xf[None] + (pf - xf)[None] * mu.float()[:, None, :]).to(x.dtype)
+
+
+def wkv_scan(r, k, v, decay, u, h):
+    """Sequential WKV recurrence.  ``r, k, v, decay [T, H, D]`` fp32, ``u [H, D]``, ``h [H, V, K]`` -> ``(o [T, H, V], h)``."""
+    out = []
+    for t in range(r.shape[0]):
+        kv = v[t][:, :, None] * k[t][:, None, :]
+        out.append(((h + u.float()[:, None, :] * kv) * r[t][:, None, :]).sum(-1))
+        h = h * decay[t][:, None, :] + kv
+    return torch.stack(out), h
+
+
+def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool):
+    """``norm(y * silu(z)) * w`` or ``norm(y) * w * silu(z)``, RMS over groups of ``group`` channels."""
+    gate = F.silu(z.float())
+    v = y.float() * gate if gate_first else y.float()
+    g = v.reshape(*v.shape[:-1], -1, group)
+    v = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).reshape(v.shape) * w.float()
+    return (v if gate_first else v * gate).to(y.dtype)
+
+
 # ----------------------------------------------------------------------------- activations
+def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    i = gate_up.shape[-1] // 2
+    g, u = gate_up[..., :i].float().clamp(max=limit), gate_up[..., i:].float().clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(gate_up.dtype)
+
+
 def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     """``[T, 2I]`` (gate | up) -> ``silu(gate) * up`` ``[T, I]``."""
     i = gate_up.shape[-1] // 2
@@ -343,7 +399,7 @@ def causal_conv1d(x: torch.Tensor, conv_state: torch.Tensor, weight: torch.Tenso
         y = y + bias.float()
     if activation:
         y = F.silu(y)
-    new_state = full[-(W - 1):].t().contiguous().to(conv_state.dtype)
+    new_state = full[full.shape[0] - (W - 1):].t().contiguous().to(conv_state.dtype)
     return y.to(x.dtype), new_state
 
 

@@ -15,6 +15,7 @@ import torch
 
 from .config import EngineConfig
 from .models import CacheStore, DecoderLM, ForwardBatch
+from .models.decoder import attention_of
 from .sched import SchedulerOutput
 
 _GRAPH_BATCH_SIZES = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256)
@@ -53,7 +54,7 @@ class ModelRunner:
         """Size the split-K decode attention scratch for the largest case any later step can ask for, so that the
         buffers captured into CUDA graphs are never replaced."""
         from .ops import cuda as K
-        mixers = [l.mixer for l in self.model.layers if l.kind == "attention"]
+        mixers = [a for a in map(attention_of, self.model.layers) if a is not None]
         if getattr(self.model, "mtp", None) is not None and getattr(self.model.mtp, "layer", None) is not None:
             mixers.append(self.model.mtp.layer.mixer)
         if not mixers:
@@ -242,8 +243,8 @@ class ModelRunner:
 
     def copy_state(self, src_slot: int, dst_slot: int) -> None:
         for st in self.cache.states.values():
-            st["conv"][dst_slot].copy_(st["conv"][src_slot])
-            st["h"][dst_slot].copy_(st["h"][src_slot])
+            for t in st.values():
+                t[dst_slot].copy_(t[src_slot])
 
     # ------------------------------------------------------------------ CUDA graphs (decode)
     def _forward_graph(self, batch: ForwardBatch) -> torch.Tensor:

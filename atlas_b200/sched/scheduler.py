@@ -337,6 +337,32 @@ class Scheduler:
             self._last_decode_time = now
         return out
 
+    # ------------------------------------------------------------------ externally driven steps (trace replay)
+    def admit_now(self, seq: Sequence) -> None:
+        """Admit ``seq`` past the queue: it owns a state slot (recurrent models) and gets blocks as it is fed."""
+        if len(self.prefilling) + len(self.running) >= self.cfg.max_num_seqs:
+            raise RuntimeError("no sequence slot free")
+        if self.hybrid and self.state_pool is not None:
+            seq.state_slot = self.state_pool.alloc()
+            if seq.state_slot is None:
+                raise RuntimeError("no recurrent-state slot free")
+            seq.has_state = False
+        seq.status = SeqStatus.PREFILL
+        self.prefilling.append(seq)
+
+    def plan_fed(self, seqs: List[Sequence]) -> SchedulerOutput:
+        """One step over every token that ``seqs`` hold beyond their computed context: single tokens of sequences with a
+        context are decode rows (first in the step, like in :meth:`schedule`), everything else is a prefill chunk."""
+        out = SchedulerOutput()
+        for s in seqs:
+            if not self._ensure_blocks(s, s.num_tokens):
+                raise RuntimeError(f"KV cache exhausted ({self.pool.num_free} of {self.pool.num_blocks} blocks free)")
+        decode = [s for s in seqs if s.num_computed > 0 and s.num_uncomputed == 1]
+        chunks = [s for s in seqs if not (s.num_computed > 0 and s.num_uncomputed == 1)]
+        out.items = [ScheduledSeq(s, s.num_computed, 1, True, True) for s in decode]
+        out.items += [ScheduledSeq(s, s.num_computed, s.num_uncomputed, True, False) for s in chunks]
+        return out
+
     def _pick_victim(self, exclude: Sequence) -> Optional[Sequence]:
         for pool in (self.prefilling, self.running):
             for s in reversed(pool):
