@@ -57,7 +57,8 @@ class LLMEngine:
         num_blocks = self.cfg.num_kv_blocks or self._profile_num_blocks()
         n_active = self.cfg.max_num_seqs if self.hybrid else 0
         n_snap = self.cfg.ssm_cache_slots if (self.hybrid and self.cfg.enable_prefix_caching) else 0
-        self.cache: CacheStore = model.alloc_cache(num_blocks, self.cfg.block_size, self.kv_dtype, n_active + n_snap,
+        self.cache: CacheStore = model.alloc_cache(num_blocks, self.cfg.block_size, self.kv_dtype,
+                                                   n_active + n_snap + (1 if self.hybrid else 0),      # + padding rows of decode graphs
                                                    high_precision_layers=self.cfg.kv_high_precision_layers)
         if os.environ.get("ATLAS_NATIVE_RUNTIME", "0") not in ("0", "", "false"):
             from .runtime_native import NativeBlockPool          # C++ pool, same interface

@@ -62,6 +62,18 @@ class _Meta:
         self.chunk_ok = limit is None and max(qlens, default=0) >= CHUNK_MIN_ROWS
 
 
+    @classmethod
+    def decode(cls, qsl: torch.Tensor, slots: torch.Tensor, live: torch.Tensor) -> "_Meta":
+        """Metadata of a decode step whose slots live in fixed device buffers (CUDA graphs): one row per sequence."""
+        self = cls.__new__(cls)
+        n = slots.shape[0]
+        self.qsl, self.slots, self.has, self.limit = qsl, slots, live, None
+        self.seq_of = torch.arange(n, dtype=torch.int32, device=slots.device)
+        self.snap_rows = self.snap_slots = torch.zeros(1, dtype=torch.int32, device=slots.device)
+        self.B, self.T, self.snaps, self.chunk_ok, self.one_row = n, n, 0, False, 1
+        return self
+
+
 def _run(layer, mixed, a, b, meta: _Meta, state, commit: bool):
     lib, st = _lib(), K._stream()
     K._dev(mixed)

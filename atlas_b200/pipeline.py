@@ -132,6 +132,13 @@ class DecodePipeline:
             r.h2d_bytes += P * 8
         else:
             g.ids[:B].copy_(self.dev_ids, non_blocking=True)          # last step's samples, device to device
+        if g.state_slots is not None:
+            st = self._pin("state_slots", (P,), torch.int32)
+            snp = st.numpy()
+            snp[:B] = [s.state_slot for s in seqs]
+            snp[B:] = r.pad_state_slot
+            g.state_slots.copy_(st, non_blocking=True)
+            r.h2d_bytes += P * 4
         g.pos.copy_(pos, non_blocking=True)
         g.slots.copy_(slots, non_blocking=True)
         g.seq_lens.copy_(sl, non_blocking=True)

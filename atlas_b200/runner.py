@@ -15,7 +15,7 @@ import torch
 
 from .config import EngineConfig
 from .models import CacheStore, DecoderLM, ForwardBatch
-from .models.decoder import attention_of
+from .models.decoder import attention_of, recurrent_of
 from .sched import SchedulerOutput
 
 _GRAPH_BATCH_SIZES = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256)
@@ -40,6 +40,11 @@ class ModelRunner:
         self.d2h_bytes = 0
         self.graph_replays = 0
         self._pin: Dict[str, torch.Tensor] = {}
+        # decode graphs of recurrent models read state slots from a device buffer; the kernels that take everything they
+        # need from there are those of recurrent.cu
+        self._states_graph_safe = all(l.kind in ("mamba2", "wkv", "parallel") for l in model.layers if recurrent_of(l) is not None)
+        # slot of padding rows: the last one, which the engine allocates beyond those it hands out
+        self.pad_state_slot = next((t.shape[0] - 1 for st in cache.states.values() for t in st.values()), None)
         if self.on_gpu:
             self._reserve_attention_scratch()
 
@@ -218,7 +223,8 @@ class ModelRunner:
         return (self.on_gpu and self.cfg.use_cuda_graphs and batch.num_seqs > 0
                 and batch.num_decodes == batch.num_seqs and not batch.spec_verify and batch.adapter_rows is None
                 and batch.positions3 is None
-                and getattr(self.model, "graph_safe", True) and not self.model.gdn_layers())
+                and getattr(self.model, "graph_safe", True) and self._states_graph_safe and not batch.snapshot_plan
+                and all(batch.has_state_host))
 
     def forward(self, batch: ForwardBatch) -> torch.Tensor:
         if self._can_graph(batch):
@@ -270,14 +276,22 @@ class _DecodeGraph:
         self.tables = torch.zeros(padded, mb, dtype=torch.int32, device=dev)
         self.seq_lens = torch.ones(padded, dtype=torch.int32, device=dev)
         self.qsl = torch.arange(padded + 1, dtype=torch.int32, device=dev)
+        self.state_slots: Optional[torch.Tensor] = None
+        if runner.pad_state_slot is not None:
+            self.state_slots = torch.full((padded,), runner.pad_state_slot, dtype=torch.int32, device=dev)
+            self.live = torch.ones(padded, dtype=torch.uint8, device=dev)
         self.graph: Optional[torch.cuda.CUDAGraph] = None
         self.out: Optional[torch.Tensor] = None
         self.num_kernels = 0
 
     def _batch(self, max_seq_len: int) -> ForwardBatch:
-        return ForwardBatch(input_ids=self.ids, positions=self.pos, slot_mapping=self.slots, block_tables=self.tables,
-                            seq_lens=self.seq_lens, query_start_loc=self.qsl, num_decodes=self.P, max_query_len=1,
-                            max_seq_len=max_seq_len, seq_lens_host=[1] * self.P, query_lens_host=[1] * self.P)
+        fb = ForwardBatch(input_ids=self.ids, positions=self.pos, slot_mapping=self.slots, block_tables=self.tables,
+                          seq_lens=self.seq_lens, query_start_loc=self.qsl, num_decodes=self.P, max_query_len=1,
+                          max_seq_len=max_seq_len, seq_lens_host=[1] * self.P, query_lens_host=[1] * self.P)
+        if self.state_slots is not None:
+            from .ops.cuda_gdn import _Meta
+            fb._gdn_meta = _Meta.decode(self.qsl, self.state_slots, self.live)
+        return fb
 
     def _load(self, b: ForwardBatch) -> None:
         n = b.num_seqs
@@ -286,6 +300,9 @@ class _DecodeGraph:
         self.slots[:n].copy_(b.slot_mapping, non_blocking=True)
         self.seq_lens[:n].copy_(b.seq_lens, non_blocking=True)
         self.tables[:n, :b.block_tables.shape[1]].copy_(b.block_tables, non_blocking=True)
+        if self.state_slots is not None:
+            self.state_slots[:n].copy_(b.state_slots, non_blocking=True)
+            self.state_slots[n:].fill_(self.r.pad_state_slot)
         if n < self.P:
             self.slots[n:].fill_(-1)
             self.seq_lens[n:].fill_(1)
@@ -298,6 +315,8 @@ class _DecodeGraph:
         if self.graph is None:
             # the graph must be valid for any later sequence length: kernels read lengths from device memory
             fb = self._batch(r.cfg.max_seq_len)
+            if self.state_slots is not None:
+                self.state_slots.fill_(r.pad_state_slot)      # the eager passes below must not advance anybody's state
             s = torch.cuda.Stream()
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
