@@ -279,7 +279,9 @@ class _DecodeGraph:
         self.state_slots: Optional[torch.Tensor] = None
         if runner.pad_state_slot is not None:
             self.state_slots = torch.full((padded,), runner.pad_state_slot, dtype=torch.int32, device=dev)
-            self.live = torch.ones(padded, dtype=torch.uint8, device=dev)
+            from .ops.cuda_gdn import _Meta
+            # captured kernels keep these addresses: the tensors live as long as the graph
+            self.state_meta = _Meta.decode(self.qsl, self.state_slots, torch.ones(padded, dtype=torch.uint8, device=dev))
         self.graph: Optional[torch.cuda.CUDAGraph] = None
         self.out: Optional[torch.Tensor] = None
         self.num_kernels = 0
@@ -289,8 +291,7 @@ class _DecodeGraph:
                           seq_lens=self.seq_lens, query_start_loc=self.qsl, num_decodes=self.P, max_query_len=1,
                           max_seq_len=max_seq_len, seq_lens_host=[1] * self.P, query_lens_host=[1] * self.P)
         if self.state_slots is not None:
-            from .ops.cuda_gdn import _Meta
-            fb._gdn_meta = _Meta.decode(self.qsl, self.state_slots, self.live)
+            fb._gdn_meta = self.state_meta
         return fb
 
     def _load(self, b: ForwardBatch) -> None:
