@@ -47,7 +47,7 @@ def _run(cmd: List[str]) -> None:
 
 # translation units every library holds, and those of the mixers, residual forms and activation types
 _UNITS_BASE = ("runtime",)
-_UNITS_BF16 = ("gemm", "elementwise", "attention")
+_UNITS_BF16 = ("gemm", "elementwise", "attention", "attention_tc16")
 _UNITS_F32 = ("attention_f32",)
 _UNITS_STREAMS = ("streams", "recurrent")
 

@@ -461,7 +461,7 @@ ATLAS_DEVICE uint32_t movmatrix_trans(uint32_t v) {
 // dims mt*16 + rq (+8), columns = heads 2c, 2c+1); `acc_scale` undoes a fixed scaling of the P operand.
 template <int D>
 ATLAS_DEVICE void decode_merge_store(const AttnParams& p, uint8_t* ring, const float (&o)[D / 16][4], const float (&m_run)[2],
-                                     const float (&l_run)[2], int warp, int lane, int G, int kvh, int split, int b, int q_row0,
+                                     const float (&l_run)[2], int warp, int lane, int G, int head0, int split, int b, int q_row0,
                                      float acc_scale) {
   constexpr int MT = D / 16;
   const int c = lane & 3, rq = lane >> 2;
@@ -504,7 +504,7 @@ ATLAS_DEVICE void decode_merge_store(const AttnParams& p, uint8_t* ring, const f
       acc += f * sm_o[(w * 8 + r) * D + d] * acc_scale;
       l += f * sm_l[w * 8 + r];
     }
-    const int head = kvh * G + r;
+    const int head = head0 + r;
     if (q8) {
       // a warp's 32 consecutive idx lie inside one head (D and the thread count are multiples of 32): the value is
       // parked in the first warp's slot, which only this thread reads, and the head's maximum is gathered per warp
@@ -516,6 +516,7 @@ ATLAS_DEVICE void decode_merge_store(const AttnParams& p, uint8_t* ring, const f
       for (int off = 16; off > 0; off >>= 1) a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, off));
       if (lane == 0) atomicMax(&sm_amax[r], __float_as_int(a));
     } else if (p.num_splits == 1) {
+      if (p.sinks) acc *= add_sink(p.sinks[head], m, l);
       const float inv = l > 0.f ? p.v_scale / l : 0.f;
       p.out[(long long)q_row0 * p.ldo + head * D + d] = __float2bfloat16_rn(acc * inv);
     } else {
@@ -531,7 +532,7 @@ ATLAS_DEVICE void decode_merge_store(const AttnParams& p, uint8_t* ring, const f
     __syncthreads();
     for (int idx = threadIdx.x * 4; idx < G * D; idx += (int)blockDim.x * 4) {
       const int r = idx / D, d = idx % D;
-      const int head = kvh * G + r;
+      const int head = head0 + r;
       const float sc = fmaxf(__int_as_float(sm_amax[r]), 1e-10f) / 448.f;
       const float inv = __frcp_rn(sc);
       const float4 v = *reinterpret_cast<const float4*>(sm_o + r * D + d);
@@ -724,7 +725,7 @@ attn_decode_kernel(const AttnParams p, int stages, status_t* status) {
     }
   }
 
-  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, kvh, split, b, q_row0, 1.f);
+  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, kvh * G, split, b, q_row0, 1.f);
 }
 
 // ---- e4m3 tensor-core tiles (used by the e4m3 decode variants below)
@@ -762,30 +763,38 @@ constexpr int kCpThreads = 128;
 // F8: FP8 pages go to e4m3 tensor-core tiles as they are (mma.m16n8k32, no widening); Q and P, which are not cached bytes,
 // are fed as two e4m3 terms each (see attn_decode_f8_kernel).  One page per step: the upper half of the 32-wide k
 // dimension of the PV product stays zero, which costs tensor-pipe slots this kernel has to spare.
-template <int D, int BS, int kCpDepth, bool KV4 = false, bool F8 = false>       // BS: block size known at compile time (0 = runtime)
+// KV16: bf16 pages meet the bf16 query and probabilities as they are; scores are scaled in fp32.  K rows are stored with their
+// 16-byte pieces permuted (kv16_piece) so that the eight lanes of a read phase hit different banks.  The query heads of a kv
+// head are taken eight at a time (grid.x = Hkv * groups of eight).
+ATLAS_DEVICE int kv16_piece(int piece, int token) { return (piece & ~7) | ((piece & 7) ^ ((piece >> 3) << 1) ^ (token & 1)); }
+template <int D, int BS, int kCpDepth, bool KV4 = false, bool F8 = false, bool KV16 = false>   // BS: block size known at compile time (0 = runtime)
 __global__ void __launch_bounds__(kCpThreads)
 attn_decode_cp_kernel(const AttnParams p) {
   constexpr int KS = D / 16, MT = D / 16, DQ = D / 4;
   constexpr float kPScale = 256.f;
   extern __shared__ __align__(128) uint8_t dsm[];
   const int bs = BS ? BS : p.block_size;
-  const int stage_bytes = KV4 ? 2 * (bs * D * 9 / 16) : 2 * bs * D;
+  const int stage_bytes = KV4 ? 2 * (bs * D * 9 / 16) : 2 * bs * D * (KV16 ? 2 : 1);
   int* bt_sm = reinterpret_cast<int*>(dsm);
   uint8_t* ring = dsm + kBtSmemEntries * 4;
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int c = lane & 3, rq = lane >> 2;
-  const int G = p.Hq / p.Hkv;
-  const int b = p.seq_base + blockIdx.z, kvh = blockIdx.x, split = blockIdx.y;
+  const int Gall = p.Hq / p.Hkv;
+  const int groups = KV16 ? (Gall + 7) / 8 : 1;
+  const int b = p.seq_base + blockIdx.z, kvh = blockIdx.x / groups, split = blockIdx.y;
+  const int g0 = (blockIdx.x % groups) * 8;
+  const int G = KV16 ? min(8, Gall - g0) : Gall;               // this CTA's query heads: [head0, head0 + G)
+  const int head0 = kvh * Gall + g0;
   chain_trigger();
   chain_wait();                       // global memory is only touched from here on
   const int L = p.seq_lens[b];
   const int q_row0 = p.query_start_loc[b];
-  const int n_blocks = (L + bs - 1) / bs;
-  const int per_split = (n_blocks + p.num_splits - 1) / p.num_splits;
-  int blk_lo = split * per_split;
-  const int blk_hi = min(n_blocks, (split + 1) * per_split);
-  if (p.window > 0) blk_lo = max(blk_lo, max(0, L - p.window) / bs);
+  const int first_tok = first_visible(p, L - 1);
+  const int n_blocks = (L + bs - 1) / bs, blk_first = first_tok / bs;
+  const int per_split = (n_blocks - blk_first + p.num_splits - 1) / p.num_splits;      // the splits share the visible pages
+  const int blk_lo = blk_first + split * per_split;
+  const int blk_hi = min(n_blocks, blk_first + (split + 1) * per_split);
   const int n_mine = max(0, blk_hi - blk_lo);
   const int* bt = p.block_tables + (long long)b * p.bt_ld + blk_lo;
   for (int i = threadIdx.x; i < min(n_mine, kBtSmemEntries); i += kCpThreads) bt_sm[i] = bt[i];
@@ -803,10 +812,16 @@ attn_decode_cp_kernel(const AttnParams p) {
     // dim permutation: MMA k index kk of k-step ks <-> dim c'*DQ + ks*4 + ..., matching the K bytes a thread reads.
     uint32_t qb[KS][2];
     {
-      const __nv_bfloat16* qrow = rq < G ? p.q + (long long)q_row0 * p.ldq + (kvh * G + rq) * D : nullptr;
+      const __nv_bfloat16* qrow = rq < G ? p.q + (long long)q_row0 * p.ldq + (head0 + rq) * D : nullptr;
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks) {
         float v[4] = {0.f, 0.f, 0.f, 0.f};
+        if (KV16) {
+          const uint2 raw = qrow ? *reinterpret_cast<const uint2*>(qrow + c * DQ + ks * 4) : make_uint2(0u, 0u);
+          qb[ks][0] = raw.x;
+          qb[ks][1] = raw.y;
+          continue;
+        }
         if (qrow) {
           const uint2 raw = *reinterpret_cast<const uint2*>(qrow + c * DQ + ks * 4);
           const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x);
@@ -857,14 +872,14 @@ attn_decode_cp_kernel(const AttnParams p) {
       sq[0] = __shfl_sync(0xffffffffu, qs, (2 * c) * 4);
       sq[1] = __shfl_sync(0xffffffffu, qs, (2 * c + 1) * 4);
     }
-    const int win_lo = p.window > 0 ? L - 1 - p.window : -1;  // tokens <= win_lo are outside the window
+    const int win_lo = first_tok - 1;                         // tokens <= win_lo are not visible
     // this thread's two token rows inside a page
     const int tok_r0 = (rq >> 1) * 4 + (rq & 1);
     const int tok_r1 = tok_r0 + 2;
     // this warp's pages: i = warp + 4 k, slot k % kCpDepth of its private ring
     uint8_t* myring = ring + (size_t)warp * kCpDepth * stage_bytes;
     const int n_w = n_mine > warp ? (n_mine - warp + 3) / 4 : 0;
-    const int half_bytes = KV4 ? bs * D * 9 / 16 : bs * D;          // one page of K or of V
+    const int half_bytes = KV4 ? bs * D * 9 / 16 : bs * D * (KV16 ? 2 : 1);          // one page of K or of V
     auto issue = [&](int k) {
       const int i = warp + 4 * k;
       const int blk = i < kBtSmemEntries ? bt_sm[i] : bt[i];
@@ -873,7 +888,9 @@ attn_decode_cp_kernel(const AttnParams p) {
       const uint8_t* ks = p.k_cache + off;
       const uint8_t* vs = p.v_cache + off;
       for (int o16 = lane * 16; o16 < half_bytes; o16 += 512) {
-        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + o16), "l"(ks + o16) : "memory");
+        const int tok = o16 / (2 * D);
+        const int k16 = KV16 ? tok * 2 * D + kv16_piece((o16 % (2 * D)) >> 4, tok) * 16 : o16;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + k16), "l"(ks + o16) : "memory");
         asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(dst + half_bytes + o16), "l"(vs + o16) : "memory");
       }
     };
@@ -913,6 +930,19 @@ attn_decode_cp_kernel(const AttnParams p) {
             }
           }
           s[0] *= sq[0]; s[1] *= sq[1]; s[2] *= sq[0]; s[3] *= sq[1];
+        } else if constexpr (KV16) {
+          const int ta = sub * 16 + tok_r0, tb = sub * 16 + tok_r1;
+          const uint4* ka = reinterpret_cast<const uint4*>(kblk + ta * 2 * D);
+          const uint4* kb = reinterpret_cast<const uint4*>(kblk + tb * 2 * D);
+#pragma unroll
+          for (int v4 = 0; v4 < DQ / 8; ++v4) {                // eight bf16 = two k-steps
+            const uint4 ra = ka[kv16_piece(c * (DQ / 8) + v4, ta)], rb = kb[kv16_piece(c * (DQ / 8) + v4, tb)];
+            const uint32_t a0[4] = {ra.x, rb.x, ra.y, rb.y}, a1[4] = {ra.z, rb.z, ra.w, rb.w};
+            mma_bf16(s, a0, qb[v4 * 2][0], qb[v4 * 2][1]);
+            mma_bf16(s, a1, qb[v4 * 2 + 1][0], qb[v4 * 2 + 1][1]);
+          }
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[e] *= p.qk_scale_log2;
         } else if constexpr (KV4) {
           const int ta = sub * 16 + tok_r0, tb = sub * 16 + tok_r1;
           const uint8_t* ka = kblk + ta * (D / 2) + c * (DQ / 2);
@@ -975,8 +1005,8 @@ attn_decode_cp_kernel(const AttnParams p) {
         l_run[0] = l_run[0] * alpha[0] + pv[0] + pv[2];
         l_run[1] = l_run[1] * alpha[1] + pv[1] + pv[3];
         // P^T as the B operand of the PV product: transpose the two 8x8 (token x head) blocks
-        const uint32_t pb0 = movmatrix_trans(pack_f16x2(pv[0], pv[1]));
-        const uint32_t pb1 = movmatrix_trans(pack_f16x2(pv[2], pv[3]));
+        const uint32_t pb0 = movmatrix_trans(KV16 ? pack_bf16x2(pv[0], pv[1]) : pack_f16x2(pv[0], pv[1]));
+        const uint32_t pb1 = movmatrix_trans(KV16 ? pack_bf16x2(pv[2], pv[3]) : pack_f16x2(pv[2], pv[3]));
         // after the transpose this thread holds head rq, tokens c*4+{0,1} (pb0) and c*4+{2,3} (pb1)
         uint32_t vmask = 0xFFFFFFFFu;
         {
@@ -991,8 +1021,22 @@ attn_decode_cp_kernel(const AttnParams p) {
         // rescale only when some head's running max moved (the accumulator's columns are heads c*2, c*2+1)
         const bool rescale = __any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f);
         // ---- O^T += V^T P^T : rows = dims, k = tokens
-        const uint8_t* vsub = vblk + sub * 16 + c * 4;
-        if constexpr (F8) {
+        const uint8_t* vsub = vblk + (sub * 16 + c * 4) * (KV16 ? 2 : 1);
+        if constexpr (KV16) {
+          const uint32_t m0 = ((vmask & 0xFFu) ? 0xFFFFu : 0u) | ((vmask & 0xFF00u) ? 0xFFFF0000u : 0u);
+          const uint32_t m1 = ((vmask & 0xFF0000u) ? 0xFFFFu : 0u) | ((vmask & 0xFF000000u) ? 0xFFFF0000u : 0u);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            const uint2 w0 = *reinterpret_cast<const uint2*>(vsub + (mt * 16 + rq) * bs * 2);
+            const uint2 w1 = *reinterpret_cast<const uint2*>(vsub + (mt * 16 + rq + 8) * bs * 2);
+            const uint32_t a[4] = {w0.x & m0, w1.x & m0, w0.y & m1, w1.y & m1};
+            if (rescale) {
+              o[mt][0] *= alpha[0]; o[mt][1] *= alpha[1];
+              o[mt][2] *= alpha[0]; o[mt][3] *= alpha[1];
+            }
+            mma_bf16(o[mt], a, pb0, pb1);
+          }
+        } else if constexpr (F8) {
           // P^T as two e4m3 terms: a b16 unit carries one head's values of this thread's two token rows; the 8x8 transpose
           // leaves head rq's tokens 4c, 4c+2, 4c+1, 4c+3 in a register, a byte permute puts them in order
           uint32_t h0, l0, h1, l1;
@@ -1059,7 +1103,7 @@ attn_decode_cp_kernel(const AttnParams p) {
     }
   }
 
-  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, kvh, split, b, q_row0, F8 ? 1.f / kPScale : 1.f);
+  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, head0, split, b, q_row0, F8 ? 1.f / kPScale : 1.f);
 }
 
 // ----------------------------------------------------------------------------- decode on FP8 tensor-core tiles
@@ -1294,7 +1338,7 @@ attn_decode_f8_kernel(const AttnParams p, int stages, status_t* status) {
       l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 16);
     }
   }
-  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, kvh, split, b, q_row0, 1.f / kPScale);
+  decode_merge_store<D>(p, ring, o, m_run, l_run, warp, lane, G, kvh * G, split, b, q_row0, 1.f / kPScale);
 }
 
 // Merge split partials: grid (Hq, B), D threads.
@@ -1412,15 +1456,15 @@ static int decode_cp_depth() {
   return v;
 }
 
-template <int D, int BS, int kCpDepth, bool KV4 = false, bool F8 = false>
+template <int D, int BS, int kCpDepth, bool KV4 = false, bool F8 = false, bool KV16 = false>
 static int launch_decode_cp(const AttnParams& p, int B, cudaStream_t st) {
-  const int stage_bytes = KV4 ? 2 * (p.block_size * D * 9 / 16) : 2 * p.block_size * D;
+  const int stage_bytes = KV4 ? 2 * (p.block_size * D * 9 / 16) : 2 * p.block_size * D * (KV16 ? 2 : 1);
   const int merge_bytes = (64 + 4 * 8 * D + 8) * (int)sizeof(float);
   const int ring_bytes = 4 * kCpDepth * stage_bytes > merge_bytes ? 4 * kCpDepth * stage_bytes : merge_bytes;
   const int smem = kBtSmemEntries * 4 + ring_bytes;
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(attn_decode_cp_kernel<D, BS, kCpDepth, KV4, F8>), smem) != cudaSuccess) return -20;
-  dim3 grid(p.Hkv, p.num_splits, B);
-  if (launch_chain(attn_decode_cp_kernel<D, BS, kCpDepth, KV4, F8>, grid, dim3(kCpThreads), (size_t)smem, st, p) != cudaSuccess) return -21;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(attn_decode_cp_kernel<D, BS, kCpDepth, KV4, F8, KV16>), smem) != cudaSuccess) return -20;
+  dim3 grid(p.Hkv * (KV16 ? (p.Hq / p.Hkv + 7) / 8 : 1), p.num_splits, B);
+  if (launch_chain(attn_decode_cp_kernel<D, BS, kCpDepth, KV4, F8, KV16>, grid, dim3(kCpThreads), (size_t)smem, st, p) != cudaSuccess) return -21;
   if (p.num_splits > 1) {
     dim3 g2(p.Hq, B);
     if (launch_chain(attn_merge_kernel, g2, dim3(D), 0, st, p.part_o, p.part_ml, p.out, p.ldo, p.query_start_loc, p.seq_base,
@@ -1556,6 +1600,12 @@ static int launch_kv16(const AttnParams& p, int B, bool prefill, cudaStream_t st
     dim3 grid((p.num_tiles + 3) / 4, p.Hq);
     paged_attn_kernel<D, true, true><<<grid, 128, 0, st>>>(p);
     return cudaGetLastError() == cudaSuccess ? 0 : -21;
+  }
+  // decode rows: the cp.async pipeline when the warps' page rings fit, the general kernel otherwise
+  constexpr int kDepth = D > 128 ? 2 : 3;
+  if (decode_cpasync_enabled() && 4 * kDepth * 4 * p.block_size * D <= 200 * 1024) {
+    if (p.block_size == 16) return launch_decode_cp<D, 16, kDepth, false, false, true>(p, B, st);
+    return launch_decode_cp<D, 0, kDepth, false, false, true>(p, B, st);
   }
   const int smem = (128 + 4 * 16 * D) * (int)sizeof(float);
   if (ensure_dynamic_smem(reinterpret_cast<const void*>(paged_attn_kernel<D, false, true>), smem) != cudaSuccess) return -20;

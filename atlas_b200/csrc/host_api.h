@@ -140,6 +140,11 @@ int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, long long l
                             const int* tile_q0, int num_tiles, float scale, int Hq, int Hkv, int D, int block_size, int window,
                             void* stream, int chunk, const float* sinks);
 
+int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
+                            const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
+                            const int* tile_q0, int num_tiles, int total_tokens, float scale, int Hq, int Hkv, int D, int block_size,
+                            int chunk, const float* sinks, unsigned long long* status, void* stream);
+
 // ---- 32-bit attention (attention_f32.cu)
 int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const int* positions,
                             const float* rope, float* k_cache, float* v_cache, const int* slot_mapping, int T, int Hq, int Hkv, int D,

@@ -717,7 +717,7 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
     bt, st, nd = batch.block_tables, _stream(), batch.num_decodes
     if nd > 0:
         visible = min(batch.max_seq_len, chunk or batch.max_seq_len, window or batch.max_seq_len)
-        splits = decode_splits(nd, Hkv * ((Hq // Hkv + 15) // 16), visible, _num_sms[d])
+        splits = decode_splits(nd, Hkv if fp4 else Hkv * ((Hq // Hkv + 7) // 8), visible, _num_sms[d])
         po = pml = None
         if splits > 1:
             po = scratch("attn_part_o", nd * Hq * splits * D * 4, q.device)
@@ -732,6 +732,20 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
                                             bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                             0, nd, float(scale), Hq, Hkv, D, bs, window, splits, _ptr(po), _ptr(pml), st, chunk,
                                             _ptr(sinks)), "attn_decode_kv16")
+    if batch.num_seqs > nd and not fp4 and _TC_PREFILL and not window and bs == 16 and D <= 128 and Hq // Hkv <= 128:
+        # tcgen05 tiles of 128 // G query tokens; 1 = a shape the kernel does not take
+        tdev, n_tiles, _ = _tc_tiles(q, batch, nd, 128 // (Hq // Hkv))
+        if not getattr(L, "_tc16_bound", False):
+            L.atlas_attn_prefill_tc16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _i, _i,
+                                                  _i, _vp, _vp, _vp]
+            L._tc16_bound = True
+        rc = L.atlas_attn_prefill_tc16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
+                                       bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
+                                       tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, T, float(scale), Hq, Hkv, D, bs, chunk,
+                                       _ptr(sinks), _status_ptr[d], st)
+        if rc != 1:
+            _check(rc, "attn_prefill_tc16")
+            return out
     if batch.num_seqs > nd:
         tiles = getattr(batch, "_attn_tiles", None)
         if tiles is None:
