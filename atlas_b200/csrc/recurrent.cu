@@ -6,7 +6,7 @@
 //                   y[p] = sum_n r[n] * (S[p][n] + u[n] * k[n] * v[p]);   S[p][n] = w[n] * S[p][n] + k[n] * v[p]
 //
 //   linear_scan_kernel   one CTA per (head, block of columns p, sequence).  KS lanes share a column; each holds NK state
-//                        entries in registers (entry j*4+e of lane s is n = (j * KS + s) * 4 + e).  Four warps walk the rows
+//                        entries of CPT columns in registers (entry j*4+e of lane s is n = (j * KS + s) * 4 + e).  Four warps walk the rows
 //                        while four more load the next kScanRows rows from global memory and turn them into the fp32
 //                        coefficients (softplus, exponentials, row constants) in the other half of a double buffer.
 //   linear_step_kernel   the same for one row per sequence (decode): no staging of rows, the state streams through.
@@ -48,7 +48,7 @@ constexpr int kScanRows = 16;
 
 ATLAS_DEVICE float softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 
-// one head's coefficients of one row, computed by one thread per element n (or column p)
+// one head's coefficients of one row, element n (or column p)
 template <typename T, int MODE>
 ATLAS_DEVICE void row_key(const ScanParams<T>& p, int head, long long t, int n, float dtv, float* k, float* q, float* w) {
   if (n >= p.N) { *k = 0.f; *q = 0.f; *w = 0.f; return; }
@@ -70,6 +70,37 @@ ATLAS_DEVICE float row_col(const ScanParams<T>& p, int head, long long t, int co
   return MODE == kMamba ? to_f32(p.a[t * p.lda + head * p.P + col]) : to_f32(p.c[t * p.ldc + head * p.P + col]);
 }
 
+// One row's raw inputs as a warp holds them: element n = lane + 32 i of the keys, column lane + 32 i of the values.
+template <int NI, int CI>
+struct RowIn {
+  float k[NI], q[NI], w[NI], x[CI], dt;
+};
+template <typename T, int MODE, int NI, int CI>
+ATLAS_DEVICE void load_row(const ScanParams<T>& p, int head, long long t, int col0, int cols, int lane, RowIn<NI, CI>& in) {
+#pragma unroll
+  for (int i = 0; i < NI; ++i) {
+    const int n = lane + 32 * i;
+    in.k[i] = in.q[i] = in.w[i] = 0.f;
+    if (n < p.N) {
+      if (MODE == kMamba) {
+        const T* row = p.a + t * p.lda + p.H * p.P + (head / (p.H / p.G)) * p.N;
+        in.k[i] = to_f32(row[n]);
+        in.q[i] = to_f32(row[p.G * p.N + n]);
+      } else {
+        in.k[i] = to_f32(p.b[t * p.ldb + head * p.N + n]);
+        if (p.a) in.q[i] = to_f32(p.a[t * p.lda + head * p.N + n]);
+        in.w[i] = to_f32(p.d[t * p.ldd + head * p.N + n]);
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < CI; ++i) {
+    const int c = lane + 32 * i;
+    in.x[i] = c < cols ? row_col<T, MODE>(p, head, t, col0 + c) : 0.f;
+  }
+  in.dt = MODE == kMamba ? to_f32(p.b[t * p.ldb + head]) : 0.f;
+}
+
 // WKV: rows of `x` that become a slot's previous-token row; the head CTAs share the W channels
 template <typename T>
 ATLAS_DEVICE void store_shift(const ScanParams<T>& p, int head, long long row, long long slot, int tid, int threads) {
@@ -77,11 +108,12 @@ ATLAS_DEVICE void store_shift(const ScanParams<T>& p, int head, long long row, l
   for (int i = lo + tid; i < hi; i += threads) p.shift[slot * p.W + i] = p.x[row * p.ldx + i];
 }
 
-template <typename T, int MODE, int NK, int KS>
+template <typename T, int MODE, int NK, int KS, int CPT>
 __global__ void __launch_bounds__(256)
 linear_scan_kernel(const ScanParams<T> p) {
-  constexpr int NP = NK * KS, CB = 128 / KS;
+  constexpr int NP = NK * KS, CL = 128 / KS, CB = CL * CPT;     // lanes' columns: c0 + i * CL
   constexpr int kRowF = NP * (MODE == kWkv ? 3 : 2) + CB;       // key, query (, decay) and column values of a row
+  constexpr int NI = (NP + 31) / 32, CI = (CB + 31) / 32;
   extern __shared__ float sm[];                                 // [2][kScanRows][kRowF] then [2][kScanRows] row scalars
   float* scal = sm + 2 * kScanRows * kRowF;
   const int head = blockIdx.x, bseq = blockIdx.z;
@@ -91,55 +123,75 @@ linear_scan_kernel(const ScanParams<T> p) {
   if (n_rows <= 0) return;
   const long long slot = p.state_slots[bseq];
   const bool walker = threadIdx.x < 128;
-  const int tid = threadIdx.x & 127;
-  const int col = blockIdx.y * CB + tid / KS, s = tid % KS;
-  const bool live = walker && col < p.P;
+  const int tid = threadIdx.x & 127, warp = tid >> 5, lane = tid & 31;
+  const int c0 = blockIdx.y * CB + tid / KS, s = tid % KS;
   const float neg_a = MODE == kMamba ? -expf(p.A_log[head]) : 0.f;
   const float dskip = MODE == kMamba ? p.D[head] : 0.f;
   const float dtb = MODE == kMamba ? p.dt_bias[head] : 0.f;
 
-  auto fill = [&](int buf, int r0) {                            // loader warps: rows [r0, r0 + kScanRows) of the chunk
+  // loader warps: rows [r0, r0 + kScanRows) of the chunk, two rows of a warp in flight together
+  auto fill = [&](int buf, int r0) {
     const int m = min(kScanRows, n_rows - r0);
-    const int warp = tid >> 5, lane = tid & 31;
-    for (int r = warp; r < m; r += 4) {
-      const long long t = q0 + r0 + r;
-      float* row = sm + (buf * kScanRows + r) * kRowF;
-      float sc = 0.f, dtv = 0.f;
-      if (MODE == kMamba) {
-        dtv = fmaxf(softplus(to_f32(p.b[t * p.ldb + head]) + dtb), p.dt_min);
-        sc = expf(neg_a * dtv);
-      }
+    for (int r = warp; r < m; r += 8) {
+      RowIn<NI, CI> in[2];
 #pragma unroll
-      for (int n = lane; n < NP; n += 32) {
-        float k, q, w;
-        row_key<T, MODE>(p, head, t, n, dtv, &k, &q, &w);
-        row[n] = k;
-        row[NP + n] = q;
-        if (MODE == kWkv) {
-          row[2 * NP + n] = w;
-          if (n < p.N) sc += q * p.u[head * p.N + n] * k;       // the bonus term's weight on v is the same for every column
+      for (int d = 0; d < 2; ++d)
+        if (r + 4 * d < m) load_row<T, MODE, NI, CI>(p, head, q0 + r0 + r + 4 * d, blockIdx.y * CB, CB, lane, in[d]);
+#pragma unroll
+      for (int d = 0; d < 2; ++d) {
+        if (r + 4 * d >= m) break;
+        float* row = sm + (buf * kScanRows + r + 4 * d) * kRowF;
+        float sc = 0.f, dtv = 1.f;
+        if (MODE == kMamba) {
+          dtv = fmaxf(softplus(in[d].dt + dtb), p.dt_min);
+          sc = expf(neg_a * dtv);
         }
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const int n = lane + 32 * i;
+          if (NP % 32 != 0 && n >= NP) break;
+          row[n] = in[d].k[i] * dtv;
+          row[NP + n] = in[d].q[i];
+          if (MODE == kWkv) {
+            float w = 0.f;
+            if (n < p.N) {
+              w = expf(-expf(in[d].w[i] + p.w0[head * p.N + n]));
+              sc += in[d].q[i] * p.u[head * p.N + n] * in[d].k[i];   // the bonus term's weight on v, the same for every column
+            }
+            row[2 * NP + n] = w;
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < CI; ++i)
+          if (lane + 32 * i < CB) row[kRowF - CB + lane + 32 * i] = in[d].x[i];
+        if (MODE == kWkv) sc = warp_sum(sc);
+        if (lane == 0) scal[buf * kScanRows + r + 4 * d] = sc;
       }
-      for (int c = lane; c < CB; c += 32) row[kRowF - CB + c] = row_col<T, MODE>(p, head, t, blockIdx.y * CB + c);
-      if (MODE == kWkv) sc = warp_sum(sc);
-      if (lane == 0) scal[buf * kScanRows + r] = sc;
     }
   };
 
-  float h[NK];
-  float* hs = p.h + (((long long)slot * p.H + head) * p.P + col) * p.N;
-  auto each = [&](auto fn) {
+  float h[CPT][NK];
+  auto each = [&](long long slot_of, auto fn) {                 // this thread's live state entries and their addresses
+    if (!walker) return;
 #pragma unroll
-    for (int j = 0; j < NK / 4; ++j)
+    for (int i = 0; i < CPT; ++i) {
+      const int col = c0 + i * CL;
+      if (col >= p.P) break;
+      float* base = p.h + ((slot_of * p.H + head) * p.P + col) * p.N;
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int n = (j * KS + s) * 4 + e;
-        if (n < p.N) fn(j * 4 + e, n);
-      }
+      for (int j = 0; j < NK / 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int n = (j * KS + s) * 4 + e;
+          if (n < p.N) fn(h[i][j * 4 + e], base[n]);
+        }
+    }
   };
 #pragma unroll
-  for (int i = 0; i < NK; ++i) h[i] = 0.f;
-  if (live && p.has_state[bseq]) each([&](int i, int n) { h[i] = hs[n]; });
+  for (int i = 0; i < CPT; ++i)
+#pragma unroll
+    for (int j = 0; j < NK; ++j) h[i][j] = 0.f;
+  if (p.has_state[bseq]) each(slot, [](float& reg, float& mem) { reg = mem; });
 
   if (!walker) fill(0, 0);
   __syncthreads();
@@ -152,8 +204,9 @@ linear_scan_kernel(const ScanParams<T> p) {
       for (int r = 0; r < m; ++r) {
         const float* row = sm + (buf * kScanRows + r) * kRowF;
         const float sc = scal[buf * kScanRows + r];
-        const float xv = row[kRowF - CB + tid / KS];
-        float acc = 0.f;
+        float xv[CPT], acc[CPT];
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) { xv[i] = row[kRowF - CB + tid / KS + i * CL]; acc[i] = 0.f; }
 #pragma unroll
         for (int j = 0; j < NK / 4; ++j) {
           const float4 k4 = *reinterpret_cast<const float4*>(row + (j * KS + s) * 4);
@@ -161,35 +214,40 @@ linear_scan_kernel(const ScanParams<T> p) {
           const float k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
           if constexpr (MODE == kMamba) {
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              h[j * 4 + e] = fmaf(h[j * 4 + e], sc, k[e] * xv);
-              acc = fmaf(h[j * 4 + e], q[e], acc);
-            }
+            for (int i = 0; i < CPT; ++i)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], sc, k[e] * xv[i]);
+                acc[i] = fmaf(h[i][j * 4 + e], q[e], acc[i]);
+              }
           } else {
             const float4 w4 = *reinterpret_cast<const float4*>(row + 2 * NP + (j * KS + s) * 4);
             const float w[4] = {w4.x, w4.y, w4.z, w4.w};
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              acc = fmaf(h[j * 4 + e], q[e], acc);
-              h[j * 4 + e] = fmaf(h[j * 4 + e], w[e], k[e] * xv);
-            }
+            for (int i = 0; i < CPT; ++i)
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                acc[i] = fmaf(h[i][j * 4 + e], q[e], acc[i]);
+                h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], w[e], k[e] * xv[i]);
+              }
           }
         }
 #pragma unroll
-        for (int off = KS / 2; off > 0; off >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
-        if (live && s == 0 && p.out)
-          p.out[(long long)(q0 + r0 + r) * p.ldo + head * p.P + col] = from_f32<T>(fmaf(MODE == kMamba ? dskip : sc, xv, acc));
-        for (int i = 0; i < p.num_snaps_per_seq; ++i) {
-          if (live && p.snap_rows[bseq * p.num_snaps_per_seq + i] == r0 + r + 1) {
-            float* dst = p.h + (((long long)p.snap_slots[bseq * p.num_snaps_per_seq + i] * p.H + head) * p.P + col) * p.N;
-            each([&](int q, int n) { dst[n] = h[q]; });
-          }
+        for (int i = 0; i < CPT; ++i) {
+#pragma unroll
+          for (int off = KS / 2; off > 0; off >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], off);
+          const int col = c0 + i * CL;
+          if (s == 0 && col < p.P && p.out)
+            p.out[(long long)(q0 + r0 + r) * p.ldo + head * p.P + col] = from_f32<T>(fmaf(MODE == kMamba ? dskip : sc, xv[i], acc[i]));
         }
+        for (int i = 0; i < p.num_snaps_per_seq; ++i)
+          if (p.snap_rows[bseq * p.num_snaps_per_seq + i] == r0 + r + 1)
+            each(p.snap_slots[bseq * p.num_snaps_per_seq + i], [](float& reg, float& mem) { mem = reg; });
       }
     }
     __syncthreads();
   }
-  if (p.commit && live) each([&](int i, int n) { hs[n] = h[i]; });
+  if (p.commit) each(slot, [](float& reg, float& mem) { mem = reg; });
   if (MODE == kWkv && blockIdx.y == 0) {
     for (int i = 0; i < p.num_snaps_per_seq; ++i) {
       const int r = p.snap_rows[bseq * p.num_snaps_per_seq + i];
@@ -304,6 +362,16 @@ linear_step_kernel(const ScanParams<T> p) {
   if (MODE == kWkv && p.commit && blockIdx.y == 0) store_shift(p, head, t, slot, tid, 128);
 }
 
+template <typename T, int MODE, int NK, int KS, int CPT>
+static int launch_rows(const ScanParams<T>& p, int B, cudaStream_t st) {
+  constexpr int CB = 128 / KS * CPT, NP = NK * KS;
+  constexpr int smem = (2 * kScanRows * (NP * (MODE == kWkv ? 3 : 2) + CB) + 2 * kScanRows) * (int)sizeof(float);
+  auto k = linear_scan_kernel<T, MODE, NK, KS, CPT>;
+  if (smem > 40 * 1024 && ensure_dynamic_smem(reinterpret_cast<const void*>(k), smem) != cudaSuccess) return -20;
+  k<<<dim3(p.H, (p.P + CB - 1) / CB, B), 256, smem, st>>>(p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
 template <typename T, int MODE, int NK, int KS>
 static int launch_scan(const ScanParams<T>& p, int B, int one_row, cudaStream_t st) {
   if (one_row) {
@@ -311,12 +379,11 @@ static int launch_scan(const ScanParams<T>& p, int B, int one_row, cudaStream_t 
     launch_chain_if(true, linear_step_kernel<T, MODE, NK, KS>, dim3(p.H, (p.P + CB - 1) / CB, B), dim3(128), 0, st, p);
     return cudaGetLastError() == cudaSuccess ? 0 : -21;
   }
-  constexpr int CB = 128 / KS, NP = NK * KS;
-  constexpr int smem = (2 * kScanRows * (NP * (MODE == kWkv ? 3 : 2) + CB) + 2 * kScanRows) * (int)sizeof(float);
-  auto k = linear_scan_kernel<T, MODE, NK, KS>;
-  if (smem > 40 * 1024 && ensure_dynamic_smem(reinterpret_cast<const void*>(k), smem) != cudaSuccess) return -20;
-  k<<<dim3(p.H, (p.P + CB - 1) / CB, B), 256, smem, st>>>(p);
-  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+  // four columns per thread where that still gives most SMs a CTA: fewer shared-memory reads per state entry
+  const long long lanes = (long long)p.H * B;
+  if (lanes * ((p.P + 4 * (128 / KS) - 1) / (4 * (128 / KS))) >= 100) return launch_rows<T, MODE, NK, KS, 4>(p, B, st);
+  if (lanes * ((p.P + 2 * (128 / KS) - 1) / (2 * (128 / KS))) >= 48) return launch_rows<T, MODE, NK, KS, 2>(p, B, st);
+  return launch_rows<T, MODE, NK, KS, 1>(p, B, st);
 }
 
 // `one_row`: every sequence of the step has exactly one row, no row limit and no snapshot
