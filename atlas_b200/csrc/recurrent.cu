@@ -70,35 +70,30 @@ ATLAS_DEVICE float row_col(const ScanParams<T>& p, int head, long long t, int co
   return MODE == kMamba ? to_f32(p.a[t * p.lda + head * p.P + col]) : to_f32(p.c[t * p.ldc + head * p.P + col]);
 }
 
-// One row's raw inputs as a warp holds them: element n = lane + 32 i of the keys, column lane + 32 i of the values.
-template <int NI, int CI>
+// One row's raw inputs as a warp holds them: element n = lane + 32 i of the keys, column lane + 32 i of the values.  The
+// loads are unconditional (indices are clamped into the row, what lies outside is dropped when the row is used), so that all
+// of them are in flight together.
+template <typename T, int NI, int CI>
 struct RowIn {
-  float k[NI], q[NI], w[NI], x[CI], dt;
+  T k[NI], q[NI], w[NI], x[CI], dt;
 };
 template <typename T, int MODE, int NI, int CI>
-ATLAS_DEVICE void load_row(const ScanParams<T>& p, int head, long long t, int col0, int cols, int lane, RowIn<NI, CI>& in) {
+ATLAS_DEVICE void load_row(const ScanParams<T>& p, int head, long long t, int col0, int lane, RowIn<T, NI, CI>& in) {
+  const T* qrow = MODE == kMamba ? p.a + t * p.lda + p.H * p.P + (p.G + head / (p.H / p.G)) * p.N
+                                 : (p.a ? p.a + t * p.lda : p.b + t * p.ldb) + head * p.N;
+  const T* krow = MODE == kMamba ? qrow - p.G * p.N : p.b + t * p.ldb + head * p.N;
+  const T* wrow = MODE == kMamba ? krow : p.d + t * p.ldd + head * p.N;
+  const T* xrow = (MODE == kMamba ? p.a + t * p.lda : p.c + t * p.ldc) + head * p.P;
 #pragma unroll
   for (int i = 0; i < NI; ++i) {
-    const int n = lane + 32 * i;
-    in.k[i] = in.q[i] = in.w[i] = 0.f;
-    if (n < p.N) {
-      if (MODE == kMamba) {
-        const T* row = p.a + t * p.lda + p.H * p.P + (head / (p.H / p.G)) * p.N;
-        in.k[i] = to_f32(row[n]);
-        in.q[i] = to_f32(row[p.G * p.N + n]);
-      } else {
-        in.k[i] = to_f32(p.b[t * p.ldb + head * p.N + n]);
-        if (p.a) in.q[i] = to_f32(p.a[t * p.lda + head * p.N + n]);
-        in.w[i] = to_f32(p.d[t * p.ldd + head * p.N + n]);
-      }
-    }
+    const int n = min(lane + 32 * i, p.N - 1);
+    in.k[i] = krow[n];
+    in.q[i] = qrow[n];
+    if (MODE == kWkv) in.w[i] = wrow[n];
   }
 #pragma unroll
-  for (int i = 0; i < CI; ++i) {
-    const int c = lane + 32 * i;
-    in.x[i] = c < cols ? row_col<T, MODE>(p, head, t, col0 + c) : 0.f;
-  }
-  in.dt = MODE == kMamba ? to_f32(p.b[t * p.ldb + head]) : 0.f;
+  for (int i = 0; i < CI; ++i) in.x[i] = xrow[min(col0 + lane + 32 * i, p.P - 1)];
+  if (MODE == kMamba) in.dt = p.b[t * p.ldb + head];
 }
 
 // WKV: rows of `x` that become a slot's previous-token row; the head CTAs share the W channels
@@ -129,44 +124,51 @@ linear_scan_kernel(const ScanParams<T> p) {
   const float dskip = MODE == kMamba ? p.D[head] : 0.f;
   const float dtb = MODE == kMamba ? p.dt_bias[head] : 0.f;
 
-  // loader warps: rows [r0, r0 + kScanRows) of the chunk, two rows of a warp in flight together
+  float w0[MODE == kWkv ? NI : 1], un[MODE == kWkv ? NI : 1];
+  if (MODE == kWkv) {
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+      const int n = lane + 32 * i;
+      w0[i] = n < p.N ? p.w0[head * p.N + n] : 0.f;
+      un[i] = n < p.N ? p.u[head * p.N + n] : 0.f;
+    }
+  }
+  // Loader warps: warp w owns rows w, w + 4, .. of every kScanRows-row block.  Their raw values are fetched one block before
+  // they are turned into coefficients, so a whole block's time hides the memory latency.
+  RowIn<T, NI, CI> in[kScanRows / 4];
+  auto fetch = [&](int r0) {
+#pragma unroll
+    for (int d = 0; d < kScanRows / 4; ++d)
+      load_row<T, MODE, NI, CI>(p, head, q0 + min(r0 + warp + 4 * d, n_rows - 1), blockIdx.y * CB, lane, in[d]);
+  };
   auto fill = [&](int buf, int r0) {
-    const int m = min(kScanRows, n_rows - r0);
-    for (int r = warp; r < m; r += 8) {
-      RowIn<NI, CI> in[2];
 #pragma unroll
-      for (int d = 0; d < 2; ++d)
-        if (r + 4 * d < m) load_row<T, MODE, NI, CI>(p, head, q0 + r0 + r + 4 * d, blockIdx.y * CB, CB, lane, in[d]);
-#pragma unroll
-      for (int d = 0; d < 2; ++d) {
-        if (r + 4 * d >= m) break;
-        float* row = sm + (buf * kScanRows + r + 4 * d) * kRowF;
-        float sc = 0.f, dtv = 1.f;
-        if (MODE == kMamba) {
-          dtv = fmaxf(softplus(in[d].dt + dtb), p.dt_min);
-          sc = expf(neg_a * dtv);
-        }
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-          const int n = lane + 32 * i;
-          if (NP % 32 != 0 && n >= NP) break;
-          row[n] = in[d].k[i] * dtv;
-          row[NP + n] = in[d].q[i];
-          if (MODE == kWkv) {
-            float w = 0.f;
-            if (n < p.N) {
-              w = expf(-expf(in[d].w[i] + p.w0[head * p.N + n]));
-              sc += in[d].q[i] * p.u[head * p.N + n] * in[d].k[i];   // the bonus term's weight on v, the same for every column
-            }
-            row[2 * NP + n] = w;
-          }
-        }
-#pragma unroll
-        for (int i = 0; i < CI; ++i)
-          if (lane + 32 * i < CB) row[kRowF - CB + lane + 32 * i] = in[d].x[i];
-        if (MODE == kWkv) sc = warp_sum(sc);
-        if (lane == 0) scal[buf * kScanRows + r + 4 * d] = sc;
+    for (int d = 0; d < kScanRows / 4; ++d) {
+      if (r0 + warp + 4 * d >= n_rows) break;
+      float* row = sm + (buf * kScanRows + warp + 4 * d) * kRowF;
+      float sc = 0.f, dtv = 1.f;
+      if (MODE == kMamba) {
+        dtv = fmaxf(softplus(to_f32(in[d].dt) + dtb), p.dt_min);
+        sc = expf(neg_a * dtv);
       }
+#pragma unroll
+      for (int i = 0; i < NI; ++i) {
+        const int n = lane + 32 * i;
+        if (NP % 32 != 0 && n >= NP) break;
+        const bool in_row = n < p.N;
+        const float k = in_row ? to_f32(in[d].k[i]) : 0.f, q = in_row && (MODE == kMamba || p.a) ? to_f32(in[d].q[i]) : 0.f;
+        row[n] = k * dtv;
+        row[NP + n] = q;
+        if (MODE == kWkv) {
+          row[2 * NP + n] = in_row ? expf(-expf(to_f32(in[d].w[i]) + w0[i])) : 0.f;
+          sc += q * un[i] * k;                                   // the bonus term's weight on v, the same for every column
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < CI; ++i)
+        if (lane + 32 * i < CB) row[kRowF - CB + lane + 32 * i] = to_f32(in[d].x[i]);
+      if (MODE == kWkv) sc = warp_sum(sc);
+      if (lane == 0) scal[buf * kScanRows + warp + 4 * d] = sc;
     }
   };
 
@@ -193,11 +195,16 @@ linear_scan_kernel(const ScanParams<T> p) {
     for (int j = 0; j < NK; ++j) h[i][j] = 0.f;
   if (p.has_state[bseq]) each(slot, [](float& reg, float& mem) { reg = mem; });
 
-  if (!walker) fill(0, 0);
+  if (!walker) {
+    fetch(0);
+    fill(0, 0);
+    fetch(kScanRows);
+  }
   __syncthreads();
   for (int r0 = 0, buf = 0; r0 < n_rows; r0 += kScanRows, buf ^= 1) {
     if (!walker) {
-      if (r0 + kScanRows < n_rows) fill(buf ^ 1, r0 + kScanRows);
+      fill(buf ^ 1, r0 + kScanRows);
+      fetch(r0 + 2 * kScanRows);
     } else {
       const int m = min(kScanRows, n_rows - r0);
 #pragma unroll 2
@@ -381,8 +388,10 @@ static int launch_scan(const ScanParams<T>& p, int B, int one_row, cudaStream_t 
   }
   // four columns per thread where that still gives most SMs a CTA: fewer shared-memory reads per state entry
   const long long lanes = (long long)p.H * B;
-  if (lanes * ((p.P + 4 * (128 / KS) - 1) / (4 * (128 / KS))) >= 100) return launch_rows<T, MODE, NK, KS, 4>(p, B, st);
-  if (lanes * ((p.P + 2 * (128 / KS) - 1) / (2 * (128 / KS))) >= 48) return launch_rows<T, MODE, NK, KS, 2>(p, B, st);
+  if constexpr (KS >= 4) {                     // (fewer lanes per column already give a block of columns per CTA)
+    if (lanes * ((p.P + 4 * (128 / KS) - 1) / (4 * (128 / KS))) >= 100) return launch_rows<T, MODE, NK, KS, 4>(p, B, st);
+    if (lanes * ((p.P + 2 * (128 / KS) - 1) / (2 * (128 / KS))) >= 48) return launch_rows<T, MODE, NK, KS, 2>(p, B, st);
+  }
   return launch_rows<T, MODE, NK, KS, 1>(p, B, st);
 }
 
