@@ -44,7 +44,7 @@ struct ScanParams {
   int H, P, N, G, commit;
 };
 
-constexpr int kScanRows = 16;
+constexpr int kScanRows = 16, kGroup = 4;
 
 ATLAS_DEVICE float softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 
@@ -206,50 +206,71 @@ linear_scan_kernel(const ScanParams<T> p) {
       fill(buf ^ 1, r0 + kScanRows);
       fetch(r0 + 2 * kScanRows);
     } else {
+      // rows in groups of kGroup: the sums over the lanes of a column are formed for a whole group together
       const int m = min(kScanRows, n_rows - r0);
-#pragma unroll 2
-      for (int r = 0; r < m; ++r) {
-        const float* row = sm + (buf * kScanRows + r) * kRowF;
-        const float sc = scal[buf * kScanRows + r];
-        float xv[CPT], acc[CPT];
+      for (int rg = 0; rg < m; rg += kGroup) {
+        float acc[kGroup][CPT], skip[kGroup][CPT];
 #pragma unroll
-        for (int i = 0; i < CPT; ++i) { xv[i] = row[kRowF - CB + tid / KS + i * CL]; acc[i] = 0.f; }
+        for (int g = 0; g < kGroup; ++g) {
+          const int r = rg + g;
+          if (r >= m) break;
+          const float* row = sm + (buf * kScanRows + r) * kRowF;
+          const float sc = scal[buf * kScanRows + r];
+          float xv[CPT], part[CPT][4];
 #pragma unroll
-        for (int j = 0; j < NK / 4; ++j) {
-          const float4 k4 = *reinterpret_cast<const float4*>(row + (j * KS + s) * 4);
-          const float4 q4 = *reinterpret_cast<const float4*>(row + NP + (j * KS + s) * 4);
-          const float k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
-          if constexpr (MODE == kMamba) {
+          for (int i = 0; i < CPT; ++i) {
+            xv[i] = row[kRowF - CB + tid / KS + i * CL];
+            skip[g][i] = (MODE == kMamba ? dskip : sc) * xv[i];
 #pragma unroll
-            for (int i = 0; i < CPT; ++i)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], sc, k[e] * xv[i]);
-                acc[i] = fmaf(h[i][j * 4 + e], q[e], acc[i]);
-              }
-          } else {
-            const float4 w4 = *reinterpret_cast<const float4*>(row + 2 * NP + (j * KS + s) * 4);
-            const float w[4] = {w4.x, w4.y, w4.z, w4.w};
-#pragma unroll
-            for (int i = 0; i < CPT; ++i)
-#pragma unroll
-              for (int e = 0; e < 4; ++e) {
-                acc[i] = fmaf(h[i][j * 4 + e], q[e], acc[i]);
-                h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], w[e], k[e] * xv[i]);
-              }
+            for (int e = 0; e < 4; ++e) part[i][e] = 0.f;
           }
+#pragma unroll
+          for (int j = 0; j < NK / 4; ++j) {
+            const float4 k4 = *reinterpret_cast<const float4*>(row + (j * KS + s) * 4);
+            const float4 q4 = *reinterpret_cast<const float4*>(row + NP + (j * KS + s) * 4);
+            const float k[4] = {k4.x, k4.y, k4.z, k4.w}, q[4] = {q4.x, q4.y, q4.z, q4.w};
+            if constexpr (MODE == kMamba) {
+#pragma unroll
+              for (int i = 0; i < CPT; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], sc, k[e] * xv[i]);
+                  part[i][e] = fmaf(h[i][j * 4 + e], q[e], part[i][e]);
+                }
+            } else {
+              const float4 w4 = *reinterpret_cast<const float4*>(row + 2 * NP + (j * KS + s) * 4);
+              const float w[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+              for (int i = 0; i < CPT; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  part[i][e] = fmaf(h[i][j * 4 + e], q[e], part[i][e]);
+                  h[i][j * 4 + e] = fmaf(h[i][j * 4 + e], w[e], k[e] * xv[i]);
+                }
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < CPT; ++i) acc[g][i] = (part[i][0] + part[i][1]) + (part[i][2] + part[i][3]);
+          for (int i = 0; i < p.num_snaps_per_seq; ++i)
+            if (p.snap_rows[bseq * p.num_snaps_per_seq + i] == r0 + r + 1)
+              each(p.snap_slots[bseq * p.num_snaps_per_seq + i], [](float& reg, float& mem) { mem = reg; });
         }
 #pragma unroll
-        for (int i = 0; i < CPT; ++i) {
+        for (int off = KS / 2; off > 0; off >>= 1)
 #pragma unroll
-          for (int off = KS / 2; off > 0; off >>= 1) acc[i] += __shfl_xor_sync(0xffffffffu, acc[i], off);
-          const int col = c0 + i * CL;
-          if (s == 0 && col < p.P && p.out)
-            p.out[(long long)(q0 + r0 + r) * p.ldo + head * p.P + col] = from_f32<T>(fmaf(MODE == kMamba ? dskip : sc, xv[i], acc[i]));
+          for (int g = 0; g < kGroup; ++g)
+#pragma unroll
+            for (int i = 0; i < CPT; ++i) acc[g][i] += __shfl_xor_sync(0xffffffffu, acc[g][i], off);
+        if (s == 0 && p.out) {
+#pragma unroll
+          for (int g = 0; g < kGroup; ++g)
+#pragma unroll
+            for (int i = 0; i < CPT; ++i) {
+              const int col = c0 + i * CL;
+              if (rg + g < m && col < p.P)
+                p.out[(long long)(q0 + r0 + rg + g) * p.ldo + head * p.P + col] = from_f32<T>(acc[g][i] + skip[g][i]);
+            }
         }
-        for (int i = 0; i < p.num_snaps_per_seq; ++i)
-          if (p.snap_rows[bseq * p.num_snaps_per_seq + i] == r0 + r + 1)
-            each(p.snap_slots[bseq * p.num_snaps_per_seq + i], [](float& reg, float& mem) { mem = reg; });
       }
     }
     __syncthreads();
