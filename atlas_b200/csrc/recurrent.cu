@@ -432,7 +432,7 @@ static int scan(const ScanParams<T>& p, int B, int one_row, cudaStream_t st) {
 }
 
 // ----------------------------------------------------------------------------- gated group norm
-// TPG threads per (row, group): a warp for small groups, a whole block for wide ones
+// TPG threads per (row, group): a quarter of a warp for head-sized groups, a warp, or a whole block for wide ones
 template <typename T, int TPG, int V, bool kGateFirst>
 __global__ void __launch_bounds__(256)
 group_norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ z, long long ldz,
@@ -441,9 +441,9 @@ group_norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restri
   chain_trigger();
   chain_wait();
   const long long unit = (long long)blockIdx.x * (256 / TPG) + threadIdx.x / TPG;
-  if (unit >= (long long)rows * groups) return;                 // TPG == 256: the whole block leaves together
+  const bool live = unit < (long long)rows * groups;            // every lane stays for the warp's sums
   const int tid = threadIdx.x % TPG;
-  const long long t = unit / groups;
+  const long long t = live ? unit / groups : 0;
   const int g0 = (int)(unit % groups) * gsize;
   const T* yr = y + t * ldy + g0;
   const T* zr = z + t * ldz + g0;
@@ -459,7 +459,8 @@ group_norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restri
 #pragma unroll
     for (int i = 0; i < V; ++i) ss += f[i] * f[i];
   }
-  ss = warp_sum(ss);
+#pragma unroll
+  for (int off = (TPG < 32 ? TPG : 32) / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
   if (TPG > 32) {
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
     __syncthreads();
@@ -467,6 +468,7 @@ group_norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restri
 #pragma unroll
     for (int i = 0; i < 8; ++i) ss += red[i];
   }
+  if (!live) return;
   const float rstd = 1.f / sqrtf(ss / (float)gsize + eps);
   for (int e = tid * V; e < gsize; e += TPG * V) {
     float f[V], g[V], wv[V];
@@ -488,6 +490,9 @@ static int launch_gnorm(const void* y, long long ldy, const void* z, long long l
   if (gsize >= 1024)
     launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 256, V, kGateFirst>, dim3((unsigned)units), dim3(256), 0, st, yp, ldy, zp, ldz, w,
                     reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps);
+  else if (gsize <= 128)
+    launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 8, V, kGateFirst>, dim3((unsigned)((units + 31) / 32)), dim3(256), 0, st, yp, ldy,
+                    zp, ldz, w, reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps);
   else
     launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 32, V, kGateFirst>, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, st, yp, ldy,
                     zp, ldz, w, reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps);
@@ -497,6 +502,9 @@ static int launch_gnorm(const void* y, long long ldy, const void* z, long long l
 template <typename T>
 static int gnorm(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
                  int groups, int gsize, float eps, int gate_first, cudaStream_t st) {
+  if (sizeof(T) == 2 && gsize % 8 == 0 && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(z, ldz) && vec_ok<T, 8>(out, ldo))
+    return gate_first ? launch_gnorm<T, 8, true>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st)
+                      : launch_gnorm<T, 8, false>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st);
   const bool vec = gsize % 4 == 0 && vec_ok<T, 4>(y, ldy) && vec_ok<T, 4>(z, ldz) && vec_ok<T, 4>(out, ldo);
   if (vec) return gate_first ? launch_gnorm<T, 4, true>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st)
                              : launch_gnorm<T, 4, false>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st);

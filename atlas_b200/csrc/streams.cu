@@ -165,9 +165,9 @@ static int hyper_norm(float* x, int rows, int S, int W, const void* y, long long
 }
 
 // ----------------------------------------------------------------------------- token shift
-constexpr int kShiftRows = 8;                  // consecutive rows of one thread: mu stays in registers, the previous row too
+constexpr int kShiftRows = 8;                  // consecutive rows of one thread (1 for few rows): mu and the previous row stay in registers
 
-template <typename T, int S, int V>
+template <typename T, int S, int V, int R>
 __global__ void __launch_bounds__(256)
 token_shift_mix_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ mu, const T* __restrict__ shift,
                        const int* __restrict__ seq_of_token, const int* __restrict__ query_start_loc,
@@ -179,7 +179,7 @@ token_shift_mix_kernel(const T* __restrict__ x, long long ldx, const float* __re
   float m[S][V];
 #pragma unroll
   for (int s = 0; s < S; ++s) load_vec<V>(mu + (long long)s * W + e, m[s]);
-  const int t0 = blockIdx.x * kShiftRows, t1 = min(rows, t0 + kShiftRows);
+  const int t0 = blockIdx.x * R, t1 = min(rows, t0 + R);
   float prev[V];
   for (int t = t0; t < t1; ++t) {
     const int b = seq_of_token[t];
@@ -210,9 +210,14 @@ token_shift_mix_kernel(const T* __restrict__ x, long long ldx, const float* __re
 template <typename T, int V>
 static int launch_shift(const void* x, long long ldx, const float* mu, const void* shift, const int* seq, const int* qsl,
                         const int* slots, const unsigned char* has, void* out, int rows, int W, cudaStream_t st) {
-  dim3 grid((rows + kShiftRows - 1) / kShiftRows, (W + 256 * V - 1) / (256 * V));
-  launch_chain_if(rows <= 256, token_shift_mix_kernel<T, 5, V>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(x), ldx, mu,
-                  reinterpret_cast<const T*>(shift), seq, qsl, slots, has, reinterpret_cast<T*>(out), rows, W);
+  const unsigned gy = (W + 256 * V - 1) / (256 * V);
+  if (rows <= 256)
+    launch_chain_if(true, token_shift_mix_kernel<T, 5, V, 1>, dim3(rows, gy), dim3(256), 0, st, reinterpret_cast<const T*>(x), ldx, mu,
+                    reinterpret_cast<const T*>(shift), seq, qsl, slots, has, reinterpret_cast<T*>(out), rows, W);
+  else
+    launch_chain_if(false, token_shift_mix_kernel<T, 5, V, kShiftRows>, dim3((rows + kShiftRows - 1) / kShiftRows, gy), dim3(256), 0, st,
+                    reinterpret_cast<const T*>(x), ldx, mu, reinterpret_cast<const T*>(shift), seq, qsl, slots, has,
+                    reinterpret_cast<T*>(out), rows, W);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 

@@ -25,7 +25,18 @@ ATLAS_DEVICE void load_vec(const float* p, float (&f)[V]) {
 }
 template <int V>
 ATLAS_DEVICE void load_vec(const __nv_bfloat16* p, float (&f)[V]) {
-  if constexpr (V % 4 == 0) {
+  if constexpr (V % 8 == 0) {
+#pragma unroll
+    for (int i = 0; i < V; i += 8) {
+      const uint4 r = *reinterpret_cast<const uint4*>(p + i);
+      const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&w[j]));
+        f[i + 2 * j] = a.x; f[i + 2 * j + 1] = a.y;
+      }
+    }
+  } else if constexpr (V % 4 == 0) {
 #pragma unroll
     for (int i = 0; i < V; i += 4) {
       const uint2 r = *reinterpret_cast<const uint2*>(p + i);
@@ -50,7 +61,12 @@ ATLAS_DEVICE void store_vec(float* p, const float (&f)[V]) {
 }
 template <int V>
 ATLAS_DEVICE void store_vec(__nv_bfloat16* p, const float (&f)[V]) {
-  if constexpr (V % 4 == 0) {
+  if constexpr (V % 8 == 0) {
+#pragma unroll
+    for (int i = 0; i < V; i += 8)
+      *reinterpret_cast<uint4*>(p + i) = make_uint4(pack_bf16x2(f[i], f[i + 1]), pack_bf16x2(f[i + 2], f[i + 3]),
+                                                    pack_bf16x2(f[i + 4], f[i + 5]), pack_bf16x2(f[i + 6], f[i + 7]));
+  } else if constexpr (V % 4 == 0) {
 #pragma unroll
     for (int i = 0; i < V; i += 4)
       *reinterpret_cast<uint2*>(p + i) = make_uint2(pack_bf16x2(f[i], f[i + 1]), pack_bf16x2(f[i + 2], f[i + 3]));
@@ -63,7 +79,7 @@ ATLAS_DEVICE void store_vec(__nv_bfloat16* p, const float (&f)[V]) {
 // rows of stride `ld` at `p` can be read V elements at a time (a null pointer can)
 template <typename T, int V>
 inline bool vec_ok(const void* p, long long ld) {
-  const size_t unit = (V * sizeof(T) > 16) ? 16 : (V * sizeof(T) >= 8 && sizeof(T) == 2 ? 8 : V * sizeof(T));
+  const size_t unit = V * sizeof(T) > 16 ? 16 : V * sizeof(T);
   return p == nullptr || ((reinterpret_cast<uintptr_t>(p) % unit) == 0 && (ld * (long long)sizeof(T)) % (long long)unit == 0);
 }
 
