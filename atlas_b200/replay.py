@@ -63,6 +63,9 @@ def replay(engine, lines, out_dir: str, answer) -> int:
         if wanted:
             path = os.path.join(out_dir, f"{step['step']}.f32")
             np.concatenate([p.numpy() for p in wanted]).astype("<f4").tofile(path)
+        elif engine.model.device.type == "cuda":
+            import torch
+            torch.cuda.synchronize()                 # "done" means that the step has run
         answer(f"done {step['step']}")
         n += 1
     return n

@@ -18,6 +18,7 @@ from .models import CacheStore, DecoderLM, ForwardBatch
 from .models.decoder import attention_of, recurrent_of
 from .sched import SchedulerOutput
 
+_PIN_RING = 3              # staging buffers per tensor: how many steps the host may run ahead
 _GRAPH_BATCH_SIZES = (1, 2, 4, 8, 16, 24, 32, 48, 64, 96, 128, 192, 256)
 
 
@@ -39,7 +40,8 @@ class ModelRunner:
         self.h2d_bytes = 0
         self.d2h_bytes = 0
         self.graph_replays = 0
-        self._pin: Dict[str, torch.Tensor] = {}
+        self._pin: Dict[str, list] = {}              # per name: a ring of (pinned buffer, event after its last copy)
+        self._pin_turn: Dict[str, int] = {}
         # decode graphs of recurrent models read state slots from a device buffer; the kernels that take everything they
         # need from there are those of recurrent.cu
         self._states_graph_safe = all(l.kind in ("mamba2", "wkv", "parallel") for l in model.layers if recurrent_of(l) is not None)
@@ -78,22 +80,29 @@ class ModelRunner:
 
     # ------------------------------------------------------------------ batch assembly
     def _stage(self, name: str, data, dtype: torch.dtype) -> torch.Tensor:
-        """Host list / numpy array -> device tensor through a reusable pinned buffer (one async H2D copy)."""
+        """Host list / numpy array -> device tensor through a reusable pinned buffer (one async H2D copy).  A buffer is
+        written again only after the copy that read it has run: steps that read nothing back (prompt portions, fed tokens)
+        let the host run ahead of the device."""
         src = torch.from_numpy(data) if isinstance(data, np.ndarray) else torch.tensor(data, dtype=dtype)
         if src.dtype != dtype:
             src = src.to(dtype)
         n = src.numel()
         if not self.on_gpu:
             return src.reshape(-1)
-        buf = self._pin.get(name)
-        if buf is None or buf.numel() < n or buf.dtype != dtype:
+        ring = self._pin.setdefault(name, [None] * _PIN_RING)
+        self._pin_turn[name] = turn = (self._pin_turn.get(name, -1) + 1) % _PIN_RING
+        if ring[turn] is not None:
+            ring[turn][1].synchronize()
+        if ring[turn] is None or ring[turn][0].numel() < n or ring[turn][0].dtype != dtype:
             cap = max(1024, 1 << (max(n, 1) - 1).bit_length())
-            buf = torch.empty(cap, dtype=dtype, pin_memory=True)
-            self._pin[name] = buf
+            ring[turn] = (torch.empty(cap, dtype=dtype, pin_memory=True), torch.cuda.Event())
+        buf, copied = ring[turn]
         host = buf[:n]
         host.copy_(src.reshape(-1))
         self.h2d_bytes += n * host.element_size()
-        return host.to(self.device, non_blocking=True)
+        out = host.to(self.device, non_blocking=True)
+        copied.record()
+        return out
 
     @staticmethod
     def _blocks_np(seq) -> np.ndarray:

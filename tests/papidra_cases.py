@@ -44,6 +44,8 @@ CASES = {
     # more query heads per kv head than one tile holds, wide state, five streams, five taps, sizes off the vector widths
     "wide": (model(77, 100, 5, [par_layer(attn(20, 1, 72, 40, 33, 36), mamba(2, 20, 136, 2, 1, 5), ff(36, 1.5)),
                                 wkv_layer(2, 72)]), 12),
+    # everything divides by two (tensor parallelism)
+    "even": (model(96, 64, 2, [wkv_layer(2, 16), par_layer(attn(4, 2, 32, 48, 24, 16), mamba(4, 24, 24, 2, 2, 3), ff(256, 1.0))]), 8),
     "odd": (model(61, 90, 3, [wkv_layer(3, 10), par_layer(attn(3, 3, 20, 12, 19, 6), mamba(3, 14, 13, 1, 3, 2), ff(45, 0.7))]), 5),
 }
 

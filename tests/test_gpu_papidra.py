@@ -340,6 +340,24 @@ def test_models_in_portions_and_batches(folder, name, dtype):
     eng.pool.check_invariants()
 
 
+@pytest.mark.parametrize("graphs", [True, False])
+def test_steps_that_read_nothing_back(folder, graphs):
+    """Only the last token's logits are asked for, so nothing makes the host wait for the device in between: every step
+    still runs on its own tokens, positions and pages."""
+    from atlas_b200.replay import build_engine
+    path, cfg, toks, want = folder("mixed")
+    eng = build_engine(path, "float32", 384, use_cuda_graphs=graphs)
+    for _ in range(3):
+        for i, t in toks.items():
+            cuts = PC.portions(len(t), [2] + [1] * 200)
+            at = 0
+            for n in cuts:
+                last = at + n == len(t)
+                got = eng.feed([(f"r{i}", t[at:at + n], [n - 1] if last else [])], [f"r{i}"] if last else [])[0]
+                at += n
+            assert PC.spread(got, want[i][-1:]) < MODEL_TOL["float32"]
+
+
 def test_decode_graph_equals_eager_decode(folder):
     from atlas_b200.replay import build_engine
     path, cfg, toks, want = folder("mixed")

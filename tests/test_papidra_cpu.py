@@ -121,6 +121,22 @@ def test_rejected_drafts_leave_the_state_alone(folder):
     assert PC.spread(got, want[23:]) < TOL
 
 
+def test_two_tensor_parallel_ranks_reproduce_the_whole_model(folder):
+    from atlas_b200.layers import ParallelCtx
+    from atlas_b200.parallel.comm import FakeWorld
+    path, cfg, w = folder("even")
+    toks = PC.tokens(cfg, 40, 8)
+    world = FakeWorld(2, timeout_s=60.0)
+
+    def rank(r):
+        comm = world.comm(r)
+        model = load_model(path, ParallelCtx(tp_rank=r, tp_size=2, comm=comm, ep_comm=comm), dtype="float32", max_pos=64)
+        return model.forward_dense_reference(toks)
+    want = O.forward(cfg, w, toks)
+    for got in world.run(rank):
+        assert PC.spread(got, want) < TOL
+
+
 def test_configuration_reads_every_size():
     cfg, _ = PC.CASES["wide"]
     c = ModelConfig.from_hf(cfg)
