@@ -502,7 +502,7 @@ static int launch_gnorm(const void* y, long long ldy, const void* z, long long l
 template <typename T>
 static int gnorm(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
                  int groups, int gsize, float eps, int gate_first, cudaStream_t st) {
-  if (sizeof(T) == 2 && gsize % 8 == 0 && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(z, ldz) && vec_ok<T, 8>(out, ldo))
+  if (sizeof(T) == 2 && gsize % 8 == 0 && (gsize < 1024 || gsize >= 2048) && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(z, ldz) && vec_ok<T, 8>(out, ldo))
     return gate_first ? launch_gnorm<T, 8, true>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st)
                       : launch_gnorm<T, 8, false>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, st);
   const bool vec = gsize % 4 == 0 && vec_ok<T, 4>(y, ldy) && vec_ok<T, 4>(z, ldz) && vec_ok<T, 4>(out, ldo);
