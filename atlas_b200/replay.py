@@ -30,8 +30,7 @@ def build_engine(path: str, dtype: str, max_tokens: int, device=None, use_cuda_g
     from .config import EngineConfig, ModelConfig
     from .loader import Checkpoint, load_weights
     from .models import build_model
-    if device is None:
-        device = "cuda:0" if torch.cuda.is_available() else "cpu"
+    device = device or "cuda:0"
     cfg = ModelConfig.from_pretrained(path)
     cfg.dtype = dtype
     if str(device).startswith("cuda"):
@@ -77,12 +76,13 @@ def main(argv=None) -> int:
     ap.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder that receives <step>.f32")
     ap.add_argument("--max-tokens", type=int, required=True, help="tokens that live requests hold at most at any time")
+    ap.add_argument("--device", default="cuda:0", help="cuda:N, or cpu for the plain PyTorch path")
     args = ap.parse_args(argv)
     # libraries may print to descriptor 1 on their own: keep it for the answers
     sys.stdout.flush()
     answers = os.fdopen(os.dup(1), "w")
     os.dup2(2, 1)
-    engine = build_engine(args.model, args.dtype, args.max_tokens)
+    engine = build_engine(args.model, args.dtype, args.max_tokens, device=args.device)
 
     def answer(text: str) -> None:
         answers.write(text + "\n")

@@ -222,7 +222,7 @@ def test_snapshots_and_row_limits(kind):
 
 # ------------------------------------------------------------------------------------------------- attention
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("H,G,D,size", [(4, 2, 64, 24), (3, 3, 128, 16), (20, 1, 64, 33), (8, 1, 256, 200), (2, 1, 64, 1), (4, 4, 64, 0)])
+@pytest.mark.parametrize("H,G,D,size", [(4, 2, 64, 24), (3, 3, 128, 16), (20, 1, 64, 33), (6, 1, 256, 160), (2, 1, 64, 1), (4, 4, 64, 0)])
 def test_chunked_attention_with_sinks(dtype, H, G, D, size):
     """Rows of prompts and decode rows over scattered pages.  One key near every edge of a chunk is aligned with all queries,
     so that a key too many or too few changes the output by its whole value; the sink is far from negligible."""

@@ -172,3 +172,40 @@ def test_random_preset_serves_through_the_command_line_loader():
     eng = LLMEngine(model, EngineConfig(num_kv_blocks=32, max_num_seqs=2, max_seq_len=128, kv_cache_dtype="fp8"))
     out = eng.generate([[1, 2, 3]], SamplingParams(max_tokens=5, ignore_eos=True))
     assert len(out[0].output_tokens) == 5
+
+
+def test_trace_runner_writes_what_was_asked_for(folder, tmp_path):
+    """The command itself: steps on standard input, one file per step with wanted places, an answer after every step."""
+    import json
+    import os
+    import subprocess
+    import sys
+
+    import numpy as np
+    path, cfg, w = folder("ones")
+    toks = PC.tokens(cfg, 12, 4)
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:9], "want": []}], "end": []},
+             {"step": 1, "entries": [{"id": "y", "tokens": toks[:4], "want": [3, 0]}, {"id": "x", "tokens": toks[9:], "want": [1]}], "end": ["x"]},
+             {"step": 7, "entries": [{"id": "y", "tokens": toks[4:5], "want": [0]}], "end": ["y"]}]
+    runner = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "bin", "trace_run")
+    r = subprocess.run([sys.executable, runner, "--model", path, "--dtype", "float32", "--out", str(tmp_path), "--max-tokens", "128",
+                        "--device", "cpu"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=300)
+    assert r.returncode == 0, r.stderr
+    assert r.stdout.split("\n")[:3] == ["done 0", "done 1", "done 7"] and sorted(os.listdir(tmp_path)) == ["1.f32", "7.f32"]
+    want = O.forward(cfg, w, toks)
+    got = torch.from_numpy(np.fromfile(tmp_path / "1.f32", dtype="<f4")).view(3, -1)
+    assert PC.spread(got, want[[3, 0, 10]]) < TOL
+    assert PC.spread(torch.from_numpy(np.fromfile(tmp_path / "7.f32", dtype="<f4")).view(1, -1), want[4:5]) < TOL
+
+
+@pytest.mark.parametrize("kind", ["wkv", "parallel"])
+def test_models_of_one_layer_kind(tmp_path, kind):
+    layer = PC.wkv_layer(2, 24, PC.ff(32, 1.0)) if kind == "wkv" else PC.par_layer(PC.attn(2, 2, 16, 16, 20, 8), PC.mamba(2, 16, 16, 2, 1, 4))
+    PC.CASES["one kind"] = (PC.model(50, 48, 3, [layer, layer]), 8)
+    try:
+        cfg, w = PC.write(str(tmp_path), "one kind")
+    finally:
+        del PC.CASES["one kind"]
+    toks = PC.tokens(cfg, 45, 1)
+    eng = build_engine(str(tmp_path), "float32", 64, device="cpu")
+    assert PC.spread(PC.feed_alone(eng, "a", toks, PC.portions(45, [7, 1, 20])), O.forward(cfg, w, toks)) < TOL
