@@ -49,7 +49,9 @@ def _run(cmd: List[str]) -> None:
 _UNITS_BASE = ("runtime",)
 _UNITS_BF16 = ("gemm", "elementwise", "attention", "attention_tc16")
 _UNITS_F32 = ("attention_f32",)
-_UNITS_STREAMS = ("streams", "recurrent")
+_UNITS_LISTED = ("streams",)                   # residual forms of models that list their layers
+_UNITS_OF_KIND = {"wkv": ("recurrent",), "parallel": ("recurrent",), "mamba2": ("recurrent",), "mlstm": ("mlstm",),
+                  "latent_attention": ("latent",)}
 
 
 def units_for(cfg) -> Optional[List[str]]:
@@ -57,7 +59,12 @@ def units_for(cfg) -> Optional[List[str]]:
     them.  Known for models that list their layers."""
     if not cfg.layer_specs or cfg.quant.method != "none":
         return None
-    return sorted(_UNITS_BASE + (_UNITS_F32 if cfg.dtype == "float32" else _UNITS_BF16) + _UNITS_STREAMS)
+    units = set(_UNITS_BASE + (_UNITS_F32 if cfg.dtype == "float32" else _UNITS_BF16) + _UNITS_LISTED)
+    for i, spec in enumerate(cfg.layer_specs):
+        units.update(_UNITS_OF_KIND.get(spec.kind, ()))
+        if cfg.is_moe_layer(i):
+            units.add("moe")
+    return sorted(units)
 
 
 def _sources() -> List[str]:

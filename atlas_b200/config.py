@@ -27,7 +27,7 @@ _FAMILY_ALIASES = {
     "holo3_1_moe": "hybrid",
     "nemotron_h": "hybrid", "nemotron_h_puzzle": "hybrid",
     "deepseek_v2": "moe", "deepseek_v3": "moe", "deepseek_v32": "moe", "kimi_k2": "moe",
-    "papidra": "hybrid",
+    "papidra": "hybrid", "tomizen": "hybrid",
 }
 
 # widths the attention kernels are instantiated for; heads of any other size are zero-padded to the next one
@@ -124,6 +124,7 @@ class ModelConfig:
     attn_output_gate: bool = False    # Qwen3-Next gated attention (q_proj emits q and gate)
     sliding_window: Optional[int] = None
     norm_plus_one: bool = False       # (1 + weight) RMSNorm convention (Qwen3-Next, Gemma)
+    qk_norm_plus_one: Optional[bool] = None   # the same for the q / k head norms (None = as the other norms)
     # MoE
     num_experts: int = 0
     num_experts_per_tok: int = 0
@@ -131,6 +132,7 @@ class ModelConfig:
     shared_expert_intermediate_size: int = 0
     norm_topk_prob: bool = True
     router_scoring: str = "softmax"   # softmax | sigmoid | sqrtsoftplus
+    router_f32: bool = False          # router logits leave their matrix product in fp32
     routed_scaling_factor: float = 1.0
     router_n_group: int = 0           # group-limited routing (DeepSeek-V3): experts split into n_group groups ...
     router_topk_group: int = 0        # ... of which the topk_group best stay eligible
@@ -152,6 +154,8 @@ class ModelConfig:
     layer_specs: List[LayerSpec] = field(default_factory=list)
     # hyper-connections: number of residual streams (0 = one plain residual stream in the activations' dtype)
     residual_streams: int = 0
+    # norms on the sublayers' outputs only: every sublayer reads the (fp32) residual stream itself
+    output_norms: bool = False
     mamba_num_heads: int = 0
     mamba_head_dim: int = 64
     ssm_state_size: int = 128
@@ -162,6 +166,11 @@ class ModelConfig:
     # WKV recurrence (RWKV-style time mixing)
     wkv_num_heads: int = 0
     wkv_head_dim: int = 0
+    # mLSTM (matrix memory with exponential gates)
+    mlstm_num_heads: int = 0
+    mlstm_head_dim: int = 0
+    mlstm_value_dim: int = 0
+    mlstm_gate_cap: float = 0.0       # bound on the raw gates (cap * tanh(. / cap))
     mlp_activation: str = "silu_glu"  # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down) | clamped_glu
     glu_limit: float = 0.0            # clamped_glu: bound on the gate (above) and on the up branch (both sides)
     glu_alpha: float = 1.702          # clamped_glu: slope inside the gate's sigmoid
@@ -169,6 +178,8 @@ class ModelConfig:
     # denominator, the number of rotated dimensions when it is not a fraction of head_dim
     attn_chunk: int = 0
     attn_sinks: bool = False
+    attn_softcap: float = 0.0         # scores become cap * tanh(score / cap) before the softmax (0 = off)
+    attn_head_gate: bool = False      # every head's output times the sigmoid of one number per head
     rotary_dims: Optional[int] = None
     attn_cache_width: int = 0         # padded width of cached heads (0 = head_dim)
     # multi-head latent attention (DeepSeek): 0 = plain GQA.  head_dim is then the padded cache width
@@ -220,7 +231,7 @@ class ModelConfig:
         return dataclasses.replace(self, layer_specs=[], **self.layer_specs[i].overrides)
 
     def layer_kind(self, i: int) -> str:
-        """Mixer kind of layer ``i``: ``attention``, ``gdn``, ``mamba2``, ``wkv``, ``parallel`` or ``none`` (an FFN-only block)."""
+        """Mixer kind of layer ``i``: ``attention``, ``gdn``, ``none`` (an FFN-only block) or one of ``layers.MIXERS``."""
         if self.layer_specs:
             return self.layer_specs[i].kind
         if self.block_types:
@@ -232,6 +243,8 @@ class ModelConfig:
         return "attention" if (i + 1) % self.full_attention_interval == 0 else "gdn"
 
     def is_moe_layer(self, i: int) -> bool:
+        if self.layer_specs:
+            return self.layer_specs[i].has_mlp and self.for_layer(i).num_experts > 0
         if self.block_types:
             return self.block_types[i] == "moe"
         if self.num_experts <= 0 or i in self.mlp_only_layers or i < self.first_k_dense_replace:
@@ -282,7 +295,9 @@ class ModelConfig:
     def _spec_layer_params(self, spec: LayerSpec) -> int:
         """Projection weights of one layer described by a :class:`LayerSpec` (``self`` is the layer's own view)."""
         h = self.hidden_size
-        n = 3 * h * self.intermediate_size if spec.has_mlp else 0
+        n = 3 * h * self.intermediate_size if spec.has_mlp and not self.num_experts else 0
+        if spec.has_mlp and self.num_experts:
+            n += self.num_experts * (h + (2 if self.mlp_activation == "relu2" else 3) * h * self.moe_intermediate_size)
         if spec.kind in ("attention", "parallel"):
             dv = self.v_head_dim or self.head_dim
             n += h * (self.q_size + self.kv_size + self.num_key_value_heads * dv) + self.num_attention_heads * dv * h
@@ -291,6 +306,12 @@ class ModelConfig:
             n += h * (2 * di + 2 * self.mamba_n_groups * self.ssm_state_size + self.mamba_num_heads) + di * h
         if spec.kind == "wkv":
             n += 5 * h * self.wkv_num_heads * self.wkv_head_dim
+        if spec.kind == "mlstm":
+            n += h * self.mlstm_num_heads * (2 * self.mlstm_head_dim + 3 * self.mlstm_value_dim + 2)
+        if spec.kind == "latent_attention":
+            qk, H = self.qk_nope_head_dim + self.qk_rope_head_dim, self.num_attention_heads
+            n += h * (H * qk + self.kv_lora_rank + self.qk_rope_head_dim + H * self.v_head_dim)
+            n += self.kv_lora_rank * H * (self.qk_nope_head_dim + self.v_head_dim)
         return n
 
     # ------------------------------------------------------------------ parsing
@@ -465,8 +486,7 @@ def _rotary_overrides(rot: Optional[Dict[str, Any]]) -> Dict[str, Any]:
 def _attention_overrides(m: Dict[str, Any]) -> Dict[str, Any]:
     d, dv = int(m["dim"]), int(m.get("vdim", m["dim"]))
     return {"num_attention_heads": int(m["heads"]), "num_key_value_heads": int(m["kv_heads"]), "head_dim": d, "v_head_dim": dv,
-            "attn_cache_width": padded_head_width(d, dv), "attn_scale": float(m["scale"]), "attn_sinks": True,
-            "attn_chunk": int((m.get("mask") or {}).get("size", 0)), **_rotary_overrides(m.get("rot"))}
+            "attn_cache_width": padded_head_width(d, dv), "attn_scale": float(m["scale"]), **_rotary_overrides(m.get("rot"))}
 
 
 def _mamba2_overrides(m: Dict[str, Any]) -> Dict[str, Any]:
@@ -481,7 +501,7 @@ def _papidra_layer(lc: Dict[str, Any]) -> LayerSpec:
     if kind == "wkv":
         over.update(wkv_num_heads=int(m["heads"]), wkv_head_dim=int(m["dim"]))
     elif kind == "parallel":
-        over.update(_attention_overrides(m["left"]))
+        over.update(_attention_overrides(m["left"]), attn_sinks=True, attn_chunk=int((m["left"].get("mask") or {}).get("size", 0)))
         over.update(_mamba2_overrides(m["right"]))
     else:
         raise ValueError(f"unsupported Papidra layer type '{kind}'")
@@ -502,16 +522,68 @@ def papidra_config(cfg: Dict[str, Any]) -> ModelConfig:
                     residual_streams=int(cfg["streams"]), tie_word_embeddings=True, layer_specs=specs,
                     mlp_activation="clamped_glu", dtype=str(cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))),
                     quant=QuantConfig(kv_cache_dtype="bf16"), bos_token_id=cfg.get("bos_token_id"), eos_token_id=cfg.get("eos_token_id"))
-    for s in specs:
-        if "num_attention_heads" in s.overrides:            # the model-wide view sizes buffers by the widest heads
+    return _size_by_heads(c)
+
+
+def _size_by_heads(c: ModelConfig) -> ModelConfig:
+    """The model-wide view of a list of layers carries the head sizes of the first attention layer (it sizes buffers)."""
+    for s in c.layer_specs:
+        if "num_attention_heads" in s.overrides:
             for k in ("num_attention_heads", "num_key_value_heads", "head_dim"):
                 setattr(c, k, s.overrides[k])
             break
     return c
 
 
+def _latent_overrides(m: Dict[str, Any]) -> Dict[str, Any]:
+    d, dr, dv = int(m["dim"]), int(m["rot_dim"]), int(m["vdim"])
+    mask = m.get("mask")
+    return {"num_attention_heads": int(m["heads"]), "num_key_value_heads": 1, "head_dim": d + dr, "qk_nope_head_dim": d,
+            "qk_rope_head_dim": dr, "v_head_dim": dv, "kv_lora_rank": int(m["kv_rank"]), "attn_scale": float(m["scale"]),
+            "attn_cache_width": padded_head_width(d + dr, dv), "sliding_window": int(mask["size"]) if mask else None,
+            **_rotary_overrides(m.get("rot"))}
+
+
+def _expert_overrides(mlp: Dict[str, Any]) -> Dict[str, Any]:
+    if mlp.get("kind") != "moe":
+        raise ValueError(f"unsupported Tomizen feed-forward '{mlp.get('kind')}'")
+    r = mlp["router"]
+    return {"num_experts": int(r["experts"]), "num_experts_per_tok": int(r["top"]), "moe_intermediate_size": int(mlp["expert"]["ff"]),
+            "norm_topk_prob": False, "router_scoring": "softmax", "router_f32": True, "mlp_activation": "relu2"}
+
+
+def _tomizen_layer(lc: Dict[str, Any]) -> LayerSpec:
+    kind, m, mlp = str(lc["type"]), lc["mixer"], lc.get("mlp")
+    if kind == "mlstm":
+        over = {"mlstm_num_heads": int(m["heads"]), "mlstm_head_dim": int(m["dim"]), "mlstm_value_dim": int(m["vdim"]),
+                "mlstm_gate_cap": float(m["gate_cap"])}
+    elif kind == "latent_attention":
+        over = _latent_overrides(m)
+    elif kind == "attention":
+        over = _attention_overrides(m)
+        over.update(attn_softcap=float(m["softcap"]), attn_head_gate=True, qk_norm=True, qk_norm_plus_one=False)
+    else:
+        raise ValueError(f"unsupported Tomizen layer type '{kind}'")
+    if mlp is not None:
+        over.update(_expert_overrides(mlp))
+    return LayerSpec(kind, mlp is not None, over)
+
+
+def tomizen_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """Tomizen: mLSTM, latent-attention and soft-capped attention layers with experts, norms on the sublayers' outputs."""
+    specs = [_tomizen_layer(lc) for lc in cfg["layers"]]
+    widest = lambda k: max([s.overrides.get(k, 0) for s in specs] + [0])
+    c = ModelConfig(model_type="tomizen", family="hybrid", vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                    intermediate_size=max(1, widest("moe_intermediate_size")), num_hidden_layers=len(specs), num_attention_heads=1,
+                    num_key_value_heads=1, head_dim=64, rms_norm_eps=float(cfg["norm"]["eps"]), norm_plus_one=True, output_norms=True,
+                    layer_specs=specs, dtype=str(cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))),
+                    quant=QuantConfig(kv_cache_dtype="bf16"), bos_token_id=cfg.get("bos_token_id"), eos_token_id=cfg.get("eos_token_id"))
+    c.moe_intermediate_size = c.intermediate_size
+    return _size_by_heads(c)
+
+
 # ``architecture`` of a config.json that lists its layers one by one -> its reader
-_NATIVE_ARCHITECTURES = {"papidra": papidra_config}
+_NATIVE_ARCHITECTURES = {"papidra": papidra_config, "tomizen": tomizen_config}
 
 
 # ---------------------------------------------------------------------------- presets
@@ -640,12 +712,41 @@ def nemotron_h_8b(quant: str = "none") -> ModelConfig:
                        max_position_embeddings=8192, quant=QuantConfig(method=quant, kv_cache_dtype="fp8"))
 
 
+def _tomizen(vocab: int, width: int, pattern: str, mlstm: tuple, latent: tuple, attn: tuple, experts: tuple, dtype: str) -> ModelConfig:
+    """``pattern``: ``m`` = mLSTM, ``l`` = latent attention, ``a`` = attention; ``mlstm`` (heads, dim, vdim), ``latent`` (heads, dim,
+    rot_dim, vdim, rank, window), ``attn`` (heads, kv heads, dim), ``experts`` (count, top, ff)."""
+    lh, ld, lr, lv, rank, window = latent
+    mixers = {
+        "m": ("mlstm", {"heads": mlstm[0], "dim": mlstm[1], "vdim": mlstm[2], "gate_cap": 15.0}),
+        "l": ("latent_attention", {"heads": lh, "dim": ld, "rot_dim": lr, "vdim": lv, "kv_rank": rank, "scale": (ld + lr) ** -0.5,
+                                   "mask": {"size": window}, "rot": {"base": 5e5, "dims": lr, "scaling": {
+                                       "factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}),
+        "a": ("attention", {"heads": attn[0], "kv_heads": attn[1], "dim": attn[2], "vdim": attn[2], "scale": attn[2] ** -0.5, "softcap": 30.0})}
+    mlp = {"kind": "moe", "expert": {"ff": experts[2]}, "router": {"experts": experts[0], "top": experts[1]}}
+    return tomizen_config({"vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "dtype": dtype,
+                           "layers": [{"type": mixers[ch][0], "mixer": mixers[ch][1], "mlp": mlp} for ch in pattern]})
+
+
+def tiny_tomizen(dtype: str = "float32") -> ModelConfig:
+    c = _tomizen(1024, 192, "mlam", (3, 32, 48), (6, 40, 24, 56, 96, 72), (6, 2, 64), (8, 3, 96), dtype)
+    c.max_position_embeddings = 4096
+    return c
+
+
+def tomizen_16b(quant: str = "none") -> ModelConfig:
+    """Layers of the size of a 16B mixture-of-experts decoder: width 2048, 16 mLSTM heads of 128 / 256, 16 latent heads on rank 512,
+    16 attention heads of 128 (2 kv), 64 experts of 1408 (6 per token)."""
+    c = _tomizen(131072, 2048, "mlam" * 8, (16, 128, 256), (16, 64, 64, 128, 512, 4096), (16, 2, 128), (64, 6, 1408), "bfloat16")
+    c.quant = QuantConfig(method=quant, kv_cache_dtype="bf16")
+    return c
+
+
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "tiny-hybrid": tiny_hybrid,
     "llama3-8b": llama3_8b, "llama3-70b": llama3_70b,
     "qwen3-30b-a3b": qwen3_30b_a3b, "qwen3-next-80b": qwen3_next_80b,
     "tiny-nemotron-h": tiny_nemotron_h, "nemotron-h-8b": nemotron_h_8b, "tiny-deepseek": tiny_deepseek,
-    "tiny-papidra": tiny_papidra, "papidra-8b": papidra_8b,
+    "tiny-papidra": tiny_papidra, "papidra-8b": papidra_8b, "tiny-tomizen": tiny_tomizen, "tomizen-16b": tomizen_16b,
 }
 
 

@@ -20,6 +20,7 @@
 #include "common.cuh"
 #include "host_api.h"
 #include "no_alloc_api.h"
+#include "tc_util.cuh"
 
 namespace atlas {
 
@@ -35,6 +36,7 @@ struct AttnParams {
   int Hq, Hkv, block_size, window;
   int chunk;                                    // > 0: a row sees keys of its own chunk-token block of the sequence only
   const float* sinks;                           // [Hq] or null: exp(sink) joins the softmax denominator
+  float cap_in, cap_out;                        // bounded scores (bf16 cache): see capped_score in tc_util.cuh; cap_out 0 = off
   // decode
   int num_splits;
   float* part_o;                                // [B, Hq, splits, D]
@@ -92,6 +94,10 @@ ATLAS_DEVICE int first_visible(const AttnParams& p, int pos) {
   if (p.chunk > 0) lo = max(lo, pos - pos % p.chunk);
   return lo;
 }
+// q . k of a bf16 cache -> score in the exp2 domain
+ATLAS_DEVICE float score_log2(const AttnParams& p, float s) {
+  return p.cap_out > 0.f ? capped_score(s, p.cap_in, p.cap_out) : s * p.qk_scale_log2;
+}
 // A sink joins the denominator of a row with running maximum m (log2 units) and sum l.  Returns the factor on what was
 // accumulated so far.
 ATLAS_DEVICE float add_sink(float sink, float& m, float& l) {
@@ -133,7 +139,7 @@ paged_attn_kernel(const AttnParams p) {
   q_row0 = p.query_start_loc[b];
   q_len = p.query_start_loc[b + 1] - q_row0;
   // a bf16 cache keeps the query as it is and scales the fp32 scores instead
-  const float q_scale = KV16 ? 1.f : p.qk_scale_log2, s_scale = KV16 ? p.qk_scale_log2 : 1.f;
+  const float q_scale = KV16 ? 1.f : p.qk_scale_log2;
 
   // ---- query fragments (scaled, f16)
   uint32_t qf[KS][4];
@@ -261,7 +267,7 @@ paged_attn_kernel(const AttnParams p) {
         for (int h = 0; h < 2; ++h) {
           const bool ok = tok <= qpos[h] && tok < L && tok >= lo_pos[h];
           float& sv = s[i][2 * h + j];
-          sv = ok ? sv * s_scale : -INFINITY;
+          sv = ok ? (KV16 ? score_log2(p, sv) : sv) : -INFINITY;
           mx[h] = fmaxf(mx[h], sv);
         }
       }
@@ -942,7 +948,7 @@ attn_decode_cp_kernel(const AttnParams p) {
             mma_bf16(s, a1, qb[v4 * 2 + 1][0], qb[v4 * 2 + 1][1]);
           }
 #pragma unroll
-          for (int e = 0; e < 4; ++e) s[e] *= p.qk_scale_log2;
+          for (int e = 0; e < 4; ++e) s[e] = score_log2(p, s[e]);
         } else if constexpr (KV4) {
           const int ta = sub * 16 + tok_r0, tb = sub * 16 + tok_r1;
           const uint8_t* ka = kblk + ta * (D / 2) + c * (DQ / 2);
@@ -1520,7 +1526,7 @@ static int fill_common(AttnParams& p, const void* q, long long ldq, void* out, l
   p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.window = window;
   p.num_splits = 1; p.part_o = nullptr; p.part_ml = nullptr; p.tile_seq = nullptr; p.tile_q0 = nullptr; p.num_tiles = 0;
   p.q_out = nullptr; p.ldqo = 0; p.s_out = nullptr; p.s_ld = 0;
-  p.chunk = 0; p.sinks = nullptr;
+  p.chunk = 0; p.sinks = nullptr; p.cap_in = p.cap_out = 0.f;
   return 0;
 }
 
@@ -1688,18 +1694,20 @@ extern "C" int atlas_attn_prefill_kv4(const void* q, long long ldq, void* out, l
 }
 
 // Same contracts as atlas_attn_decode / atlas_attn_prefill with a bf16 cache (K [nb, Hkv, bs, D], V [nb, Hkv, D, bs]), any
-// number of query heads per kv head, and optional chunked visibility (`chunk` > 0) and softmax sinks (fp32 [Hq]).
+// number of query heads per kv head, and optional chunked visibility (`chunk` > 0), softmax sinks (fp32 [Hq]) and bounded
+// scores (`softcap` > 0: softcap * tanh(score / softcap)).
 extern "C" int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache,
                                       const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                       const int* query_start_loc, int seq_base, int B, float scale, int Hq, int Hkv, int D,
                                       int block_size, int window, int num_splits, float* part_o, float* part_ml, void* stream,
-                                      int chunk, const float* sinks) {
+                                      int chunk, const float* sinks, float softcap) {
   if (B <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, seq_base, scale,
                        1.f, 1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
   p.chunk = chunk; p.sinks = sinks;
+  if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   if (p.num_splits > 1 && (!part_o || !part_ml)) return -3;
   p.part_o = part_o; p.part_ml = part_ml;
@@ -1713,13 +1721,14 @@ extern "C" int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, 
                                        const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                        const int* query_start_loc, const int* tile_seq, const int* tile_q0, int num_tiles,
                                        float scale, int Hq, int Hkv, int D, int block_size, int window, void* stream, int chunk,
-                                       const float* sinks) {
+                                       const float* sinks, float softcap) {
   if (num_tiles <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, 0, scale, 1.f,
                        1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
   p.chunk = chunk; p.sinks = sinks;
+  if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.num_tiles = num_tiles;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (D == 64) return launch_kv16<64>(p, 0, true, st);

@@ -1,9 +1,10 @@
 // 32-bit attention: rotation + paged cache write and attention over an fp32 cache, for models served in float32.
 //
-//   rope_kv_write_f32_kernel  one warp per (token, head of q | k | v): rotates q in place and k on its way into the cache
+//   rope_kv_write_f32_kernel  one warp per (token, head of q | k | v): head norms of q and k, then rotates q in place and k on
+//                             its way into the cache
 //   attn_f32_kernel           one warp per (query row, head), prompt rows and decode rows alike: 32 keys a step, one per
 //                             lane, online softmax, then every lane accumulates its own output dimensions.  Sliding window,
-//                             chunked visibility and softmax sinks as in paged_attn_kernel (attention.cu).
+//                             chunked visibility, softmax sinks and bounded scores as in paged_attn_kernel (attention.cu).
 //
 // Cache layout: K [blocks, Hkv, block_size, D], V [blocks, Hkv, D, block_size].
 #include "common.cuh"
@@ -14,7 +15,8 @@ namespace atlas {
 __global__ void __launch_bounds__(128)
 rope_kv_write_f32_kernel(float* q, long long ldq, const float* __restrict__ k, long long ldk, const float* __restrict__ v, long long ldv,
                          const int* __restrict__ positions, const float* __restrict__ rope, float* k_cache, float* v_cache,
-                         const int* __restrict__ slot_mapping, int T, int Hq, int Hkv, int D, int rotary, int block_size) {
+                         const int* __restrict__ slot_mapping, int T, int Hq, int Hkv, int D, int rotary, int block_size,
+                         const float* __restrict__ q_norm, const float* __restrict__ k_norm, int norm_dim, int plus_one, float eps) {
   extern __shared__ float sm[];                 // [4 warps][D]
   chain_trigger();
   chain_wait();
@@ -30,6 +32,13 @@ rope_kv_write_f32_kernel(float* q, long long ldq, const float* __restrict__ k, l
   if (!is_q && slot < 0) return;
   float* buf = sm + warp * D;
   for (int d = lane; d < D; d += 32) buf[d] = src[d];
+  const float* nw = is_q ? q_norm : (is_k ? k_norm : nullptr);
+  if (nw) {
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) ss += buf[d] * buf[d];
+    const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)norm_dim + eps);
+    for (int d = lane; d < D; d += 32) buf[d] = buf[d] * rstd * (plus_one ? 1.f + nw[d] : nw[d]);
+  }
   __syncwarp();
   const int half = rotary >> 1;
   const float* cs = rope + (long long)positions[t] * rotary;
@@ -53,7 +62,7 @@ struct AttnF32Params {
   const int* seq_lens; const int* query_start_loc;
   const float* sinks;
   int B, T, Hq, Hkv, block_size, window, chunk;
-  float scale;
+  float scale, softcap;
 };
 
 template <int D>
@@ -95,6 +104,7 @@ attn_f32_kernel(const AttnF32Params p) {
         const float4 kv = __ldg(kr + d);
         s += kv.x * sq[warp][d * 4] + kv.y * sq[warp][d * 4 + 1] + kv.z * sq[warp][d * 4 + 2] + kv.w * sq[warp][d * 4 + 3];
       }
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     }
     const float top = fmaxf(m, warp_max(s));
     const float f = m == -INFINITY ? 0.f : expf(m - top);
@@ -121,13 +131,14 @@ using namespace atlas;
 
 extern "C" int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv,
                                        const int* positions, const float* rope, float* k_cache, float* v_cache,
-                                       const int* slot_mapping, int T, int Hq, int Hkv, int D, int rotary, int block_size, void* stream) {
+                                       const int* slot_mapping, int T, int Hq, int Hkv, int D, int rotary, int block_size,
+                                       const float* q_norm, const float* k_norm, int norm_dim, int plus_one, float eps, void* stream) {
   if (T <= 0) return 0;
   if (rotary > D || rotary % 2 || D > 1024) return -1;
   const long long units = (long long)T * (Hq + 2 * Hkv);
   launch_chain_if(T <= 256, rope_kv_write_f32_kernel, dim3((unsigned)((units + 3) / 4)), dim3(128), 4 * D * sizeof(float),
                   reinterpret_cast<cudaStream_t>(stream), q, ldq, k, ldk, v, ldv, positions, rope, k_cache, v_cache, slot_mapping, T, Hq,
-                  Hkv, D, rotary, block_size);
+                  Hkv, D, rotary, block_size, q_norm, k_norm, norm_dim, plus_one, eps);
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }
 
@@ -135,11 +146,11 @@ extern "C" int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, 
 extern "C" int atlas_attn_f32(const float* q, long long ldq, float* out, long long ldo, const float* k_cache, const float* v_cache,
                               const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int B, int T,
                               float scale, int Hq, int Hkv, int D, int block_size, int window, int chunk, const float* sinks,
-                              void* stream) {
+                              float softcap, void* stream) {
   if (T <= 0 || B <= 0) return 0;
   if (Hq % Hkv || block_size < 1) return -1;
   AttnF32Params p = {q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, sinks, B, T, Hq, Hkv,
-                     block_size, window, chunk, scale};
+                     block_size, window, chunk, scale, softcap};
   const dim3 grid((unsigned)(((long long)T * Hq + 3) / 4));
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (D == 64) attn_f32_kernel<64><<<grid, 128, 0, st>>>(p);

@@ -1,5 +1,6 @@
 // Prefill (chunk) attention over the paged bf16 KV cache on the 5th-generation tensor cores: head_dim 64 or 128, 16-token
-// pages, any number of query heads per kv head up to 128, causal with optional chunked visibility and softmax sinks.
+// pages, any number of query heads per kv head up to 128, causal with optional chunked visibility, sliding window, softmax
+// sinks and bounded scores.
 //
 // One CTA per (128-row query tile, kv head); the G query heads that share the kv head are packed into the tile's rows
 // (row = token * G + head; rows past G * floor(128 / G) stay unused).  The cached bytes are MMA operands as they are, so
@@ -30,9 +31,16 @@ struct Tc16Params {
   const int* tile_seq; const int* tile_q0;
   const float* sinks;
   float scale_log2;
-  int Hkv, G, chunk;
+  float cap_in, cap_out;                      // bounded scores (cap_out 0 = off)
+  int Hkv, G, chunk, window;
   status_t* status;
 };
+
+// first position a row at `pos` can see
+ATLAS_DEVICE int first_visible16(const Tc16Params& p, int pos) {
+  const int lo = p.chunk > 0 ? pos - pos % p.chunk : 0;
+  return p.window > 0 ? max(lo, pos - p.window + 1) : lo;
+}
 
 ATLAS_DEVICE void cp16(uint32_t dst, const void* src, bool live) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
@@ -76,7 +84,7 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
   const int ctx0 = L - q_len;
   const int first_pos = ctx0 + q0;
   const int kv_hi = min(L, ctx0 + min(q0 + tpt, q_len));         // causal bound of the tile's last live token
-  const int kv_lo = (p.chunk > 0 ? first_pos - first_pos % p.chunk : 0) / kT16Kv * kT16Kv;
+  const int kv_lo = first_visible16(p, first_pos) / kT16Kv * kT16Kv;
   const int n_kv = (kv_hi - kv_lo + kT16Kv - 1) / kT16Kv;        // at least 1: the tile's first token sees itself
 
   if (threadIdx.x == 0) {
@@ -233,7 +241,9 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
     const int tok = q0 + row / G;
     const bool row_live = row < G * tpt && tok < q_len;
     const int pos = ctx0 + tok;
-    const int lo_pos = p.chunk > 0 ? pos - pos % p.chunk : 0;
+    const int lo_pos = first_visible16(p, pos);
+    const bool capped = p.cap_out > 0.f;
+    const float s_mul = capped ? 1.f : p.scale_log2;
     float m = -INFINITY, l = 0.f;                                 // m: reference point in the exp2 domain
     const int sw = row & 7;
     uint8_t* prow = sP + half * kT16Sub + (row >> 3) * 1024 + sw * 128;
@@ -250,6 +260,12 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[sb]);
+      if (capped) {
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(capped_score(__uint_as_float(sr[c][i]), p.cap_in, p.cap_out));
+      }
       const bool full = __all_sync(0xffffffffu, vis >= col0 + 64 && hid <= col0);
       if (!full) {
 #pragma unroll
@@ -268,7 +284,7 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
       const float mine = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       float theirs;
       if (!exchange(mine, theirs)) { ok = false; break; }
-      const float mx = fmaxf(mine, theirs) * p.scale_log2;       // a positive scale: checked by the host
+      const float mx = fmaxf(mine, theirs) * s_mul;              // a positive scale: checked by the host
       float m_new = m, alpha = 1.f;
       if (mx > m + 8.f) {
         m_new = mx;
@@ -299,7 +315,7 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
           float e[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            e[i] = fast_exp2(fmaf(__uint_as_float(sr[c][q * 8 + i]), p.scale_log2, -mref));
+            e[i] = fast_exp2(fmaf(__uint_as_float(sr[c][q * 8 + i]), s_mul, -mref));
             sum4[i & 3] += e[i];
           }
           uint4 o;
@@ -366,8 +382,8 @@ using namespace atlas;
 extern "C" int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                                        const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc,
                                        const int* tile_seq, const int* tile_q0, int num_tiles, int total_tokens, float scale, int Hq,
-                                       int Hkv, int D, int block_size, int chunk, const float* sinks, unsigned long long* status,
-                                       void* stream) {
+                                       int Hkv, int D, int block_size, int chunk, int window, const float* sinks, float softcap,
+                                       unsigned long long* status, void* stream) {
   if (num_tiles <= 0) return 0;
   if ((D != 64 && D != 128) || block_size != kT16Page || Hq % Hkv || Hq / Hkv > kT16Rows || !(scale > 0.f)) return 1;
   if ((reinterpret_cast<uintptr_t>(q) & 15) || (ldq % 8) || (ldo % 8) || (reinterpret_cast<uintptr_t>(out) & 15)) return 1;
@@ -387,7 +403,9 @@ extern "C" int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, 
   p.k_cache = reinterpret_cast<const __nv_bfloat16*>(k_cache); p.v_cache = reinterpret_cast<const __nv_bfloat16*>(v_cache);
   p.block_tables = block_tables; p.bt_ld = bt_ld; p.seq_lens = seq_lens; p.query_start_loc = query_start_loc;
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f;
-  p.Hkv = Hkv; p.G = G; p.chunk = chunk; p.status = status;
+  p.Hkv = Hkv; p.G = G; p.chunk = chunk; p.window = window; p.status = status;
+  p.cap_in = p.cap_out = 0.f;
+  if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return D == 64 ? launch_tc16<64>(tq, p, num_tiles, st) : launch_tc16<128>(tq, p, num_tiles, st);
 }

@@ -212,6 +212,7 @@ struct RopeKvParams {
   void* k_cache; void* v_cache;
   const int* slot_mapping;
   int T, Hq, Hkv, D, rotary_dim, block_size, kv_fp8, plus_one;
+  int norm_dim;            // channels a head norm counts (D, or less for zero-padded heads)
   int v_separate;          // V rows are written by v_write_pages_kernel (prefill-size batches), not here
   int rotate;              // Walsh-Hadamard rotation of every q / k / v head before the write (head_dim-128 kernel only)
   float eps, inv_k_scale, inv_v_scale;
@@ -246,7 +247,7 @@ rope_kv_write_kernel(const RopeKvParams p) {
   const __nv_bfloat16* nw = is_q ? p.q_norm_w : (is_k ? p.k_norm_w : nullptr);
   if (nw) {
     ss = warp_sum(ss);
-    const float rstd = rsqrtf(ss / (float)D + p.eps);
+    const float rstd = rsqrtf(ss / (float)p.norm_dim + p.eps);
     for (int e = lane * 2; e < D; e += 64) {
       float2 wv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(nw + e));
       if (p.plus_one) { wv.x += 1.f; wv.y += 1.f; }
@@ -723,7 +724,7 @@ extern "C" int atlas_rope_kv_write(void* q, long long ldq, const void* k, long l
                                    const int* positions, const float* rope, const void* q_norm_w,
                                    const void* k_norm_w, void* k_cache, void* v_cache, const int* slot_mapping, int T,
                                    int Hq, int Hkv, int D, int rotary_dim, int block_size, int kv_fp8, int plus_one,
-                                   float eps, float k_scale, float v_scale, void* stream) {
+                                   float eps, float k_scale, float v_scale, void* stream, int norm_dim) {
   if (T <= 0) return 0;
   if (D % 64 || D > 512 || rotary_dim > D || rotary_dim % 2) return -1;
   RopeKvParams p;
@@ -735,6 +736,7 @@ extern "C" int atlas_rope_kv_write(void* q, long long ldq, const void* k, long l
   p.k_norm_w = reinterpret_cast<const __nv_bfloat16*>(k_norm_w);
   p.k_cache = k_cache; p.v_cache = v_cache; p.slot_mapping = slot_mapping;
   p.T = T; p.Hq = Hq; p.Hkv = Hkv; p.D = D; p.rotary_dim = rotary_dim; p.block_size = block_size;
+  p.norm_dim = norm_dim > 0 ? norm_dim : D;
   p.rotate = (kv_fp8 & 8) ? 1 : 0;           // bit 3 of the cache mode asks for the Hadamard rotation
   kv_fp8 &= 7;
   p.kv_fp8 = kv_fp8; p.plus_one = plus_one; p.eps = eps; p.inv_k_scale = 1.f / k_scale; p.inv_v_scale = 1.f / v_scale;
@@ -743,7 +745,7 @@ extern "C" int atlas_rope_kv_write(void* q, long long ldq, const void* k, long l
                   (reinterpret_cast<uintptr_t>(v) & 7) == 0) ? 1 : 0;
   const long long units = (long long)T * (Hq + (p.v_separate ? 1 : 2) * Hkv);
   const int grid = (int)((units + 3) / 4);
-  const bool d128 = D == 128 && rotary_dim == 128 && (ldq % 4) == 0 && (ldk % 4) == 0 && (ldv % 4) == 0 &&
+  const bool d128 = D == 128 && rotary_dim == 128 && p.norm_dim == D && (ldq % 4) == 0 && (ldk % 4) == 0 && (ldv % 4) == 0 &&
                     ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 7) == 0 &&
                     (reinterpret_cast<uintptr_t>(rope) & 15) == 0;
   if (p.rotate && !d128) return -2;                                   // so is the rotation

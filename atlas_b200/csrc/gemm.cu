@@ -69,6 +69,9 @@ struct GemmParams {
   int m_tiles, n_tiles;
   int b_scale_ld;           // k-groups per row of b_scale
   int vec_ok;               // 16-byte stores into C are legal
+  // bf16 kernels: columns from tail_col on are stored as fp32 in `tail` [M, N - tail_col] (null = off); relu2 squares the
+  // positive part of every value before the store
+  float* tail; long long tail_ld; int tail_col, tail_vec, relu2;
   int cluster_splits;       // > 1: the K splits of a tile are the CTAs of one thread-block cluster (one item per CTA, a
                             // single m-tile): partials meet in distributed shared memory instead of the workspace and
                             // every CTA finishes 128 / cluster_splits rows of the tile (see cluster_tail)
@@ -1008,9 +1011,31 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
       } else
       if (store_now && m < M_rows) {
         __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)m * p.ldc;
+        if (!FP8 && p.relu2) {
+#pragma unroll
+          for (int i = 0; i < HALF; ++i) {
+            const float r = fmaxf(acc[i], 0.f);
+            acc[i] = r * r;
+          }
+        }
 #pragma unroll
         for (int j = 0; j < HALF; j += 8) {
           const int n = n_base + j;
+          if (!FP8 && p.tail != nullptr && n + 8 > p.tail_col) {
+            float* trow = p.tail + (size_t)m * p.tail_ld - p.tail_col;
+            if (p.tail_vec && n >= p.tail_col && n + 8 <= p.N) {
+              *reinterpret_cast<float4*>(trow + n) = make_float4(acc[j], acc[j + 1], acc[j + 2], acc[j + 3]);
+              *reinterpret_cast<float4*>(trow + n + 4) = make_float4(acc[j + 4], acc[j + 5], acc[j + 6], acc[j + 7]);
+            } else {
+#pragma unroll
+              for (int i = 0; i < 8; ++i) {
+                if (n + i >= p.N) continue;
+                if (n + i >= p.tail_col) trow[n + i] = acc[j + i];
+                else crow[n + i] = __float2bfloat16_rn(acc[j + i]);
+              }
+            }
+            continue;
+          }
           if (p.vec_ok && n + 8 <= p.N) {
             uint4 v;
             v.x = pack_bf16x2(acc[j + 0], acc[j + 1]);
@@ -1257,7 +1282,8 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
                      long long sa_k, const float* b_scale, int b_scale_ld, int M, int N, int K, long long lda,
                      long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters,
                      int num_sms, unsigned long long* status, void* stream, const uint32_t* a_ready,
-                     const unsigned int* a_ready_epoch, long long max_cycles, const AtlasEpilogue* epi = nullptr) {
+                     const unsigned int* a_ready_epoch, long long max_cycles, const AtlasEpilogue* epi = nullptr,
+                     float* tail = nullptr, long long tail_ld = 0, int tail_col = 0) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const uint32_t esize = kind == 1 ? 1 : 2;
   const int elems_per_row = 128 / esize;
@@ -1289,6 +1315,8 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
   p.C = C; p.a_scale = a_scale; p.b_scale = b_scale; p.workspace = workspace; p.counters = counters;
   p.status = status; p.ldc = ldc; p.sa_k = sa_k; p.M = M; p.N = N; p.K = K;
   p.epi_mode = epi_mode;
+  p.tail = tail; p.tail_ld = tail_ld; p.tail_col = tail_col;
+  p.tail_vec = tail_col % 4 == 0 && tail_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(tail) & 15) == 0 ? 1 : 0;
   if (epi) {
     p.act_cols = N / 2; p.q_out = reinterpret_cast<uint8_t*>(epi->q_out); p.ldq = epi->ldq; p.s_out = epi->s_out; p.s_ld = epi->s_ld;
     p.residual = reinterpret_cast<__nv_bfloat16*>(epi->residual); p.ldr = epi->ldr;
@@ -1321,7 +1349,7 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
   // and meet in distributed shared memory (cluster_tail) instead of in the global workspace.
   p.cluster_splits = 1;
   if (cluster_splitk_enabled() && p.m_tiles == 1 && block_n == 128 && (p.splits == 2 || p.splits == 4) && items <= num_sms &&
-      (epi_mode == 2 || (epi_mode == 0 && p.vec_ok)) && (N % 128) == 0 && a_ready == nullptr)
+      (epi_mode == 2 || (epi_mode == 0 && p.vec_ok && tail == nullptr)) && (N % 128) == 0 && a_ready == nullptr)
     p.cluster_splits = p.splits;
   p.prefetch_b = p.m_tiles <= 2 ? prefetch_depth() : 0;      // weights read once from HBM: run ahead of the ring in L2
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
@@ -1342,6 +1370,15 @@ extern "C" int atlas_gemm(int kind, const void* A, const void* B, void* C, const
                           int num_sms, unsigned long long* status, void* stream) {
   return gemm_impl(kind, A, B, C, a_scale, sa_m, sa_k, b_scale, b_scale_ld, M, N, K, lda, ldb, ldc, block_n, splits, workspace,
                    counters, num_sms, status, stream, nullptr, nullptr, 0);
+}
+
+// bf16 GEMM in two parts: columns [0, n_main) of the product to C as bf16, the others to `tail` [M, N - n_main] as fp32.
+extern "C" int atlas_gemm_tail(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, int M, int N, int K,
+                               long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters,
+                               int num_sms, unsigned long long* status, void* stream) {
+  if (n_main < 0 || n_main > N || (n_main > 0 && !C) || (n_main < N && (!tail || tail_ld < N - n_main))) return -45;
+  return gemm_impl(0, A, B, C, nullptr, 0, 0, nullptr, 0, M, N, K, lda, ldb, ldc, block_n, splits, workspace, counters, num_sms, status,
+                   stream, nullptr, nullptr, 0, nullptr, n_main < N ? tail : nullptr, tail_ld, n_main);
 }
 
 // All-gather -> GEMM: the rows of A (and their scales) are written into this rank's memory by the ranks that own them;
@@ -1376,7 +1413,8 @@ extern "C" int atlas_gemm_fused(int kind, const void* A, const void* B, void* C,
 extern "C" int atlas_gemm_grouped(int kind, const void* A, const void* B, void* C, const float* a_scale, long long sa_k,
                                   const float* b_scale, int max_rows, int N, int K, int E, long long lda, long long ldb,
                                   long long ldc, int block_n, const int* tile_expert, const int* num_m_tiles,
-                                  int num_sms, unsigned long long* status, void* stream) {
+                                  int num_sms, unsigned long long* status, void* stream, int relu2) {
+  if (relu2 && kind != 0) return -11;
   if (max_rows <= 0 || N <= 0 || K <= 0 || E <= 0) return 0;
   if (max_rows % kBlockM) return -9;
   const uint32_t esize = kind == 1 ? 1 : 2;
@@ -1402,6 +1440,7 @@ extern "C" int atlas_gemm_grouped(int kind, const void* A, const void* B, void* 
   p.n_tiles = N / block_n;
   p.b_scale_ld = p.k_blocks;
   p.vec_ok = ((ldc % 8) == 0 && (reinterpret_cast<uintptr_t>(C) & 15) == 0) ? 1 : 0;
+  p.relu2 = relu2;
   p.tile_expert = tile_expert; p.num_m_tiles_ptr = num_m_tiles; p.expert_n = N;
   p.ar_state = nullptr; p.ar_world = 1; p.ar_rank = 0; p.ar_mode = 0; p.ar_parity_stride = 0; p.prefetch_b = 0;
   p.rs_tiles_per_rank = 1; p.a_ready = nullptr; p.a_ready_epoch = nullptr; p.ar_max_cycles = kMbarMaxCycles;

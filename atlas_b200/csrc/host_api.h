@@ -52,7 +52,7 @@ int atlas_rope_kv_write(void* q, long long ldq, const void* k, long long ldk, co
                         const int* positions, const float* rope, const void* q_norm_w, const void* k_norm_w,
                         void* k_cache, void* v_cache, const int* slot_mapping, int T, int Hq, int Hkv, int D,
                         int rotary_dim, int block_size, int kv_fp8, int plus_one, float eps, float k_scale,
-                        float v_scale, void* stream);
+                        float v_scale, void* stream, int norm_dim);
 int atlas_wht_d128(void* x, long long ld, int T, int H, void* stream);
 int atlas_gated_rmsnorm(const void* x, long long ldx, const void* z, long long ldz, const void* w, void* y,
                         long long ldy, int T, int H, int D, float eps, void* stream);
@@ -87,7 +87,14 @@ int atlas_gemm_w4a16_grouped(const void* A, const void* packed, const void* bsca
 int atlas_gemm_grouped(int kind, const void* A, const void* B, void* C, const float* a_scale, long long sa_k,
                        const float* b_scale, int max_rows, int N, int K, int E, long long lda, long long ldb,
                        long long ldc, int block_n, const int* tile_expert, const int* num_m_tiles, int num_sms,
-                       unsigned long long* status, void* stream);
+                       unsigned long long* status, void* stream, int relu2);
+int atlas_gemm_tail(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, int M, int N, int K, long long lda,
+                    long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,
+                    unsigned long long* status, void* stream);
+int atlas_moe_plain_gemm(const void* x, long long ldx, const void* w, const int* row_token, const int* tile_expert, const int* num_tiles,
+                         int max_rows, int gather, int relu2, int N, int K, void* y, long long ldy, int f32, void* stream);
+int atlas_moe_plain_combine(const void* y, long long ldy, const int* slot_of, const float* topk_w, int T, int k, int H, void* out,
+                            long long ldo, int f32, void* stream);
 
 // ---- Gated DeltaNet (gdn.cu)
 int atlas_gdn_conv(const void* x, long long ldx, const void* w, int C, int W, const void* conv_state,
@@ -134,24 +141,26 @@ int atlas_attn_prefill(const void* q, long long ldq, void* out, long long ldo, c
 int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                            const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int seq_base, int B,
                            float scale, int Hq, int Hkv, int D, int block_size, int window, int num_splits, float* part_o,
-                           float* part_ml, void* stream, int chunk, const float* sinks);
+                           float* part_ml, void* stream, int chunk, const float* sinks, float softcap);
 int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                             const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
                             const int* tile_q0, int num_tiles, float scale, int Hq, int Hkv, int D, int block_size, int window,
-                            void* stream, int chunk, const float* sinks);
+                            void* stream, int chunk, const float* sinks, float softcap);
 
 int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                             const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
                             const int* tile_q0, int num_tiles, int total_tokens, float scale, int Hq, int Hkv, int D, int block_size,
-                            int chunk, const float* sinks, unsigned long long* status, void* stream);
+                            int chunk, int window, const float* sinks, float softcap, unsigned long long* status, void* stream);
 
 // ---- 32-bit attention (attention_f32.cu)
 int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const int* positions,
                             const float* rope, float* k_cache, float* v_cache, const int* slot_mapping, int T, int Hq, int Hkv, int D,
-                            int rotary, int block_size, void* stream);
+                            int rotary, int block_size, const float* q_norm, const float* k_norm, int norm_dim, int plus_one, float eps,
+                            void* stream);
 int atlas_attn_f32(const float* q, long long ldq, float* out, long long ldo, const float* k_cache, const float* v_cache,
                    const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int B, int T, float scale, int Hq,
-                   int Hkv, int D, int block_size, int window, int chunk, const float* sinks, void* stream);
+                   int Hkv, int D, int block_size, int window, int chunk, const float* sinks, float softcap,
+                   void* stream);
 
 // ---- residual streams, token shift, clamped gated unit (streams.cu); f32 = activations are fp32 instead of bf16
 int atlas_hyper_norm(float* x, int rows, int S, int W, const void* y, long long ldy, const void* y2, long long ldy2, const float* w1,
@@ -173,7 +182,43 @@ int atlas_wkv_scan(const void* r, long long ldr, const void* k, long long ldk, c
                    const int* qsl, const int* slots, const unsigned char* has, const int* limit, const int* snap_rows,
                    const int* snap_slots, int snaps, int B, int H, int D, int commit, int one_row, int f32, void* stream);
 int atlas_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
-                          int groups, int gsize, float eps, int gate_first, int f32, void* stream);
+                          int groups, int gsize, float eps, int gate_first, int sigmoid, const float* den, int f32, void* stream);
+int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const float* w,
+                     const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store, float eps, int f32, void* stream);
+int atlas_head_gate(void* x, long long ldx, const float* g, long long ldg, int rows, int H, int D, int f32, void* stream);
+
+// ---- mLSTM (mlstm.cu)
+int atlas_mlstm_gates(const float* raw, long long ld, const float* bias, float cap, float* m, float* la, float* lb, float* top, const int* qsl,
+                      const int* slots, const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B,
+                      int H, int commit, void* stream);
+int atlas_mlstm_scan(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const float* la, const float* lb,
+                     const float* top, float q_scale, float* h, void* out, long long ldo, float* den, const int* qsl, const int* slots,
+                     const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B, int H, int V,
+                     int D, int commit, int one_row, int f32, void* stream);
+int atlas_mlstm_chunk(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const float* la, const float* lb,
+                      const float* top, float scale, float* h, void* out, long long ldo, float* den, const int* qsl, const int* slots,
+                      const unsigned char* has, const int* snap_rows, const int* snap_slots, int snaps, int B, int H, int V, int D, int commit,
+                      void* stream);
+
+// ---- latent attention (latent.cu)
+int atlas_latent_rows(const void* q, long long ldq, const float* ckv, long long ldc, const float* norm_w, const int* positions, const float* rope,
+                      const int* slot_mapping, const int* row_map, void* cache, void* qa, void* qx, int rows, int H, int nope, int rope_dim,
+                      int rotary, int rank, int rp, int ep, int dx, float eps, int f32, void* stream);
+int atlas_head_gemm(const void* in, long long in_row, int in_head, const void* w, void* out, long long out_row, int out_head, const int* in_rows,
+                    const int* out_rows, int rows, int H, int N, int K, void* stream);
+int atlas_latent_attn(const void* q, const void* cache, void* out, float* part_o, float* part_ml, const int* block_tables, int bt_ld,
+                      const int* seq_lens, const int* query_start_loc, const int* row_start, const int* tile_seq, const int* tile_r0, int tiles,
+                      int B, int rows, int H, int rp, int ep, int block_size, int window, int splits, int mt, float scale, void* stream);
+int atlas_latent_attn_f32(const float* q, const float* cache, float* out, const int* block_tables, int bt_ld, const int* seq_lens,
+                          const int* query_start_loc, int B, int T, int H, int rp, int ep, int block_size, int window, float scale, void* stream);
+int atlas_latent_gather(const void* cache, const int* block_tables, int bt_ld, const int* seq_lens, const int* page_seq, const int* page_idx,
+                        int pages, int block_size, int rp, int W, void* out, void* stream);
+int atlas_latent_pages(const void* kv, const void* cache, const int* block_tables, int bt_ld, const int* seq_lens, const int* page_seq,
+                       const int* page_idx, int pages, int block_size, int H, int nope, int rope, int vd, int rp, int W, int dx, void* k_pages,
+                       void* v_pages, void* stream);
+int atlas_latent_unpad(const void* in, const int* rows, int n, int H, int vd, int dx, void* out, void* stream);
+
+// ---- recurrences (recurrent.cu), continued
 int atlas_conv1d_bias_silu(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                            const int* seq_of_token, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
                            int rows, int f32, void* stream);

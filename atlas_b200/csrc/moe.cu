@@ -4,6 +4,8 @@
 //                       m-tile -> expert worklist and the live tile count (all on device: graph-capturable)
 //   moe_gather_kernel   expert-sorted activation rows (bf16 copy, or FP8 + k-group-major scales)
 //   moe_combine_kernel  out[t] = sum_j w[t,j] * y[slot(t,j)]  (+ optional addend, e.g. shared expert / residual)
+//   moe_plain_gemm_kernel  the grouped product on the CUDA cores, fp32 sums, any sizes: fp32 models, and bf16 shapes that the
+//                       tensor-core tiles do not take
 // Reference ops replaced: kernels/gb10/common/{moe_topk,moe_topk_sigmoid,moe_permute}.cu
 // (moe_count_experts, moe_sort_by_expert, moe_permute_tokens, moe_build_tile_worklist, moe_unpermute_reduce).
 #include "common.cuh"
@@ -28,10 +30,13 @@ struct RouteOpts {
   float out_scale;
 };
 
-__device__ __forceinline__ float route_score(float x, float mx, int mode) {
-  if (mode == 1) return 1.f / (1.f + __expf(-x));
-  if (mode == 2) return sqrtf(x > 20.f ? x : log1pf(__expf(x)));
-  return __expf(x - mx);
+__device__ __forceinline__ float route_exp(float x, const __nv_bfloat16*) { return __expf(x); }
+__device__ __forceinline__ float route_exp(float x, const float*) { return expf(x); }       // 32-bit logits keep 32-bit scores
+template <typename T>
+__device__ __forceinline__ float route_score(float x, float mx, int mode, const T* kind) {
+  if (mode == 1) return 1.f / (1.f + route_exp(-x, kind));
+  if (mode == 2) return sqrtf(x > 20.f ? x : log1pf(route_exp(x, kind)));
+  return route_exp(x - mx, kind);
 }
 
 // one warp per token; E <= 1024
@@ -58,7 +63,7 @@ moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int 
 #pragma unroll
   for (int i = 0; i < kMaxPer; ++i) {
     if (i < per && v[i] > -INFINITY) {
-      v[i] = route_score(v[i], mx, o.score_mode);
+      v[i] = route_score(v[i], mx, o.score_mode, logits);
       sum += o.score_mode == 0 ? v[i] : 0.f;
     }
   }
@@ -76,7 +81,7 @@ moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int 
     const int tok = o.token_ids[t];
     int my_e = lane < k ? o.hash_table[(long long)tok * k + lane] : 0;
     my_e = min(max(my_e, 0), E - 1);
-    const float my_w = lane < k ? route_score((float)logits[t * ld + my_e], mx, o.score_mode) * inv : 0.f;
+    const float my_w = lane < k ? route_score((float)logits[t * ld + my_e], mx, o.score_mode, logits) * inv : 0.f;
     float wsum = warp_sum(lane < k ? my_w : 0.f);
     if (lane < k) {
       w_out[(long long)t * k + lane] = (norm ? my_w / (wsum + 1e-20f) : my_w) * o.out_scale;
@@ -290,6 +295,66 @@ moe_combine_kernel(const __nv_bfloat16* __restrict__ y, long long ldy, const int
   *reinterpret_cast<uint4*>(out + (long long)t * ldo + e) = o;
 }
 
+// y[r, n] = act(sum_k x[src(r), k] w[e, n, k]) for the live rows r of the expert-sorted buffer; src(r) = row_token[r] with `gather`, r
+// otherwise.  32 rows x 64 columns per CTA, four 32-row blocks per 128-row tile.
+constexpr int kPgRows = 32, kPgCols = 64, kPgK = 32;
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_plain_gemm_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const int* __restrict__ row_token,
+                      const int* __restrict__ tile_expert, const int* __restrict__ num_tiles, int gather, int relu2, int N, int K, T* y,
+                      long long ldy) {
+  __shared__ float xs[kPgRows][kPgK + 1], ws[kPgCols][kPgK + 1];
+  const int tile = blockIdx.y >> 2, r0 = tile * 128 + (blockIdx.y & 3) * kPgRows, n0 = blockIdx.x * kPgCols;
+  if (tile >= *num_tiles) return;
+  if (row_token[r0] < 0) return;               // live rows are the leading ones of a tile
+  const T* we = w + (long long)tile_expert[tile] * N * K;
+  const int tid = threadIdx.x, c = tid & 63, rg = tid >> 6;      // column, rows rg, rg + 4, ..
+  float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  for (int k0 = 0; k0 < K; k0 += kPgK) {
+    for (int i = tid; i < kPgRows * kPgK; i += 256) {
+      const int r = i / kPgK, k = i % kPgK, tok = row_token[r0 + r];
+      xs[r][k] = tok >= 0 && k0 + k < K ? (float)x[(gather ? (long long)tok : (long long)(r0 + r)) * ldx + k0 + k] : 0.f;
+    }
+    for (int i = tid; i < kPgCols * kPgK; i += 256) {
+      const int n = i / kPgK, k = i % kPgK;
+      ws[n][k] = n0 + n < N && k0 + k < K ? (float)we[(long long)(n0 + n) * K + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int k = 0; k < kPgK; ++k) {
+      const float wv = ws[c][k];
+#pragma unroll
+      for (int i = 0; i < 8; ++i) acc[i] = fmaf(xs[rg + 4 * i][k], wv, acc[i]);
+    }
+    __syncthreads();
+  }
+  if (n0 + c >= N) return;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int r = r0 + rg + 4 * i;
+    if (row_token[r] < 0) continue;
+    float v = acc[i];
+    if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+    y[(long long)r * ldy + n0 + c] = (T)v;
+  }
+}
+
+// out[t] = sum_j w[t, j] y[slot(t, j)], any width
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_plain_combine_kernel(const T* __restrict__ y, long long ldy, const int* __restrict__ slot_of, const float* __restrict__ topk_w, int k, int H,
+                         T* out, long long ldo) {
+  const long long t = blockIdx.x;
+  for (int e = threadIdx.x; e < H; e += 256) {
+    float acc = 0.f;
+    for (int j = 0; j < k; ++j) {
+      const int s = slot_of[t * k + j];
+      if (s >= 0) acc = fmaf(topk_w[t * k + j], (float)y[s * ldy + e], acc);
+    }
+    out[t * ldo + e] = (T)acc;
+  }
+}
+
 // ---------------------------------------------------------------------------- expert-parallel dispatch
 // Rank r owns experts [r * experts_per_rank, (r + 1) * experts_per_rank).  One block: histogram of destination ranks
 // over all (token, k) pairs, prefix sums -> send_off[world + 1], and the position of every pair inside its
@@ -400,6 +465,33 @@ extern "C" int atlas_moe_combine(const void* y, long long ldy, const int* slot_o
   moe_combine_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
       reinterpret_cast<const __nv_bfloat16*>(y), ldy, slot_of, topk_w, k, H, reinterpret_cast<const __nv_bfloat16*>(addend),
       ld_add, reinterpret_cast<__nv_bfloat16*>(out), ldo);
+  return cudaGetLastError() == cudaSuccess ? 0 : -20;
+}
+
+// Grouped product on the CUDA cores (see moe_plain_gemm_kernel): rows sorted by moe_align, w [E, N, K]
+extern "C" int atlas_moe_plain_gemm(const void* x, long long ldx, const void* w, const int* row_token, const int* tile_expert,
+                                    const int* num_tiles, int max_rows, int gather, int relu2, int N, int K, void* y, long long ldy, int f32,
+                                    void* stream) {
+  if (max_rows <= 0) return 0;
+  if (max_rows % 128 || N < 1 || K < 1 || max_rows / 32 > 65535) return -1;
+  dim3 grid((N + kPgCols - 1) / kPgCols, max_rows / 32);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) moe_plain_gemm_kernel<float><<<grid, 256, 0, st>>>(reinterpret_cast<const float*>(x), ldx, reinterpret_cast<const float*>(w), row_token,
+                                                               tile_expert, num_tiles, gather, relu2, N, K, reinterpret_cast<float*>(y), ldy);
+  else moe_plain_gemm_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx,
+                                                                  reinterpret_cast<const __nv_bfloat16*>(w), row_token, tile_expert, num_tiles,
+                                                                  gather, relu2, N, K, reinterpret_cast<__nv_bfloat16*>(y), ldy);
+  return cudaGetLastError() == cudaSuccess ? 0 : -20;
+}
+
+extern "C" int atlas_moe_plain_combine(const void* y, long long ldy, const int* slot_of, const float* topk_w, int T, int k, int H, void* out,
+                                       long long ldo, int f32, void* stream) {
+  if (T <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) moe_plain_combine_kernel<float><<<T, 256, 0, st>>>(reinterpret_cast<const float*>(y), ldy, slot_of, topk_w, k, H,
+                                                              reinterpret_cast<float*>(out), ldo);
+  else moe_plain_combine_kernel<__nv_bfloat16><<<T, 256, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(y), ldy, slot_of, topk_w, k, H,
+                                                                  reinterpret_cast<__nv_bfloat16*>(out), ldo);
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }
 

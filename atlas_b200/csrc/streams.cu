@@ -8,6 +8,11 @@
 //                           each; at the start of the model the streams are set to the scaled embedding instead.
 //   token_shift_mix_kernel  out[s] = x + (x_prev - x) * mu[s] for S mixes, x_prev = the previous token's row (from the
 //                           sequence's state slot for the first row of a chunk, zeros at the start of a sequence)
+//   group_norm_gate_kernel  rms norm over channel groups joined with a gate: norm(y * silu(z)) * w (Mamba-2),
+//                           norm(y) * w * silu(z) (WKV) or norm(y / den) * w * sigmoid(z) (mLSTM)
+//   add_normed_kernel       one CTA per token: x += rmsnorm(y) * w on an fp32 residual, y being a sublayer's output or the weighted
+//                           sum of expert rows; hands the new x on in the activations' dtype, normed again where asked
+//   head_gate_kernel        x[t, h, :] *= sigmoid(g[t, h])
 //   clamped_glu_kernel      g = min(gate, limit), u = clamp(up, +-limit):  g * sigmoid(alpha g) * (u + 1)
 //
 // Every kernel exists for bf16 and fp32 activations (template parameter T).
@@ -221,6 +226,224 @@ static int launch_shift(const void* x, long long ldx, const float* mu, const voi
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
+// ----------------------------------------------------------------------------- gated group norm
+// TPG threads per (row, group): a quarter of a warp for head-sized groups, a warp, or a whole block for wide ones
+// kGate: 0 silu before the norm, 1 silu after it, 2 sigmoid after it.  `den` [rows, groups] (may be null): divisor of the group.
+enum { kSiluFirst = 0, kSiluAfter = 1, kSigmoidAfter = 2 };
+template <typename T, int TPG, int V, int kGate>
+__global__ void __launch_bounds__(256)
+group_norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ z, long long ldz,
+                       const float* __restrict__ w, T* out, long long ldo, int rows, int groups, int gsize, float eps,
+                       const float* __restrict__ den) {
+  constexpr bool kGateFirst = kGate == kSiluFirst;
+  __shared__ float red[8];
+  chain_trigger();
+  chain_wait();
+  const long long unit = (long long)blockIdx.x * (256 / TPG) + threadIdx.x / TPG;
+  const bool live = unit < (long long)rows * groups;            // every lane stays for the warp's sums
+  const int tid = threadIdx.x % TPG;
+  const long long t = live ? unit / groups : 0;
+  const int g0 = (int)(unit % groups) * gsize;
+  const T* yr = y + t * ldy + g0;
+  const T* zr = z + t * ldz + g0;
+  const float inv = den && live ? 1.f / den[unit] : 1.f;
+  float ss = 0.f;
+  for (int e = tid * V; e < gsize; e += TPG * V) {
+    float f[V], g[V];
+    load_vec<V>(yr + e, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] *= inv;
+    if (kGateFirst) {
+      load_vec<V>(zr + e, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) f[i] *= g[i] / (1.f + expf(-g[i]));
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += f[i] * f[i];
+  }
+#pragma unroll
+  for (int off = (TPG < 32 ? TPG : 32) / 2; off > 0; off >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, off);
+  if (TPG > 32) {
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ss += red[i];
+  }
+  if (!live) return;
+  const float rstd = inv / sqrtf(ss / (float)gsize + eps);
+  for (int e = tid * V; e < gsize; e += TPG * V) {
+    float f[V], g[V], wv[V];
+    load_vec<V>(yr + e, f);
+    load_vec<V>(zr + e, g);
+#pragma unroll
+    for (int i = 0; i < V; ++i) wv[i] = w[g0 + e + i];
+#pragma unroll
+    for (int i = 0; i < V; ++i) f[i] = f[i] * rstd * wv[i] * ((kGate == kSigmoidAfter ? 1.f : g[i]) / (1.f + expf(-g[i])));
+    store_vec<V>(out + t * ldo + g0 + e, f);
+  }
+}
+
+template <typename T, int V, int kGate>
+static int launch_gnorm(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo,
+                        int rows, int groups, int gsize, float eps, const float* den, cudaStream_t st) {
+  const long long units = (long long)rows * groups;
+  const T *yp = reinterpret_cast<const T*>(y), *zp = reinterpret_cast<const T*>(z);
+  if (gsize >= 1024)
+    launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 256, V, kGate>, dim3((unsigned)units), dim3(256), 0, st, yp, ldy, zp, ldz, w,
+                    reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps, den);
+  else if (gsize <= 128)
+    launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 8, V, kGate>, dim3((unsigned)((units + 31) / 32)), dim3(256), 0, st, yp, ldy,
+                    zp, ldz, w, reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps, den);
+  else
+    launch_chain_if(rows <= 256, group_norm_gate_kernel<T, 32, V, kGate>, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, st, yp, ldy,
+                    zp, ldz, w, reinterpret_cast<T*>(out), ldo, rows, groups, gsize, eps, den);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+template <typename T, int V>
+static int launch_gnorm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
+                             int groups, int gsize, float eps, int kind, const float* den, cudaStream_t st) {
+  if (kind == kSiluFirst) return launch_gnorm<T, V, kSiluFirst>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, den, st);
+  if (kind == kSiluAfter) return launch_gnorm<T, V, kSiluAfter>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, den, st);
+  return launch_gnorm<T, V, kSigmoidAfter>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, den, st);
+}
+
+template <typename T>
+static int gnorm(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
+                 int groups, int gsize, float eps, int kind, const float* den, cudaStream_t st) {
+  if (sizeof(T) == 2 && gsize % 8 == 0 && (gsize < 1024 || gsize >= 2048) && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(z, ldz) && vec_ok<T, 8>(out, ldo))
+    return launch_gnorm_gate<T, 8>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st);
+  const bool vec = gsize % 4 == 0 && vec_ok<T, 4>(y, ldy) && vec_ok<T, 4>(z, ldz) && vec_ok<T, 4>(out, ldo);
+  if (vec) return launch_gnorm_gate<T, 4>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st);
+  return launch_gnorm_gate<T, 1>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st);
+}
+
+// ----------------------------------------------------------------------------- normed outputs on an fp32 residual
+template <typename T>
+struct AddNormedParams {
+  float* x; long long ldx;                     // [T, W]
+  const T* y; long long ldy;
+  const int* slot_of; const float* pick_w; int picks;      // picks > 0: y = sum_j pick_w[t, j] * rows slot_of[t, j] (>= 0) of `y`
+  const float* w; const float* out_w;          // w null: x = y (start of the model); out_w null: out = x
+  T* out; long long ldo;
+  int W, plus_one, store;
+  float eps;
+};
+
+// NI pieces of V elements per thread, the row stays in registers
+template <typename T, int V, int NI>
+__global__ void __launch_bounds__(1024)
+add_normed_kernel(const AddNormedParams<T> p) {
+  __shared__ float red[32];
+  chain_trigger();
+  chain_wait();
+  const long long t = blockIdx.x;
+  const int step = blockDim.x * V;
+  float y[NI][V];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    const int e = threadIdx.x * V + k * step;
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[k][i] = 0.f;
+    if (e >= p.W) continue;
+    if (p.picks == 0) {
+      load_vec<V>(p.y + t * p.ldy + e, y[k]);
+    } else {
+      for (int j = 0; j < p.picks; ++j) {
+        const int row = p.slot_of[t * p.picks + j];
+        if (row < 0) continue;
+        const float wj = p.pick_w[t * p.picks + j];
+        float f[V];
+        load_vec<V>(p.y + row * p.ldy + e, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] = fmaf(wj, f[i], y[k][i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += y[k][i] * y[k][i];
+  }
+  const float plus = p.plus_one ? 1.f : 0.f;
+  if (p.w) {
+    const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps);
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NI; ++k) {
+      const int e = threadIdx.x * V + k * step;
+      if (e >= p.W) continue;
+      float w[V], x[V];
+      load_vec<V>(p.w + e, w);
+      load_vec<V>(p.x + t * p.ldx + e, x);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        y[k][i] = fmaf(y[k][i] * rstd, w[i] + plus, x[i]);
+        ss += y[k][i] * y[k][i];
+      }
+    }
+  }
+  const float orstd = p.out_w ? 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps) : 1.f;
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    const int e = threadIdx.x * V + k * step;
+    if (e >= p.W) continue;
+    if (p.store) store_vec<V>(p.x + t * p.ldx + e, y[k]);
+    if (p.out_w) {
+      float w[V];
+      load_vec<V>(p.out_w + e, w);
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[k][i] = y[k][i] * orstd * (w[i] + plus);
+    }
+    store_vec<V>(p.out + t * p.ldo + e, y[k]);
+  }
+}
+
+template <typename T>
+static int add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const float* w,
+                      const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store, float eps, cudaStream_t st) {
+  AddNormedParams<T> p = {x, ldx, reinterpret_cast<const T*>(y), ldy, slot_of, pick_w, picks, w, out_w, reinterpret_cast<T*>(out), ldo, W, plus_one,
+                          store, eps};
+  const bool vec = W % 8 == 0 && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(out, ldo) && vec_ok<float, 4>(x, ldx) && vec_ok<float, 4>(w, 0) &&
+                   vec_ok<float, 4>(out_w, 0);
+  const int v = vec ? 8 : 1, pieces = (W + v - 1) / v;
+  void (*k)(const AddNormedParams<T>) = nullptr;
+  int ni = 1;
+  if (vec) {
+    ni = pieces <= 1024 ? 1 : 4;
+    k = ni == 1 ? add_normed_kernel<T, 8, 1> : add_normed_kernel<T, 8, 4>;
+  } else {
+    ni = pieces <= 1024 ? 1 : 32;
+    k = ni == 1 ? add_normed_kernel<T, 1, 1> : add_normed_kernel<T, 1, 32>;
+  }
+  const int threads = ((pieces + ni - 1) / ni + 31) / 32 * 32;
+  if (threads > 1024) return -2;
+  launch_chain_if(rows <= 256, k, dim3(rows), dim3(threads), 0, st, p);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+head_gate_kernel(T* x, long long ldx, const float* __restrict__ g, long long ldg, int H, int D) {
+  chain_trigger();
+  chain_wait();
+  const long long t = blockIdx.x;
+  const int e = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (e >= H * D) return;
+  const float s = 1.f / (1.f + expf(-g[t * ldg + e / D]));
+  float f[V];
+  load_vec<V>(x + t * ldx + e, f);
+#pragma unroll
+  for (int i = 0; i < V; ++i) f[i] *= s;
+  store_vec<V>(x + t * ldx + e, f);
+}
+
+template <typename T, int V>
+static int launch_head_gate(void* x, long long ldx, const float* g, long long ldg, int rows, int H, int D, cudaStream_t st) {
+  launch_chain_if(rows <= 256, head_gate_kernel<T, V>, dim3(rows, (H * D + 256 * V - 1) / (256 * V)), dim3(256), 0, st, reinterpret_cast<T*>(x), ldx, g,
+                  ldg, H, D);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
 // ----------------------------------------------------------------------------- clamped gated unit, tanh
 template <typename T, int V>
 __global__ void __launch_bounds__(256)
@@ -314,4 +537,38 @@ extern "C" int atlas_tanh(void* x, long long n, int f32, void* stream) {
   if (f32) launch_chain_if(n <= 65536, tanh_kernel<float>, grid, dim3(256), 0, st, reinterpret_cast<float*>(x), n);
   else launch_chain_if(n <= 65536, tanh_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, reinterpret_cast<__nv_bfloat16*>(x), n);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+// gate_first: silu(z) before the norm; otherwise silu(z), or with `sigmoid` sigmoid(z), after it
+extern "C" int atlas_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo,
+                                     int rows, int groups, int gsize, float eps, int gate_first, int sigmoid, const float* den, int f32,
+                                     void* stream) {
+  if (rows <= 0) return 0;
+  if (gate_first && sigmoid) return -1;
+  const int kind = gate_first ? kSiluFirst : (sigmoid ? kSigmoidAfter : kSiluAfter);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return f32 ? gnorm<float>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st)
+             : gnorm<__nv_bfloat16>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st);
+}
+
+// fp32 residual x [rows, W]: x += rmsnorm(y) * w (w null: x = y), out = x or rmsnorm(x) * out_w.  picks > 0: y [*, W] holds expert rows,
+// slot_of / pick_w [rows, picks].  With plus_one the weights are stored around zero; store = 0 leaves x as it is.
+extern "C" int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks,
+                                const float* w, const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store,
+                                float eps, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  if (W < 1 || W > 32768 || picks < 0 || (picks > 0 && (!slot_of || !pick_w))) return -1;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  return f32 ? add_normed<float>(x, ldx, y, ldy, slot_of, pick_w, picks, w, out_w, out, ldo, rows, W, plus_one, store, eps, st)
+             : add_normed<__nv_bfloat16>(x, ldx, y, ldy, slot_of, pick_w, picks, w, out_w, out, ldo, rows, W, plus_one, store, eps, st);
+}
+
+// x [rows, H, D] (row stride ldx) times sigmoid(g [rows, H]), in place
+extern "C" int atlas_head_gate(void* x, long long ldx, const float* g, long long ldg, int rows, int H, int D, int f32, void* stream) {
+  if (rows <= 0) return 0;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) return D % 4 == 0 && vec_ok<float, 4>(x, ldx) ? launch_head_gate<float, 4>(x, ldx, g, ldg, rows, H, D, st)
+                                                         : launch_head_gate<float, 1>(x, ldx, g, ldg, rows, H, D, st);
+  using B = __nv_bfloat16;
+  return D % 8 == 0 && vec_ok<B, 8>(x, ldx) ? launch_head_gate<B, 8>(x, ldx, g, ldg, rows, H, D, st) : launch_head_gate<B, 1>(x, ldx, g, ldg, rows, H, D, st);
 }

@@ -30,6 +30,16 @@ ATLAS_DEVICE float fast_exp2(float x) {
   return y;
 }
 
+// Bounded scores: cap * tanh(s * scale / cap) in the exp2 domain, with tanh(x) = 1 - 2 / (1 + e^(2x)).
+//   cap_in = 2 log2(e) scale / cap,  cap_out = cap log2(e)
+ATLAS_DEVICE float capped_score(float s, float cap_in, float cap_out) {
+  return cap_out - __fdividef(2.f * cap_out, 1.f + exp2f(s * cap_in));
+}
+inline void cap_constants(float scale, float cap, float* cap_in, float* cap_out) {
+  *cap_in = (float)(2.0 * 1.4426950408889634 * (double)scale / (double)cap);
+  *cap_out = (float)(1.4426950408889634 * (double)cap);
+}
+
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*,
                                   const cuuint64_t*, const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);

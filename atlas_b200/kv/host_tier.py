@@ -137,6 +137,8 @@ class HostKVTier:
         for l, (k, v) in cache.kv.items():
             for which, t in (("k", k), ("v", v)):
                 n = t[0].numel() * t.element_size()
+                if n == 0:
+                    continue                                  # a latent cache has one pool
                 self.layout.append((l, which, off, n))
                 off += n
         self.record_bytes = off
@@ -146,7 +148,7 @@ class HostKVTier:
         self.states: Dict[int, Dict[str, torch.Tensor]] = {}
         for l, st in cache.states.items():
             self.states[l] = {name: torch.empty((self.num_state_slots,) + tuple(t.shape[1:]), dtype=t.dtype, pin_memory=self.on_gpu)
-                              for name, t in st.items() if name in ("conv", "h")}
+                              for name, t in st.items()}
         self.stream = torch.cuda.Stream(device=self.device) if self.on_gpu else None
         self._staging: Optional[torch.Tensor] = None
         self.blocks_out = 0

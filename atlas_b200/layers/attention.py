@@ -17,7 +17,7 @@ from .. import ops
 from ..config import ModelConfig
 from ..ops import Act, LinearWeight
 from ..lora import GATE_SUFFIX, add_delta
-from .common import ParallelCtx, make_weight, randn_weight, shard_cols, shard_rows
+from .common import ParallelCtx, TailLinear, make_weight, randn_weight, shard_cols, shard_rows
 
 
 class Attention:
@@ -36,6 +36,9 @@ class Attention:
         self.scale = cfg.attn_scale or self.dqk ** -0.5
         self.chunk = cfg.attn_chunk         # > 0: a token sees keys of its own ``chunk``-token block of the sequence only
         self.sinks: Optional[torch.Tensor] = None       # [hq] fp32: extra term exp(sink) of the softmax denominator
+        self.softcap = cfg.attn_softcap     # > 0: scores are bounded before the softmax
+        self.norm_plus_one = cfg.norm_plus_one if cfg.qk_norm_plus_one is None else cfg.qk_norm_plus_one
+        self.gated_qkv: Optional[TailLinear] = None     # head gates: q | k | v with one gate number per head as an fp32 tail
         # models with per-layer attention kinds (Gemma): only "sliding_attention" layers use the window
         kinds = cfg.layer_types if (cfg.family != "hybrid" and cfg.layer_types) else None
         self.local = bool(kinds) and kinds[layer_idx] == "sliding_attention"
@@ -58,11 +61,13 @@ class Attention:
         return w[head * self.d:(head + self.hkv) * self.d]
 
     def load(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, o: torch.Tensor,
-             q_norm=None, k_norm=None, qkv_bias=None, sinks: Optional[torch.Tensor] = None) -> None:
+             q_norm=None, k_norm=None, qkv_bias=None, sinks: Optional[torch.Tensor] = None, head_gate: Optional[torch.Tensor] = None) -> None:
         """Takes full (unsharded) HF-layout tensors; slices for this rank, fuses, quantizes."""
         cfg, tp, r = self.cfg, self.pctx.tp_size, self.pctx.tp_rank
         if self.d != self.dqk or self.d != self.dv:
-            assert not self.gated and q_norm is None and qkv_bias is None, "padded heads: plain q / k / v projections only"
+            assert not self.gated and qkv_bias is None, "padded heads: plain q / k / v projections only"
+            pad = lambda n: None if n is None else torch.nn.functional.pad(n, (0, self.d - self.dqk))
+            q_norm, k_norm = pad(q_norm), pad(k_norm)
             q, k, v = self._pad_rows(q, self.dqk), self._pad_rows(k, self.dqk), self._pad_rows(v, self.dv)
             o = self._pad_rows(o.t(), self.dv).t()
         if sinks is not None:
@@ -74,7 +79,12 @@ class Attention:
         if self.gated:
             parts.append(shard_rows(gate, r, tp))
         fused = torch.cat(parts, 0)
-        self.qkv = make_weight(fused, self.quant_kind, qkv_bias)
+        if head_gate is not None:
+            assert qkv_bias is None
+            self.gated_qkv = TailLinear(fused, shard_rows(head_gate, r, tp), self.quant_kind)
+            self.qkv = self.gated_qkv.w
+        else:
+            self.qkv = make_weight(fused, self.quant_kind, qkv_bias)
         self.o = make_weight(shard_cols(o, r, tp).contiguous(), self.quant_kind)
         self.q_norm, self.k_norm = q_norm, k_norm
 
@@ -95,17 +105,18 @@ class Attention:
         o = randn_weight(gen, h, cfg.num_attention_heads * self.dv, std, dtype, device)
         qn = kn = None
         if cfg.qk_norm:
-            base = 0.0 if cfg.norm_plus_one else 1.0
-            qn = torch.full((self.d,), base, dtype=dtype, device=device)
-            kn = torch.full((self.d,), base, dtype=dtype, device=device)
+            base = float(not self.norm_plus_one)
+            qn = torch.full((self.dqk,), base, dtype=dtype, device=device)
+            kn = torch.full((self.dqk,), base, dtype=dtype, device=device)
         sinks = torch.zeros(cfg.num_attention_heads, dtype=torch.float32, device=device) if cfg.attn_sinks else None
-        self.load(q, k, v, o, qn, kn, sinks=sinks)
+        gate = randn_weight(gen, cfg.num_attention_heads, h, std, dtype, device) if cfg.attn_head_gate else None
+        self.load(q, k, v, o, qn, kn, sinks=sinks, head_gate=gate)
 
     @property
     def plain(self) -> bool:
-        """No chunked visibility and no sink: every cache dtype and attention kernel applies.  Otherwise the layer keeps a
-        cache in the model's own dtype."""
-        return not self.chunk and not self.cfg.attn_sinks
+        """No chunked visibility, sink or bounded scores: every cache dtype and attention kernel applies.  Otherwise the layer
+        keeps a cache in the model's own dtype."""
+        return not self.chunk and not self.cfg.attn_sinks and not self.softcap
 
     # ------------------------------------------------------------------ forward
     def forward(self, act: Act, batch, kv: Tuple[torch.Tensor, torch.Tensor, float, float],
@@ -124,7 +135,7 @@ class Attention:
         ``Act`` holding its FP8 form when the attention kernel quantised it)."""
         cfg = self.cfg
         k_cache, v_cache, k_scale, v_scale = kv
-        qkv = ops.linear(act, self.qkv)
+        qkv, head_gate = self.gated_qkv(act) if self.gated_qkv is not None else (ops.linear(act, self.qkv), None)
         T = qkv.shape[0]
         nq, nkv = self.hq * self.d, self.hkv * self.d
         if self.lora is not None and batch.adapter_rows is not None:
@@ -140,21 +151,24 @@ class Attention:
         rope_pos, rope_cache = batch.rope_inputs(rope_cache, cfg.mrope_section)
         q = ops.qk_norm_rope_kv_write(q, k, v, rope_pos, rope_cache, cfg.rotary_dim, k_cache, v_cache,
                                       batch.slot_mapping, k_scale, v_scale, self.q_norm, self.k_norm,
-                                      cfg.rms_norm_eps, cfg.norm_plus_one, rotate=self.kv_rotate)
+                                      cfg.rms_norm_eps, self.norm_plus_one, rotate=self.kv_rotate, norm_dim=self.dqk)
         if self.selector is not None:
             from ..kv.sparse_select import attend_selected
             self.selector.on_write(self.layer_idx, k_cache, batch, k_scale)
             out = attend_selected(ops.paged_attention, self.selector, self.layer_idx, q, k_cache, v_cache, batch, self.scale,
                                   k_scale, v_scale, self.window)
         else:
-            if (self.o.kind == "fp8_block" and not self.gated and self.o.bias is None and not self.kv_rotate
+            if (self.o.kind == "fp8_block" and not self.gated and head_gate is None and self.o.bias is None and not self.kv_rotate
                     and (self.lora is None or batch.adapter_rows is None) and self.plain):
                 a = ops.paged_attention_fp8_out(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window)
                 if a is not None:
                     return a                  # decode step: rows already quantised for the output projection
-            out = ops.paged_attention(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window, self.chunk, self.sinks)
+            out = ops.paged_attention(q, k_cache, v_cache, batch, self.scale, k_scale, v_scale, self.window, self.chunk, self.sinks,
+                                      self.softcap)
         if self.kv_rotate:
             out = ops.head_rotate(out)        # sum_j p_j (H v_j) = H o, and H is its own inverse
+        if head_gate is not None:
+            out = ops.head_gate(out, head_gate)
         out = out.reshape(T, nq)
         if self.gated:
             gate = qkv[:, nq + 2 * nkv:]

@@ -78,6 +78,26 @@ class ParallelCtx:
         return t
 
 
+class TailLinear:
+    """Two projections of the same input in one matrix product: ``main`` in the activations' dtype and ``tail``, whose results
+    stay in fp32 (gates, logits and whatever else is computed in 32 bits from there on).  A quantised main part leaves the tail
+    a product of its own."""
+
+    def __init__(self, main: torch.Tensor, tail: torch.Tensor, kind: str):
+        self.n_main = main.shape[0]
+        w = make_weight(main, kind)
+        self.fused = w.kind == "dense"
+        self.w = LinearWeight("dense", torch.cat([main, tail], 0).contiguous()) if self.fused else w
+        self.tail = None if self.fused else LinearWeight("dense", tail.contiguous())
+
+    def __call__(self, act):
+        """``(main [T, n_main], tail [T, n_tail] fp32)``"""
+        from .. import ops
+        if self.fused:
+            return ops.linear_tail(act, self.w, self.n_main)
+        return ops.linear(act, self.w), ops.linear_tail(act, self.tail, 0)[1]
+
+
 def shard_rows(w: torch.Tensor, rank: int, size: int) -> torch.Tensor:
     """Column-parallel slice (output features)."""
     if size == 1:

@@ -17,6 +17,7 @@ from dataclasses import dataclass
 from typing import List, Optional
 
 import torch
+import torch.nn.functional as F
 
 from .. import ops, quant as Q
 from ..config import ModelConfig
@@ -28,7 +29,7 @@ from .mlp import DenseMLP
 
 @dataclass
 class ExpertWeights:
-    """Stacked local experts. ``w13 [E,2I,H]`` (gate rows then up rows), ``w2 [E,H,I]``.
+    """Stacked local experts. ``w13 [E,2I,H]`` (gate rows then up rows; ``[E,I,H]`` for experts without a gate), ``w2 [E,H,I]``.
 
     kind ``dense`` keeps the model dtype; ``fp8_block`` adds ``*_scale [E, ceil(N/128), ceil(K/128)]``;
     ``nvfp4`` stores packed nibbles ``[E,N,K/2]``, e4m3 ``*_scale [E,N,K/16]`` and fp32 ``*_gscale [E]`` (or ``[E,N]``, one per output row).
@@ -94,6 +95,8 @@ class MoE:
         self.cfg, self.pctx = cfg, pctx
         self.expert_kind, self.dense_kind = expert_kind, dense_kind
         self.top_k = cfg.num_experts_per_tok
+        self.activation = "relu2" if cfg.mlp_activation == "relu2" else "silu_glu"      # silu(gate) * up, or relu(up)^2
+        self.router_f32 = cfg.router_f32
         self.e_lo, self.e_hi = cfg.local_expert_range(pctx.ep_rank, pctx.ep_size)
         self.ep_mode = ep_mode
         self.router: Optional[LinearWeight] = None
@@ -113,6 +116,10 @@ class MoE:
         self.router = LinearWeight("dense", router.contiguous())
         if w13.shape[0] == self.cfg.num_experts and self.pctx.ep_size > 1:
             w13, w2 = w13[self.e_lo:self.e_hi], w2[self.e_lo:self.e_hi]
+        if self.activation == "relu2" and w2.shape[2] % 64:
+            # whole GEMM tiles: hidden channels of zero weights stay zero through the activation
+            pad = 64 - w2.shape[2] % 64
+            w13, w2 = F.pad(w13, (0, 0, 0, pad)), F.pad(w2, (0, pad))
         self.experts = ExpertWeights.from_dense(w13, w2, self.expert_kind)
 
     def init_random(self, gen, std, dtype, device) -> None:
@@ -123,25 +130,25 @@ class MoE:
         n_local = self.e_hi - self.e_lo
         w13_l, w2_l = [], []
         for e in range(cfg.num_experts):
-            a = torch.randn(2 * i, h, generator=gen, dtype=torch.float32, device=gen.device) * std
+            a = torch.randn(i if self.activation == "relu2" else 2 * i, h, generator=gen, dtype=torch.float32, device=gen.device) * std
             b = torch.randn(h, i, generator=gen, dtype=torch.float32, device=gen.device) * std
             if self.e_lo <= e < self.e_hi:
                 w13_l.append(a.to(device=device, dtype=dtype))
                 w2_l.append(b.to(device=device, dtype=dtype))
         assert len(w13_l) == n_local
-        self.router = LinearWeight("dense", router)
         if cfg.router_selection_bias:
             self.router_bias = (torch.rand(cfg.num_experts, generator=gen, device=gen.device) * 0.1).to(device)
-        self.experts = ExpertWeights.from_dense(torch.stack(w13_l), torch.stack(w2_l), self.expert_kind)
+        self.load(router, torch.stack(w13_l), torch.stack(w2_l))
         if self.shared is not None:
             self.shared.init_random(gen, std, dtype, device)
             self.shared_gate = randn_weight(gen, 1, h, std, dtype, device)
 
     # ------------------------------------------------------------------ forward
-    def forward(self, act: Act, token_ids: Optional[torch.Tensor] = None, batch=None) -> torch.Tensor:
+    def forward(self, act: Act, token_ids: Optional[torch.Tensor] = None, batch=None, rows_ok: bool = False):
+        """``rows_ok``: the caller takes the weighted sum itself, so the result may be an :class:`ops.ExpertRows`."""
         x = act.plain()
         cfg = self.cfg
-        logits = ops.linear(x, self.router)
+        logits = ops.linear_tail(x, self.router, 0)[1] if self.router_f32 else ops.linear(x, self.router)
         adapters = self.lora is not None and batch is not None and batch.adapter_rows is not None and bool(self.lora_prefix)
         if adapters:
             add_delta(logits, self.lora, self.lora_prefix + "gate", x, batch)
@@ -149,7 +156,11 @@ class MoE:
                                          cfg.router_n_group, cfg.router_topk_group, cfg.routed_scaling_factor,
                                          self.hash_table, token_ids if self.hash_table is not None else None)
         if ops.on_gpu(x):
-            y = ops.cuda_ops().moe_forward(x, topk_w, topk_ids, self.experts, self.e_lo, self.pctx, self.ep_mode)
+            rows_ok = rows_ok and not adapters and self.shared is None and self.pctx.ep_size == 1
+            y = ops.cuda_ops().moe_forward(x, topk_w, topk_ids, self.experts, self.e_lo, self.pctx, self.ep_mode,
+                                           activation=self.activation, rows_ok=rows_ok)
+            if rows_ok:
+                return y
         else:
             y = self._forward_ref(x, topk_w, topk_ids)
         if adapters:
@@ -185,7 +196,7 @@ class MoE:
             return y
         xr, ids, wts, slot_r = x[rows].float(), topk_ids[rows].long(), topk_w[rows].float(), adapter_rows[rows]
         part = torch.zeros(rows.numel(), x.shape[1], dtype=torch.float32, device=x.device)
-        inter = self.cfg.moe_intermediate_size
+        inter = self.experts.w2.shape[-1] if self.experts.kind == "dense" else self.cfg.moe_intermediate_size
 
         def pair(ad, e, leaf):
             w = ad.weights.get(f"{self.lora_prefix}experts.{e}.{leaf}")
@@ -205,10 +216,13 @@ class MoE:
                     continue
                 xe = xr[sel]
                 h = xe @ w13.float().t()
-                g = h[:, :inter] + low_rank(xe, pair(ad, e, "gate_proj"))
-                u = h[:, inter:] + low_rank(xe, pair(ad, e, "up_proj"))
-                a = (torch.nn.functional.silu(g) * u).to(x.dtype).float()
-                o = a @ w2.float().t() + low_rank(a, pair(ad, e, "down_proj"))
+                if self.activation == "relu2":
+                    up = low_rank(xe, pair(ad, e, "up_proj"))
+                    h = h + (F.pad(up, (0, inter - up.shape[1])) if torch.is_tensor(up) else up)
+                else:
+                    h = torch.cat([h[:, :inter] + low_rank(xe, pair(ad, e, "gate_proj")), h[:, inter:] + low_rank(xe, pair(ad, e, "up_proj"))], 1)
+                a = ref.expert_act(h, self.activation).to(x.dtype).float()
+                o = a @ w2.float().t() + low_rank(a[:, :self.cfg.moe_intermediate_size], pair(ad, e, "down_proj"))
                 part.index_add_(0, sel, o * (wts[sel] * hit[sel]).sum(-1, keepdim=True))
         p = self.pctx
         comm = p.ep_comm if p.ep_comm is not None else p.comm
@@ -225,9 +239,9 @@ class MoE:
         comm = p.ep_comm if p.ep_comm is not None else p.comm
         mode = self.ep_mode if self.ep_mode != "auto" else "allreduce"
         if p.ep_size == 1 or comm is None:
-            return ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo)
+            return ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation)
         if mode == "allreduce":
-            return comm.all_reduce(ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo))
+            return comm.all_reduce(ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation))
         return self._forward_alltoall_ref(x, topk_w, topk_ids, w13, w2, comm)
 
     def _forward_alltoall_ref(self, x, topk_w, topk_ids, w13, w2, comm) -> torch.Tensor:
@@ -254,7 +268,7 @@ class MoE:
                 continue
             ids = meta[:, 1:2].to(torch.int32)
             ones = torch.ones(rows.shape[0], 1, dtype=torch.float32, device=rows.device)
-            outs.append(ref.moe_experts(rows, w13, w2, ones, ids, self.e_lo))
+            outs.append(ref.moe_experts(rows, w13, w2, ones, ids, self.e_lo, self.activation))
         back = comm.all_to_all(outs)
         y = torch.zeros(T, H, dtype=torch.float32, device=x.device)
         for r in range(p.ep_size):

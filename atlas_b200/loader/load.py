@@ -293,9 +293,35 @@ def _load_papidra(model: DecoderLM, ck: Checkpoint) -> None:
     ck.close()
 
 
+def _load_tomizen(model: DecoderLM, ck: Checkpoint) -> None:
+    """Tomizen naming: ``embed``, ``l<i>.{norm1, norm2, mix.*, mlp.router, mlp.e<j>.{up, down}}``, ``final.norm``, ``head``."""
+    wt = lambda name: ck.get(name).to(device=model.device, dtype=model.dtype)
+    f32 = lambda name: ck.get(name).to(device=model.device, dtype=torch.float32).contiguous()
+    model.embed = wt("embed").contiguous()
+    for i, layer in enumerate(model.layers):
+        pre, mx = f"l{i}.", layer.mixer
+        m = pre + "mix."
+        layer.input_norm = f32(pre + "norm1")
+        if layer.kind == "mlstm":
+            mx.load(*(wt(m + n) for n in "qkvg"), wt(m + "i"), f32(m + "i.b"), wt(m + "f"), f32(m + "f.b"), f32(m + "norm"), wt(m + "o"), model.device)
+        elif layer.kind == "latent_attention":
+            mx.load(wt(m + "q"), wt(m + "dkv"), f32(m + "dkv.norm"), wt(m + "uk"), wt(m + "uv"), wt(m + "o"))
+        else:
+            mx.load(*(wt(m + n) for n in "qkvo"), wt(m + "q.norm"), wt(m + "k.norm"), head_gate=wt(m + "g"))
+        if layer.ffn is not None:
+            layer.post_norm = f32(pre + "norm2")
+            local = range(layer.ffn.e_lo, layer.ffn.e_hi)
+            layer.ffn.load(wt(pre + "mlp.router"), *(torch.stack([wt(f"{pre}mlp.e{e}.{n}") for e in local]) for n in ("up", "down")))
+    model.final_norm = f32("final.norm")
+    model.set_lm_head(wt("head"))
+    ck.close()
+
+
 def load_weights(model: DecoderLM, ck: Checkpoint) -> None:
     cfg = model.cfg
     dense_kind, expert_kind = quant_kinds(cfg)
+    if cfg.model_type == "tomizen":
+        return _load_tomizen(model, ck)
     if cfg.model_type == "papidra":
         return _load_papidra(model, ck)
     if cfg.block_types:

@@ -1,8 +1,8 @@
 """Generic decoder-only LM assembled from the layer blocks.
 
 One class covers the dense (Llama/Mistral/Qwen2/Qwen3), MoE (Qwen3-MoE) and hybrid
-(Qwen3-Next: Gated DeltaNet + gated attention + MoE + MTP head) families; ``ModelConfig`` decides
-the mixer and FFN kind of every layer.
+(Qwen3-Next: Gated DeltaNet + gated attention + MoE + MTP head; models given by a list of layers) families;
+``ModelConfig`` decides the mixer and FFN kind of every layer and the form of the residual.
 
 Reference parity: ``crates/spark-model/src/model/`` (``TransformerModel``), the decode program in
 ``model/trait_impl/decode_a2.rs`` and the chunked prefill program in ``model/trait_impl/prefill_b.rs``.
@@ -20,7 +20,7 @@ from ..config import ModelConfig
 from ..layers import (MIXERS, Attention, DenseMLP, GatedDeltaNet, HyperConnection, Mamba2Mixer, MLAttention, MoE, ParallelCtx,
                       ParallelMixer)
 from ..layers.common import make_weight, randn_weight, shard_rows
-from ..ops import Act, LinearWeight, StreamDelta, reference as ref
+from ..ops import Act, LinearWeight, NormDelta, StreamDelta, reference as ref
 from .batch import ForwardBatch
 
 # tensor-parallel steps with at least this many rows run sequence-parallel (reduce-scatter / all-gather fused into the
@@ -301,16 +301,67 @@ class StreamLayer:
         return x, streams
 
 
+class OutputNormLayer:
+    """A layer whose norms sit on the sublayers' outputs: ``x += norm(mixer(x))``, then ``x += norm(ffn(x))`` where the layer has a
+    feed-forward, on an fp32 residual stream that the sublayers read itself.  Same ``forward`` protocol as
+    :class:`DecoderLayer`, with the pending :class:`NormDelta` in place of the previous layer's output."""
+
+    def __init__(self, cfg: ModelConfig, idx: int, pctx: ParallelCtx, ep_mode: str = "auto"):
+        spec = cfg.layer_specs[idx]
+        self.cfg, self.idx = cfg.for_layer(idx), idx
+        dense_kind, expert_kind = quant_kinds(cfg)
+        self.kind, self.is_moe = spec.kind, cfg.is_moe_layer(idx)
+        self.mixer = MIXERS[spec.kind](self.cfg, idx, pctx, dense_kind)
+        self.ffn = None
+        if spec.has_mlp:
+            self.ffn = MoE(self.cfg, pctx, expert_kind, dense_kind, ep_mode) if self.is_moe else DenseMLP(self.cfg, pctx, dense_kind)
+        self.input_norm: Optional[torch.Tensor] = None         # fp32, on the mixer's output
+        self.post_norm: Optional[torch.Tensor] = None          # fp32, on the feed-forward's output
+        self.rope_override: Optional[torch.Tensor] = None      # this layer's own rotary table
+
+    def init_random(self, gen, std, dtype, device):
+        fresh = lambda: torch.full((self.cfg.hidden_size,), 0.0 if self.cfg.norm_plus_one else 1.0, dtype=torch.float32, device=device)
+        self.mixer.init_random(gen, std, dtype, device)
+        self.input_norm = fresh()
+        if self.ffn is not None:
+            self.ffn.init_random(gen, std, dtype, device)
+            self.post_norm = fresh()
+
+    def accepts_prenormed(self) -> bool:
+        return False
+
+    def forward(self, x: NormDelta, stream: Optional[torch.Tensor], batch: ForwardBatch, cache: CacheStore, rope_cache, next_norm=None):
+        eps, p1 = self.cfg.rms_norm_eps, self.cfg.norm_plus_one
+        rope_cache = rope_cache if self.rope_override is None else self.rope_override
+        h, stream = ops.add_normed(stream, x, eps, p1)
+        if attention_of(self) is not None:
+            y = self.mixer.forward(Act(x=h), batch, cache.layer_kv(self.idx), rope_cache)
+        else:
+            y = self.mixer.forward(Act(x=h), batch, cache.states[self.idx])
+        x = NormDelta(y, self.input_norm)
+        if self.ffn is not None:
+            h, stream = ops.add_normed(stream, x, eps, p1)
+            y = self.ffn.forward(Act(x=h), batch=batch, rows_ok=True) if self.is_moe else self.ffn.forward(Act(x=h), batch=batch)
+            x = NormDelta(y, self.post_norm)
+        return x, stream
+
+
 def attention_of(layer):
     """The attention block of a layer (None without one): the owner of the layer's KV cache."""
     if layer.kind == "parallel":
         return layer.mixer.left
-    return layer.mixer if layer.kind == "attention" else None
+    return layer.mixer if layer.kind in ("attention", "latent_attention") else None
 
 
 def recurrent_of(layer):
     """The mixer of a layer that owns a recurrent state slot (None without one)."""
-    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel") else None
+    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel", "mlstm") else None
+
+
+def kv_elements_of(attn) -> int:
+    """Cached numbers per token of an attention block: a key and a value per head unless the block says otherwise."""
+    n = getattr(attn, "kv_elements", None)
+    return 2 * attn.hkv * attn.d if n is None else n
 
 
 class DecoderLM:
@@ -321,9 +372,10 @@ class DecoderLM:
         self.device = torch.device(device)
         self.dtype = torch_dtype(cfg.dtype)
         if cfg.layer_specs:
-            if cfg.residual_streams < 1:
-                raise ValueError("a model given by a list of layers runs on hyper-connected residual streams")
-            self.layers = [StreamLayer(cfg, i, self.pctx) for i in range(cfg.num_hidden_layers)]
+            if bool(cfg.residual_streams) == cfg.output_norms:
+                raise ValueError("a model given by a list of layers runs on hyper-connected residual streams or on normed outputs")
+            self.layers = [OutputNormLayer(cfg, i, self.pctx, ep_mode) if cfg.output_norms else StreamLayer(cfg, i, self.pctx)
+                           for i in range(cfg.num_hidden_layers)]
         elif cfg.block_types:
             self.layers = [SingleBlock(cfg, i, self.pctx) for i in range(cfg.num_hidden_layers)]
         else:
@@ -357,7 +409,7 @@ class DecoderLM:
         for layer in self.layers:
             layer.init_random(gen, std, dt, dev)
         base = 0.0 if cfg.norm_plus_one else 1.0
-        self.final_norm = torch.full((cfg.hidden_size,), base, dtype=torch.float32 if cfg.residual_streams else dt, device=dev)
+        self.final_norm = torch.full((cfg.hidden_size,), base, dtype=torch.float32 if cfg.layer_specs else dt, device=dev)
         head = self.embed if cfg.tie_word_embeddings else randn_weight(gen, cfg.vocab_size, cfg.hidden_size, std, dt, dev)
         self.set_lm_head(head)
         if self.mtp is not None:
@@ -371,7 +423,7 @@ class DecoderLM:
         if getattr(self, "lora", None) is None:
             self.lora = LoraSet(max_slots)
             for l in self.layers:
-                if attention_of(l) is not None:
+                if attention_of(l) is not None and l.kind != "latent_attention":
                     attention_of(l).lora = self.lora
                 if l.ffn is None:
                     continue
@@ -449,7 +501,7 @@ class DecoderLM:
     def kv_bytes_per_block(self, block_size: int, kv_dtype: torch.dtype, high_precision_layers=()) -> int:
         if self.cfg.layer_specs:
             owners = [(l, attention_of(l)) for l in self.layers if attention_of(l) is not None]
-            return int(sum(2 * block_size * a.hkv * a.d * kv_element_bytes(self._cache_dtype(l, kv_dtype, set(high_precision_layers)))
+            return int(sum(block_size * kv_elements_of(a) * kv_element_bytes(self._cache_dtype(l, kv_dtype, set(high_precision_layers)))
                            for l, a in owners))
         n_attn = len(self.attention_layers()) + (1 if self.mtp is not None else 0)
         hkv = self.layers[self.attention_layers()[0]].mixer.hkv if n_attn else 0
@@ -466,7 +518,10 @@ class DecoderLM:
         for l in self.layers:
             a = attention_of(l)
             if a is not None:
-                store.kv[l.idx] = alloc_kv(num_blocks, block_size, a.hkv, a.d, self._cache_dtype(l, kv_dtype, hi), self.device)
+                dt = self._cache_dtype(l, kv_dtype, hi)
+                own = getattr(a, "alloc_kv", None)
+                store.kv[l.idx] = (own(num_blocks, block_size, dt, self.device) if own is not None
+                                   else alloc_kv(num_blocks, block_size, a.hkv, a.d, dt, self.device))
                 store.kv_scales[l.idx] = (1.0, 1.0)
             if recurrent_of(l) is not None:
                 store.states[l.idx] = l.mixer.alloc_state(max(1, state_slots), self.device, self.dtype)
@@ -554,6 +609,8 @@ class DecoderLM:
         residual = None
         if self.cfg.residual_streams:
             x = StreamDelta(x, scale=self.cfg.embed_scale)      # fp32 streams start from the scaled embedding
+        elif self.cfg.output_norms:
+            x = NormDelta(x)                  # so does the fp32 stream that takes normed outputs
         elif batch.inputs_embeds is not None:
             x = x.clone()                     # fused epilogues update the residual stream in place
         if layer_ids is not None:
@@ -569,7 +626,7 @@ class DecoderLM:
             nxt = self.layers[i + 1] if i + 1 < n else None
             next_norm = nxt.input_norm if (nxt is not None and nxt.accepts_prenormed()) else None
             x, residual = layer.forward(x, residual, batch, cache, self.rope_cache, next_norm=next_norm)
-            if i in self.capture_layers and isinstance(x, StreamDelta):
+            if i in self.capture_layers and isinstance(x, (StreamDelta, NormDelta)):
                 self.aux_hidden.append(self._stream_sum(x, residual))
             elif i in self.capture_layers:
                 # the stream after layer i: already summed when the layer's epilogue handed over normalised activations
@@ -581,6 +638,8 @@ class DecoderLM:
         if isinstance(x, StreamDelta):
             y, _ = ops.hyper_norm(residual, x, self._stream_ones, self.final_norm, self.cfg.rms_norm_eps, write=False)
             return y
+        if isinstance(x, NormDelta):
+            return ops.add_normed(residual, x, self.cfg.rms_norm_eps, self.cfg.norm_plus_one, self.final_norm, write=False)[0]
         y, _ = ops.rmsnorm(x, self.final_norm, self.cfg.rms_norm_eps, residual, self.cfg.norm_plus_one)
         return y
 
@@ -591,8 +650,10 @@ class DecoderLM:
             t = self._ones = torch.ones(self.cfg.residual_streams, dtype=torch.float32, device=self.device)
         return t
 
-    def _stream_sum(self, x: StreamDelta, streams: torch.Tensor) -> torch.Tensor:
+    def _stream_sum(self, x, streams: torch.Tensor) -> torch.Tensor:
         """Sum of the residual streams with a pending update applied (fp32)."""
+        if isinstance(x, NormDelta):
+            return ops.add_normed(streams.clone(), x, self.cfg.rms_norm_eps, self.cfg.norm_plus_one)[1]
         _, after = ops.hyper_norm(streams.clone(), x, self._stream_ones, self.final_norm, self.cfg.rms_norm_eps)
         return after.sum(1)
 

@@ -136,6 +136,33 @@ def hyper_norm(streams: Optional[torch.Tensor], delta: StreamDelta, read: torch.
     return ref.hyper_norm(streams, delta, read, norm_w, eps)
 
 
+@dataclass
+class ExpertRows:
+    """Expert outputs before their weighted sum: ``y`` holds one row per (token, choice) pair, ``slot_of [T * k]`` the row of each
+    pair (-1: nothing to add), ``w [T, k]`` its weight."""
+    y: torch.Tensor
+    slot_of: torch.Tensor
+    w: torch.Tensor
+
+
+@dataclass
+class NormDelta:
+    """What the last sublayer leaves for an fp32 residual stream that takes normed outputs: ``stream += rmsnorm(y) * norm``, with
+    ``y`` given as it is or as :class:`ExpertRows`.  Start of the model (``norm`` is None): the stream is ``y``."""
+    y: object
+    norm: Optional[torch.Tensor] = None
+
+
+def add_normed(stream: Optional[torch.Tensor], delta: NormDelta, eps: float, plus_one: bool, out_norm: Optional[torch.Tensor] = None,
+               write: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Apply ``delta`` to ``stream [T, W]`` (fp32, in place; None at the start) and return ``(h, stream)``: ``h`` is the stream in
+    the activations' dtype, normed with ``out_norm`` where one is given.  ``write=False`` leaves the stream as it is."""
+    y = delta.y.y if isinstance(delta.y, ExpertRows) else delta.y
+    if on_gpu(y):
+        return cuda_ops().add_normed(stream, delta, eps, plus_one, out_norm, write)
+    return ref.add_normed(stream, delta, eps, plus_one, out_norm, write)
+
+
 # ----------------------------------------------------------------------------- elementwise / norm
 def quant_fp8(x: torch.Tensor, group: int = 128):
     if on_gpu(x):
@@ -197,12 +224,21 @@ def tanh_(x: torch.Tensor) -> torch.Tensor:
     return x.tanh_()
 
 
-def group_norm_gate(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, group: int, eps: float, gate_first: bool) -> torch.Tensor:
-    """RMS norm over groups of ``group`` channels joined with a SiLU gate: ``norm(y * silu(z)) * w`` with ``gate_first``
-    (Mamba-2), ``norm(y) * w * silu(z)`` otherwise (WKV).  ``z`` may be a column slice."""
+def group_norm_gate(y: torch.Tensor, z: torch.Tensor, w: torch.Tensor, group: int, eps: float, gate_first: bool, gate: str = "silu",
+                    den: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """RMS norm over groups of ``group`` channels joined with a gate: ``norm(y * gate(z)) * w`` with ``gate_first`` (Mamba-2),
+    ``norm(y) * w * gate(z)`` otherwise (WKV, mLSTM); ``gate`` is silu or sigmoid.  ``z`` may be a column slice.  ``den [T, groups]``
+    (fp32) divides every group of ``y`` first."""
     if on_gpu(y):
-        return cuda_ops().group_norm_gate(y, z, w, group, eps, gate_first)
-    return ref.group_norm_gate(y, z, w, group, eps, gate_first)
+        return cuda_ops().group_norm_gate(y, z, w, group, eps, gate_first, gate, den)
+    return ref.group_norm_gate(y, z, w, group, eps, gate_first, gate, den)
+
+
+def head_gate(x: torch.Tensor, g: torch.Tensor) -> torch.Tensor:
+    """``x [T, H, D]`` times ``sigmoid(g [T, H])`` (fp32 gate numbers; in place on the GPU)."""
+    if on_gpu(x):
+        return cuda_ops().head_gate(x, g)
+    return (x.float() * torch.sigmoid(g.float())[..., None]).to(x.dtype)
 
 
 def silu_mul_act(gate_up: torch.Tensor, want_fp8=False) -> Act:
@@ -256,6 +292,17 @@ def linear(a, w: LinearWeight, out: Optional[torch.Tensor] = None) -> torch.Tens
     return y
 
 
+def linear_tail(a, w: LinearWeight, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``a @ W^T`` of an unquantised weight in two parts: the first ``n_main`` columns in the activations' dtype, the others as the
+    fp32 sums that the product forms.  Returns ``(main, tail)``."""
+    x = a.plain() if isinstance(a, Act) else a
+    assert w.kind == "dense" and w.bias is None
+    if on_gpu(x) and x.dtype == torch.bfloat16:
+        return cuda_ops().linear_tail(x, w.weight, n_main)
+    y = torch.nn.functional.linear(x.float(), w.weight.float())
+    return y[:, :n_main].to(x.dtype), y[:, n_main:]
+
+
 # NVFP4 weights: quantise the activations to NVFP4 too and run the block-scaled FP4 x FP4 tensor-core GEMM (what an
 # "NVFP4" ModelOpt checkpoint is calibrated for); off = weight-only (activations stay bf16)
 NVFP4_ACTIVATIONS = os.environ.get("ATLAS_NVFP4_W4A4", "0") == "1"
@@ -302,15 +349,15 @@ def linear_residual_norm(a, w: LinearWeight, residual: torch.Tensor, norm_w: tor
 
 # ----------------------------------------------------------------------------- attention
 def qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping,
-                          k_scale=1.0, v_scale=1.0, q_norm_w=None, k_norm_w=None, eps=1e-6, norm_plus_one=False, rotate=False):
+                          k_scale=1.0, v_scale=1.0, q_norm_w=None, k_norm_w=None, eps=1e-6, norm_plus_one=False, rotate=False, norm_dim=0):
     """``rotate``: every q / k / v head goes through the orthonormal Walsh-Hadamard transform after RoPE, so the cache
     holds rotated keys and values (the "turbo8" cache: rotation + FP8) and the attention output comes out rotated too
-    (``head_rotate`` takes it back)."""
+    (``head_rotate`` takes it back).  ``norm_dim``: channels of a head that its norm counts (0 = all; the rest is zero padding)."""
     if on_gpu(q):
         return cuda_ops().qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache,
-                                                slot_mapping, k_scale, v_scale, q_norm_w, k_norm_w, eps, norm_plus_one, rotate)
+                                                slot_mapping, k_scale, v_scale, q_norm_w, k_norm_w, eps, norm_plus_one, rotate, norm_dim)
     return ref.qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping,
-                                     k_scale, v_scale, q_norm_w, k_norm_w, eps, norm_plus_one, rotate)
+                                     k_scale, v_scale, q_norm_w, k_norm_w, eps, norm_plus_one, rotate, norm_dim)
 
 
 def head_rotate(x: torch.Tensor) -> torch.Tensor:
@@ -321,13 +368,14 @@ def head_rotate(x: torch.Tensor) -> torch.Tensor:
 
 
 def paged_attention(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None, chunk=0,
-                    sinks=None) -> torch.Tensor:
+                    sinks=None, softcap=0.0) -> torch.Tensor:
     """Attention of the step's query rows over the paged cache. ``batch`` is a ``ForwardBatch``.  ``chunk`` > 0: a token sees
-    only keys of its own ``chunk``-token block of the sequence; ``sinks [Hq]``: ``exp(sink)`` joins the softmax denominator."""
+    only keys of its own ``chunk``-token block of the sequence; ``sinks [Hq]``: ``exp(sink)`` joins the softmax denominator;
+    ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)``."""
     if on_gpu(q):
-        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk, sinks)
+        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap)
     return ref.paged_attention(q, k_cache, v_cache, batch.block_tables, batch.seq_lens, batch.query_start_loc,
-                               scale, k_scale, v_scale, sliding_window, chunk, sinks)
+                               scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap)
 
 
 def paged_attention_fp8_out(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None) -> Optional[Act]:

@@ -76,7 +76,7 @@ def load() -> None:
     lib.atlas_silu_mul.argtypes = [_vp, _ll, _i, _i, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp]
     lib.atlas_quant_fp8.argtypes = [_vp, _ll, _i, _i, _vp, _ll, _vp, _ll, _vp]
     lib.atlas_rope_kv_write.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i,
-                                        _i, _i, _i, _i, _f, _f, _f, _vp]
+                                        _i, _i, _i, _i, _f, _f, _f, _vp, _i]
     lib.atlas_gated_rmsnorm.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _vp]
     lib.atlas_wht_d128.argtypes = [_vp, _ll, _i, _i, _vp]
     lib.atlas_attn_decode.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _f, _f, _i, _i, _i,
@@ -454,6 +454,34 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None) -> torch.Tensor:
     return _gemm(0, x, w, None, None, out)
 
 
+def linear_tail(x: torch.Tensor, w: torch.Tensor, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """bf16 product whose columns from ``n_main`` on stay fp32: ``(main [M, n_main] bf16, tail [M, N - n_main] fp32)``."""
+    assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.stride(1) == 1
+    M, K = x.shape
+    N = w.shape[0]
+    d = _dev(x)
+    if K % 8:                          # rows that TMA cannot address (16-byte strides): vendor products
+        return torch.nn.functional.linear(x, w[:n_main]), torch.nn.functional.linear(x.float(), w[n_main:].float())
+    if x.stride(1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
+        x = x.contiguous()
+    main = torch.empty(M, n_main, dtype=torch.bfloat16, device=x.device)
+    tail = torch.empty(M, N - n_main, dtype=torch.float32, device=x.device)
+    L = lib()
+    if not getattr(L, "_tail_bound", False):
+        L.atlas_gemm_tail.argtypes = [_vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
+        L._tail_bound = True
+    sms = _num_sms[d]
+    bn, splits = gemm_plan(M, N, K, 0, sms)
+    ws = cnt = None
+    if splits > 1:
+        ws = scratch("gemm_ws", _GEMM_WS_BYTES, x.device)
+        cnt = scratch("gemm_counters", 1 << 18, x.device)
+    _check(L.atlas_gemm_tail(x.data_ptr(), w.data_ptr(), main.data_ptr() if n_main else None, tail.data_ptr() if n_main < N else None, N - n_main,
+                             n_main, M, N, K, x.stride(0), w.stride(0), n_main, bn, splits, _ptr(ws), _ptr(cnt), sms, _status_ptr[d], _stream()),
+           "gemm_tail")
+    return main, tail
+
+
 def gemm_fp8_block(xq: torch.Tensor, xs: torch.Tensor, wq: torch.Tensor, ws: torch.Tensor, out=None, ready=None) -> torch.Tensor:
     assert xq.dtype == FP8 and wq.dtype == FP8
     return _gemm(1, xq, wq, xs, ws, out, ready)
@@ -516,18 +544,19 @@ def wht_d128(x: torch.Tensor) -> torch.Tensor:
 
 
 def qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, k_scale, v_scale,
-                          q_norm_w, k_norm_w, eps, norm_plus_one, rotate=False):
+                          q_norm_w, k_norm_w, eps, norm_plus_one, rotate=False, norm_dim=0):
     T, Hq, D = q.shape
     Hkv = k.shape[1]
     _dev(q)
     _kv_layout_ok(k_cache, v_cache)
     if q.dtype == torch.float32:
-        if q_norm_w is not None or rotate:
-            raise KernelError("32-bit attention has neither head norms nor a rotated cache")
+        if rotate:
+            raise KernelError("32-bit attention has no rotated cache")
         if checked.ENABLED:
             checked.kv_write(slot_mapping, positions, k_cache.shape[0], k_cache.shape[1], rope_cache.shape[0] if rotary_dim else 0)
         from . import cuda_recurrent
-        return cuda_recurrent.rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping)
+        return cuda_recurrent.rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm_w,
+                                                k_norm_w, norm_dim or D, norm_plus_one, eps)
     assert q.stride(2) == 1 and q.stride(1) == D and k.stride(1) == D and v.stride(1) == D
     assert positions.dtype == torch.int32 and slot_mapping.dtype == torch.int32 and rope_cache.dtype == torch.float32
     bs = k_cache.shape[1]
@@ -540,7 +569,7 @@ def qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v
                                      positions.data_ptr(), rope_cache.data_ptr(), _ptr(q_norm_w), _ptr(k_norm_w),
                                      k_cache.data_ptr(), v_cache.data_ptr(), slot_mapping.data_ptr(), T, Hq, Hkv, D,
                                      rotary_dim, bs, kv_mode, 1 if norm_plus_one else 0, float(eps), float(k_scale),
-                                     float(v_scale), _stream()), "rope_kv_write")
+                                     float(v_scale), _stream(), int(norm_dim or D)), "rope_kv_write")
     return q
 
 
@@ -557,7 +586,7 @@ def decode_splits(B: int, hkv: int, max_seq_len: int, sms: int) -> int:
     return int(max(1, min((2 * sms + ctas - 1) // ctas, (pages + 7) // 8, 64)))
 
 
-def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk=0, sinks=None):
+def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk=0, sinks=None, softcap=0.0):
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     d = _dev(q)
@@ -573,11 +602,11 @@ def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding
         raise KernelError("attention sinks are one fp32 value per query head")
     if k_cache.dtype == torch.float32:
         from . import cuda_recurrent
-        return cuda_recurrent.attention_f32(q, k_cache, v_cache, batch, scale, window, int(chunk), sinks)
+        return cuda_recurrent.attention_f32(q, k_cache, v_cache, batch, scale, window, int(chunk), sinks, float(softcap))
     if k_cache.dtype == torch.bfloat16:
-        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, chunk=int(chunk), sinks=sinks)
-    if chunk or sinks is not None:
-        raise KernelError("chunked attention and softmax sinks need a bf16 or fp32 KV cache")
+        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, chunk=int(chunk), sinks=sinks, softcap=float(softcap))
+    if chunk or sinks is not None or softcap:
+        raise KernelError("chunked attention, softmax sinks and bounded scores need a bf16 or fp32 KV cache")
     if is_nvfp4_kv(k_cache):
         return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=(float(k_scale), float(v_scale)))
     if nd > 0:
@@ -694,7 +723,7 @@ def _tc_tiles(q, batch, nd: int, tok: int):
     return tiles
 
 
-def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None, chunk=0, sinks=None):
+def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None, chunk=0, sinks=None, softcap=0.0):
     """bf16 KV cache (or, with ``scales = (k_scale, v_scale)``, an NVFP4 one): the general mma.sync kernel serves decode
     rows (split-K + merge) and prefill tiles."""
     T, Hq, D = q.shape
@@ -711,8 +740,8 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
         raise KernelError("the NVFP4 KV cache is implemented for head_dim 128")
     if not getattr(L, "_kv16_bound", False):
         L.atlas_attn_decode_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i,
-                                             _vp, _vp, _vp, _i, _vp]
-        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp, _i, _vp]
+                                             _vp, _vp, _vp, _i, _vp, _f]
+        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp, _i, _vp, _f]
         L._kv16_bound = True
     bt, st, nd = batch.block_tables, _stream(), batch.num_decodes
     if nd > 0:
@@ -731,18 +760,18 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
             _check(L.atlas_attn_decode_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                             bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                             0, nd, float(scale), Hq, Hkv, D, bs, window, splits, _ptr(po), _ptr(pml), st, chunk,
-                                            _ptr(sinks)), "attn_decode_kv16")
-    if batch.num_seqs > nd and not fp4 and _TC_PREFILL and not window and bs == 16 and D <= 128 and Hq // Hkv <= 128:
+                                            _ptr(sinks), softcap), "attn_decode_kv16")
+    if batch.num_seqs > nd and not fp4 and _TC_PREFILL and bs == 16 and D <= 128 and Hq // Hkv <= 128:
         # tcgen05 tiles of 128 // G query tokens; 1 = a shape the kernel does not take
         tdev, n_tiles, _ = _tc_tiles(q, batch, nd, 128 // (Hq // Hkv))
         if not getattr(L, "_tc16_bound", False):
             L.atlas_attn_prefill_tc16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _i, _i,
-                                                  _i, _vp, _vp, _vp]
+                                                  _i, _i, _vp, _f, _vp, _vp]
             L._tc16_bound = True
         rc = L.atlas_attn_prefill_tc16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                        bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                        tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, T, float(scale), Hq, Hkv, D, bs, chunk,
-                                       _ptr(sinks), _status_ptr[d], st)
+                                       window, _ptr(sinks), softcap, _status_ptr[d], st)
         if rc != 1:
             _check(rc, "attn_prefill_tc16")
             return out
@@ -767,7 +796,7 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
             _check(L.atlas_attn_prefill_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                              bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                              tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, float(scale), Hq, Hkv, D, bs, window, st, chunk,
-                                             _ptr(sinks)), "attn_prefill_kv16")
+                                             _ptr(sinks), softcap), "attn_prefill_kv16")
     return out
 
 
@@ -865,9 +894,9 @@ def moe_route(logits, top_k, norm_topk, scoring, bias=None, n_group=0, topk_grou
     return cuda_ext.moe_route(logits, top_k, norm_topk, scoring, bias, n_group, topk_group, scale, hash_table, token_ids)
 
 
-def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode):
+def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation="silu_glu", rows_ok=False):
     from . import cuda_ext
-    return cuda_ext.moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode)
+    return cuda_ext.moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation=activation, rows_ok=rows_ok)
 
 
 def gdn_forward(layer, mixed, a, b, batch, state, commit):
@@ -900,9 +929,34 @@ def wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted
     return cuda_recurrent.wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted_rows)
 
 
-def group_norm_gate(y, z, w, group, eps, gate_first):
+def mlstm_forward(layer, q, k, v, raw, batch, state, commit):
     from . import cuda_recurrent
-    return cuda_recurrent.group_norm_gate(y, z, w, group, eps, gate_first)
+    return cuda_recurrent.mlstm_forward(layer, q, k, v, raw, batch, state, commit)
+
+
+def mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_rows):
+    from . import cuda_recurrent
+    return cuda_recurrent.mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_rows)
+
+
+def latent_attention(layer, q, ckv, batch, cache, rope_cache):
+    from . import cuda_latent
+    return cuda_latent.latent_attention(layer, q, ckv, batch, cache, rope_cache)
+
+
+def group_norm_gate(y, z, w, group, eps, gate_first, gate="silu", den=None):
+    from . import cuda_recurrent
+    return cuda_recurrent.group_norm_gate(y, z, w, group, eps, gate_first, gate, den)
+
+
+def add_normed(stream, delta, eps, plus_one, out_norm, write):
+    from . import cuda_recurrent
+    return cuda_recurrent.add_normed(stream, delta, eps, plus_one, out_norm, write)
+
+
+def head_gate(x, g):
+    from . import cuda_recurrent
+    return cuda_recurrent.head_gate(x, g)
 
 
 def hyper_norm(streams, delta, read, norm_w, eps, write):

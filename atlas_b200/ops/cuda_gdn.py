@@ -56,6 +56,7 @@ class _Meta:
         self.limit = dev[o:o + B] if limit is not None else None
         self.has = torch.tensor([1 if h else 0 for h in has_state], dtype=torch.uint8).pin_memory().to(device, non_blocking=True)
         self.B, self.T, self.snaps = B, len(seq_of), snaps
+        self.longest = max(qlens, default=0)
         # every sequence brings exactly one row and no row limit or snapshot applies (decode)
         self.one_row = int(limit is None and self.snaps == 0 and all(n == 1 for n in qlens))
         # the chunked (64-token, tensor-core) kernel takes prefill-sized steps (a snapshot row just ends a chunk early)
@@ -70,7 +71,7 @@ class _Meta:
         self.qsl, self.slots, self.has, self.limit = qsl, slots, live, None
         self.seq_of = torch.arange(n, dtype=torch.int32, device=slots.device)
         self.snap_rows = self.snap_slots = torch.zeros(1, dtype=torch.int32, device=slots.device)
-        self.B, self.T, self.snaps, self.chunk_ok, self.one_row = n, n, 0, False, 1
+        self.B, self.T, self.snaps, self.chunk_ok, self.one_row, self.longest = n, n, 0, False, 1, 1
         return self
 
 

@@ -1,5 +1,5 @@
 """Binding of the residual-stream, recurrence and 32-bit attention kernels (``csrc/streams.cu``, ``csrc/recurrent.cu``,
-``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
+``csrc/mlstm.cu``, ``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
 from __future__ import annotations
 
 import ctypes as C
@@ -25,11 +25,16 @@ def _lib():
         lib.atlas_mamba2_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp] + [_i] * 9 + [_vp]
         lib.atlas_wkv_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _vp, _vp, _vp,
                                        _vp, _vp, _vp] + [_i] * 7 + [_vp]
-        lib.atlas_group_norm_gate.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _i, _i, _vp]
+        lib.atlas_group_norm_gate.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _i, _i, _vp, _i, _vp]
+        lib.atlas_add_normed.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _i, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _f, _i, _vp]
+        lib.atlas_head_gate.argtypes = [_vp, _ll, _vp, _ll, _i, _i, _i, _i, _vp]
+        lib.atlas_mlstm_gates.argtypes = [_vp, _ll, _vp, _f] + [_vp] * 10 + [_i] * 4 + [_vp]
+        lib.atlas_mlstm_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll] + [_vp] * 7 + [_i] * 8 + [_vp]
+        lib.atlas_mlstm_chunk.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll] + [_vp] * 6 + [_i] * 6 + [_vp]
         lib.atlas_conv1d_bias_silu.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _vp]
         lib.atlas_conv1d_state.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]
-        lib.atlas_rope_kv_write_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp]
-        lib.atlas_attn_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp, _vp]
+        lib.atlas_rope_kv_write_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _f, _vp]
+        lib.atlas_attn_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp, _f, _vp]
         _bound = True
     return lib
 
@@ -102,15 +107,17 @@ def tanh_(x):
 
 
 # ----------------------------------------------------------------------------- recurrences
-def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool):
+def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool, gate: str = "silu", den=None):
     T, n = y.shape
     K._dev(y)
     f32 = _f32(y)
     assert z.dtype == y.dtype and z.shape == y.shape and z.stride(1) == 1 and n % group == 0
+    assert den is None or (den.dtype == torch.float32 and den.is_contiguous() and den.numel() == T * (n // group))
     wf = w if w.dtype == torch.float32 else _float_cached(w)
     out = torch.empty(T, n, dtype=y.dtype, device=y.device)
     K._check(_lib().atlas_group_norm_gate(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), wf.data_ptr(), out.data_ptr(), n, T,
-                                          n // group, group, float(eps), 1 if gate_first else 0, f32, K._stream()), "group_norm_gate")
+                                          n // group, group, float(eps), 1 if gate_first else 0, 1 if gate == "sigmoid" else 0, K._ptr(den),
+                                          f32, K._stream()), "group_norm_gate")
     return out
 
 
@@ -186,21 +193,99 @@ def wkv_commit(layer, x, k, v, raw, qlens, slots, has_state, state, num_accepted
     _wkv_run(layer, x, None, k, v, raw, meta, state, True)
 
 
+MLSTM_CHUNKED = True         # tests switch this off to compare the two forms
+MLSTM_CHUNK_MIN_ROWS = 16    # longest portion of a step from which the chunked kernel takes the step
+
+
+def _mlstm_run(layer, q, k, v, raw, meta: _Meta, state, commit: bool):
+    lib, st = _lib(), K._stream()
+    K._dev(k)
+    f32 = _f32(k)
+    h, m = state["h"], state["m"]
+    T, H, dev = k.shape[0], layer.h, k.device
+    for t in (k, v) + ((q,) if q is not None else ()):
+        assert t.dtype == k.dtype and t.stride(1) == 1
+    assert raw.dtype == layer.gate_bias.dtype == torch.float32 and raw.stride(1) == 1
+    assert h.dtype == m.dtype == torch.float32 and h.is_contiguous() and m.is_contiguous()
+    la, lb, top = torch.empty(3, T, H, dtype=torch.float32, device=dev)
+    seq = (meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr())
+    snaps = (meta.snap_rows.data_ptr(), meta.snap_slots.data_ptr(), meta.snaps, meta.B)
+    K._check(lib.atlas_mlstm_gates(raw.data_ptr(), raw.stride(0), layer.gate_bias.data_ptr(), float(layer.cap), m.data_ptr(), la.data_ptr(),
+                                   lb.data_ptr(), top.data_ptr(), *seq, K._ptr(meta.limit), *snaps, H, 1 if commit else 0, st), "mlstm_gates")
+    num = den = None
+    if q is not None:
+        num = torch.empty(T, layer.nv, dtype=k.dtype, device=dev)
+        den = torch.empty(T, H, dtype=torch.float32, device=dev)
+    rows = (K._ptr(q), q.stride(0) if q is not None else 0, k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), la.data_ptr(), lb.data_ptr(),
+            top.data_ptr(), float(layer.scale), h.data_ptr(), K._ptr(num), layer.nv, K._ptr(den)) + seq
+    rc = 1
+    if MLSTM_CHUNKED and not f32 and q is not None and meta.limit is None and meta.T >= MLSTM_CHUNK_MIN_ROWS and meta.longest >= MLSTM_CHUNK_MIN_ROWS:
+        rc = lib.atlas_mlstm_chunk(*rows, *snaps, H, layer.v, layer.d, 1 if commit else 0, st)
+        if rc != 1:
+            K._check(rc, "mlstm_chunk")
+    if rc == 1:
+        K._check(lib.atlas_mlstm_scan(*rows, K._ptr(meta.limit), *snaps, H, layer.v, layer.d, 1 if commit else 0, meta.one_row, f32, st),
+                 "mlstm_scan")
+    return num, den
+
+
+def mlstm_forward(layer, q, k, v, raw, batch, state, commit):
+    return _mlstm_run(layer, q, k, v, raw, step_meta(batch, k.device), state, commit)
+
+
+def mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_rows):
+    meta = _Meta(qlens, slots, has_state, k.device, None, limit=list(num_accepted_rows))
+    _mlstm_run(layer, None, k, v, raw, meta, state, True)
+
+
+# ----------------------------------------------------------------------------- normed outputs on an fp32 residual
+def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool, out_norm, write: bool):
+    rows = delta.y if hasattr(delta.y, "slot_of") else None
+    y = rows.y if rows is not None else delta.y
+    W = y.shape[1]
+    T = rows.w.shape[0] if rows is not None else y.shape[0]
+    K._dev(y)
+    f32 = _f32(y)
+    if stream is None:
+        assert delta.norm is None
+        stream, write = torch.empty(T, W, dtype=torch.float32, device=y.device), True
+    assert stream.dtype == torch.float32 and stream.shape == (T, W) and stream.is_contiguous()
+    for w in (delta.norm, out_norm):
+        assert w is None or (w.dtype == torch.float32 and w.numel() == W and w.is_contiguous())
+    if rows is not None:
+        assert rows.slot_of.dtype == torch.int32 and rows.w.dtype == torch.float32 and rows.w.is_contiguous()
+    out = torch.empty(T, W, dtype=y.dtype, device=y.device)
+    K._check(_lib().atlas_add_normed(stream.data_ptr(), W, y.data_ptr(), y.stride(0), K._ptr(rows.slot_of) if rows is not None else None,
+                                     K._ptr(rows.w) if rows is not None else None, rows.w.shape[1] if rows is not None else 0,
+                                     K._ptr(delta.norm), K._ptr(out_norm), out.data_ptr(), W, T, W, 1 if plus_one else 0, 1 if write else 0,
+                                     float(eps), f32, K._stream()), "add_normed")
+    return out, stream
+
+
+def head_gate(x, g):
+    T, H, D = x.shape
+    K._dev(x)
+    assert x.stride(2) == 1 and x.stride(1) == D and g.dtype == torch.float32 and g.shape == (T, H) and g.stride(1) == 1
+    K._check(_lib().atlas_head_gate(x.data_ptr(), x.stride(0), g.data_ptr(), g.stride(0), T, H, D, _f32(x), K._stream()), "head_gate")
+    return x
+
+
 # ----------------------------------------------------------------------------- 32-bit attention
-def rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping):
+def rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm, k_norm, norm_dim, plus_one, eps):
     T, Hq, D = q.shape
     Hkv = k.shape[1]
     K._dev(q)
     assert q.stride(2) == 1 and q.stride(1) == k.stride(1) == v.stride(1) == D and k_cache.dtype == torch.float32
     assert positions.dtype == slot_mapping.dtype == torch.int32 and rope_cache.dtype == torch.float32
+    assert q_norm is None or (q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.numel() == k_norm.numel() == D)
     K._check(_lib().atlas_rope_kv_write_f32(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
                                             positions.data_ptr(), rope_cache.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
-                                            slot_mapping.data_ptr(), T, Hq, Hkv, D, rotary_dim, k_cache.shape[1], K._stream()),
-             "rope_kv_write_f32")
+                                            slot_mapping.data_ptr(), T, Hq, Hkv, D, rotary_dim, k_cache.shape[1], K._ptr(q_norm),
+                                            K._ptr(k_norm), int(norm_dim), 1 if plus_one else 0, float(eps), K._stream()), "rope_kv_write_f32")
     return q
 
 
-def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, sinks):
+def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, sinks, softcap: float = 0.0):
     T, Hq, D = q.shape
     K._dev(q)
     assert k_cache.dtype == torch.float32 and q.stride(2) == 1 and q.stride(1) == D
@@ -209,5 +294,5 @@ def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, si
     K._check(_lib().atlas_attn_f32(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                    bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                    batch.num_seqs, T, float(scale), Hq, k_cache.shape[2], D, k_cache.shape[1], window, chunk,
-                                   K._ptr(sinks), K._stream()), "attn_f32")
+                                   K._ptr(sinks), softcap, K._stream()), "attn_f32")
     return out

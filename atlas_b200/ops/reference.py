@@ -124,9 +124,10 @@ def apply_rope(x: torch.Tensor, positions: torch.Tensor, cache: torch.Tensor, ro
     return out.to(x.dtype)
 
 
-def head_rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, plus_one: bool) -> torch.Tensor:
+def head_rmsnorm(x: torch.Tensor, w: torch.Tensor, eps: float, plus_one: bool, dim: int = 0) -> torch.Tensor:
+    """``dim``: channels the mean counts (0 = all)."""
     xf = x.float()
-    var = xf.pow(2).mean(-1, keepdim=True)
+    var = xf.pow(2).sum(-1, keepdim=True) / (dim or x.shape[-1])
     wf = w.float() + 1.0 if plus_one else w.float()
     return (xf * torch.rsqrt(var + eps) * wf).to(x.dtype)
 
@@ -155,15 +156,15 @@ def qk_norm_rope_kv_write(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos
                           k_cache: torch.Tensor, v_cache: torch.Tensor, slot_mapping: torch.Tensor,
                           k_scale: float = 1.0, v_scale: float = 1.0,
                           q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None,
-                          eps: float = 1e-6, norm_plus_one: bool = False, rotate: bool = False) -> torch.Tensor:
+                          eps: float = 1e-6, norm_plus_one: bool = False, rotate: bool = False, norm_dim: int = 0) -> torch.Tensor:
     """Fused (q/k head RMSNorm) + RoPE + (head rotation) + (FP8 quant) + paged cache write.
 
     ``q [T,Hq,D]``, ``k,v [T,Hkv,D]``.  Returns the roped ``q``; k/v go to the cache at
     ``slot_mapping`` (rows with slot < 0 are skipped).
     """
     if q_norm_w is not None:
-        q = head_rmsnorm(q, q_norm_w, eps, norm_plus_one)
-        k = head_rmsnorm(k, k_norm_w, eps, norm_plus_one)
+        q = head_rmsnorm(q, q_norm_w, eps, norm_plus_one, norm_dim)
+        k = head_rmsnorm(k, k_norm_w, eps, norm_plus_one, norm_dim)
     q = apply_rope(q, positions, rope_cache, rotary_dim)
     k = apply_rope(k, positions, rope_cache, rotary_dim)
     if rotate:
@@ -186,11 +187,11 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     block_tables: torch.Tensor, seq_lens: torch.Tensor, query_start_loc: torch.Tensor,
                     scale: float, k_scale: float = 1.0, v_scale: float = 1.0,
                     sliding_window: Optional[int] = None, chunk: int = 0,
-                    sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
     """Causal attention of new query rows over the paged cache (prefill chunks and decode alike).
 
     ``chunk`` > 0 limits a row to keys of its own ``chunk``-token block (counted from the sequence's first token);
-    ``sinks [Hq]`` adds ``exp(sink)`` to every row's softmax denominator.
+    ``sinks [Hq]`` adds ``exp(sink)`` to every row's softmax denominator; ``softcap`` > 0 bounds the scores.
 
     Sequence ``b`` owns query rows ``query_start_loc[b]:query_start_loc[b+1]``; its last row sits
     at position ``seq_lens[b]-1``.  ``q [T,Hq,D]`` -> ``out [T,Hq,D]``.
@@ -212,6 +213,8 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         vv = v_cache[blocks].reshape(nblk * bs, Hkv, D)[:L].float() * v_scale
         qq = q[q0:q1].float().view(ql, Hkv, G, D)
         s = torch.einsum("qhgd,khd->hgqk", qq, kk) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(L - ql, L, device=q.device)[:, None]
         kpos = torch.arange(L, device=q.device)[None, :]
         mask = kpos <= qpos
@@ -261,13 +264,96 @@ def wkv_scan(r, k, v, decay, u, h):
     return torch.stack(out), h
 
 
-def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool):
-    """``norm(y * silu(z)) * w`` or ``norm(y) * w * silu(z)``, RMS over groups of ``group`` channels."""
-    gate = F.silu(z.float())
-    v = y.float() * gate if gate_first else y.float()
+def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool, gate: str = "silu", den=None):
+    """``norm(y * gate(z)) * w`` or ``norm(y) * w * gate(z)``, RMS over groups of ``group`` channels, each divided by ``den`` first."""
+    gz = (torch.sigmoid if gate == "sigmoid" else F.silu)(z.float())
+    v = y.float() * gz if gate_first else y.float()
     g = v.reshape(*v.shape[:-1], -1, group)
+    if den is not None:
+        g = g / den[..., None]
     v = (g * torch.rsqrt(g.pow(2).mean(-1, keepdim=True) + eps)).reshape(v.shape) * w.float()
-    return (v if gate_first else v * gate).to(y.dtype)
+    return (v if gate_first else v * gz).to(y.dtype)
+
+
+# ----------------------------------------------------------------------------- mLSTM, latent attention, normed outputs
+MLSTM_EPS = 1e-6            # joins the denominator of the memory's output
+
+
+def mlstm_gates(raw, bias, cap: float, m):
+    """Raw gates ``[T, 2 H]`` (input, forget) -> per row the log factors on the old state and on the new token, and the running
+    maximum: ``la = f + m_prev - m <= 0``, ``lb = i - m <= 0``, ``m`` (all ``[T, H]``).  ``m`` carries on from ``m [H]``."""
+    z = cap * torch.tanh((raw.float() + bias) / cap)
+    i, f = z.chunk(2, -1)
+    f = F.logsigmoid(f)
+    la, lb, ms = [], [], []
+    for t in range(raw.shape[0]):
+        new = torch.maximum(f[t] + m, i[t])
+        la.append(f[t] + m - new)
+        lb.append(i[t] - new)
+        ms.append(new)
+        m = new
+    return torch.stack(la), torch.stack(lb), torch.stack(ms)
+
+
+def mlstm_scan(q, k, v, la, lb, h):
+    """Sequential memory.  ``q`` (scaled), ``k [T, H, D]``, ``v [T, H, V]``, ``h [H, V + 1, D]`` (last row: the normaliser) ->
+    ``(S q [T, H, V], n . q [T, H], h)``."""
+    one = torch.ones(v.shape[1], 1, dtype=v.dtype, device=v.device)
+    out = []
+    for t in range(k.shape[0]):
+        new = torch.cat([v[t], one], -1)[:, :, None] * k[t][:, None, :]
+        h = h * torch.exp(la[t])[:, None, None] + torch.exp(lb[t])[:, None, None] * new
+        out.append((h * q[t][:, None, :]).sum(-1))
+    o = torch.stack(out)
+    return o[..., :-1], o[..., -1], h
+
+
+def latent_rows(ckv, q_rope, norm_w, rank: int, rp: int, ep: int, positions, rope_cache, rotary: int, eps: float):
+    """``(cache rows [T, rp + ep], rotated query parts [T, H, ep])`` of a step, fp32, zero-padded to the cache row's widths."""
+    c = ckv[:, :rank].float()
+    c = c * torch.rsqrt(c.pow(2).mean(-1, keepdim=True) + eps) * norm_w
+    turn = (lambda x: apply_rope(x.float(), positions, rope_cache, rotary)) if rotary else (lambda x: x.float())
+    r = turn(ckv[:, None, rank:])[:, 0]
+    pad = lambda x, n: F.pad(x, (0, n - x.shape[-1]))
+    return torch.cat([pad(c, rp), pad(r, ep)], -1), pad(turn(q_rope), ep)
+
+
+def latent_attention(q, cache, rp: int, block_tables, seq_lens, query_start_loc, scale: float, window: Optional[int] = None):
+    """Absorbed form: ``q [T, H, rp + ep]`` against cache rows of the same width, values the rows' first ``rp`` numbers."""
+    out = torch.zeros(*q.shape[:2], rp, dtype=torch.float32, device=q.device)
+    qsl, sl, bs = query_start_loc.tolist(), seq_lens.tolist(), cache.shape[1]
+    for b, L in enumerate(sl):
+        q0, q1 = qsl[b], qsl[b + 1]
+        n = q1 - q0
+        if n <= 0 or L <= 0:
+            continue
+        rows = cache[block_tables[b, :(L + bs - 1) // bs].long()].reshape(-1, cache.shape[-1])[:L].float()
+        s = torch.einsum("qhw,kw->hqk", q[q0:q1].float(), rows) * scale
+        qpos, kpos = torch.arange(L - n, L, device=q.device)[:, None], torch.arange(L, device=q.device)[None, :]
+        see = kpos <= qpos
+        if window:
+            see &= kpos > qpos - window
+        p = torch.softmax(s.masked_fill(~see, float("-inf")), -1)
+        out[q0:q1] = torch.einsum("hqk,kr->qhr", p, rows[:, :rp])
+    return out
+
+
+def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool):
+    """See ``ops.add_normed``."""
+    if hasattr(delta.y, "slot_of"):
+        e = delta.y
+        T, k = e.w.shape
+        slots = e.slot_of.view(T, k).long()
+        picked = e.y.float()[slots.clamp_min(0)] * (slots >= 0)[..., None]
+        y, dtype = (picked * e.w[..., None]).sum(1), e.y.dtype
+    else:
+        y, dtype = delta.y.float(), delta.y.dtype
+    unit = lambda t, w: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + 1.0 if plus_one else w.float())
+    x = y.clone() if delta.norm is None else stream + unit(y, delta.norm)
+    if write and stream is not None:
+        stream.copy_(x)
+    h = x if out_norm is None else unit(x, out_norm)
+    return h.to(dtype), (x if stream is None else stream)
 
 
 # ----------------------------------------------------------------------------- activations
@@ -357,11 +443,19 @@ def _topk_low_ties(x: torch.Tensor, k: int) -> torch.Tensor:
     return torch.sort(x, dim=-1, descending=True, stable=True).indices[..., :k]
 
 
+def expert_act(h: torch.Tensor, activation: str) -> torch.Tensor:
+    """``silu_glu``: silu(gate) * up of ``[gate | up]``; ``relu2``: squared relu of a single up projection."""
+    if activation == "relu2":
+        return torch.relu(h).square()
+    i = h.shape[-1] // 2
+    return F.silu(h[..., :i]) * h[..., i:]
+
+
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
-                topk_ids: torch.Tensor, expert_lo: int = 0) -> torch.Tensor:
+                topk_ids: torch.Tensor, expert_lo: int = 0, activation: str = "silu_glu") -> torch.Tensor:
     """Dense-math MoE over local experts ``[expert_lo, expert_lo+E_local)``.
 
-    ``w13 [E,2I,H]`` (gate rows then up rows), ``w2 [E,H,I]`` already dequantized.
+    ``w13 [E,2I,H]`` (gate rows then up rows; ``relu2``: ``[E,I,H]``), ``w2 [E,H,I]`` already dequantized.
     Tokens routed to non-local experts contribute zero (their owner rank adds them).
     """
     T, H = x.shape
@@ -375,8 +469,7 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
             continue
         wgt = (topk_w * sel).sum(-1)[tok]
         h = xf[tok] @ w13[e].float().t()
-        i = h.shape[-1] // 2
-        a = (F.silu(h[:, :i]) * h[:, i:]).to(x.dtype).float()
+        a = expert_act(h, activation).to(x.dtype).float()
         y = a @ w2[e].float().t()
         out.index_add_(0, tok, y * wgt[:, None])
     return out.to(x.dtype)

@@ -14,6 +14,7 @@ import numpy as np
 import torch
 
 from .config import EngineConfig
+from .layers import LatentAttention
 from .models import CacheStore, DecoderLM, ForwardBatch
 from .models.decoder import attention_of, recurrent_of
 from .sched import SchedulerOutput
@@ -44,7 +45,7 @@ class ModelRunner:
         self._pin_turn: Dict[str, int] = {}
         # decode graphs of recurrent models read state slots from a device buffer; the kernels that take everything they
         # need from there are those of recurrent.cu
-        self._states_graph_safe = all(l.kind in ("mamba2", "wkv", "parallel") for l in model.layers if recurrent_of(l) is not None)
+        self._states_graph_safe = all(l.kind in ("mamba2", "wkv", "parallel", "mlstm") for l in model.layers if recurrent_of(l) is not None)
         # slot of padding rows: the last one, which the engine allocates beyond those it hands out
         self.pad_state_slot = next((t.shape[0] - 1 for st in cache.states.values() for t in st.values()), None)
         if self.on_gpu:
@@ -71,7 +72,16 @@ class ModelRunner:
         top = max(self.graph_batch_sizes())            # eager mixed steps can carry any number of decode rows up to this
         sizes = list(range(1, top + 1))
         po = pml = 0
+        latent = [m for m in mixers if isinstance(m, LatentAttention)]
+        if latent:
+            from .ops import cuda_latent
+            lo, lml = (max(x) for x in zip(*(cuda_latent.scratch_bytes(sizes, m, self.cfg.max_seq_len, sms) for m in latent)))
+            if lo:
+                K.reserve_scratch("latent_part_o", lo, self.device)
+                K.reserve_scratch("latent_part_ml", lml, self.device)
         for m in mixers:
+            if isinstance(m, LatentAttention):
+                continue
             a, b = K.attention_scratch_bytes(sizes, m.hq, m.hkv, m.d, self.cfg.max_seq_len, sms)
             po, pml = max(po, a), max(pml, b)
         if po:
