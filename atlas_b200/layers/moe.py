@@ -74,6 +74,8 @@ class ExpertWeights:
 
     @staticmethod
     def from_dense(w13: torch.Tensor, w2: torch.Tensor, kind: str) -> "ExpertWeights":
+        if kind == "fp8_block" and (w13.shape[2] % 128 or w2.shape[2] % 128):
+            kind = "dense"                             # rows that are not whole quantisation groups stay as they are
         if kind in ("dense", "none"):
             return ExpertWeights("dense", w13.contiguous(), w2.contiguous())
         E = w13.shape[0]

@@ -8,6 +8,7 @@ model.
 """
 from __future__ import annotations
 
+import gc
 from typing import Dict, List, Optional, Tuple
 
 import numpy as np
@@ -347,8 +348,17 @@ class _DecodeGraph:
             from .ops import cuda as K
             K.freeze_scratch()
             n0 = K.launch_count
-            with torch.cuda.graph(self.graph):
-                self.out = r.model.forward(fb, r.cache)
+            # a collection during the capture could destroy events, pinned buffers or graphs of other engines, which the
+            # capturing stream forbids
+            gc.collect()
+            collecting = gc.isenabled()
+            gc.disable()
+            try:
+                with torch.cuda.graph(self.graph):
+                    self.out = r.model.forward(fb, r.cache)
+            finally:
+                if collecting:
+                    gc.enable()
             self.num_kernels = K.launch_count - n0
             self._load(b)
         self.graph.replay()

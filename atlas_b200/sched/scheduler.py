@@ -44,6 +44,7 @@ class Scheduler:
         self.running: List[Sequence] = []
         self.finished_queue: List[Sequence] = []
         self.num_preemptions = 0
+        self._fresh_snapshots: set = set()        # snapshot slots that the step being planned will fill
         self.snapshot_interval = max(self.bs, (cfg.ssm_checkpoint_interval + self.bs - 1) // self.bs * self.bs)
         self._last_decode_time: Optional[float] = None
 
@@ -231,7 +232,9 @@ class Scheduler:
         need = self._admission_blocks(seq, cached)
         avail = self.pool.num_free + (self.radix.evictable_blocks() if self.radix is not None else 0)
         avail -= self._outstanding_prefill_blocks()
-        if need > avail:
+        # a snapshot planned in this step is filled by this step's forward: whoever wants it is admitted in the next one
+        fresh = match is not None and match.snapshot_slot is not None and match.snapshot_slot in self._fresh_snapshots
+        if need > avail or fresh:
             if match is not None and match.nodes:
                 self.radix.release(match.nodes)
                 self.pool.free(match.blocks)
@@ -258,6 +261,7 @@ class Scheduler:
         """``now`` / ``expire=False`` let a multi-process leader impose its clock and its expiry decisions on the
         follower replicas so that every rank plans the same step."""
         out = SchedulerOutput()
+        self._fresh_snapshots.clear()
         cfg = self.cfg
         now = time.monotonic() if now is None else now
         if expire:
@@ -404,6 +408,7 @@ class Scheduler:
                 continue
             slot = self.radix.attach_snapshot(nodes[-1])
             if slot is not None:
+                self._fresh_snapshots.add(slot)
                 out.snapshot_requests.append((item_index, p - lo, slot))
 
     def expire(self, now: float) -> List[Sequence]:

@@ -1,0 +1,504 @@
+"""Tomizen on the GPU: every kernel of its mechanisms against the plain statement, then whole models through the engine in
+bf16 and fp32 (portions, unequal batches, reused pages and slots, decode graphs, generation)."""
+import math
+from types import SimpleNamespace
+
+import pytest
+import torch
+
+import tomizen_cases as TC
+import tomizen_oracle as O
+
+pytestmark = pytest.mark.gpu
+DTYPES = [torch.bfloat16, torch.float32]
+REL = {torch.bfloat16: 1.2e-2, torch.float32: 2e-5}
+
+
+def rnd(*shape, seed=0, std=1.0):
+    return torch.randn(*shape, generator=torch.Generator().manual_seed(seed)) * std
+
+
+def close(got, want, dtype, what="", factor=1.0):
+    got, want = got.detach().cpu().double(), want.double()
+    err = (got - want).abs().max().item()
+    assert err <= factor * REL[dtype] * max(want.abs().max().item(), 1e-3), f"{what}: {err} of {want.abs().max().item()}"
+
+
+def batch_of(lens, live, slots):
+    """The part of a ForwardBatch that recurrent layers read."""
+    return SimpleNamespace(query_lens_host=list(lens), state_slots_host=list(slots), has_state_host=list(live), snapshot_plan={})
+
+
+# ------------------------------------------------------------------------------------------------- norms and gates
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("W,T", [(64, 3), (90, 4), (2048, 5), (1101, 2), (12288, 2)])
+def test_add_normed(dtype, W, T):
+    from atlas_b200 import ops
+    eps = 1e-5
+    x, y = rnd(T, W, seed=1, std=3.0), rnd(T, W, seed=2).to(dtype)
+    w, ow = rnd(W, seed=3, std=0.3), rnd(W, seed=4, std=0.3)
+    slots = torch.tensor([[3, -1, 0], [1, 2, 4], [0, 0, 5], [6, -1, -1], [2, 7, 1]], dtype=torch.int32)[:T]
+    rows, pick = rnd(8, W, seed=5).to(dtype), rnd(T, 3, seed=6).abs()
+    summed = sum(rows.double()[slots[:, j].clamp_min(0).long()] * (slots[:, j] >= 0)[:, None] * pick[:, j:j + 1].double() for j in range(3))
+    experts = ops.ExpertRows(rows.cuda(), slots.reshape(-1).cuda(), pick.cuda())
+    for plus in (True, False):
+        norm = lambda t, k: O.output_norm(t, k.double() - (0.0 if plus else 1.0), eps)
+        for arg, plain in ((y.cuda(), y.double()), (experts, summed)):
+            h, s = ops.add_normed(x.cuda(), ops.NormDelta(arg, w.cuda()), eps, plus)
+            want = x.double() + norm(plain, w)
+            close(s, want, torch.float32, "stream", factor=2)
+            close(h, want, dtype, "handed on")
+            h, s = ops.add_normed(x.cuda(), ops.NormDelta(arg, w.cuda()), eps, plus, ow.cuda(), write=False)
+            close(h, norm(want, ow), dtype, "normed again")
+            assert torch.equal(s.cpu(), x)
+    h, s = ops.add_normed(None, ops.NormDelta(y.cuda()), eps, True)
+    assert torch.equal(s.cpu(), y.float()) and torch.equal(h.cpu(), y)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("groups,size", [(1, 8), (3, 10), (4, 64), (16, 256), (2, 1100)])
+def test_group_norm_with_sigmoid_gate_and_denominator(dtype, groups, size):
+    from atlas_b200 import ops
+    n, eps = groups * size, 1e-5
+    y, zz, w, den = rnd(5, n, seed=1, std=1e-2).to(dtype), rnd(5, n + 6, seed=2).to(dtype), rnd(n, seed=3), rnd(5, groups, seed=4).abs() + 0.3
+    for off in (0, 3):
+        z = zz[:, off:off + n]
+        unit = O.unit_rms(y.double().view(5, groups, size) / den.double()[..., None], eps).reshape(5, n)
+        got = ops.group_norm_gate(y.cuda(), zz.cuda()[:, off:off + n], w.cuda(), size, eps, False, gate="sigmoid", den=den.cuda())
+        close(got, unit * w.double() * O.sigmoid(z.double()), dtype)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,D", [(1, 64), (5, 20), (6, 256)])
+def test_head_gate(dtype, H, D):
+    from atlas_b200 import ops
+    x, g = rnd(7, H, D).to(dtype), rnd(7, H + 2, seed=1, std=3.0)
+    close(ops.head_gate(x.cuda(), g.cuda()[:, 1:H + 1]), x.double() * O.sigmoid(g[:, 1:H + 1].double())[..., None], dtype)
+
+
+@pytest.mark.parametrize("T,K,N,main", [(1, 256, 100, 64), (5, 96, 77, 0), (130, 2048, 4100, 4096), (300, 136, 40, 40), (64, 1024, 130, 3), (9, 90, 21, 8)])
+def test_linear_with_an_fp32_tail(T, K, N, main):
+    """The tail keeps the product's fp32 sums: far closer to the exact product than a bf16 result."""
+    from atlas_b200 import ops
+    x, w = rnd(T, K).to(torch.bfloat16), rnd(N, K, seed=1, std=K ** -0.5).to(torch.bfloat16)
+    a, b = ops.linear_tail(x.cuda(), ops.LinearWeight("dense", w.cuda()), main)
+    want = x.double() @ w.double().T
+    assert a.dtype == torch.bfloat16 and b.dtype == torch.float32 and a.shape == (T, main) and b.shape == (T, N - main)
+    if main:
+        close(a, want[:, :main], torch.bfloat16)
+    if main < N:
+        close(b, want[:, main:], torch.float32, factor=2)
+
+
+# ------------------------------------------------------------------------------------------------- experts
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("T,H,I,E,top", [(1, 64, 64, 1, 1), (7, 128, 40, 6, 2), (150, 256, 192, 16, 4), (33, 100, 36, 5, 5), (700, 64, 128, 3, 1)])
+def test_experts_without_a_gate(dtype, T, H, I, E, top):
+    from atlas_b200 import ops
+    from atlas_b200.config import ModelConfig
+    from atlas_b200.layers import MoE, ParallelCtx
+    cfg = ModelConfig(hidden_size=H, num_experts=E, num_experts_per_tok=top, moe_intermediate_size=I, norm_topk_prob=False, router_f32=True,
+                      mlp_activation="relu2")
+    moe = MoE(cfg, ParallelCtx(), "dense", "dense")
+    router, up, down = rnd(E, H, seed=1, std=2 * H ** -0.5).to(dtype), rnd(E, I, H, seed=2, std=H ** -0.5).to(dtype), rnd(E, H, I, seed=3, std=I ** -0.5).to(dtype)
+    moe.load(router.cuda(), up.cuda(), down.cuda())
+    x = rnd(T, H, seed=4).to(dtype)
+    w = {"router": router.double()}
+    for e in range(E):
+        w[f"e{e}.up"], w[f"e{e}.down"] = up[e].double(), down[e].double()
+    want = O.experts(x.double(), w, "", {"router": {"top": top}})
+    close(moe.forward(ops.Act(x=x.cuda())), want, dtype, factor=1.5)
+    rows = moe.forward(ops.Act(x=x.cuda()), rows_ok=True)
+    assert isinstance(rows, ops.ExpertRows)
+    stream, nw = rnd(T, H, seed=5), rnd(H, seed=6, std=0.2)
+    _, s = ops.add_normed(stream.cuda(), ops.NormDelta(rows, nw.cuda()), 1e-5, True)
+    close(s - stream.cuda(), O.output_norm(want, nw.double(), 1e-5), dtype, factor=1.5)
+
+
+def test_router_scores_in_32_bit():
+    """Logits that differ by less than a bf16 step are told apart."""
+    from atlas_b200 import ops
+    from atlas_b200.config import ModelConfig
+    from atlas_b200.layers import MoE, ParallelCtx
+    H, E = 128, 4
+    moe = MoE(ModelConfig(hidden_size=H, num_experts=E, num_experts_per_tok=1, moe_intermediate_size=64, norm_topk_prob=False, router_f32=True,
+                          mlp_activation="relu2"), ParallelCtx(), "dense", "dense")
+    router = torch.zeros(E, H)
+    router[:, 0] = 64.0                                     # a large common part, then 1 / 16 for the winner of each row
+    for e in range(E):
+        router[e, 1 + e] = 0.0625
+    up = torch.zeros(E, 64, H)
+    up[:, :, 0] = 1.0
+    down = torch.stack([torch.full((H, 64), float(e + 1)) for e in range(E)])
+    moe.load(*(t.to(torch.bfloat16).cuda() for t in (router, up, down)))
+    x = torch.zeros(E, H)
+    x[:, 0] = 1.0
+    x[torch.arange(E), 1 + torch.arange(E)] = 1.0
+    y = moe.forward(ops.Act(x=x.to(torch.bfloat16).cuda())).float().cpu()
+    assert (y[:, 0] / y[0, 0]).sub(torch.arange(1, E + 1).float()).abs().max() < 0.05
+
+
+# ------------------------------------------------------------------------------------------------- mLSTM
+LENS = [([1, 1, 1], [True, False, True]), ([37, 1, 2, 18], [False, True, True, False]), ([64, 65, 130], [True, True, False]),
+        ([2, 2], [True, False])]
+
+
+@pytest.mark.parametrize("form", ["bf16 chunks", "bf16 scan", "fp32"])
+@pytest.mark.parametrize("lens,live", LENS, ids=["decode", "mixed", "chunk edges", "two rows"])
+@pytest.mark.parametrize("H,D,V", [(1, 8, 8), (3, 24, 40), (2, 64, 136), (2, 128, 64), (1, 200, 24), (1, 10, 7), (1, 256, 72), (1, 300, 16)])
+def test_matrix_memory(form, lens, live, H, D, V):
+    """State and running maximum carried in, unequal lengths, closed and open forget gates, input gates that jump."""
+    from atlas_b200.ops import cuda as K, cuda_recurrent as R
+    dtype = torch.float32 if form == "fp32" else torch.bfloat16
+    T, cap = sum(lens), 12.0
+    q, k = (rnd(T, H * D, seed=i).to(dtype) for i in range(2))
+    v = rnd(T, H * V, seed=2).to(dtype)
+    raw = rnd(T, 2 * H, seed=3, std=3.0)
+    bias = torch.cat([torch.full((H,), -1.0), torch.linspace(1.0, 6.0, H)])
+    raw[::7, H:] -= 12.0                                    # now and then nearly everything is forgotten
+    raw[5::11, :H] += 9.0
+    slots = [4, 1, 0, 2][:len(lens)]
+    h0, m0 = rnd(5, H, V + 1, D, seed=7), rnd(5, H, seed=8)
+    layer = SimpleNamespace(gate_bias=bias.cuda(), cap=cap, scale=D ** -0.5, nv=H * V, h=H, v=V, d=D)
+    state = {"h": h0.cuda(), "m": m0.cuda()}
+    args = [t.cuda() for t in (q, k, v, raw)]
+    R.MLSTM_CHUNKED = form == "bf16 chunks"
+    try:
+        dry = K.mlstm_forward(layer, *args, batch_of(lens, live, slots), state, False)
+        assert torch.equal(state["h"].cpu(), h0) and torch.equal(state["m"].cpu(), m0)
+        num, den = K.mlstm_forward(layer, *args, batch_of(lens, live, slots), state, True)
+    finally:
+        R.MLSTM_CHUNKED = True
+    assert torch.equal(dry[0], num) and torch.equal(dry[1], den)
+    i, f = O.log_gates((raw[:, :H] + bias[:H]).double(), (raw[:, H:] + bias[H:]).double(), cap)
+    got, t0 = num.cpu().double().view(T, H, V) / den.cpu().double()[..., None], 0
+    for n, a, s in zip(lens, live, slots):
+        rows = slice(t0, t0 + n)
+        at = (h0[s, :, :V].transpose(1, 2).double(), h0[s, :, V].double(), m0[s].double()) if a else None
+        want, (S, nn, m) = O.matrix_memory(q[rows].double().view(n, H, D) * D ** -0.5, k[rows].double().view(n, H, D),
+                                           v[rows].double().view(n, H, V), i[rows], f[rows], at)
+        # relative to each row: a row whose denominator is small is as exact as any other
+        err = (got[rows] - want).abs().amax(-1) / want.abs().amax(-1).clamp_min(1e-3)
+        assert err.max() < (1.5e-2 if dtype == torch.bfloat16 else 4e-4), (s, err.max())
+        tol = 2e-4 if form == "bf16 chunks" else 2e-5
+        assert (state["h"][s, :, :V].cpu().transpose(1, 2) - S).abs().max() < tol * S.abs().max()
+        assert (state["h"][s, :, V].cpu() - nn).abs().max() < tol * max(1.0, nn.abs().max())
+        assert (state["m"][s].cpu() - m).abs().max() < 1e-4
+        t0 += n
+    for s in set(range(5)) - set(slots):
+        assert torch.equal(state["h"][s].cpu(), h0[s]) and torch.equal(state["m"][s].cpu(), m0[s])
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_memory_snapshots_and_accepted_rows(dtype):
+    """A snapshot inside a portion and the fold of accepted rows both equal the state after exactly that many rows."""
+    from atlas_b200.ops import cuda as K
+    H, D, V, T, cut = 2, 32, 48, 100, 48
+    layer = SimpleNamespace(gate_bias=torch.tensor([0.0, 0.5, 3.0, 5.0]).cuda(), cap=9.0, scale=D ** -0.5, nv=H * V, h=H, v=V, d=D)
+    q, k, v = (rnd(T, H * n, seed=j).to(dtype).cuda() for j, n in enumerate((D, D, V)))
+    raw = rnd(T, 2 * H, seed=9, std=2.0).cuda()
+    fresh = lambda: {"h": torch.zeros(4, H, V + 1, D).cuda(), "m": torch.zeros(4, H).cuda()}
+    want, snap, part = fresh(), fresh(), fresh()
+    K.mlstm_forward(layer, q[:cut], k[:cut], v[:cut], raw[:cut], batch_of([cut], [False], [0]), want, True)
+    b = batch_of([T], [False], [0])
+    b.snapshot_plan = {0: [(cut, 3)]}
+    K.mlstm_forward(layer, q, k, v, raw, b, snap, True)
+    K.mlstm_commit(layer, k, v, raw, [T], [0], [False], part, [cut])
+    for n in want:
+        top = want[n][0].abs().max()
+        assert (snap[n][3] - want[n][0]).abs().max() < 1e-4 * top and (part[n][0] - want[n][0]).abs().max() < 1e-4 * top
+
+
+# ------------------------------------------------------------------------------------------------- attention
+REQS = [(150, 1), (97, 1), (64, 1), (210, 77), (49, 2), (40, 40), (300, 130), (129, 97)]      # (tokens after the step, new rows)
+
+
+def paged(reqs, nd):
+    bs = 16
+    nblk = sum((L + bs - 1) // bs for L, _ in reqs)
+    perm = torch.randperm(nblk, generator=torch.Generator().manual_seed(3)).tolist()
+    tables = torch.zeros(len(reqs), max((L + bs - 1) // bs for L, _ in reqs), dtype=torch.int32)
+    for i, (L, _) in enumerate(reqs):
+        blocks = [perm.pop() for _ in range((L + bs - 1) // bs)]
+        tables[i, :len(blocks)] = torch.tensor(blocks, dtype=torch.int32)
+    lens = [n for _, n in reqs]
+    qsl = torch.tensor([0] + lens).cumsum(0).to(torch.int32)
+    pos = torch.cat([torch.arange(L - n, L) for L, n in reqs]).to(torch.int32)
+    slot = torch.cat([tables[i][torch.arange(L - n, L) // bs].long() * bs + torch.arange(L - n, L) % bs for i, (L, n) in enumerate(reqs)])
+    batch = SimpleNamespace(block_tables=tables.cuda(), seq_lens=torch.tensor([L for L, _ in reqs], dtype=torch.int32).cuda(),
+                            query_start_loc=qsl.cuda(), num_decodes=nd, num_seqs=len(reqs), query_lens_host=lens,
+                            seq_lens_host=[L for L, _ in reqs], max_seq_len=max(L for L, _ in reqs), positions=pos.cuda(),
+                            slot_mapping=slot.to(torch.int32).cuda())
+    return batch, tables, nblk, qsl
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,G,D,cap,window", [(4, 2, 64, 5.0, 0), (3, 3, 128, 30.0, 0), (20, 1, 64, 2.0, 0), (6, 1, 256, 8.0, 0), (8, 1, 128, 20.0, 0),
+                                              (4, 4, 64, 0.0, 37), (2, 2, 128, 3.0, 128), (2, 1, 64, 0.0, 1)])
+def test_bounded_scores_and_windows(dtype, H, G, D, cap, window):
+    """Rows of prompts and decode rows over scattered pages.  Keys far back, at page borders and around every window's edge are
+    aligned with all queries: one of them too many or too few, or scores without their bound, change whole values."""
+    from atlas_b200 import ops
+    from atlas_b200.ops import cuda as K
+    batch, tables, nblk, qsl = paged(REQS, 3)
+    kc, vc = K.alloc_kv_cache(nblk, 16, G, D, dtype, "cuda")
+    dirn = torch.nn.functional.normalize(rnd(D, seed=11), dim=0) * math.sqrt(D)
+    scale, qs, ks, vs = D ** -0.5, [], [], []
+    for i, (L, n) in enumerate(REQS):
+        k, v, q = rnd(L, G, D, seed=20 + i, std=0.3), rnd(L, G, D, seed=40 + i), rnd(n, H, D, seed=60 + i, std=0.3) + dirn * 0.5
+        marks = set(range(0, L, 16)) | {1, 15, 17} | ({p for e in range(L - n, L) for p in (e - window, e - window + 1)} if window and n < 5 else set())
+        for p in marks:
+            if 0 <= p < L:
+                k[p] = dirn * (0.5 + 0.02 * (p % 13))
+        qs.append(q.to(dtype)); ks.append(k.to(dtype)); vs.append(v.to(dtype))
+        at = torch.arange(L)
+        kc[tables[i][at // 16].long().cuda(), (at % 16).cuda()] = ks[-1].cuda()
+        vc[tables[i][at // 16].long().cuda(), (at % 16).cuda()] = vs[-1].cuda()
+    run = lambda: ops.paged_attention(torch.cat(qs).cuda(), kc, vc, batch, scale, sliding_window=window or None, softcap=cap)
+    got = run()
+    for i, (L, n) in enumerate(REQS):
+        vis = (O.window(L, window) if window else O.causal(L))[L - n:]
+        for h in range(H):
+            s = (qs[i][:, h].double() @ ks[i][:, h // (H // G)].double().T) * scale
+            p = O.softmax_visible(O.soft_cap(s, cap) if cap else s, vis)
+            close(got[qsl[i]:qsl[i + 1], h], p @ vs[i][:, h // (H // G)].double(), dtype, f"request {i} head {h}", factor=2)
+    K._FORCE_DECODE_SPLITS, keep = 3, K._FORCE_DECODE_SPLITS        # decode split over several CTAs, as with a long context
+    try:
+        close(run(), got.cpu(), dtype, factor=1.5)
+    finally:
+        K._FORCE_DECODE_SPLITS = keep
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("D,dim", [(64, 64), (64, 40), (128, 72), (256, 130)])
+def test_head_norms_of_padded_heads(dtype, D, dim):
+    """The norm counts the head's own channels, not the zeros that pad it to the cache's width."""
+    from atlas_b200 import ops
+    from atlas_b200.ops import cuda as K
+    T, H, G, eps = 9, 3, 1, 1e-3
+    pad = lambda t: torch.nn.functional.pad(t, (0, D - dim))
+    q, k, v = rnd(T, H, dim, std=0.05).to(dtype), rnd(T, G, dim, seed=1, std=0.05).to(dtype), rnd(T, G, dim, seed=2).to(dtype)
+    qw, kw = rnd(dim, seed=3).to(dtype), rnd(dim, seed=4).to(dtype)
+    kc, vc = K.alloc_kv_cache(2, 16, G, D, dtype, "cuda")
+    slot, pos = torch.arange(3, 3 + T, dtype=torch.int32).cuda(), torch.arange(T, dtype=torch.int32).cuda()
+    got = ops.qk_norm_rope_kv_write(pad(q).cuda(), pad(k).cuda(), pad(v).cuda(), pos, torch.zeros(T, 0).cuda(), 0, kc, vc, slot, 1.0, 1.0,
+                                    pad(qw).cuda(), pad(kw).cuda(), eps, False, norm_dim=dim)
+    close(got[..., :dim], O.unit_rms(q.double(), eps) * qw.double(), dtype)
+    at = torch.arange(3, 3 + T)
+    close(kc[at // 16, at % 16][..., :dim], O.unit_rms(k.double(), eps) * kw.double(), dtype)
+    close(vc[at // 16, at % 16][..., :dim], v.double(), dtype)
+    assert got[..., dim:].abs().sum() == 0 and kc[..., dim:].abs().sum() == 0
+
+
+LATENT = [(4, 32, 32, 64, 64, 40), (1, 8, 2, 8, 8, 1), (20, 72, 20, 130, 136, 33), (3, 9, 6, 11, 13, 19), (16, 64, 64, 128, 512, 100), (6, 20, 12, 28, 96, 0),
+          (40, 32, 16, 32, 256, 128), (2, 16, 16, 16, 700, 50)]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,size", LATENT)
+def test_latent_attention(dtype, H, dim, rot, vdim, rank, size):
+    """Decode rows, short portions (absorbed form) and long ones (expanded form) of unequal requests over scattered pages.  Latents at
+    page borders and around the window's edges of the decode rows stand out for every head, so that one key too many or too few
+    moves the output by its whole value."""
+    from atlas_b200.config import _rotary_overrides
+    from atlas_b200.layers.mla import deinterleave_rows
+    from atlas_b200.layers import LatentAttention, ParallelCtx
+    from atlas_b200.config import ModelConfig
+    from atlas_b200.config import padded_head_width
+    from atlas_b200.ops import cuda as K, cuda_latent, reference as ref
+    eps = 1e-5
+    rd = {"dims": rot, "base": 1e3, "scaling": {"factor": 3.0, "original": 64, "fast": 8.0, "slow": 1.0}}
+    cfg = ModelConfig(hidden_size=64, num_attention_heads=H, num_key_value_heads=1, head_dim=dim + rot, qk_nope_head_dim=dim, qk_rope_head_dim=rot,
+                      v_head_dim=vdim, kv_lora_rank=rank, attn_scale=1.0, attn_cache_width=padded_head_width(dim + rot, vdim),
+                      sliding_window=size or None, rms_norm_eps=eps, **_rotary_overrides(rd))
+    lay = LatentAttention(cfg, 0, ParallelCtx(), "dense")
+    uk, uv = rnd(H * dim, rank, seed=1, std=rank ** -0.5).to(dtype), rnd(H * vdim, rank, seed=2, std=rank ** -0.5).to(dtype)
+    cn = rnd(rank, seed=3, std=0.2) + 1.0
+    lay.load(torch.zeros(H * (dim + rot), 64, dtype=dtype).cuda(), torch.zeros(rank + rot, 64, dtype=dtype).cuda(), cn.cuda(), uk.cuda(), uv.cuda(),
+             torch.zeros(64, H * vdim, dtype=dtype).cuda())
+    table = ref.build_rope_cache(rot, 400, rd["base"], cfg.rope_scaling).cuda()
+    batch, tables, nblk, qsl = paged(REQS, 3)
+    cache, _ = lay.alloc_kv(nblk, 16, dtype, "cuda")
+    lift = rnd(rank, seed=5)
+    aim = (uk.double().view(H, dim, rank) @ (O.unit_rms(lift.double(), eps) * cn.double()))          # what W_uk makes of the marked latent
+    aim = aim / aim.pow(2).sum(-1, keepdim=True).sqrt().clamp_min(1e-6)
+    turn = lambda x: deinterleave_rows(x.movedim(-1, 0), rot).movedim(0, -1)
+    qs, downs, wants = [], [], []
+    for i, (L, n) in enumerate(REQS):
+        down = rnd(L, rank + rot, seed=10 + i)
+        w = size or 50
+        marks = set(range(0, L, 16)) | {1, 15} | {p for e in range(L - n, L) for p in (e - w, e - w + 1)} if n < 5 else set(range(0, L, 9))
+        for p in marks:
+            if 0 <= p < L:
+                down[p, :rank] = lift + 0.05 * rnd(rank, seed=100 + p)
+        q = rnd(L, H, dim + rot, seed=30 + i, std=0.4)
+        q[..., :dim] += 3.0 * aim.float()
+        q, rows = q.to(dtype), slice(L - n, L)
+        d = down.double()
+        c = O.unit_rms(d[:, :rank], eps) * cn.double()
+        pos = torch.arange(L)
+        o = O.latent_heads(q.double()[..., :dim], O.rotate_pairs(q.double()[..., dim:], rd, pos), c, O.rotate_pairs(d[:, None, rank:], rd, pos)[:, 0],
+                           uk.double(), uv.double(), 1.0, O.window(L, size) if size else O.causal(L))
+        wants.append(o[rows])
+        qs.append(torch.cat([turn(q[rows, :, dim:]), q[rows, :, :dim]], -1).reshape(n, -1))
+        downs.append(torch.cat([down[:, :rank], turn(down[:, rank:])], -1))
+        if n < L:                                # what earlier steps have left in the cache
+            row, _ = ref.latent_rows(downs[-1], torch.zeros(L, 1, rot), cn, rank, lay.rp, lay.ep, pos, table.cpu(), rot, eps)
+            at = torch.arange(L - n)
+            cache[tables[i][at // 16].long().cuda(), (at % 16).cuda(), 0] = row[:L - n].to(dtype).cuda()
+    q, down = torch.cat(qs).cuda(), torch.cat([dn[-n:] for dn, (_, n) in zip(downs, REQS)]).cuda()
+    run = lambda: K.latent_attention(lay, q, down, batch, cache, table)
+    got = run().view(-1, H, vdim)
+    factor = 3 if dtype == torch.bfloat16 else 5
+    for i, (L, n) in enumerate(REQS):
+        close(got[qsl[i]:qsl[i + 1]], wants[i], dtype, f"request {i}", factor=factor)
+    if dtype == torch.bfloat16:
+        # the same rows in one form only, and with the keys of decode rows split
+        for rows, splits in ((10 ** 9, None), (2, None), (96, 3)):
+            keep = cuda_latent.EXPAND_MIN_ROWS, cuda_latent.decode_splits
+            cuda_latent.EXPAND_MIN_ROWS = rows
+            if splits:
+                cuda_latent.decode_splits = lambda *a: splits
+            batch._latent_plans = {}
+            try:
+                again = run().view(-1, H, vdim)
+            finally:
+                cuda_latent.EXPAND_MIN_ROWS, cuda_latent.decode_splits = keep
+            for i in range(len(REQS)):
+                close(again[qsl[i]:qsl[i + 1]], wants[i], dtype, f"request {i}, forms from {rows}", factor=factor)
+
+
+@pytest.mark.parametrize("rows,H,N,K_", [(1, 3, 64, 32), (5, 2, 100, 40), (65, 1, 16, 300), (130, 4, 72, 9)])
+def test_products_per_head(rows, H, N, K_):
+    from atlas_b200.ops import cuda as K, cuda_latent  # noqa: F401
+    x, w = rnd(rows + 3, H, K_ + 8).to(torch.bfloat16), rnd(H, N, K_, seed=1, std=K_ ** -0.5).to(torch.bfloat16)
+    pick = torch.randperm(rows + 3, generator=torch.Generator().manual_seed(1))[:rows].to(torch.int32)
+    out = torch.zeros(rows + 3, H, N + 4, dtype=torch.bfloat16).cuda()
+    K._dev(out)
+    cuda_latent._head_gemm(x.cuda(), H * (K_ + 8), K_ + 8, w.cuda(), out, H * (N + 4), N + 4, rows, in_rows=pick.cuda(), out_rows=pick.flip(0).contiguous().cuda(),
+                           offset=8)
+    want = torch.einsum("rhk,hnk->rhn", x.double()[pick.long(), :, 8:], w.double())
+    close(out[pick.flip(0).long()][..., :N], want, torch.bfloat16)
+    left = [r for r in range(rows + 3) if r not in set(pick.tolist())]
+    assert out[..., N:].abs().sum() == 0 and out[left].abs().sum() == 0
+
+
+# ------------------------------------------------------------------------------------------------- whole models
+@pytest.fixture(scope="module")
+def folder(tmp_path_factory):
+    root = tmp_path_factory.mktemp("tomizen_gpu")
+    made = {}
+
+    def get(name):
+        if name not in made:
+            path = str(root / name)
+            cfg, w = TC.write(path, name)
+            toks = {i: TC.tokens(cfg, n, i) for i, n in enumerate((150, 41, 90, 7))}
+            made[name] = (path, cfg, toks, {i: O.forward(cfg, w, t) for i, t in toks.items()}, w)
+        return made[name]
+    return get
+
+
+# fp32 is the sharp comparison.  In bf16 the choice of an expert can turn on rounding, which moves a whole token: the typical row is
+# compared there, and rows may not be off everywhere
+MODEL_TOL = {"bfloat16": 0.12, "float32": 3e-4}
+SHAPES = {"whole": [[1000], [1000], [1000], [1000]], "decode": [[100, 1], [9, 1], [1], [2, 1]], "portions": [[2, 33, 1, 16], [3, 2], [17, 24], [2]],
+          "long portions": [[110, 2], [40], [3, 80], [7]]}
+
+
+def off(got, want, dtype):
+    if dtype == "float32":
+        return TC.spread(got, want)
+    d = got.double() - want.double()
+    d = d - d.mean(-1, keepdim=True)
+    return (d.pow(2).mean(-1).sqrt().quantile(0.8) / want.double().std()).item()
+
+
+@pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
+@pytest.mark.parametrize("name", list(TC.CASES))
+def test_models_in_portions_and_batches(folder, name, dtype):
+    """Each request alone and all together, in one piece, decoded and in portions, on one engine whose pages and slots are used
+    again and again."""
+    from atlas_b200.replay import build_engine
+    path, cfg, toks, want, _ = folder(name)
+    eng = build_engine(path, dtype, 384)
+    tol = MODEL_TOL[dtype]
+    cut = lambda i, shape: ([SHAPES[shape][i][0]] + [1] * 200 if shape == "decode" else SHAPES[shape][i])
+    for shape in SHAPES:
+        plans = {}
+        for i, t in toks.items():
+            c = TC.portions(len(t), cut(i, shape))
+            plans[f"r{i}"] = (t, c, i)
+            assert off(TC.feed_alone(eng, f"a{i}", t, c), want[i], dtype) < tol, (shape, i)
+        for r, lg in TC.feed_together(eng, plans).items():
+            assert off(lg, want[int(r[1:])], dtype) < tol, (shape, r, "together")
+    assert eng.runner.graph_replays > 0 and eng.pool.num_free == eng.pool.num_blocks
+    eng.pool.check_invariants()
+
+
+@pytest.mark.parametrize("graphs", [True, False])
+def test_long_decoding_with_nothing_read_back(folder, graphs):
+    """A prompt of two tokens, then single tokens only, past windows and pages; only the last logits are asked for."""
+    from atlas_b200.replay import build_engine
+    path, cfg, toks, want, _ = folder("mixed")
+    eng = build_engine(path, "float32", 384, use_cuda_graphs=graphs)
+    for i, t in toks.items():
+        at = 0
+        for n in TC.portions(len(t), [2] + [1] * 200):
+            last = at + n == len(t)
+            got = eng.feed([(f"r{i}", t[at:at + n], [n - 1] if last else [])], [f"r{i}"] if last else [])[0]
+            at += n
+        assert TC.spread(got, want[i][-1:]) < MODEL_TOL["float32"]
+
+
+def test_decode_graph_equals_eager_decode(folder):
+    from atlas_b200.replay import build_engine
+    path, cfg, toks, want, _ = folder("aligned")
+    for dtype in ("float32", "bfloat16"):
+        a = build_engine(path, dtype, 384)
+        b = build_engine(path, dtype, 384, use_cuda_graphs=False)
+        plans = {f"r{i}": (t, TC.portions(len(t), [20] + [1] * 200), 0) for i, t in toks.items()}
+        x, y = TC.feed_together(a, plans), TC.feed_together(b, plans)
+        assert a.runner.graph_replays > 0 and b.runner.graph_replays == 0
+        for r in plans:
+            assert off(x[r], y[r].double(), dtype) < (1e-4 if dtype == "float32" else 0.05)
+
+
+@pytest.mark.parametrize("options", [{}, {"max_prefill_tokens": 16}, {"num_kv_blocks": 13, "admission_watermark_tokens": 0},
+                                     {"num_kv_blocks": 13, "admission_watermark_tokens": 0, "swap_space_gb": 0.01},
+                                     {"ngram_speculative": True, "num_drafts": 3, "mtp_gate": False}], ids=["plain", "portions", "preempt", "swap", "spec"])
+def test_greedy_generation_through_the_scheduler(folder, options):
+    """Engine, scheduler, sampler and the lag-one decode pipeline in fp32: the continuation is the exact model's argmax."""
+    from atlas_b200.config import EngineConfig
+    from atlas_b200.engine import LLMEngine
+    from atlas_b200.loader.load import load_model
+    from atlas_b200.sampling import SamplingParams
+    path, cfg, toks, _, w = folder("mixed")
+    prompts = [toks[1], toks[3], toks[2][:60]]
+    prompts.append(prompts[0][:35] + TC.tokens(cfg, 6, 99))
+    eng = LLMEngine(load_model(path, device="cuda", dtype="float32", max_pos=256),
+                    EngineConfig(**{**{"num_kv_blocks": 64, "max_num_seqs": 4, "max_seq_len": 160, "ssm_checkpoint_interval": 16}, **options}))
+    sp = SamplingParams(max_tokens=24, temperature=0.0, ignore_eos=True)
+    for _ in range(2):
+        for p, o in zip(prompts, eng.generate(prompts, sp)):
+            full = p + o.output_tokens
+            best = O.forward(cfg, w, full)[len(p) - 1:-1]
+            top = best.max(-1).values
+            picked = best.gather(-1, torch.tensor(o.output_tokens)[:, None])[:, 0]
+            assert len(o.output_tokens) == 24 and (top - picked).max() < 1e-3
+
+
+def test_sampled_serving_preset_runs_in_bf16():
+    from atlas_b200.config import EngineConfig, _tomizen, tiny_tomizen
+    from atlas_b200.engine import LLMEngine
+    from atlas_b200.models import build_model
+    from atlas_b200.ops import cuda as K
+    from atlas_b200.sampling import SamplingParams
+    for quant in ("none", "fp8_block", "nvfp4"):
+        cfg = tiny_tomizen("bfloat16") if quant == "none" else _tomizen(
+            1024, 256, "mlam", (2, 64, 128), (4, 32, 32, 64, 128, 72), (4, 2, 64), (8, 2, 128), "bfloat16")
+        cfg.max_position_embeddings, cfg.quant.method = 4096, quant
+        model = build_model(cfg, device="cuda").init_random(0)
+        eng = LLMEngine(model, EngineConfig(num_kv_blocks=64, max_num_seqs=4, max_seq_len=256, kv_cache_dtype="fp8"))
+        outs = eng.generate([[1, 2, 3] * 9, [4, 5]], SamplingParams(max_tokens=30, temperature=0.8, top_p=0.9, seed=1, ignore_eos=True))
+        assert all(len(o.output_tokens) == 30 for o in outs) and K.check_status() == 0
