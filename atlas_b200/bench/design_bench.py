@@ -1,11 +1,16 @@
-"""Prefill and decode throughput of Papidra layers beside Nemotron-H blocks of equal size, and the rooflines of their kernels.
+"""Prefill and decode throughput of a design's layers beside the closest other model at equal size, and the rooflines of their
+kernels.
 
-    python bench.py --design papidra            # or: python -m atlas_b200.bench.design_bench
+    python bench.py --design papidra|tomizen    # or: python -m atlas_b200.bench.design_bench --design ...
 
-Both models have the same width, feed-forward size, attention heads, Mamba-2 heads, vocabulary and cache dtype and random bf16
-weights.  One period is, for Papidra, a WKV layer and a layer with attention beside Mamba-2 plus a feed-forward; for
-Nemotron-H the blocks with the same work: Mamba-2, attention, Mamba-2, MLP.  Steps are timed with CUDA events around a
-captured step (L2 flushed in between), kernels the same way one by one.
+``papidra`` beside Nemotron-H: the same width, feed-forward size, attention heads, Mamba-2 heads, vocabulary and cache dtype.  One
+period is, for Papidra, a WKV layer and a layer with attention beside Mamba-2 plus a feed-forward; for Nemotron-H the blocks with
+the same work: Mamba-2, attention, Mamba-2, MLP.
+
+``tomizen`` (tomizen_bench.py) beside Qwen3-Next, and its latent attention beside DeepSeek's.
+
+All with random bf16 weights.  Steps are timed with CUDA events around a captured step (L2 flushed in between), kernels the same
+way one by one.
 """
 from __future__ import annotations
 
@@ -156,31 +161,39 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
     return rows
 
 
-def run(sizes: Optional[List[str]] = None, kernels: bool = True) -> dict:
+def designs() -> dict:
+    """name -> (name of the model beside it, sizes, configuration of both by size, kernel table, layers)"""
+    from . import tomizen_bench as T
+    return {"papidra": ("nemotron_h", SIZES, papidra, nemotron, kernel_table, f"{PERIODS} periods"),
+            "tomizen": ("qwen3_next", T.SIZES, T.tomizen, T.beside, T.kernel_table, "4 layers")}
+
+
+def run(sizes: Optional[List[str]] = None, kernels: bool = True, design: str = "papidra") -> dict:
     from ..ops import cuda as K
     from .microbench import Timer, load_peaks
     K.load()
     timer, peaks = Timer(), load_peaks()
-    out: dict = {"design": "papidra", "beside": "nemotron_h", "dtype": "bf16 weights and KV cache", "data": "synthetic: random weights and tokens",
+    other, all_sizes, mine, theirs, table, layers = designs()[design]
+    out: dict = {"design": design, "beside": other, "dtype": "bf16 weights and KV cache", "data": "synthetic: random weights and tokens",
                  "l2": "flushed between timed steps", "peaks": peaks, "sizes": {}}
     with torch.inference_mode():
-        for s in sizes or list(SIZES):
-            a, b = papidra(s), nemotron(s)
-            out["sizes"][s] = {"papidra": throughput(a, timer), "nemotron_h": throughput(b, timer), "layers": f"{PERIODS} periods",
+        for s in sizes or list(all_sizes):
+            a, b = mine(s), theirs(s)
+            out["sizes"][s] = {design: throughput(a, timer), other: throughput(b, timer), "layers": layers,
                                "params_m": [round(c.param_count() / 1e6, 1) for c in (a, b)]}
             if kernels:
-                out["sizes"][s]["kernels"] = kernel_table(s, timer, peaks)
+                out["sizes"][s]["kernels"] = table(s, timer, peaks)
     assert K.check_status() == 0
     return out
 
 
 def report(res: dict) -> str:
-    lines = []
+    lines, (a, b) = [], (res["design"], res["beside"])
     for s, r in res["sizes"].items():
         lines.append(f"width {s}, {r['layers']}, parameters (M) {r['params_m'][0]} / {r['params_m'][1]}")
-        for key, v in r["papidra"].items():
-            w = r["nemotron_h"][key]
-            lines.append(f"  {key:<18} papidra {v['ms']:>9} ms {v['tok_s']:>9} tok/s    nemotron_h {w['ms']:>9} ms {w['tok_s']:>9} tok/s")
+        for key, v in r[a].items():
+            w = r[b][key]
+            lines.append(f"  {key:<18} {a} {v['ms']:>9} ms {v['tok_s']:>9} tok/s    {b} {w['ms']:>9} ms {w['tok_s']:>9} tok/s")
         for k in r.get("kernels", ()):
             lines.append(f"  {k['pair']:<11} {k['kernel']:<38} {k['shape']:<20} {k['us']:>9} us  {k['roofline']:.3f} of roofline")
     return "\n".join(lines)
@@ -188,11 +201,12 @@ def report(res: dict) -> str:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--sizes", default=",".join(SIZES))
+    ap.add_argument("--design", default="papidra", choices=["papidra", "tomizen"])
+    ap.add_argument("--sizes", default="", help="widths (default: all of the design)")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--out")
     a = ap.parse_args(argv)
-    res = run(a.sizes.split(","), not a.no_kernels)
+    res = run([s for s in a.sizes.split(",") if s], not a.no_kernels, a.design)
     print(report(res))
     if a.out:
         with open(a.out, "w") as f:

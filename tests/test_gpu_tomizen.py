@@ -399,19 +399,10 @@ def folder(tmp_path_factory):
     return get
 
 
-# fp32 is the sharp comparison.  In bf16 the choice of an expert can turn on rounding, which moves a whole token: the typical row is
-# compared there, and rows may not be off everywhere
-MODEL_TOL = {"bfloat16": 0.12, "float32": 3e-4}
+# rounding of a whole bf16 model against the exact logits; fp32 is the sharp comparison
+MODEL_TOL = {"bfloat16": 0.15, "float32": 3e-4}
 SHAPES = {"whole": [[1000], [1000], [1000], [1000]], "decode": [[100, 1], [9, 1], [1], [2, 1]], "portions": [[2, 33, 1, 16], [3, 2], [17, 24], [2]],
           "long portions": [[110, 2], [40], [3, 80], [7]]}
-
-
-def off(got, want, dtype):
-    if dtype == "float32":
-        return TC.spread(got, want)
-    d = got.double() - want.double()
-    d = d - d.mean(-1, keepdim=True)
-    return (d.pow(2).mean(-1).sqrt().quantile(0.8) / want.double().std()).item()
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
@@ -429,9 +420,9 @@ def test_models_in_portions_and_batches(folder, name, dtype):
         for i, t in toks.items():
             c = TC.portions(len(t), cut(i, shape))
             plans[f"r{i}"] = (t, c, i)
-            assert off(TC.feed_alone(eng, f"a{i}", t, c), want[i], dtype) < tol, (shape, i)
+            assert TC.spread(TC.feed_alone(eng, f"a{i}", t, c), want[i]) < tol, (shape, i)
         for r, lg in TC.feed_together(eng, plans).items():
-            assert off(lg, want[int(r[1:])], dtype) < tol, (shape, r, "together")
+            assert TC.spread(lg, want[int(r[1:])]) < tol, (shape, r, "together")
     assert eng.runner.graph_replays > 0 and eng.pool.num_free == eng.pool.num_blocks
     eng.pool.check_invariants()
 
@@ -461,7 +452,7 @@ def test_decode_graph_equals_eager_decode(folder):
         x, y = TC.feed_together(a, plans), TC.feed_together(b, plans)
         assert a.runner.graph_replays > 0 and b.runner.graph_replays == 0
         for r in plans:
-            assert off(x[r], y[r].double(), dtype) < (1e-4 if dtype == "float32" else 0.05)
+            assert TC.spread(x[r], y[r]) < (1e-4 if dtype == "float32" else 0.08)
 
 
 @pytest.mark.parametrize("options", [{}, {"max_prefill_tokens": 16}, {"num_kv_blocks": 13, "admission_watermark_tokens": 0},

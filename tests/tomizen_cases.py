@@ -51,8 +51,9 @@ CASES = {
 
 
 def weights(cfg, seed=0):
-    """Random weights (rounded to bf16, like a checkpoint), scaled so that attention is peaked, scores meet their bound, memories
-    are short and long, and the experts a token takes stand out from the others."""
+    """Random weights (rounded to bf16, like a checkpoint), scaled so that attention is peaked, scores meet their bound and memories
+    are short and long.  The routers read channels of the embedding that no sublayer writes (their norm weights are zero there),
+    so that no choice of an expert turns on rounding."""
     g = torch.Generator().manual_seed(seed)
     W = cfg["width"]
     out = {}
@@ -63,12 +64,14 @@ def weights(cfg, seed=0):
         else:
             t = torch.randn(*shape, generator=g) * (std if std is not None else shape[-1] ** -0.5) + mean
         out[name] = t.to(torch.bfloat16)
+    kept = W - max(4, min(16, W // 4))
     put("embed", cfg["vocab"], W, std=1.0)
     put("final.norm", W, std=0.2)
     put("head", cfg["vocab"], W)
     for i, l in enumerate(cfg["layers"]):
         p, m = f"l{i}.", l["mixer"]
         put(p + "norm1", W, std=0.2)
+        out[p + "norm1"][kept:] = -1.0
         x = p + "mix."
         H = m["heads"]
         if l["type"] == "mlstm":
@@ -97,8 +100,10 @@ def weights(cfg, seed=0):
             put(x + "o", W, H * m["vdim"])
         if l["mlp"] is not None:
             put(p + "norm2", W, std=0.2)
+            out[p + "norm2"][kept:] = -1.0
             n = l["mlp"]["expert"]["ff"]
-            put(p + "mlp.router", l["mlp"]["router"]["experts"], W, std=2.0 * W ** -0.5)
+            put(p + "mlp.router", l["mlp"]["router"]["experts"], W, std=(W - kept) ** -0.5)
+            out[p + "mlp.router"][:, :kept] = 0.0
             for e in range(l["mlp"]["router"]["experts"]):
                 put(f"{p}mlp.e{e}.up", n, W)
                 put(f"{p}mlp.e{e}.down", W, n)
