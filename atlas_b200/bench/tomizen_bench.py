@@ -159,7 +159,7 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
         add("latent block", "expanded cache (existing)", shape, lambda: mla.mix(act, fb, (kx, vx, 1.0, 1.0), table),
             wb + io + nseq * L * lh * (dn + dr + lv) * 2, pw_flops + core + expand)
         if decode:
-            mt = KL.row_tiles(lh)
+            mt = KL.row_tiles(la)
             qq, lat = rn(T, lh, la.width), torch.empty(T, lh, la.rp, dtype=bf, device=dev)
             splits = KL.decode_splits(nseq, lh, mt, vis, K._num_sms[K._dev(qq)])
             po, pml = torch.empty(T * lh * splits * la.rp, device=dev), torch.empty(T * lh * splits * 2, device=dev)

@@ -5,9 +5,8 @@
 //                          expanded form's padded heads (expanded rows)
 //   head_gemm_kernel       out[row, head, :] = W[head] in[row, head, :], mma.sync, 64 rows x 64 columns of one head per CTA: the
 //                          absorbed W_uk on the query side and W_uv on the output side
-//   latent_attn_kernel     absorbed attention (bf16): 16 or 32 (token, head) rows per CTA against 64-token tiles of the cache, which
-//                          serve as keys (full width) and values (first rp columns).  Eight warps: 8 keys each for the scores,
-//                          an eighth of the latent each for the output.  Split over the keys where the grid is small
+//   latent_attn_kernel     absorbed attention (bf16): 16 or 32 (token, head) rows per CTA against tiles of the cache, which serve
+//                          as keys (full width) and values (first rp columns).  Split over the keys where the grid is small
 //                          (latent_merge_kernel).  Decode rows and short portions alike.
 //   latent_attn_f32_kernel the same in fp32, one warp per (row, head)
 //   latent_gather_kernel, latent_pages_kernel   expanded form: visible cache rows as a matrix; its product with [W_uk; W_uv] to
@@ -167,7 +166,7 @@ head_gemm_kernel(const HeadGemmParams p) {
 }
 
 // ----------------------------------------------------------------------------- absorbed attention
-constexpr int kLtTok = 64, kLtWarps = 8, kLtPS = kLtTok + 8;
+constexpr int kLtKG = 4, kLtMaxStages = 6;     // groups of warps that share a row's width
 
 template <typename T>
 struct LatentAttnParams {
@@ -179,21 +178,32 @@ struct LatentAttnParams {
   const int* seq_lens; const int* query_start_loc;
   const int* row_start;                        // [B] first row of a sequence in q / out (null = query_start_loc)
   const int* tile_seq; const int* tile_r0;     // (sequence, first flattened (token, head) row); null: tile z of sequence blockIdx.x
-  int H, rp, ep, block_size, window, splits, stages;
+  int H, rp, ep, block_size, bs_shift, window, splits, stages;   // bs_shift: log2 of the block size, -1 if it is none
   float scale;
 };
 
-template <int NT, int MT>
-__global__ void __launch_bounds__(32 * kLtWarps)
+// A tile of TOK keys goes through three steps, each one tile behind the other, with one barrier per tile:
+//   scores    warp (kg, tg): k-steps of group kg for the HK keys of part tg -> partial sums in shared memory
+//   softmax   TPR threads per row add the kLtKG partial sums, keep the row's maximum and sum, write the probabilities (bf16)
+//   output    every warp its NT * 8 columns of the latent over the tile's keys
+// so between two barriers the warps work on the scores of tile p + 1, the softmax of tile p and the output of tile p - 1.  Tiles
+// arrive through a ring of `stages` (>= 4) buffers.
+// KPG: k-steps per warp (HK = 8: taken in pairs), MT: 16-row units
+template <int KPG, int NT, int MT, int WARPS, int TOK>
+__global__ void __launch_bounds__(32 * WARPS)
 latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
-  constexpr int M = 16 * MT;
+  constexpr int M = 16 * MT, THREADS = 32 * WARPS, TPR = THREADS / M, KPT = TOK / TPR;
+  constexpr int TG = WARPS / kLtKG, HK = TOK / TG, RPW = TOK / WARPS;
+  constexpr int PS = TOK + 8, SS = TOK + 4;    // padded rows of the probabilities and of the partial sums
+  static_assert(HK == 8 || HK == 16, "eight or sixteen keys per warp");
+  static_assert(HK == 16 || KPG % 2 == 0, "pairs of k-steps");
   extern __shared__ __align__(16) uint8_t lt_smem[];
-  const int W = p.rp + p.ep, WS = W + 8;
-  __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(lt_smem);                 // [M][WS]
-  __nv_bfloat16* sp = sq + M * WS;                                               // [M][kLtPS]
-  float* smax = reinterpret_cast<float*>(sp + M * kLtPS);                        // [8][M]
-  float* ssum = smax + kLtWarps * M;
-  __nv_bfloat16* skv = reinterpret_cast<__nv_bfloat16*>(ssum + kLtWarps * M);    // [stages][64][WS]
+  const int W = p.rp + p.ep, WS = W + 8, CW = W / 8;
+  float* spart = reinterpret_cast<float*>(lt_smem);                              // [2][kLtKG][M][SS]
+  __nv_bfloat16* sp = reinterpret_cast<__nv_bfloat16*>(spart + 2 * kLtKG * M * SS);        // [2][M][PS]
+  float* salpha = reinterpret_cast<float*>(sp + 2 * M * PS);                     // [2][M]
+  float* ssum = salpha + 2 * M;                                                  // [M]
+  __nv_bfloat16* skv = reinterpret_cast<__nv_bfloat16*>(ssum + M);               // [stages][TOK][WS]
   chain_trigger();
   chain_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
@@ -207,165 +217,212 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
   auto low = [&](int pos) { return p.window > 0 ? max(0, pos - p.window + 1) : 0; };
   const int last = min(r0 + M, n_flat) - 1;
   const int key_lo = low(ctx + r0 / p.H), key_hi = ctx + last / p.H + 1;         // keys some row of the tile sees
-  const int tiles = (key_hi - key_lo + kLtTok - 1) / kLtTok, per = (tiles + p.splits - 1) / p.splits;
-  const int j0 = split * per, j1 = min(tiles, j0 + per);
+  const int tiles = (key_hi - key_lo + TOK - 1) / TOK, per = (tiles + p.splits - 1) / p.splits;
+  const int j0 = split * per, n_tiles = max(0, min(tiles, j0 + per) - j0), kv0 = key_lo + j0 * TOK;
   const int* bt = p.block_tables + (long long)b * p.bt_ld;
+  const int S = p.stages;
 
-  // queries of the tile (zeros past the end)
-  const int CW = W / 8;
-  for (int i = tid; i < M * CW; i += 32 * kLtWarps) {
-    const int r = i / CW, c = (i % CW) * 8;
-    cp_async16(smem_u32(sq + r * WS + c), p.q + (flat0 + (r0 + r < n_flat ? r : 0)) * W + c, r0 + r < n_flat);
-  }
-  auto fetch = [&](int j, int st) {
-    const int k0 = key_lo + j * kLtTok;
-    for (int i = tid; i < kLtTok * CW; i += 32 * kLtWarps) {
-      const int r = i / CW, c = (i % CW) * 8, key = k0 + r;
-      const bool live = key < key_hi;
-      const long long row = live ? (long long)bt[key / p.block_size] * p.block_size + key % p.block_size : 0;
-      cp_async16(smem_u32(skv + ((long long)st * kLtTok + r) * WS + c), p.cache + row * W + c, live);
+  // A warp copies rows warp, warp + WARPS, .. of a tile; lane i looks up the i-th of them.  The page number is fetched one tile
+  // before it is used: nothing waits for it.
+  auto page_of = [&](int t) -> int {
+    const int key = kv0 + t * TOK + warp + WARPS * (lane & (RPW - 1));
+    return t < n_tiles && key < key_hi ? bt[p.bs_shift >= 0 ? key >> p.bs_shift : key / p.block_size] : -1;
+  };
+  auto fetch = [&](int st, int t, int page) {
+    const int key = kv0 + t * TOK + warp + WARPS * (lane & (RPW - 1));
+    const int rows = page < 0 ? -1 : page * p.block_size + (p.bs_shift >= 0 ? key & (p.block_size - 1) : key % p.block_size);
+    const uint32_t dst = smem_u32(skv + (long long)st * TOK * WS);
+#pragma unroll
+    for (int i = 0; i < RPW; ++i) {
+      const int row = __shfl_sync(0xffffffffu, rows, i);
+      const __nv_bfloat16* src = p.cache + (long long)max(row, 0) * W;
+#pragma unroll
+      for (int u = 0; u < (KPG * kLtKG * 2 + 31) / 32; ++u) {
+        const int c = u * 32 + lane;
+        if (c < CW) cp_async16(dst + ((warp + WARPS * i) * WS + c * 8) * 2, src + c * 8, row >= 0);
+      }
     }
   };
-  int pos[MT][2], lo[MT][2];
+  for (int t = 0; t < S - 2; ++t) {            // one group per tile, empty past the end
+    if (t < n_tiles) fetch(t, t, page_of(t));
+    cp_async_commit();
+  }
+  int next = page_of(S - 2);
+
+  // query fragments of this warp's k-steps stay in registers (zero past the row's width)
+  const int kg = warp % kLtKG, tg = warp / kLtKG, nks = W / 16;
+  auto kstep = [&](int i) { return HK == 8 ? 2 * (kg + kLtKG * (i >> 1)) + (i & 1) : kg + kLtKG * i; };
+  uint32_t qf[MT][KPG][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int r = r0 + m * 16 + g + 8 * h;
-      pos[m][h] = r < n_flat ? ctx + r / p.H : -1;
-      lo[m][h] = low(pos[m][h]);
-    }
-  float o[MT][NT][4], mr[MT][2], lr[MT][2];
+    for (int i = 0; i < KPG; ++i)
 #pragma unroll
-  for (int m = 0; m < MT; ++m) {
-    mr[m][0] = mr[m][1] = -INFINITY;
-    lr[m][0] = lr[m][1] = 0.f;
+      for (int e = 0; e < 4; ++e) {
+        const int r = m * 16 + g + 8 * (e & 1), k = kstep(i) * 16 + 2 * t4 + 8 * (e >> 1);
+        qf[m][i][e] = r0 + r < n_flat && k < W ? *reinterpret_cast<const uint32_t*>(p.q + (flat0 + r) * W + k) : 0u;
+      }
+  // softmax: this thread's row and keys
+  const int srow = tid / TPR, sc = (tid % TPR) * KPT;
+  const int pos = r0 + srow < n_flat ? ctx + (r0 + srow) / p.H : -1, lo = low(pos);
+  const float sl2 = p.scale * 1.4426950408889634f;
+  float mrun = -INFINITY, lrun = 0.f;
+  float o[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int j = 0; j < NT; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
-  }
-  const float sl2 = p.scale * 1.4426950408889634f;
   const int a_row = lane & 15, a_col = (lane >> 4) * 8;
-  const uint32_t uq = smem_u32(sq), up = smem_u32(sp);
+  const uint32_t ukv0 = smem_u32(skv), up0 = smem_u32(sp), stage_bytes = TOK * WS * 2;
   const int d0 = warp * NT * 8;                // this warp's latent columns
 
-  if (j0 < j1) fetch(j0, 0);
-  cp_async_commit();
-  for (int j = j0; j < j1; ++j) {
-    const int st = p.stages == 2 ? (j - j0) & 1 : 0;
-    if (p.stages == 2 && j + 1 < j1) fetch(j + 1, st ^ 1);
-    cp_async_commit();
-    cp_async_wait<1>();
-    __syncthreads();
-    const uint32_t ukv = smem_u32(skv + (long long)st * kLtTok * WS);
-    // ---- scores of keys 8 warp .. 8 warp + 7
-    float s[MT][4];
+  auto scores = [&](int st, int buf) {
+    float acc[MT][HK / 8][4];
 #pragma unroll
-    for (int m = 0; m < MT; ++m) s[m][0] = s[m][1] = s[m][2] = s[m][3] = 0.f;
-    {
-      // two k-steps per ldmatrix.x4: matrices are the key rows' columns 0..7, 8..15, 16..23, 24..31
-      const uint32_t bk = ukv + ((warp * 8 + (lane & 7)) * WS + (lane >> 3) * 8) * 2;
-      int kk = 0;
-      for (; kk + 32 <= W; kk += 32) {
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < HK / 8; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
+    const uint32_t base = ukv0 + st * stage_bytes;
+    if constexpr (HK == 16) {
+      const uint32_t bk = base + ((tg * 16 + (lane & 7) + ((lane >> 4) << 3)) * WS + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+      for (int i = 0; i < KPG; ++i) {
         uint32_t bb[4];
-        ldsm4(bk + kk * 2, bb);
+        ldsm4(bk + min(kstep(i), nks - 1) * 32, bb);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          ldsm4(uq + ((m * 16 + a_row) * WS + kk + a_col) * 2, a);
-          mma16816(s[m], a, bb[0], bb[1]);
-          ldsm4(uq + ((m * 16 + a_row) * WS + kk + 16 + a_col) * 2, a);
-          mma16816(s[m], a, bb[2], bb[3]);
+          mma16816(acc[m][0], qf[m][i], bb[0], bb[1]);
+          mma16816(acc[m][HK / 8 - 1], qf[m][i], bb[2], bb[3]);
         }
       }
-      if (kk < W) {
-        uint32_t b0, b1;
-        ldsm2(ukv + ((warp * 8 + (lane & 7)) * WS + kk + ((lane >> 3) & 1) * 8) * 2, b0, b1);
+    } else {
+      const uint32_t bk = base + ((tg * 8 + (lane & 7)) * WS + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll
+      for (int i = 0; i < KPG; i += 2) {       // eight keys, two k-steps
+        uint32_t bb[4];
+        ldsm4(bk + min(kstep(i) + (lane >> 4), nks - 1) * 32, bb);
 #pragma unroll
         for (int m = 0; m < MT; ++m) {
-          uint32_t a[4];
-          ldsm4(uq + ((m * 16 + a_row) * WS + kk + a_col) * 2, a);
-          mma16816(s[m], a, b0, b1);
+          mma16816(acc[m][0], qf[m][i], bb[0], bb[1]);
+          mma16816(acc[m][0], qf[m][i + 1], bb[2], bb[3]);
         }
       }
     }
-    const int key = key_lo + j * kLtTok + warp * 8 + 2 * t4;
+    float* dst = spart + (buf * kLtKG + kg) * M * SS + tg * HK + 2 * t4;
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
+      for (int n = 0; n < HK / 8; ++n)
 #pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          float& x = s[m][2 * h + e];
-          x = key + e <= pos[m][h] && key + e >= lo[m][h] ? x * sl2 : -INFINITY;
-        }
-        float mx = fmaxf(s[m][2 * h], s[m][2 * h + 1]);
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        if (t4 == 0) smax[warp * M + m * 16 + g + 8 * h] = mx;
+        for (int h = 0; h < 2; ++h)
+          *reinterpret_cast<float2*>(dst + (m * 16 + g + 8 * h) * SS + n * 8) = make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
+  };
+  auto softmax = [&](int t, int buf) {
+    float s[KPT], mx = mrun;
+#pragma unroll
+    for (int u = 0; u < KPT; ++u) s[u] = 0.f;
+#pragma unroll
+    for (int k = 0; k < kLtKG; ++k) {
+      float f[KPT];
+      load_vec<KPT>(spart + ((buf * kLtKG + k) * M + srow) * SS + sc, f);
+#pragma unroll
+      for (int u = 0; u < KPT; ++u) s[u] += f[u];
+    }
+#pragma unroll
+    for (int u = 0; u < KPT; ++u) {
+      const int key = kv0 + t * TOK + sc + u;
+      s[u] = key <= pos && key >= lo ? s[u] * sl2 : -INFINITY;
+      mx = fmaxf(mx, s[u]);
+    }
+#pragma unroll
+    for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    const float ref = mx == -INFINITY ? 0.f : mx, alpha = fast_exp2(mrun - ref);            // nothing seen yet: 0
+    mrun = mx;
+    lrun *= alpha;
+    __nv_bfloat16* dst = sp + (buf * M + srow) * PS + sc;
+#pragma unroll
+    for (int u = 0; u < KPT; ++u) {
+      s[u] = fast_exp2(s[u] - ref);
+      lrun += s[u];
+    }
+    store_vec<KPT>(dst, s);
+    if (sc == 0) salpha[buf * M + srow] = alpha;
+  };
+  auto output = [&](int st, int buf) {
+    if (d0 >= p.rp) return;
+    const uint32_t ukv = ukv0 + st * stage_bytes, up = up0 + buf * M * PS * 2;
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float f0 = salpha[buf * M + m * 16 + g], f1 = salpha[buf * M + m * 16 + g + 8];
+      if (__any_sync(0xffffffffu, f0 != 1.f || f1 != 1.f)) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n) { o[m][n][0] *= f0; o[m][n][1] *= f0; o[m][n][2] *= f1; o[m][n][3] *= f1; }
       }
-    __syncthreads();
+    }
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int kk = 0; kk < TOK / 16; ++kk) {
+      uint32_t a[MT][4];
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int r = m * 16 + g + 8 * h;
-        float mx = mr[m][h];
+      for (int m = 0; m < MT; ++m) ldsm4(up + ((m * 16 + a_row) * PS + kk * 16 + a_col) * 2, a[m]);
+      if constexpr (NT == 1) {
+        uint32_t b0, b1;                       // one n8 tile: matrices keys 0..7 and 8..15
+        asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
+                     : "=r"(b0), "=r"(b1) : "r"(ukv + ((kk * 16 + a_row) * WS + d0) * 2) : "memory");
 #pragma unroll
-        for (int w = 0; w < kLtWarps; ++w) mx = fmaxf(mx, smax[w * M + r]);
-        const float ref = mx == -INFINITY ? 0.f : mx, alpha = exp2f(mr[m][h] - ref);        // nothing seen yet: 0
-        const float p0 = exp2f(s[m][2 * h] - ref), p1 = exp2f(s[m][2 * h + 1] - ref);
-        lr[m][h] = lr[m][h] * alpha + p0 + p1;
-        mr[m][h] = mx;
-        *reinterpret_cast<uint32_t*>(sp + r * kLtPS + warp * 8 + 2 * t4) = pack_bf16x2(p0, p1);
+        for (int m = 0; m < MT; ++m) mma16816(o[m][0], a[m], b0, b1);
+      } else {
 #pragma unroll
-        for (int n = 0; n < NT; ++n) { o[m][n][2 * h] *= alpha; o[m][n][2 * h + 1] *= alpha; }
-      }
-    __syncthreads();
-    // ---- output: this warp's columns over all 64 keys
-    if (d0 < p.rp) {
+        for (int n = 0; n < NT / 2; ++n) {
+          uint32_t x[4];                       // columns past the latent are computed and dropped
+          ldsm4t(ukv + ((kk * 16 + a_row) * WS + min(d0 + n * 16, p.rp - 16) + a_col) * 2, x);
 #pragma unroll
-      for (int kk = 0; kk < kLtTok / 16; ++kk) {
-        uint32_t a[MT][4];
-#pragma unroll
-        for (int m = 0; m < MT; ++m) ldsm4(up + ((m * 16 + a_row) * kLtPS + kk * 16 + a_col) * 2, a[m]);
-        if constexpr (NT == 1) {
-          uint32_t b0, b1;                     // one n8 tile: matrices keys 0..7 and 8..15
-          asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
-                       : "=r"(b0), "=r"(b1) : "r"(ukv + ((kk * 16 + a_row) * WS + d0) * 2) : "memory");
-#pragma unroll
-          for (int m = 0; m < MT; ++m) mma16816(o[m][0], a[m], b0, b1);
-        } else {
-#pragma unroll
-          for (int n = 0; n < NT / 2; ++n) {
-            if (d0 + n * 16 >= p.rp) break;
-            uint32_t x[4];
-            ldsm4t(ukv + ((kk * 16 + a_row) * WS + d0 + n * 16 + a_col) * 2, x);
-#pragma unroll
-            for (int m = 0; m < MT; ++m) {
-              mma16816(o[m][2 * n], a[m], x[0], x[1]);
-              mma16816(o[m][2 * n + 1], a[m], x[2], x[3]);
-            }
+          for (int m = 0; m < MT; ++m) {
+            mma16816(o[m][2 * n], a[m], x[0], x[1]);
+            mma16816(o[m][2 * n + 1], a[m], x[2], x[3]);
           }
         }
       }
     }
-    __syncthreads();                           // the tile's buffers are free
-    if (p.stages == 1 && j + 1 < j1) {
-      fetch(j + 1, 0);
+  };
+
+  if (n_tiles > 0) {
+    cp_async_wait<0>();
+    __syncthreads();                           // the first S - 2 >= 2 tiles
+    scores(0, 0);
+    __syncthreads();
+    int s_prev = 0, s_cur = 0, s_next = 1, s_in = S - 2;         // ring positions of tiles p - 1, p, p + 1 and of the one requested
+    for (int t = 0; t < n_tiles; ++t) {
+      const int ahead = t + S - 2;
+      if (ahead < n_tiles) fetch(s_in, ahead, next);
       cp_async_commit();
+      next = page_of(ahead + 1);
+      scores(s_next, (t + 1) & 1);             // past the last tile: stale keys, never read
+      softmax(t, t & 1);
+      if (t > 0) output(s_prev, (t - 1) & 1);
+      // tile t + 2 has to be here; the S - 4 requested after it need not
+      if (S == 4) cp_async_wait<0>();
+      else if (S == 5) cp_async_wait<1>();
+      else cp_async_wait<2>();
+      __syncthreads();
+      s_prev = s_cur;
+      s_cur = s_next;
+      s_next = s_next + 1 == S ? 0 : s_next + 1;
+      s_in = s_in + 1 == S ? 0 : s_in + 1;
     }
+    output(s_prev, (n_tiles - 1) & 1);
   }
   cp_async_wait<0>();
-  // ---- sums over the warps' keys, output
+  // ---- row sums, output
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      float l = lr[m][h];
-      l += __shfl_xor_sync(0xffffffffu, l, 1);
-      l += __shfl_xor_sync(0xffffffffu, l, 2);
-      if (t4 == 0) ssum[warp * M + m * 16 + g + 8 * h] = l;
+  for (int off = TPR / 2; off > 0; off >>= 1) lrun += __shfl_xor_sync(0xffffffffu, lrun, off);
+  if (sc == 0) {
+    ssum[srow] = lrun;
+    if (p.splits > 1 && pos >= 0) {
+      float* ml = p.part_ml + ((flat0 + srow) * p.splits + split) * 2;
+      ml[0] = mrun;
+      ml[1] = lrun;
     }
+  }
   __syncthreads();
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -373,12 +430,9 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
     for (int h = 0; h < 2; ++h) {
       const int r = m * 16 + g + 8 * h;
       if (r0 + r >= n_flat) continue;
-      float l = 0.f;
-#pragma unroll
-      for (int w = 0; w < kLtWarps; ++w) l += ssum[w * M + r];
       const long long flat = flat0 + r;
       if (p.splits == 1) {
-        const float inv = 1.f / l;             // a row sees at least itself
+        const float inv = 1.f / ssum[r];       // a row sees at least itself
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           const int d = d0 + n * 8 + 2 * t4;
@@ -390,10 +444,6 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
         for (int n = 0; n < NT; ++n) {
           const int d = d0 + n * 8 + 2 * t4;
           if (d < p.rp) *reinterpret_cast<float2*>(po + d) = make_float2(o[m][n][2 * h], o[m][n][2 * h + 1]);
-        }
-        if (warp == 0 && t4 == 0) {
-          p.part_ml[(flat * p.splits + split) * 2] = mr[m][h];
-          p.part_ml[(flat * p.splits + split) * 2 + 1] = l;
         }
       }
     }
@@ -573,23 +623,33 @@ static int latent_rows(const void* q, long long ldq, const float* ckv, long long
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
-template <int NT, int MT>
+template <int KPG, int NT, int MT, int WARPS, int TOK>
 static int launch_latent(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaStream_t st) {
   constexpr int M = 16 * MT;
-  const int WS = p.rp + p.ep + 8, fixed = M * WS * 2 + M * kLtPS * 2 + 2 * kLtWarps * M * 4, stage = kLtTok * WS * 2;
-  p.stages = fixed + 2 * stage <= 220 * 1024 ? 2 : 1;
+  const int WS = p.rp + p.ep + 8, fixed = 2 * kLtKG * M * (TOK + 4) * 4 + 2 * M * (TOK + 8) * 2 + 3 * M * 4, stage = TOK * WS * 2;
+  p.stages = (227 * 1024 - fixed) / stage;
+  if (p.stages > kLtMaxStages) p.stages = kLtMaxStages;
+  if (p.stages < 4) return -3;
   const int smem = fixed + p.stages * stage;
-  if (smem > 226 * 1024) return -3;
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(latent_attn_kernel<NT, MT>), smem) != cudaSuccess) return -20;
-  return launch_chain(latent_attn_kernel<NT, MT>, grid, dim3(32 * kLtWarps), (size_t)smem, st, p) == cudaSuccess ? 0 : -21;
+  auto k = latent_attn_kernel<KPG, NT, MT, WARPS, TOK>;
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(k), smem) != cudaSuccess) return -20;
+  return launch_chain(k, grid, dim3(32 * WARPS), (size_t)smem, st, p) == cudaSuccess ? 0 : -21;
 }
-template <int MT>
-static int launch_latent_nt(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaStream_t st) {
-  if (p.rp <= 64) return launch_latent<1, MT>(p, grid, st);
-  if (p.rp <= 128) return launch_latent<2, MT>(p, grid, st);
-  if (p.rp <= 256) return launch_latent<4, MT>(p, grid, st);
-  if (p.rp <= 512) return launch_latent<8, MT>(p, grid, st);
-  return launch_latent<16, MT>(p, grid, st);
+// classes of latent and row widths: NT * 8 * WARPS columns, 16 * KPG * kLtKG numbers of a row
+static int launch_latent_1(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaStream_t st) {
+  const int W = p.rp + p.ep;
+  if (p.rp <= 128 && W <= 192) return launch_latent<4, 1, 1, 16, 32>(p, grid, st);
+  if (p.rp <= 256 && W <= 320) return launch_latent<6, 2, 1, 16, 32>(p, grid, st);
+  if (p.rp <= 512 && W <= 576) return launch_latent<10, 4, 1, 16, 32>(p, grid, st);
+  if (W <= 1088) return launch_latent<18, 16, 1, 8, 16>(p, grid, st);
+  return -5;
+}
+static int launch_latent_2(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaStream_t st) {
+  const int W = p.rp + p.ep;
+  if (p.rp <= 128 && W <= 192) return launch_latent<3, 2, 2, 8, 32>(p, grid, st);
+  if (p.rp <= 256 && W <= 320) return launch_latent<5, 4, 2, 8, 32>(p, grid, st);
+  if (p.rp <= 512 && W <= 576) return launch_latent<9, 8, 2, 8, 32>(p, grid, st);
+  return -5;
 }
 
 }  // namespace atlas
@@ -632,15 +692,18 @@ extern "C" int atlas_latent_attn(const void* q, const void* cache, void* out, fl
                                  const int* tile_r0, int tiles, int B, int rows, int H, int rp, int ep, int block_size, int window, int splits,
                                  int mt, float scale, void* stream) {
   if (B <= 0 || rows <= 0) return 0;
-  if (rp % 16 || ep % 16 || rp > 1024 || (mt != 1 && mt != 2) || block_size < 1) return -1;
+  if (rp % 16 || ep % 16 || rp > 1024 || rp + ep > 1088 || (mt != 1 && mt != 2) || block_size < 1) return -1;
+  if (mt == 2 && (rp > 512 || rp + ep > 576)) return -5;         // wider rows exist with 16-row tiles
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(cache)) & 15) return -2;
   if (splits > 1 && (!part_o || !part_ml)) return -4;
   LatentAttnParams<bf16> p = {reinterpret_cast<const bf16*>(q), reinterpret_cast<const bf16*>(cache), reinterpret_cast<bf16*>(out), part_o, part_ml,
                               block_tables, bt_ld, seq_lens, query_start_loc, row_start, tiles > 0 ? tile_seq : nullptr, tile_r0, H, rp, ep,
-                              block_size, window, splits < 1 ? 1 : splits, 1, scale};
+                              block_size, -1, window, splits < 1 ? 1 : splits, 1, scale};
+  for (int k = 0; k < 20; ++k)
+    if (block_size == 1 << k) p.bs_shift = k;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const dim3 grid(tiles > 0 ? tiles : B, p.splits, tiles > 0 ? 1 : (H + 16 * mt - 1) / (16 * mt));
-  const int rc = mt == 1 ? launch_latent_nt<1>(p, grid, st) : launch_latent_nt<2>(p, grid, st);
+  const int rc = mt == 1 ? launch_latent_1(p, grid, st) : launch_latent_2(p, grid, st);
   if (rc) return rc;
   if (p.splits > 1 &&
       launch_chain(latent_merge_kernel, dim3((unsigned)(rows * H)), dim3(128), 0, st, (const float*)part_o, (const float*)part_ml, p.out, rp, p.splits) != cudaSuccess)
@@ -655,7 +718,7 @@ extern "C" int atlas_latent_attn_f32(const float* q, const float* cache, float* 
   if (B <= 0 || T <= 0) return 0;
   if (rp % 4 || ep % 4 || rp > 32 * kLfMax || block_size < 1) return -1;
   LatentAttnParams<float> p = {q, cache, out, nullptr, nullptr, block_tables, bt_ld, seq_lens, query_start_loc, nullptr, nullptr, nullptr, H, rp, ep,
-                               block_size, window, 1, 1, scale};
+                               block_size, -1, window, 1, 1, scale};
   latent_attn_f32_kernel<<<(unsigned)(((long long)T * H + 3) / 4), 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(p, B, T);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }

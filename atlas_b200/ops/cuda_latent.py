@@ -12,7 +12,7 @@ from . import checked, cuda as K
 _vp, _ll, _i, _f = C.c_void_p, C.c_longlong, C.c_int, C.c_float
 _bound = False
 EXPAND_MIN_ROWS = 96          # portions of at least this many rows take the expanded form
-_KEYS_PER_TILE = 64
+_KEYS_PER_SPLIT = 64          # the least a split of the keys is given
 
 
 def _lib():
@@ -31,14 +31,14 @@ def _lib():
 
 
 def decode_splits(B: int, H: int, mt: int, visible: int, sms: int) -> int:
-    """Key splits of the absorbed decode kernel: about one CTA per SM, at least two key tiles each."""
+    """Key splits of the absorbed decode kernel: about one CTA per SM."""
     ctas = B * ((H + 16 * mt - 1) // (16 * mt))
-    return max(1, min(sms // max(1, ctas), (visible + 2 * _KEYS_PER_TILE - 1) // (2 * _KEYS_PER_TILE), 32))
+    return max(1, min(sms // max(1, ctas), (visible + _KEYS_PER_SPLIT - 1) // _KEYS_PER_SPLIT, 32))
 
 
-def row_tiles(H: int) -> int:
-    """16-row units per CTA: two where a token has more than sixteen heads."""
-    return 2 if H > 16 else 1
+def row_tiles(layer) -> int:
+    """16-row units per CTA: two where a token has more than sixteen heads (and the cache rows are not too wide)."""
+    return 2 if layer.hq > 16 and layer.rp <= 512 and layer.width <= 576 else 1
 
 
 def scratch_bytes(batch_sizes, layer, max_seq_len: int, sms: int):
@@ -46,16 +46,16 @@ def scratch_bytes(batch_sizes, layer, max_seq_len: int, sms: int):
     po = pml = 0
     visible = min(max_seq_len, layer.window or max_seq_len)
     for b in batch_sizes:
-        s = decode_splits(b, layer.hq, row_tiles(layer.hq), visible, sms)
+        s = decode_splits(b, layer.hq, row_tiles(layer), visible, sms)
         if s > 1:
             po, pml = max(po, b * layer.hq * s * layer.rp * 4), max(pml, b * layer.hq * s * 8)
     return po, pml
 
 
 class _Plan:
-    """Which sequences of a step take which form, shared by the step's latent layers of the same window."""
+    """Which sequences of a step take which form, shared by the step's latent layers of the same window and tiling."""
 
-    def __init__(self, batch, window: int, H: int, block_size: int, device):
+    def __init__(self, batch, window: int, H: int, mt: int, block_size: int, device):
         qlens, nd, B = batch.query_lens_host, batch.num_decodes, batch.num_seqs
         expand = [i for i in range(nd, B) if qlens[i] >= EXPAND_MIN_ROWS and block_size % 16 == 0]
         short = [i for i in range(nd, B) if qlens[i] < EXPAND_MIN_ROWS or block_size % 16]
@@ -78,7 +78,6 @@ class _Plan:
                     row_map[r] = -(len(dst) + 1) if dst is list_x else len(dst)
                     dst.append(r)
             parts += [row_map, row_start, list_a, list_x]
-        mt = row_tiles(H)
         if short:
             seqs, firsts = [], []
             for i in short:
@@ -124,13 +123,13 @@ class _Plan:
                                            max_seq_len=max(self.x_lens))
 
 
-def _plan(batch, window: int, H: int, block_size: int, device) -> _Plan:
+def _plan(batch, window: int, H: int, mt: int, block_size: int, device) -> _Plan:
     plans = getattr(batch, "_latent_plans", None)
     if plans is None:
         plans = batch._latent_plans = {}
-    key = (window, H)
+    key = (window, H, mt)
     if key not in plans:
-        plans[key] = _Plan(batch, window, H, block_size, device)
+        plans[key] = _Plan(batch, window, H, mt, block_size, device)
     return plans[key]
 
 
@@ -153,7 +152,7 @@ def latent_attention(layer, q, ckv, batch, cache, rope_cache) -> torch.Tensor:
         checked.kv_write(batch.slot_mapping, batch.positions, cache.shape[0], bs, rope_cache.shape[0] if layer.rotary else 0)
         checked.paged_read(batch.block_tables, batch.seq_lens, cache.shape[0], bs)
     window, bt = int(layer.window or 0), batch.block_tables
-    plan: Optional[_Plan] = None if f32 else _plan(batch, window, H, bs, dev)
+    plan: Optional[_Plan] = None if f32 else _plan(batch, window, H, row_tiles(layer), bs, dev)
     rows_a, rows_x = (T, 0) if f32 else (plan.rows_a, plan.rows_x)
     qa = torch.empty(rows_a, H, W, dtype=q.dtype, device=dev) if rows_a else None
     qx = torch.empty(rows_x, H, layer.dx, dtype=q.dtype, device=dev) if rows_x else None
@@ -174,7 +173,7 @@ def latent_attention(layer, q, ckv, batch, cache, rope_cache) -> torch.Tensor:
     if rows_a:
         _head_gemm(q, q.stride(0), qd, layer.uk, qa, H * W, W, rows_a, in_rows=plan.list_a, offset=layer.rope)
         lat = torch.empty(rows_a, H, rp, dtype=q.dtype, device=dev)
-        mt = row_tiles(H)
+        mt = row_tiles(layer)
         args = (bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(), K._ptr(plan.row_start))
         if plan.nd:
             visible = min(batch.max_seq_len, window or batch.max_seq_len)

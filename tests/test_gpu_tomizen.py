@@ -399,10 +399,19 @@ def folder(tmp_path_factory):
     return get
 
 
-# rounding of a whole bf16 model against the exact logits; fp32 is the sharp comparison
-MODEL_TOL = {"bfloat16": 0.15, "float32": 3e-4}
+# fp32 is the sharp comparison.  In bf16 a position now and then is ill-conditioned (the norm of a small memory output), so that
+# nine in ten positions are held to the bound
+MODEL_TOL = {"bfloat16": 0.08, "float32": 3e-4}
 SHAPES = {"whole": [[1000], [1000], [1000], [1000]], "decode": [[100, 1], [9, 1], [1], [2, 1]], "portions": [[2, 33, 1, 16], [3, 2], [17, 24], [2]],
           "long portions": [[110, 2], [40], [3, 80], [7]]}
+
+
+def off(got, want, dtype):
+    if dtype == "float32":
+        return TC.spread(got, want)
+    d = got.double() - want.double()
+    d = d - d.mean(-1, keepdim=True)
+    return (d.pow(2).mean(-1).sqrt().quantile(0.9) / want.double().std()).item()
 
 
 @pytest.mark.parametrize("dtype", ["bfloat16", "float32"])
@@ -420,9 +429,9 @@ def test_models_in_portions_and_batches(folder, name, dtype):
         for i, t in toks.items():
             c = TC.portions(len(t), cut(i, shape))
             plans[f"r{i}"] = (t, c, i)
-            assert TC.spread(TC.feed_alone(eng, f"a{i}", t, c), want[i]) < tol, (shape, i)
+            assert off(TC.feed_alone(eng, f"a{i}", t, c), want[i], dtype) < tol, (shape, i)
         for r, lg in TC.feed_together(eng, plans).items():
-            assert TC.spread(lg, want[int(r[1:])]) < tol, (shape, r, "together")
+            assert off(lg, want[int(r[1:])], dtype) < tol, (shape, r, "together")
     assert eng.runner.graph_replays > 0 and eng.pool.num_free == eng.pool.num_blocks
     eng.pool.check_invariants()
 
@@ -452,7 +461,7 @@ def test_decode_graph_equals_eager_decode(folder):
         x, y = TC.feed_together(a, plans), TC.feed_together(b, plans)
         assert a.runner.graph_replays > 0 and b.runner.graph_replays == 0
         for r in plans:
-            assert TC.spread(x[r], y[r]) < (1e-4 if dtype == "float32" else 0.08)
+            assert off(x[r], y[r], dtype) < (1e-4 if dtype == "float32" else 0.05)
 
 
 @pytest.mark.parametrize("options", [{}, {"max_prefill_tokens": 16}, {"num_kv_blocks": 13, "admission_watermark_tokens": 0},
