@@ -183,7 +183,8 @@ struct LatentAttnParams {
 };
 
 // A tile of TOK keys goes through three steps, each one tile behind the other, with one barrier per tile:
-//   scores    warp (kg, tg): k-steps of group kg for the HK keys of part tg -> partial sums in shared memory
+//   scores    warp (kg, tg): k-steps of group kg for the HK keys of part tg -> partial sums in shared memory (with sixteen warps
+//             and 32 rows: warp (kg, tg, wm), one 16-row unit each)
 //   softmax   TPR threads per row add the kLtKG partial sums, keep the row's maximum and sum, write the probabilities (bf16)
 //   output    every warp its NT * 8 columns of the latent over the tile's keys
 // so between two barriers the warps work on the scores of tile p + 1, the softmax of tile p and the output of tile p - 1.  Tiles
@@ -193,7 +194,8 @@ template <int KPG, int NT, int MT, int WARPS, int TOK>
 __global__ void __launch_bounds__(32 * WARPS)
 latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
   constexpr int M = 16 * MT, THREADS = 32 * WARPS, TPR = THREADS / M, KPT = TOK / TPR;
-  constexpr int TG = WARPS / kLtKG, HK = TOK / TG, RPW = TOK / WARPS;
+  constexpr int WM = MT == 2 && WARPS == 16 ? 2 : 1, MS = MT / WM;               // parts of the rows, 16-row units of a warp's scores
+  constexpr int TG = WARPS / kLtKG / WM, HK = TOK / TG, RPW = TOK / WARPS;
   constexpr int PS = TOK + 8, SS = TOK + 4;    // padded rows of the probabilities and of the partial sums
   static_assert(HK == 8 || HK == 16, "eight or sixteen keys per warp");
   static_assert(HK == 16 || KPG % 2 == 0, "pairs of k-steps");
@@ -250,16 +252,16 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
   int next = page_of(S - 2);
 
   // query fragments of this warp's k-steps stay in registers (zero past the row's width)
-  const int kg = warp % kLtKG, tg = warp / kLtKG, nks = W / 16;
+  const int kg = warp % kLtKG, tg = warp / kLtKG % TG, m0 = warp / (kLtKG * TG) * MS, nks = W / 16;
   auto kstep = [&](int i) { return HK == 8 ? 2 * (kg + kLtKG * (i >> 1)) + (i & 1) : kg + kLtKG * i; };
-  uint32_t qf[MT][KPG][4];
+  uint32_t qf[MS][KPG][4];
 #pragma unroll
-  for (int m = 0; m < MT; ++m)
+  for (int m = 0; m < MS; ++m)
 #pragma unroll
     for (int i = 0; i < KPG; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int r = m * 16 + g + 8 * (e & 1), k = kstep(i) * 16 + 2 * t4 + 8 * (e >> 1);
+        const int r = (m0 + m) * 16 + g + 8 * (e & 1), k = kstep(i) * 16 + 2 * t4 + 8 * (e >> 1);
         qf[m][i][e] = r0 + r < n_flat && k < W ? *reinterpret_cast<const uint32_t*>(p.q + (flat0 + r) * W + k) : 0u;
       }
   // softmax: this thread's row and keys
@@ -276,33 +278,42 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
   const uint32_t ukv0 = smem_u32(skv), up0 = smem_u32(sp), stage_bytes = TOK * WS * 2;
   const int d0 = warp * NT * 8;                // this warp's latent columns
 
-  auto scores = [&](int st, int buf) {
-    float acc[MT][HK / 8][4];
+  // ldmatrix addresses inside a tile: this warp's keys at its k-steps (clamped into the row), its latent columns (likewise)
+  constexpr int KO = HK == 16 ? KPG : KPG / 2, VO = NT == 1 ? 1 : NT / 2;
+  uint32_t key_off[KO], col_off[VO];
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+  for (int i = 0; i < KO; ++i)
+    key_off[i] = HK == 16 ? ((tg * 16 + (lane & 7) + ((lane >> 4) << 3)) * WS + ((lane >> 3) & 1) * 8 + min(kstep(i), nks - 1) * 16) * 2
+                          : ((tg * 8 + (lane & 7)) * WS + ((lane >> 3) & 1) * 8 + min(kstep(2 * i) + (lane >> 4), nks - 1) * 16) * 2;
+#pragma unroll
+  for (int n = 0; n < VO; ++n) col_off[n] = NT == 1 ? (a_row * WS + d0) * 2 : (a_row * WS + min(d0 + n * 16, p.rp - 16) + a_col) * 2;
+  const uint32_t step16 = 16 * WS * 2;
+
+  auto scores = [&](int st, int buf) {
+    float acc[MS][HK / 8][4];
+#pragma unroll
+    for (int m = 0; m < MS; ++m)
 #pragma unroll
       for (int n = 0; n < HK / 8; ++n) acc[m][n][0] = acc[m][n][1] = acc[m][n][2] = acc[m][n][3] = 0.f;
     const uint32_t base = ukv0 + st * stage_bytes;
     if constexpr (HK == 16) {
-      const uint32_t bk = base + ((tg * 16 + (lane & 7) + ((lane >> 4) << 3)) * WS + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
       for (int i = 0; i < KPG; ++i) {
         uint32_t bb[4];
-        ldsm4(bk + min(kstep(i), nks - 1) * 32, bb);
+        ldsm4(base + key_off[i], bb);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
+        for (int m = 0; m < MS; ++m) {
           mma16816(acc[m][0], qf[m][i], bb[0], bb[1]);
           mma16816(acc[m][HK / 8 - 1], qf[m][i], bb[2], bb[3]);
         }
       }
     } else {
-      const uint32_t bk = base + ((tg * 8 + (lane & 7)) * WS + ((lane >> 3) & 1) * 8) * 2;
 #pragma unroll
       for (int i = 0; i < KPG; i += 2) {       // eight keys, two k-steps
         uint32_t bb[4];
-        ldsm4(bk + min(kstep(i) + (lane >> 4), nks - 1) * 32, bb);
+        ldsm4(base + key_off[i / 2], bb);
 #pragma unroll
-        for (int m = 0; m < MT; ++m) {
+        for (int m = 0; m < MS; ++m) {
           mma16816(acc[m][0], qf[m][i], bb[0], bb[1]);
           mma16816(acc[m][0], qf[m][i + 1], bb[2], bb[3]);
         }
@@ -310,12 +321,12 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
     }
     float* dst = spart + (buf * kLtKG + kg) * M * SS + tg * HK + 2 * t4;
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+    for (int m = 0; m < MS; ++m)
 #pragma unroll
       for (int n = 0; n < HK / 8; ++n)
 #pragma unroll
         for (int h = 0; h < 2; ++h)
-          *reinterpret_cast<float2*>(dst + (m * 16 + g + 8 * h) * SS + n * 8) = make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
+          *reinterpret_cast<float2*>(dst + ((m0 + m) * 16 + g + 8 * h) * SS + n * 8) = make_float2(acc[m][n][2 * h], acc[m][n][2 * h + 1]);
   };
   auto softmax = [&](int t, int buf) {
     float s[KPT], mx = mrun;
@@ -324,7 +335,14 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
 #pragma unroll
     for (int k = 0; k < kLtKG; ++k) {
       float f[KPT];
-      load_vec<KPT>(spart + ((buf * kLtKG + k) * M + srow) * SS + sc, f);
+      const float* row = spart + ((buf * kLtKG + k) * M + srow) * SS + sc;
+      if constexpr (KPT == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(row);
+        f[0] = v.x;
+        f[KPT - 1] = v.y;
+      } else {
+        load_vec<KPT>(row, f);
+      }
 #pragma unroll
       for (int u = 0; u < KPT; ++u) s[u] += f[u];
     }
@@ -336,17 +354,21 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
     }
 #pragma unroll
     for (int off = TPR / 2; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    // the reference point follows the maximum only when it has grown by a factor of 2^8: the output is rarely rescaled
+    mx = mx > mrun + 8.f ? mx : mrun;
     const float ref = mx == -INFINITY ? 0.f : mx, alpha = fast_exp2(mrun - ref);            // nothing seen yet: 0
+    const float keep = mrun == mx ? 1.f : alpha;
     mrun = mx;
-    lrun *= alpha;
+    lrun *= keep;
     __nv_bfloat16* dst = sp + (buf * M + srow) * PS + sc;
 #pragma unroll
     for (int u = 0; u < KPT; ++u) {
       s[u] = fast_exp2(s[u] - ref);
       lrun += s[u];
     }
-    store_vec<KPT>(dst, s);
-    if (sc == 0) salpha[buf * M + srow] = alpha;
+    if constexpr (KPT == 2) *reinterpret_cast<uint32_t*>(dst) = pack_bf16x2(s[0], s[KPT - 1]);
+    else store_vec<KPT>(dst, s);
+    if (sc == 0) salpha[buf * M + srow] = keep;
   };
   auto output = [&](int st, int buf) {
     if (d0 >= p.rp) return;
@@ -367,14 +389,14 @@ latent_attn_kernel(const LatentAttnParams<__nv_bfloat16> p) {
       if constexpr (NT == 1) {
         uint32_t b0, b1;                       // one n8 tile: matrices keys 0..7 and 8..15
         asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];\n"
-                     : "=r"(b0), "=r"(b1) : "r"(ukv + ((kk * 16 + a_row) * WS + d0) * 2) : "memory");
+                     : "=r"(b0), "=r"(b1) : "r"(ukv + kk * step16 + col_off[0]) : "memory");
 #pragma unroll
         for (int m = 0; m < MT; ++m) mma16816(o[m][0], a[m], b0, b1);
       } else {
 #pragma unroll
         for (int n = 0; n < NT / 2; ++n) {
           uint32_t x[4];                       // columns past the latent are computed and dropped
-          ldsm4t(ukv + ((kk * 16 + a_row) * WS + min(d0 + n * 16, p.rp - 16) + a_col) * 2, x);
+          ldsm4t(ukv + kk * step16 + col_off[n], x);
 #pragma unroll
           for (int m = 0; m < MT; ++m) {
             mma16816(o[m][2 * n], a[m], x[0], x[1]);
@@ -646,9 +668,9 @@ static int launch_latent_1(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaSt
 }
 static int launch_latent_2(LatentAttnParams<__nv_bfloat16>& p, dim3 grid, cudaStream_t st) {
   const int W = p.rp + p.ep;
-  if (p.rp <= 128 && W <= 192) return launch_latent<3, 2, 2, 8, 32>(p, grid, st);
-  if (p.rp <= 256 && W <= 320) return launch_latent<5, 4, 2, 8, 32>(p, grid, st);
-  if (p.rp <= 512 && W <= 576) return launch_latent<9, 8, 2, 8, 32>(p, grid, st);
+  if (p.rp <= 128 && W <= 192) return launch_latent<3, 1, 2, 16, 32>(p, grid, st);
+  if (p.rp <= 256 && W <= 320) return launch_latent<5, 2, 2, 16, 32>(p, grid, st);
+  if (p.rp <= 512 && W <= 576) return launch_latent<9, 4, 2, 16, 32>(p, grid, st);
   return -5;
 }
 
