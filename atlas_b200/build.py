@@ -50,7 +50,7 @@ _UNITS_BASE = ("runtime",)
 _UNITS_BF16 = ("gemm", "elementwise", "attention", "attention_tc16")
 _UNITS_F32 = ("attention_f32",)
 _UNITS_LISTED = ("streams",)                   # residual forms of models that list their layers
-_UNITS_OF_KIND = {"wkv": ("recurrent",), "parallel": ("recurrent",), "mamba2": ("recurrent",), "mlstm": ("mlstm",),
+_UNITS_OF_KIND = {"rglru": ("recurrent", "rglru"), "wkv": ("recurrent",), "parallel": ("recurrent",), "mamba2": ("recurrent",), "mlstm": ("mlstm",),
                   "latent_attention": ("latent",)}
 
 
@@ -62,6 +62,8 @@ def units_for(cfg) -> Optional[List[str]]:
     units = set(_UNITS_BASE + (_UNITS_F32 if cfg.dtype == "float32" else _UNITS_BF16) + _UNITS_LISTED)
     for i, spec in enumerate(cfg.layer_specs):
         units.update(_UNITS_OF_KIND.get(spec.kind, ()))
+        if cfg.for_layer(i).qk_norm_rows:
+            units.add("row_norm_kv")
         if cfg.is_moe_layer(i):
             units.add("moe")
     return sorted(units)

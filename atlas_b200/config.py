@@ -27,7 +27,7 @@ _FAMILY_ALIASES = {
     "holo3_1_moe": "hybrid",
     "nemotron_h": "hybrid", "nemotron_h_puzzle": "hybrid",
     "deepseek_v2": "moe", "deepseek_v3": "moe", "deepseek_v32": "moe", "kimi_k2": "moe",
-    "papidra": "hybrid", "tomizen": "hybrid",
+    "papidra": "hybrid", "tomizen": "hybrid", "kenovik": "hybrid",
 }
 
 # widths the attention kernels are instantiated for; heads of any other size are zero-padded to the next one
@@ -45,10 +45,15 @@ def padded_head_width(*dims: int) -> int:
 @dataclass
 class LayerSpec:
     """One layer of a model whose layers differ in kind or size: the mixer's kind, whether a feed-forward sublayer
-    follows, and the :class:`ModelConfig` fields that hold for this layer only."""
+    follows, and the :class:`ModelConfig` fields that hold for this layer only.
+
+    A layer that runs several times (looped models) has one entry per run, in the order of execution.  Runs after the first
+    take the weights of an earlier entry and keep a cache or state of their own."""
     kind: str                              # a mixer kind of ``layers.MIXERS``
     has_mlp: bool = True
     overrides: Dict[str, Any] = field(default_factory=dict)
+    weights_of: int = -1                   # entry whose weights this run takes (-1: it has its own)
+    step: int = -1                         # >= 0: row of the model's step vectors added to the residual ahead of this run
 
 
 @dataclass
@@ -156,6 +161,9 @@ class ModelConfig:
     residual_streams: int = 0
     # norms on the sublayers' outputs only: every sublayer reads the (fp32) residual stream itself
     output_norms: bool = False
+    # norms on the sublayers' inputs, on an fp32 residual stream (models given by a list of layers)
+    input_norms: bool = False
+    loop_steps: int = 0               # passes of the looped layers that have a step vector
     mamba_num_heads: int = 0
     mamba_head_dim: int = 64
     ssm_state_size: int = 128
@@ -163,6 +171,10 @@ class ModelConfig:
     mamba_conv_kernel: int = 4
     mamba_dt_min: float = 0.0
     mamba_norm_groups: int = 0        # parts of the gated output norm (0 = one per B / C group)
+    # RG-LRU recurrence (gated linear recurrent unit per channel)
+    rglru_width: int = 0
+    rglru_blocks: int = 0
+    rglru_conv_kernel: int = 4
     # WKV recurrence (RWKV-style time mixing)
     wkv_num_heads: int = 0
     wkv_head_dim: int = 0
@@ -174,12 +186,21 @@ class ModelConfig:
     mlp_activation: str = "silu_glu"  # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down) | clamped_glu
     glu_limit: float = 0.0            # clamped_glu: bound on the gate (above) and on the up branch (both sides)
     glu_alpha: float = 1.702          # clamped_glu: slope inside the gate's sigmoid
+    shared_glu_limit: float = 0.0     # the same bound for the shared expert
     # attention variants: chunked visibility (a token sees its own chunk only), a learned per-head sink in the softmax
     # denominator, the number of rotated dimensions when it is not a fraction of head_dim
     attn_chunk: int = 0
     attn_sinks: bool = False
+    attn_sink_score: Optional[float] = None   # a fixed sink score of every head instead of learned ones (0: one is added)
     attn_softcap: float = 0.0         # scores become cap * tanh(score / cap) before the softmax (0 = off)
     attn_head_gate: bool = False      # every head's output times the sigmoid of one number per head
+    # a learned bias per head and distance bucket joins the scores: rows of the table and the distance from which on all
+    # keys share its last row (0 = off); the first half of the rows are single distances, the others logarithmic
+    attn_distance_rows: int = 0
+    attn_distance_reach: int = 0
+    qk_norm_rows: bool = False        # q and k are normed over all heads at once, before they are split
+    attn_query_temp: float = 0.0      # queries times 1 + c ln(floor((position + 1) / every) + 1) (0 = off)
+    attn_query_temp_every: int = 1
     rotary_dims: Optional[int] = None
     attn_cache_width: int = 0         # padded width of cached heads (0 = head_dim)
     # multi-head latent attention (DeepSeek): 0 = plain GQA.  head_dim is then the padded cache width
@@ -269,7 +290,7 @@ class ModelConfig:
         h, L = self.hidden_size, self.num_hidden_layers
         n = self.vocab_size * h * (1 if self.tie_word_embeddings else 2)
         if self.layer_specs:
-            return n + sum(self.for_layer(i)._spec_layer_params(s) for i, s in enumerate(self.layer_specs))
+            return n + sum(self.for_layer(i)._spec_layer_params(s) for i, s in enumerate(self.layer_specs) if s.weights_of < 0)
         for i in range(L):
             if self.layer_kind(i) == "attention":
                 qmul = 2 if self.attn_output_gate else 1
@@ -298,12 +319,15 @@ class ModelConfig:
         n = 3 * h * self.intermediate_size if spec.has_mlp and not self.num_experts else 0
         if spec.has_mlp and self.num_experts:
             n += self.num_experts * (h + (2 if self.mlp_activation == "relu2" else 3) * h * self.moe_intermediate_size)
+            n += 3 * h * self.shared_expert_intermediate_size
         if spec.kind in ("attention", "parallel"):
             dv = self.v_head_dim or self.head_dim
             n += h * (self.q_size + self.kv_size + self.num_key_value_heads * dv) + self.num_attention_heads * dv * h
         if spec.kind in ("mamba2", "parallel"):
             di = self.mamba_num_heads * self.mamba_head_dim
             n += h * (2 * di + 2 * self.mamba_n_groups * self.ssm_state_size + self.mamba_num_heads) + di * h
+        if spec.kind == "rglru":
+            n += 3 * h * self.rglru_width + 2 * self.rglru_width * (self.rglru_width // self.rglru_blocks)
         if spec.kind == "wkv":
             n += 5 * h * self.wkv_num_heads * self.wkv_head_dim
         if spec.kind == "mlstm":
@@ -472,10 +496,14 @@ class ModelConfig:
 
 # ---------------------------------------------------------------------------- configurations that list their layers
 def _rotary_overrides(rot: Optional[Dict[str, Any]]) -> Dict[str, Any]:
-    """``{dims, base, scaling}`` -> rotary fields; ``scaling`` is YaRN's ``{factor, original, fast, slow}``."""
+    """``{dims, base, scaling}`` -> rotary fields; ``scaling`` is YaRN's ``{factor, original, fast, slow}`` or, with a factor alone,
+    linear."""
     if not rot:
         return {"rotary_dims": 0}
     sc = rot.get("scaling")
+    if sc and "original" not in sc:
+        return {"rotary_dims": int(rot["dims"]), "rope_theta": float(rot["base"]),
+                "rope_scaling": {"rope_type": "linear", "factor": float(sc["factor"])}}
     return {"rotary_dims": int(rot["dims"]), "rope_theta": float(rot["base"]),
             "rope_scaling": None if not sc else {
                 "rope_type": "yarn", "factor": float(sc["factor"]), "original_max_position_embeddings": float(sc["original"]),
@@ -582,8 +610,77 @@ def tomizen_config(cfg: Dict[str, Any]) -> ModelConfig:
     return _size_by_heads(c)
 
 
+def _kenovik_ff(mlp: Dict[str, Any]) -> Dict[str, Any]:
+    if mlp.get("kind", "dense") == "dense":
+        return {"intermediate_size": int(mlp["ff"]), "mlp_activation": "silu_glu"}
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unsupported Kenovik feed-forward '{mlp['kind']}'")
+    r, shared = mlp["router"], mlp.get("shared")
+    groups = r.get("groups") or {"count": 1, "keep": 1}
+    if int(r["experts"]) % int(groups["count"]):
+        raise ValueError(f"{r['experts']} experts do not form {groups['count']} equal groups")
+    return {"num_experts": int(r["experts"]), "num_experts_per_tok": int(r["top"]), "moe_intermediate_size": int(mlp["expert"]["ff"]),
+            "mlp_activation": "clamped_glu", "glu_limit": float(mlp["expert"]["limit"]), "norm_topk_prob": True,
+            "router_scoring": "sigmoid", "router_selection_bias": True, "router_f32": True, "routed_scaling_factor": float(r["scale"]),
+            "router_n_group": int(groups["count"]), "router_topk_group": int(groups["keep"]),
+            "shared_expert_intermediate_size": int(shared["ff"]) if shared else 0,
+            "shared_glu_limit": float(shared["limit"]) if shared else 0.0}
+
+
+def _kenovik_layer(lc: Dict[str, Any]) -> LayerSpec:
+    kind, m, mlp = str(lc["type"]), lc["mixer"], lc.get("mlp")
+    if kind == "rglru":
+        over = {"rglru_width": int(m["width"]), "rglru_blocks": int(m["blocks"]), "rglru_conv_kernel": int(m["conv"])}
+        if over["rglru_width"] % over["rglru_blocks"]:
+            raise ValueError(f"{over['rglru_width']} channels do not form {over['rglru_blocks']} equal blocks")
+    elif kind == "attention":
+        over = {**_attention_overrides(m), "attention_bias": True, "attn_sinks": True, "attn_sink_score": 0.0}
+    elif kind == "attention_2":
+        temp = m.get("q_temp") or {"coef": 0.0, "every": 1}
+        over = {**_attention_overrides(m), "qk_norm": True, "qk_norm_rows": True, "qk_norm_plus_one": False,
+                "attn_query_temp": float(temp["coef"]), "attn_query_temp_every": int(temp["every"]),
+                "attn_distance_rows": int(m.get("bias_rows", 32)), "attn_distance_reach": int(m["bias_max"])}
+        kind = "attention"
+    else:
+        raise ValueError(f"unsupported Kenovik layer type '{kind}'")
+    if mlp is not None:
+        over.update(_kenovik_ff(mlp))
+    return LayerSpec(kind, mlp is not None, over)
+
+
+def _unrolled(specs: List[LayerSpec], loop: Optional[Dict[str, Any]]) -> List[LayerSpec]:
+    """One entry per run of a layer: layers ``start .. stop - 1`` run ``times`` times in a row on the same weights, and the first
+    one of every pass adds that pass's step vector."""
+    if not loop:
+        return list(specs)
+    a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= a < b <= len(specs) or times < 1:
+        raise ValueError(f"a loop over layers {a} .. {b - 1}, {times} times, does not fit a model of {len(specs)} layers")
+    runs = list(specs[:a])
+    for t in range(times):
+        for i in range(a, b):
+            runs.append(dataclasses.replace(specs[i], weights_of=i if t else -1, step=t if i == a else -1))
+    return runs + list(specs[b:])
+
+
+def kenovik_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """Kenovik: RG-LRU layers and two kinds of attention (biased projections with a fixed sink; distance bias with normed
+    projections and a query temperature), dense or expert feed-forwards, some of the layers run several times."""
+    loop = cfg.get("loop")
+    specs = _unrolled([_kenovik_layer(lc) for lc in cfg["layers"]], loop)
+    widest = lambda k: max([s.overrides.get(k, 0) for s in specs] + [0])
+    c = ModelConfig(model_type="kenovik", family="hybrid", vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                    intermediate_size=max(1, widest("intermediate_size"), widest("moe_intermediate_size")), num_hidden_layers=len(specs),
+                    num_attention_heads=1, num_key_value_heads=1, head_dim=64, rms_norm_eps=float(cfg["norm"]["eps"]), input_norms=True,
+                    embed_scale=float(cfg["embedding"]["scale"]), loop_steps=int(loop["times"]) if loop else 0, tie_word_embeddings=True,
+                    layer_specs=specs, dtype=str(cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))),
+                    quant=QuantConfig(kv_cache_dtype="bf16"), bos_token_id=cfg.get("bos_token_id"), eos_token_id=cfg.get("eos_token_id"))
+    c.moe_intermediate_size = widest("moe_intermediate_size")
+    return _size_by_heads(c)
+
+
 # ``architecture`` of a config.json that lists its layers one by one -> its reader
-_NATIVE_ARCHITECTURES = {"papidra": papidra_config, "tomizen": tomizen_config}
+_NATIVE_ARCHITECTURES = {"papidra": papidra_config, "tomizen": tomizen_config, "kenovik": kenovik_config}
 
 
 # ---------------------------------------------------------------------------- presets
@@ -741,12 +838,48 @@ def tomizen_16b(quant: str = "none") -> ModelConfig:
     return c
 
 
+def _kenovik(vocab: int, width: int, pattern: str, lru: tuple, attn: tuple, attn2: tuple, ff: int, experts: tuple, loop: Optional[tuple],
+             dtype: str) -> ModelConfig:
+    """``pattern``: ``r`` = RG-LRU, ``a`` = attention with a fixed sink, ``d`` = attention with a distance bias, each with experts;
+    a capital letter has a dense feed-forward of ``ff`` instead.  ``lru`` (width, blocks), ``attn`` (heads, kv heads, dim, vdim,
+    rotated), ``attn2`` (heads, kv heads, dim, vdim, reach), ``experts`` (count, top, ff, groups, kept), ``loop`` (start, stop, times)."""
+    mixers = {
+        "r": ("rglru", {"width": lru[0], "blocks": lru[1], "conv": 4}),
+        "a": ("attention", {"heads": attn[0], "kv_heads": attn[1], "dim": attn[2], "vdim": attn[3], "scale": attn[2] ** -0.5,
+                            "rot": {"base": 5e5, "dims": attn[4], "scaling": {"factor": 4.0}}}),
+        "d": ("attention_2", {"heads": attn2[0], "kv_heads": attn2[1], "dim": attn2[2], "vdim": attn2[3], "scale": attn2[2] ** -0.5,
+                              "bias_max": attn2[4], "q_temp": {"coef": 0.1, "every": 8192}})}
+    e, top, eff, groups, keep = experts
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "shared": {"ff": eff, "limit": 7.0},
+           "router": {"experts": e, "top": top, "scale": 2.5, "groups": {"count": groups, "keep": keep}}}
+    layers = [{"type": mixers[ch.lower()][0], "mixer": mixers[ch.lower()][1], "mlp": {"kind": "dense", "ff": ff} if ch.isupper() else moe}
+              for ch in pattern]
+    return kenovik_config({"vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": width ** 0.5}, "dtype": dtype,
+                           "loop": None if loop is None else dict(zip(("start", "stop", "times"), loop)), "layers": layers})
+
+
+def tiny_kenovik(dtype: str = "float32") -> ModelConfig:
+    c = _kenovik(1024, 192, "Drad", (144, 3), (6, 2, 64, 48, 32), (4, 2, 48, 64, 100), 256, (8, 3, 96, 4, 2), (1, 3, 2), dtype)
+    c.max_position_embeddings = 4096
+    return c
+
+
+def kenovik_20b(quant: str = "none") -> ModelConfig:
+    """Layers of the size of a 20B mixture-of-experts decoder: width 2048, RG-LRU of 2560 channels in 10 blocks, 16 heads of 128
+    (2 kv), 64 experts of 1408 (6 per token, 8 groups of which 4 stay open), the middle eight layers run twice."""
+    c = _kenovik(131072, 2048, "R" + "radr" * 7 + "rad", (2560, 10), (16, 2, 128, 128, 64), (16, 2, 128, 128, 4096), 8192,
+                 (64, 6, 1408, 8, 4), (12, 20, 2), "bfloat16")
+    c.quant = QuantConfig(method=quant, kv_cache_dtype="bf16")
+    return c
+
+
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "tiny-hybrid": tiny_hybrid,
     "llama3-8b": llama3_8b, "llama3-70b": llama3_70b,
     "qwen3-30b-a3b": qwen3_30b_a3b, "qwen3-next-80b": qwen3_next_80b,
     "tiny-nemotron-h": tiny_nemotron_h, "nemotron-h-8b": nemotron_h_8b, "tiny-deepseek": tiny_deepseek,
     "tiny-papidra": tiny_papidra, "papidra-8b": papidra_8b, "tiny-tomizen": tiny_tomizen, "tomizen-16b": tomizen_16b,
+    "tiny-kenovik": tiny_kenovik, "kenovik-20b": kenovik_20b,
 }
 
 

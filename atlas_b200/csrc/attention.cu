@@ -37,6 +37,7 @@ struct AttnParams {
   int chunk;                                    // > 0: a row sees keys of its own chunk-token block of the sequence only
   const float* sinks;                           // [Hq] or null: exp(sink) joins the softmax denominator
   float cap_in, cap_out;                        // bounded scores (bf16 cache): see capped_score in tc_util.cuh; cap_out 0 = off
+  const float* distance; int reach;             // bf16 cache: [Hq, reach + 1], joins the score of a key by its distance (null = off)
   // decode
   int num_splits;
   float* part_o;                                // [B, Hq, splits, D]
@@ -97,6 +98,10 @@ ATLAS_DEVICE int first_visible(const AttnParams& p, int pos) {
 // q . k of a bf16 cache -> score in the exp2 domain
 ATLAS_DEVICE float score_log2(const AttnParams& p, float s) {
   return p.cap_out > 0.f ? capped_score(s, p.cap_in, p.cap_out) : s * p.qk_scale_log2;
+}
+// distance bias of `head` for a key `back` tokens before the query, in the exp2 domain
+ATLAS_DEVICE float distance_log2(const AttnParams& p, int head, int back) {
+  return __ldg(p.distance + (long long)head * (p.reach + 1) + min(max(back, 0), p.reach)) * 1.4426950408889634f;
 }
 // A sink joins the denominator of a row with running maximum m (log2 units) and sum l.  Returns the factor on what was
 // accumulated so far.
@@ -268,6 +273,9 @@ paged_attn_kernel(const AttnParams p) {
           const bool ok = tok <= qpos[h] && tok < L && tok >= lo_pos[h];
           float& sv = s[i][2 * h + j];
           sv = ok ? (KV16 ? score_log2(p, sv) : sv) : -INFINITY;
+          if constexpr (KV16) {
+            if (p.distance && ok) sv += distance_log2(p, PREFILL ? qhead : min(kvh * G + g0 + rq + 8 * h, p.Hq - 1), qpos[h] - tok);
+          }
           mx[h] = fmaxf(mx[h], sv);
         }
       }
@@ -879,6 +887,10 @@ attn_decode_cp_kernel(const AttnParams p) {
       sq[1] = __shfl_sync(0xffffffffu, qs, (2 * c + 1) * 4);
     }
     const int win_lo = first_tok - 1;                         // tokens <= win_lo are not visible
+    // distance bias: heads c*2 and c*2+1 of this thread's score columns; keys at `reach` tokens or more share one value
+    const int bias_h[2] = {head0 + min(2 * c, G - 1), head0 + min(2 * c + 1, G - 1)};
+    float bias_far[2] = {0.f, 0.f};
+    if (KV16 && p.distance) { bias_far[0] = distance_log2(p, bias_h[0], p.reach); bias_far[1] = distance_log2(p, bias_h[1], p.reach); }
     // this thread's two token rows inside a page
     const int tok_r0 = (rq >> 1) * 4 + (rq & 1);
     const int tok_r1 = tok_r0 + 2;
@@ -949,6 +961,16 @@ attn_decode_cp_kernel(const AttnParams p) {
           }
 #pragma unroll
           for (int e = 0; e < 4; ++e) s[e] = score_log2(p, s[e]);
+          if (p.distance) {
+            const int back = L - 1 - (blk_tok0 + sub * 16);          // distance of the page's first token
+            if (back - 15 >= p.reach) {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) s[e] += bias_far[e & 1];
+            } else {
+#pragma unroll
+              for (int e = 0; e < 4; ++e) s[e] += distance_log2(p, bias_h[e & 1], back - (e < 2 ? tok_r0 : tok_r1));
+            }
+          }
         } else if constexpr (KV4) {
           const int ta = sub * 16 + tok_r0, tb = sub * 16 + tok_r1;
           const uint8_t* ka = kblk + ta * (D / 2) + c * (DQ / 2);
@@ -1526,7 +1548,7 @@ static int fill_common(AttnParams& p, const void* q, long long ldq, void* out, l
   p.Hq = Hq; p.Hkv = Hkv; p.block_size = block_size; p.window = window;
   p.num_splits = 1; p.part_o = nullptr; p.part_ml = nullptr; p.tile_seq = nullptr; p.tile_q0 = nullptr; p.num_tiles = 0;
   p.q_out = nullptr; p.ldqo = 0; p.s_out = nullptr; p.s_ld = 0;
-  p.chunk = 0; p.sinks = nullptr; p.cap_in = p.cap_out = 0.f;
+  p.chunk = 0; p.sinks = nullptr; p.cap_in = p.cap_out = 0.f; p.distance = nullptr; p.reach = 0;
   return 0;
 }
 
@@ -1695,18 +1717,19 @@ extern "C" int atlas_attn_prefill_kv4(const void* q, long long ldq, void* out, l
 
 // Same contracts as atlas_attn_decode / atlas_attn_prefill with a bf16 cache (K [nb, Hkv, bs, D], V [nb, Hkv, D, bs]), any
 // number of query heads per kv head, and optional chunked visibility (`chunk` > 0), softmax sinks (fp32 [Hq]) and bounded
-// scores (`softcap` > 0: softcap * tanh(score / softcap)).
+// scores (`softcap` > 0: softcap * tanh(score / softcap)) and a distance bias (fp32 [Hq, reach + 1], null = off).
 extern "C" int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache,
                                       const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                       const int* query_start_loc, int seq_base, int B, float scale, int Hq, int Hkv, int D,
                                       int block_size, int window, int num_splits, float* part_o, float* part_ml, void* stream,
-                                      int chunk, const float* sinks, float softcap) {
+                                      int chunk, const float* sinks, float softcap, const float* distance, int reach) {
   if (B <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, seq_base, scale,
                        1.f, 1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
-  p.chunk = chunk; p.sinks = sinks;
+  if (distance && reach < 0) return -6;
+  p.chunk = chunk; p.sinks = sinks; p.distance = distance; p.reach = reach;
   if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   p.num_splits = num_splits < 1 ? 1 : num_splits;
   if (p.num_splits > 1 && (!part_o || !part_ml)) return -3;
@@ -1721,13 +1744,14 @@ extern "C" int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, 
                                        const void* v_cache, const int* block_tables, int bt_ld, const int* seq_lens,
                                        const int* query_start_loc, const int* tile_seq, const int* tile_q0, int num_tiles,
                                        float scale, int Hq, int Hkv, int D, int block_size, int window, void* stream, int chunk,
-                                       const float* sinks, float softcap) {
+                                       const float* sinks, float softcap, const float* distance, int reach) {
   if (num_tiles <= 0) return 0;
   AttnParams p;
   int rc = fill_common(p, q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, 0, scale, 1.f,
                        1.f, Hq, Hkv, D, block_size, window);
   if (rc) return rc;
-  p.chunk = chunk; p.sinks = sinks;
+  if (distance && reach < 0) return -6;
+  p.chunk = chunk; p.sinks = sinks; p.distance = distance; p.reach = reach;
   if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.num_tiles = num_tiles;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

@@ -4,7 +4,8 @@
 //                             its way into the cache
 //   attn_f32_kernel           one warp per (query row, head), prompt rows and decode rows alike: 32 keys a step, one per
 //                             lane, online softmax, then every lane accumulates its own output dimensions.  Sliding window,
-//                             chunked visibility, softmax sinks and bounded scores as in paged_attn_kernel (attention.cu).
+//                             chunked visibility, softmax sinks, bounded scores and distance bias as in paged_attn_kernel
+//                             (attention.cu).
 //
 // Cache layout: K [blocks, Hkv, block_size, D], V [blocks, Hkv, D, block_size].
 #include "common.cuh"
@@ -61,6 +62,7 @@ struct AttnF32Params {
   const int* block_tables; int bt_ld;
   const int* seq_lens; const int* query_start_loc;
   const float* sinks;
+  const float* distance; int reach;            // [Hq, reach + 1] by the key's distance (null = off)
   int B, T, Hq, Hkv, block_size, window, chunk;
   float scale, softcap;
 };
@@ -105,6 +107,7 @@ attn_f32_kernel(const AttnF32Params p) {
         s += kv.x * sq[warp][d * 4] + kv.y * sq[warp][d * 4 + 1] + kv.z * sq[warp][d * 4 + 2] + kv.w * sq[warp][d * 4 + 3];
       }
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (p.distance) s += __ldg(p.distance + (long long)head * (p.reach + 1) + min(pos - j, p.reach));
     }
     const float top = fmaxf(m, warp_max(s));
     const float f = m == -INFINITY ? 0.f : expf(m - top);
@@ -146,10 +149,10 @@ extern "C" int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, 
 extern "C" int atlas_attn_f32(const float* q, long long ldq, float* out, long long ldo, const float* k_cache, const float* v_cache,
                               const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int B, int T,
                               float scale, int Hq, int Hkv, int D, int block_size, int window, int chunk, const float* sinks,
-                              float softcap, void* stream) {
+                              float softcap, const float* distance, int reach, void* stream) {
   if (T <= 0 || B <= 0) return 0;
-  if (Hq % Hkv || block_size < 1) return -1;
-  AttnF32Params p = {q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, sinks, B, T, Hq, Hkv,
+  if (Hq % Hkv || block_size < 1 || (distance && reach < 0)) return -1;
+  AttnF32Params p = {q, ldq, out, ldo, k_cache, v_cache, block_tables, bt_ld, seq_lens, query_start_loc, sinks, distance, reach, B, T, Hq, Hkv,
                      block_size, window, chunk, scale, softcap};
   const dim3 grid((unsigned)(((long long)T * Hq + 3) / 4));
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

@@ -1,6 +1,6 @@
 // Prefill (chunk) attention over the paged bf16 KV cache on the 5th-generation tensor cores: head_dim 64 or 128, 16-token
 // pages, any number of query heads per kv head up to 128, causal with optional chunked visibility, sliding window, softmax
-// sinks and bounded scores.
+// sinks, bounded scores and a bias per head by the key's distance.
 //
 // One CTA per (128-row query tile, kv head); the G query heads that share the kv head are packed into the tile's rows
 // (row = token * G + head; rows past G * floor(128 / G) stay unused).  The cached bytes are MMA operands as they are, so
@@ -32,6 +32,8 @@ struct Tc16Params {
   const float* sinks;
   float scale_log2;
   float cap_in, cap_out;                      // bounded scores (cap_out 0 = off)
+  const float* distance; int reach;           // [Hq, reach + 1] joins a score by the key's distance (null = off)
+  int bias_ld;                                // > 0: the group's rows fit in shared memory, this many floats apart (exp2 domain)
   int Hkv, G, chunk, window;
   status_t* status;
 };
@@ -74,6 +76,7 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
   uint64_t* x_ready = bars + 15;              // [2 parities][4 row groups]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 23);
   volatile uint32_t* abort_flag = tmem_slot + 1;
+  float* s_bias = reinterpret_cast<float*>(bars + 32);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int G = p.G, tpt = kT16Rows / G;      // query tokens per tile
@@ -100,6 +103,11 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
   }
   if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
   if (warp == 0 && lane == 0) tma_prefetch_desc(&tmap_q);
+  if (p.bias_ld > 0) {
+    const float* src = p.distance + (long long)kvh * G * (p.reach + 1);
+    for (int g = 0; g < G; ++g)
+      for (int i = threadIdx.x; i <= p.reach; i += kT16Threads) s_bias[g * p.bias_ld + i] = src[g * (p.reach + 1) + i] * 1.4426950408889634f;
+  }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -243,7 +251,12 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
     const int pos = ctx0 + tok;
     const int lo_pos = first_visible16(p, pos);
     const bool capped = p.cap_out > 0.f;
-    const float s_mul = capped ? 1.f : p.scale_log2;
+    const bool biased = p.distance != nullptr;
+    const float s_mul = capped || biased ? 1.f : p.scale_log2;
+    const int bias_head = row % G;
+    const float* bias_row = biased ? (p.bias_ld > 0 ? s_bias + bias_head * p.bias_ld : p.distance + (long long)(kvh * G + bias_head) * (p.reach + 1)) : nullptr;
+    const float bias_mul = p.bias_ld > 0 ? 1.f : 1.4426950408889634f;
+    const float bias_far = biased ? bias_row[p.reach] * bias_mul : 0.f;
     float m = -INFINITY, l = 0.f;                                 // m: reference point in the exp2 domain
     const int sw = row & 7;
     uint8_t* prow = sP + half * kT16Sub + (row >> 3) * 1024 + sw * 128;
@@ -265,6 +278,24 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
         for (int c = 0; c < 2; ++c)
 #pragma unroll
           for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(capped_score(__uint_as_float(sr[c][i]), p.cap_in, p.cap_out));
+      }
+      if (biased) {
+        const float mul = capped ? 1.f : p.scale_log2;
+        const int back = pos - kv0 - col0;                            // distance of this thread's first column
+        if (__all_sync(0xffffffffu, back - 63 >= p.reach)) {
+#pragma unroll
+          for (int c = 0; c < 2; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sr[c][i] = __float_as_uint(fmaf(__uint_as_float(sr[c][i]), mul, bias_far));
+        } else {
+#pragma unroll
+          for (int c = 0; c < 2; ++c)
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              const float bv = bias_row[min(max(back - c * 32 - i, 0), p.reach)] * bias_mul;
+              sr[c][i] = __float_as_uint(fmaf(__uint_as_float(sr[c][i]), mul, bv));
+            }
+        }
       }
       const bool full = __all_sync(0xffffffffu, vis >= col0 + 64 && hid <= col0);
       if (!full) {
@@ -368,8 +399,16 @@ attn_prefill_tc16_kernel(const __grid_constant__ CUtensorMap tmap_q, const Tc16P
 template <int D>
 static int launch_tc16(const CUtensorMap& tq, const Tc16Params& p, int num_tiles, cudaStream_t st) {
   constexpr int kSmem = (D / 64) * kT16Sub + 2 * kT16Sub + 2 * (D / 64) * kT16Sub + 4 * D * 128 + 256 + 1024;
-  if (ensure_dynamic_smem(reinterpret_cast<const void*>(attn_prefill_tc16_kernel<D>), kSmem) != cudaSuccess) return -20;
-  attn_prefill_tc16_kernel<D><<<dim3(num_tiles, p.Hkv), kT16Threads, kSmem, st>>>(tq, p);
+  Tc16Params pp = p;
+  int bytes = kSmem;
+  pp.bias_ld = 0;
+  if (p.distance) {
+    // rows 32 / G banks apart: the heads of a token meet different banks
+    const int step = p.G < 32 ? 32 / p.G : 1, ld = (p.reach + 1 + 31) / 32 * 32 + step;
+    if ((long long)kSmem + 4ll * p.G * ld <= 227 * 1024) { pp.bias_ld = ld; bytes += 4 * p.G * ld; }
+  }
+  if (ensure_dynamic_smem(reinterpret_cast<const void*>(attn_prefill_tc16_kernel<D>), bytes) != cudaSuccess) return -20;
+  attn_prefill_tc16_kernel<D><<<dim3(num_tiles, p.Hkv), kT16Threads, bytes, st>>>(tq, pp);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
@@ -383,8 +422,9 @@ extern "C" int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, 
                                        const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc,
                                        const int* tile_seq, const int* tile_q0, int num_tiles, int total_tokens, float scale, int Hq,
                                        int Hkv, int D, int block_size, int chunk, int window, const float* sinks, float softcap,
-                                       unsigned long long* status, void* stream) {
+                                       const float* distance, int reach, unsigned long long* status, void* stream) {
   if (num_tiles <= 0) return 0;
+  if (distance && reach < 0) return -2;
   if ((D != 64 && D != 128) || block_size != kT16Page || Hq % Hkv || Hq / Hkv > kT16Rows || !(scale > 0.f)) return 1;
   if ((reinterpret_cast<uintptr_t>(q) & 15) || (ldq % 8) || (ldo % 8) || (reinterpret_cast<uintptr_t>(out) & 15)) return 1;
   EncodeTiledFn enc = tc_encode_fn();
@@ -405,6 +445,7 @@ extern "C" int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, 
   p.tile_seq = tile_seq; p.tile_q0 = tile_q0; p.sinks = sinks; p.scale_log2 = scale * 1.4426950408889634f;
   p.Hkv = Hkv; p.G = G; p.chunk = chunk; p.window = window; p.status = status;
   p.cap_in = p.cap_out = 0.f;
+  p.distance = distance; p.reach = reach; p.bias_ld = 0;
   if (softcap > 0.f) cap_constants(scale, softcap, &p.cap_in, &p.cap_out);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return D == 64 ? launch_tc16<64>(tq, p, num_tiles, st) : launch_tc16<128>(tq, p, num_tiles, st);

@@ -251,6 +251,18 @@ ATLAS_DEVICE float fp8_e4m3_to_f32(uint8_t v) {
 ATLAS_DEVICE uint8_t f32_to_fp8_e4m3(float v) {
   return (uint8_t)__nv_cvt_float_to_fp8(v, __NV_SATFINITE, __NV_E4M3);
 }
+// gated unit: g = min(gate, limit), u = clamp(up, +-limit):  g sigmoid(alpha g) (u + shift).  limit = inf, alpha = 1, shift = 0 is
+// silu(gate) * up.
+struct GatedUnit { float limit, alpha, shift; };
+ATLAS_DEVICE float gated_unit(float gate, float up, const GatedUnit& k) {
+  const float g = fminf(gate, k.limit), u = fminf(fmaxf(up, -k.limit), k.limit);
+  return g / (1.f + expf(-k.alpha * g)) * (u + k.shift);
+}
+// the same for values that leave in bf16
+ATLAS_DEVICE float gated_unit_fast(float gate, float up, const GatedUnit& k) {
+  const float g = fminf(gate, k.limit), u = fminf(fmaxf(up, -k.limit), k.limit);
+  return __fdividef(g, 1.f + __expf(-k.alpha * g)) * (u + k.shift);
+}
 ATLAS_DEVICE float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

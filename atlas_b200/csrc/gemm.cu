@@ -69,9 +69,11 @@ struct GemmParams {
   int m_tiles, n_tiles;
   int b_scale_ld;           // k-groups per row of b_scale
   int vec_ok;               // 16-byte stores into C are legal
-  // bf16 kernels: columns from tail_col on are stored as fp32 in `tail` [M, N - tail_col] (null = off); relu2 squares the
-  // positive part of every value before the store
-  float* tail; long long tail_ld; int tail_col, tail_vec, relu2;
+  // bf16 kernels: columns from tail_col on are stored as fp32 in `tail` [M, N - tail_col] (null = off); `bias` [N] joins the
+  // sums; act 1 squares the positive part of every value before the store, act 2 takes neighbouring columns as gate and up of
+  // a gated unit (common.cuh) and stores N / 2 columns
+  float* tail; long long tail_ld; int tail_col, tail_vec;
+  const float* bias; int act; GatedUnit unit;
   int cluster_splits;       // > 1: the K splits of a tile are the CTAs of one thread-block cluster (one item per CTA, a
                             // single m-tile): partials meet in distributed shared memory instead of the workspace and
                             // every CTA finishes 128 / cluster_splits rows of the tile (see cluster_tail)
@@ -1011,13 +1013,35 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
       } else
       if (store_now && m < M_rows) {
         __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)m * p.ldc;
-        if (!FP8 && p.relu2) {
+        if (!FP8 && p.bias != nullptr) {
+#pragma unroll
+          for (int i = 0; i < HALF; ++i)
+            if (n_base + i < p.N) acc[i] += __ldg(p.bias + n_base + i);
+        }
+        if (!FP8 && p.act == 1) {
 #pragma unroll
           for (int i = 0; i < HALF; ++i) {
             const float r = fmaxf(acc[i], 0.f);
             acc[i] = r * r;
           }
         }
+        if (!FP8 && p.act == 2) {
+#pragma unroll
+          for (int j = 0; j < HALF; j += 16) {
+            const int n = n_base + j;
+            float o[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[i] = gated_unit_fast(acc[j + 2 * i], acc[j + 2 * i + 1], p.unit);
+            if (p.vec_ok && n + 16 <= p.N) {
+              *reinterpret_cast<uint4*>(crow + n / 2) =
+                  make_uint4(pack_bf16x2(o[0], o[1]), pack_bf16x2(o[2], o[3]), pack_bf16x2(o[4], o[5]), pack_bf16x2(o[6], o[7]));
+            } else {
+#pragma unroll
+              for (int i = 0; i < 8; ++i)
+                if (n + 2 * i < p.N) crow[n / 2 + i] = __float2bfloat16_rn(o[i]);
+            }
+          }
+        } else
 #pragma unroll
         for (int j = 0; j < HALF; j += 8) {
           const int n = n_base + j;
@@ -1283,7 +1307,8 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
                      long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters,
                      int num_sms, unsigned long long* status, void* stream, const uint32_t* a_ready,
                      const unsigned int* a_ready_epoch, long long max_cycles, const AtlasEpilogue* epi = nullptr,
-                     float* tail = nullptr, long long tail_ld = 0, int tail_col = 0) {
+                     float* tail = nullptr, long long tail_ld = 0, int tail_col = 0, const float* bias = nullptr, int act = 0,
+                     float glu_limit = 0.f, float glu_alpha = 0.f, float glu_shift = 0.f) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const uint32_t esize = kind == 1 ? 1 : 2;
   const int elems_per_row = 128 / esize;
@@ -1316,6 +1341,7 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
   p.status = status; p.ldc = ldc; p.sa_k = sa_k; p.M = M; p.N = N; p.K = K;
   p.epi_mode = epi_mode;
   p.tail = tail; p.tail_ld = tail_ld; p.tail_col = tail_col;
+  p.bias = bias; p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift};
   p.tail_vec = tail_col % 4 == 0 && tail_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(tail) & 15) == 0 ? 1 : 0;
   if (epi) {
     p.act_cols = N / 2; p.q_out = reinterpret_cast<uint8_t*>(epi->q_out); p.ldq = epi->ldq; p.s_out = epi->s_out; p.s_ld = epi->s_ld;
@@ -1349,7 +1375,7 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
   // and meet in distributed shared memory (cluster_tail) instead of in the global workspace.
   p.cluster_splits = 1;
   if (cluster_splitk_enabled() && p.m_tiles == 1 && block_n == 128 && (p.splits == 2 || p.splits == 4) && items <= num_sms &&
-      (epi_mode == 2 || (epi_mode == 0 && p.vec_ok && tail == nullptr)) && (N % 128) == 0 && a_ready == nullptr)
+      (epi_mode == 2 || (epi_mode == 0 && p.vec_ok && tail == nullptr && bias == nullptr && act == 0)) && (N % 128) == 0 && a_ready == nullptr)
     p.cluster_splits = p.splits;
   p.prefetch_b = p.m_tiles <= 2 ? prefetch_depth() : 0;      // weights read once from HBM: run ahead of the ring in L2
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
@@ -1381,6 +1407,16 @@ extern "C" int atlas_gemm_tail(const void* A, const void* B, void* C, float* tai
                    stream, nullptr, nullptr, 0, nullptr, n_main < N ? tail : nullptr, tail_ld, n_main);
 }
 
+// bf16 GEMM with a bias row (fp32 [N] or null) and / or an activation in its epilogue: act 0 none, 1 relu squared, 2 gated
+// unit (common.cuh) of alternating gate and up columns (C has N / 2 columns).
+extern "C" int atlas_gemm_bias_act(const void* A, const void* B, void* C, const float* bias, int act, float glu_limit, float glu_alpha, float glu_shift, int M,
+                                   int N, int K, long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace,
+                                   int* counters, int num_sms, unsigned long long* status, void* stream) {
+  if (act < 0 || act > 2 || (act == 2 && N % 2)) return -46;
+  return gemm_impl(0, A, B, C, nullptr, 0, 0, nullptr, 0, M, N, K, lda, ldb, ldc, block_n, splits, workspace, counters, num_sms, status,
+                   stream, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, bias, act, glu_limit, glu_alpha, glu_shift);
+}
+
 // All-gather -> GEMM: the rows of A (and their scales) are written into this rank's memory by the ranks that own them;
 // `a_ready` holds one flag per 8 rows and a row group is complete once its flag has reached *a_ready_epoch.  The TMA
 // producer polls the flags of a tile's rows before it loads the tile, so the GEMM starts on the rows that are already
@@ -1409,12 +1445,14 @@ extern "C" int atlas_gemm_fused(int kind, const void* A, const void* B, void* C,
 
 // Grouped (MoE) GEMM: C[r, :] = A[r, :] * B[e(r)]^T for expert-sorted rows.  `A` has `max_rows` rows (a multiple of
 // 128); m-tile i covers rows [128 i, 128 i + 128) and uses expert tile_expert[i]; *num_m_tiles (device memory) says how
-// many tiles are live.  `B` is the expert stack [E * N, K]; b_scale is [E, ceil(N/128), K/128].
+// many tiles are live.  `B` is the expert stack [E * N, K]; b_scale is [E, ceil(N/128), K/128].  act (bf16): see
+// atlas_gemm_bias_act.
 extern "C" int atlas_gemm_grouped(int kind, const void* A, const void* B, void* C, const float* a_scale, long long sa_k,
                                   const float* b_scale, int max_rows, int N, int K, int E, long long lda, long long ldb,
                                   long long ldc, int block_n, const int* tile_expert, const int* num_m_tiles,
-                                  int num_sms, unsigned long long* status, void* stream, int relu2) {
-  if (relu2 && kind != 0) return -11;
+                                  int num_sms, unsigned long long* status, void* stream, int act, float glu_limit,
+                                  float glu_alpha, float glu_shift) {
+  if (act < 0 || act > 2 || (act && kind != 0)) return -11;
   if (max_rows <= 0 || N <= 0 || K <= 0 || E <= 0) return 0;
   if (max_rows % kBlockM) return -9;
   const uint32_t esize = kind == 1 ? 1 : 2;
@@ -1440,7 +1478,7 @@ extern "C" int atlas_gemm_grouped(int kind, const void* A, const void* B, void* 
   p.n_tiles = N / block_n;
   p.b_scale_ld = p.k_blocks;
   p.vec_ok = ((ldc % 8) == 0 && (reinterpret_cast<uintptr_t>(C) & 15) == 0) ? 1 : 0;
-  p.relu2 = relu2;
+  p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift};
   p.tile_expert = tile_expert; p.num_m_tiles_ptr = num_m_tiles; p.expert_n = N;
   p.ar_state = nullptr; p.ar_world = 1; p.ar_rank = 0; p.ar_mode = 0; p.ar_parity_stride = 0; p.prefetch_b = 0;
   p.rs_tiles_per_rank = 1; p.a_ready = nullptr; p.a_ready_epoch = nullptr; p.ar_max_cycles = kMbarMaxCycles;

@@ -87,12 +87,16 @@ int atlas_gemm_w4a16_grouped(const void* A, const void* packed, const void* bsca
 int atlas_gemm_grouped(int kind, const void* A, const void* B, void* C, const float* a_scale, long long sa_k,
                        const float* b_scale, int max_rows, int N, int K, int E, long long lda, long long ldb,
                        long long ldc, int block_n, const int* tile_expert, const int* num_m_tiles, int num_sms,
-                       unsigned long long* status, void* stream, int relu2);
+                       unsigned long long* status, void* stream, int act, float glu_limit, float glu_alpha, float glu_shift);
+int atlas_gemm_bias_act(const void* A, const void* B, void* C, const float* bias, int act, float glu_limit, float glu_alpha, float glu_shift, int M, int N, int K,
+                        long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,
+                        unsigned long long* status, void* stream);
 int atlas_gemm_tail(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, int M, int N, int K, long long lda,
                     long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,
                     unsigned long long* status, void* stream);
 int atlas_moe_plain_gemm(const void* x, long long ldx, const void* w, const int* row_token, const int* tile_expert, const int* num_tiles,
-                         int max_rows, int gather, int relu2, int N, int K, void* y, long long ldy, int f32, void* stream);
+                         int max_rows, int gather, int act, float glu_limit, float glu_alpha, float glu_shift, int N, int K, void* y, long long ldy, int f32,
+                         void* stream);
 int atlas_moe_plain_combine(const void* y, long long ldy, const int* slot_of, const float* topk_w, int T, int k, int H, void* out,
                             long long ldo, int f32, void* stream);
 
@@ -141,16 +145,17 @@ int atlas_attn_prefill(const void* q, long long ldq, void* out, long long ldo, c
 int atlas_attn_decode_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                            const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int seq_base, int B,
                            float scale, int Hq, int Hkv, int D, int block_size, int window, int num_splits, float* part_o,
-                           float* part_ml, void* stream, int chunk, const float* sinks, float softcap);
+                           float* part_ml, void* stream, int chunk, const float* sinks, float softcap, const float* distance, int reach);
 int atlas_attn_prefill_kv16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                             const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
                             const int* tile_q0, int num_tiles, float scale, int Hq, int Hkv, int D, int block_size, int window,
-                            void* stream, int chunk, const float* sinks, float softcap);
+                            void* stream, int chunk, const float* sinks, float softcap, const float* distance, int reach);
 
 int atlas_attn_prefill_tc16(const void* q, long long ldq, void* out, long long ldo, const void* k_cache, const void* v_cache,
                             const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, const int* tile_seq,
                             const int* tile_q0, int num_tiles, int total_tokens, float scale, int Hq, int Hkv, int D, int block_size,
-                            int chunk, int window, const float* sinks, float softcap, unsigned long long* status, void* stream);
+                            int chunk, int window, const float* sinks, float softcap, const float* distance, int reach, unsigned long long* status,
+                            void* stream);
 
 // ---- 32-bit attention (attention_f32.cu)
 int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long ldk, const float* v, long long ldv, const int* positions,
@@ -160,7 +165,7 @@ int atlas_rope_kv_write_f32(float* q, long long ldq, const float* k, long long l
 int atlas_attn_f32(const float* q, long long ldq, float* out, long long ldo, const float* k_cache, const float* v_cache,
                    const int* block_tables, int bt_ld, const int* seq_lens, const int* query_start_loc, int B, int T, float scale, int Hq,
                    int Hkv, int D, int block_size, int window, int chunk, const float* sinks, float softcap,
-                   void* stream);
+                   const float* distance, int reach, void* stream);
 
 // ---- residual streams, token shift, clamped gated unit (streams.cu); f32 = activations are fp32 instead of bf16
 int atlas_hyper_norm(float* x, int rows, int S, int W, const void* y, long long ldy, const void* y2, long long ldy2, const float* w1,
@@ -168,8 +173,8 @@ int atlas_hyper_norm(float* x, int rows, int S, int W, const void* y, long long 
                      long long ldo, int init, int store, float scale, float eps, int f32, void* stream);
 int atlas_token_shift_mix(const void* x, long long ldx, const float* mu, const void* shift, const int* seq_of_token, const int* qsl,
                           const int* slots, const unsigned char* has, void* out, int rows, int W, int f32, void* stream);
-int atlas_clamped_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha, int f32,
-                      void* stream);
+int atlas_gated_unit(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha, float shift, int paired,
+                     int f32, void* stream);
 int atlas_tanh(void* x, long long n, int f32, void* stream);
 
 // ---- linear recurrences (recurrent.cu)
@@ -183,9 +188,33 @@ int atlas_wkv_scan(const void* r, long long ldr, const void* k, long long ldk, c
                    const int* snap_slots, int snaps, int B, int H, int D, int commit, int one_row, int f32, void* stream);
 int atlas_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
                           int groups, int gsize, float eps, int gate_first, int sigmoid, const float* den, int f32, void* stream);
-int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const float* w,
-                     const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store, float eps, int f32, void* stream);
+int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const void* extra,
+                     long long lde, const float* w, const float* out_w, const float* step, void* out, long long ldo, int rows, int W, int plus_one,
+                     int store, int first, float eps, float scale, int f32, void* stream);
 int atlas_head_gate(void* x, long long ldx, const float* g, long long ldg, int rows, int H, int D, int f32, void* stream);
+
+// ---- RG-LRU (rglru.cu): arguments of both forms, see the entry points
+typedef struct {
+  const void* x; long long ldx; const void* u; long long ldu;
+  const float* zr; const float* zi; long long z_row; long long z_block;
+  const void* y; long long ldy;
+  const void* conv_w; const void* conv_b; const void* conv_state; const void* tiles;
+  const float* gate_bias; const float* lam;
+  float* h; float* P; float* S; float* endP; float* endS;
+  void* out; long long ldo;
+  const int* seq_of; const int* qsl; const int* slots; const unsigned char* has;
+  const int* limit; const int* snap_rows; const int* snap_slots;
+  unsigned long long* status;
+  int snaps, rows, C, n, taps, commit, one_row;
+} AtlasRglru;
+int atlas_rglru_tc(const AtlasRglru* a, void* stream);
+int atlas_rglru_scan(const AtlasRglru* a, int f32, void* stream);
+
+// ---- norm of queries and keys over all heads (row_norm_kv.cu)
+int atlas_row_norm_kv_write(void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, const int* positions,
+                            const float* rope, const int* seq_positions, const float* qw, const float* kw, const float* sums, void* k_cache,
+                            void* v_cache, const int* slot_mapping, int T, int Hq, int Hkv, int D, int rotary, int block_size, int nq, int nk,
+                            float eps, float temp, int every, int f32, void* stream);
 
 // ---- mLSTM (mlstm.cu)
 int atlas_mlstm_gates(const float* raw, long long ld, const float* bias, float cap, float* m, float* la, float* lb, float* top, const int* qsl,
@@ -221,7 +250,7 @@ int atlas_latent_unpad(const void* in, const int* rows, int n, int H, int vd, in
 // ---- recurrences (recurrent.cu), continued
 int atlas_conv1d_bias_silu(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                            const int* seq_of_token, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
-                           int rows, int f32, void* stream);
+                           int rows, int silu, int f32, void* stream);
 int atlas_conv1d_state(const void* x, long long ldx, int C, int W, void* state, const int* qsl, const int* slots,
                        const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B, int f32,
                        void* stream);

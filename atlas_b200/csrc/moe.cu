@@ -301,8 +301,8 @@ constexpr int kPgRows = 32, kPgCols = 64, kPgK = 32;
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_plain_gemm_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const int* __restrict__ row_token,
-                      const int* __restrict__ tile_expert, const int* __restrict__ num_tiles, int gather, int relu2, int N, int K, T* y,
-                      long long ldy) {
+                      const int* __restrict__ tile_expert, const int* __restrict__ num_tiles, int gather, int act, GatedUnit unit,
+                      int N, int K, T* y, long long ldy) {
   __shared__ float xs[kPgRows][kPgK + 1], ws[kPgCols][kPgK + 1];
   const int tile = blockIdx.y >> 2, r0 = tile * 128 + (blockIdx.y & 3) * kPgRows, n0 = blockIdx.x * kPgCols;
   if (tile >= *num_tiles) return;
@@ -328,13 +328,17 @@ moe_plain_gemm_kernel(const T* __restrict__ x, long long ldx, const T* __restric
     }
     __syncthreads();
   }
-  if (n0 + c >= N) return;
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
     const int r = r0 + rg + 4 * i;
-    if (row_token[r] < 0) continue;
     float v = acc[i];
-    if (relu2) { v = fmaxf(v, 0.f); v *= v; }
+    const float up = __shfl_down_sync(0xffffffffu, v, 1);      // the next column of the same row
+    if (n0 + c >= N || row_token[r] < 0) continue;
+    if (act == 2) {                            // alternating gate and up columns
+      if ((c & 1) == 0) y[(long long)r * ldy + (n0 + c) / 2] = (T)gated_unit(v, up, unit);
+      continue;
+    }
+    if (act == 1) { v = fmaxf(v, 0.f); v *= v; }
     y[(long long)r * ldy + n0 + c] = (T)v;
   }
 }
@@ -469,18 +473,21 @@ extern "C" int atlas_moe_combine(const void* y, long long ldy, const int* slot_o
 }
 
 // Grouped product on the CUDA cores (see moe_plain_gemm_kernel): rows sorted by moe_align, w [E, N, K]
+// act: 0 none, 1 relu squared, 2 gated unit (common.cuh) of alternating gate and up columns (y has N / 2 columns)
 extern "C" int atlas_moe_plain_gemm(const void* x, long long ldx, const void* w, const int* row_token, const int* tile_expert,
-                                    const int* num_tiles, int max_rows, int gather, int relu2, int N, int K, void* y, long long ldy, int f32,
-                                    void* stream) {
+                                    const int* num_tiles, int max_rows, int gather, int act, float glu_limit, float glu_alpha, float glu_shift, int N,
+                                    int K, void* y, long long ldy, int f32, void* stream) {
   if (max_rows <= 0) return 0;
+  if (act < 0 || act > 2 || (act == 2 && N % 2)) return -2;
   if (max_rows % 128 || N < 1 || K < 1 || max_rows / 32 > 65535) return -1;
   dim3 grid((N + kPgCols - 1) / kPgCols, max_rows / 32);
+  const GatedUnit unit = {glu_limit, glu_alpha, glu_shift};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (f32) moe_plain_gemm_kernel<float><<<grid, 256, 0, st>>>(reinterpret_cast<const float*>(x), ldx, reinterpret_cast<const float*>(w), row_token,
-                                                               tile_expert, num_tiles, gather, relu2, N, K, reinterpret_cast<float*>(y), ldy);
+                                                               tile_expert, num_tiles, gather, act, unit, N, K, reinterpret_cast<float*>(y), ldy);
   else moe_plain_gemm_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx,
                                                                   reinterpret_cast<const __nv_bfloat16*>(w), row_token, tile_expert, num_tiles,
-                                                                  gather, relu2, N, K, reinterpret_cast<__nv_bfloat16*>(y), ldy);
+                                                                  gather, act, unit, N, K, reinterpret_cast<__nv_bfloat16*>(y), ldy);
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }
 

@@ -1,6 +1,6 @@
 // Mamba-2 and WKV recurrences (kernels in linear_scan.cuh) and the short convolution in front of Mamba-2:
 //
-//   conv1d_kernel        causal depth-wise convolution + bias + SiLU, window state of the last W - 1 inputs per channel
+//   conv1d_kernel        causal depth-wise convolution + bias (+ SiLU), window state of the last W - 1 inputs per channel
 //
 // Activations are bf16 or fp32 (template parameter T).
 // Reference ops replaced: kernels/gb10/common/mamba2_ssm_decode.cu, mamba2_ssd_chunk.cu, causal_conv1d.cu.
@@ -20,7 +20,7 @@ template <typename T, int kTaps, int V>
 __global__ void __launch_bounds__(256)
 conv1d_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const T* __restrict__ bias, int C, int W,
               const T* __restrict__ state, const int* __restrict__ seq_of_token, const int* __restrict__ query_start_loc,
-              const int* __restrict__ state_slots, const unsigned char* __restrict__ has_state, T* y, long long ldy, int rows) {
+              const int* __restrict__ state_slots, const unsigned char* __restrict__ has_state, T* y, long long ldy, int rows, int silu) {
   chain_trigger();
   chain_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -82,7 +82,7 @@ conv1d_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, c
       }
     }
 #pragma unroll
-    for (int v = 0; v < V; ++v) acc[v] = acc[v] / (1.f + expf(-acc[v]));
+    for (int v = 0; v < V; ++v) acc[v] = silu ? acc[v] / (1.f + expf(-acc[v])) : acc[v];
     store_vec<V>(y + (long long)t * ldy + c, acc);
   }
 }
@@ -122,28 +122,28 @@ conv1d_state_kernel(const T* __restrict__ x, long long ldx, int C, int W, T* sta
 template <typename T, int kTaps>
 static int launch_conv(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                        const int* seq, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
-                       int rows, cudaStream_t st) {
+                       int rows, int silu, cudaStream_t st) {
   const T *xp = reinterpret_cast<const T*>(x), *wp = reinterpret_cast<const T*>(w), *bp = reinterpret_cast<const T*>(bias);
   const T* sp = reinterpret_cast<const T*>(state);
   T* yp = reinterpret_cast<T*>(y);
   const unsigned gx = (rows + kConvRows - 1) / kConvRows;
   if (kTaps > 0 && rows > 256 && C % 4 == 0 && vec_ok<T, 4>(x, ldx) && vec_ok<T, 4>(y, ldy))
     launch_chain_if(false, conv1d_kernel<T, kTaps, (kTaps > 0 ? 4 : 1)>, dim3(gx, (C + 1023) / 1024), dim3(256), 0, st, xp, ldx, wp, bp, C, W,
-                    sp, seq, qsl, slots, has, yp, ldy, rows);
+                    sp, seq, qsl, slots, has, yp, ldy, rows, silu);
   else
     launch_chain_if(rows <= 256, conv1d_kernel<T, kTaps, 1>, dim3(gx, (C + 255) / 256), dim3(256), 0, st, xp, ldx, wp, bp, C, W, sp, seq, qsl,
-                    slots, has, yp, ldy, rows);
+                    slots, has, yp, ldy, rows, silu);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
 template <typename T>
 static int conv(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state, const int* seq,
-                const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy, int rows, cudaStream_t st) {
+                const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy, int rows, int silu, cudaStream_t st) {
   switch (W) {
-    case 2: return launch_conv<T, 2>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, st);
-    case 3: return launch_conv<T, 3>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, st);
-    case 4: return launch_conv<T, 4>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, st);
-    default: return launch_conv<T, 0>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, st);
+    case 2: return launch_conv<T, 2>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, silu, st);
+    case 3: return launch_conv<T, 3>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, silu, st);
+    case 4: return launch_conv<T, 4>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, silu, st);
+    default: return launch_conv<T, 0>(x, ldx, w, bias, C, W, state, seq, qsl, slots, has, y, ldy, rows, silu, st);
   }
 }
 
@@ -202,15 +202,15 @@ extern "C" int atlas_wkv_scan(const void* r, long long ldr, const void* k, long 
                          snap_slots, snaps, B, H, D, commit, one_row, st);
 }
 
-// depth-wise causal convolution + bias (may be null) + SiLU of [rows, C]; state [slots, C, W - 1]
+// depth-wise causal convolution + bias (may be null), then SiLU where `silu` says so, of [rows, C]; state [slots, C, W - 1]
 extern "C" int atlas_conv1d_bias_silu(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                                       const int* seq_of_token, const int* qsl, const int* slots, const unsigned char* has, void* y,
-                                      long long ldy, int rows, int f32, void* stream) {
+                                      long long ldy, int rows, int silu, int f32, void* stream) {
   if (rows <= 0) return 0;
   if (W < 1 || W > kMaxTaps) return -1;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return f32 ? conv<float>(x, ldx, w, bias, C, W, state, seq_of_token, qsl, slots, has, y, ldy, rows, st)
-             : conv<bf16>(x, ldx, w, bias, C, W, state, seq_of_token, qsl, slots, has, y, ldy, rows, st);
+  return f32 ? conv<float>(x, ldx, w, bias, C, W, state, seq_of_token, qsl, slots, has, y, ldy, rows, silu, st)
+             : conv<bf16>(x, ldx, w, bias, C, W, state, seq_of_token, qsl, slots, has, y, ldy, rows, silu, st);
 }
 
 extern "C" int atlas_conv1d_state(const void* x, long long ldx, int C, int W, void* state, const int* qsl, const int* slots,

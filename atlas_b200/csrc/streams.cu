@@ -1,4 +1,4 @@
-// Hyper-connected residual streams (fp32), the token-shift mixes of WKV layers and the clamped gated unit.
+// Hyper-connected residual streams (fp32), the token-shift mixes of WKV layers and gated units.
 //
 //   hyper_norm_kernel       one CTA per token: rewrites the S streams with the last sublayer's connection and output
 //                             x'[t] = sum_s mix[s, t] * x[s] + write[t] * y
@@ -10,10 +10,12 @@
 //                           sequence's state slot for the first row of a chunk, zeros at the start of a sequence)
 //   group_norm_gate_kernel  rms norm over channel groups joined with a gate: norm(y * silu(z)) * w (Mamba-2),
 //                           norm(y) * w * silu(z) (WKV) or norm(y / den) * w * sigmoid(z) (mLSTM)
-//   add_normed_kernel       one CTA per token: x += rmsnorm(y) * w on an fp32 residual, y being a sublayer's output or the weighted
-//                           sum of expert rows; hands the new x on in the activations' dtype, normed again where asked
+//   add_normed_kernel       one CTA per token: x += rmsnorm(y) * w or x += y on an fp32 residual, y being a sublayer's output or the
+//                           weighted sum of expert rows (and a shared expert's row); adds a step vector where one is given and hands
+//                           the new x on in the activations' dtype, normed again where asked
 //   head_gate_kernel        x[t, h, :] *= sigmoid(g[t, h])
-//   clamped_glu_kernel      g = min(gate, limit), u = clamp(up, +-limit):  g * sigmoid(alpha g) * (u + 1)
+//   gated_unit_kernel       g = min(gate, limit), u = clamp(up, +-limit):  g * sigmoid(alpha g) * (u + shift), of [gate | up] or of
+//                           alternating columns
 //
 // Every kernel exists for bf16 and fp32 activations (template parameter T).
 #include "common.cuh"
@@ -325,10 +327,12 @@ struct AddNormedParams {
   float* x; long long ldx;                     // [T, W]
   const T* y; long long ldy;
   const int* slot_of; const float* pick_w; int picks;      // picks > 0: y = sum_j pick_w[t, j] * rows slot_of[t, j] (>= 0) of `y`
-  const float* w; const float* out_w;          // w null: x = y (start of the model); out_w null: out = x
+  const T* extra; long long lde;               // joins y (null = off)
+  const float* w; const float* out_w;          // w null: x += y; out_w null: out = x
+  const float* step;                           // [W] added to the new x (null = off)
   T* out; long long ldo;
-  int W, plus_one, store;
-  float eps;
+  int W, plus_one, store, first;               // first: x = y * scale (start of the model)
+  float eps, scale;
 };
 
 // NI pieces of V elements per thread, the row stays in registers
@@ -348,8 +352,16 @@ add_normed_kernel(const AddNormedParams<T> p) {
 #pragma unroll
     for (int i = 0; i < V; ++i) y[k][i] = 0.f;
     if (e >= p.W) continue;
+    if (p.extra) load_vec<V>(p.extra + t * p.lde + e, y[k]);
     if (p.picks == 0) {
-      load_vec<V>(p.y + t * p.ldy + e, y[k]);
+      if (p.extra) {
+        float f[V];
+        load_vec<V>(p.y + t * p.ldy + e, f);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] += f[i];
+      } else {
+        load_vec<V>(p.y + t * p.ldy + e, y[k]);
+      }
     } else {
       for (int j = 0; j < p.picks; ++j) {
         const int row = p.slot_of[t * p.picks + j];
@@ -381,6 +393,39 @@ add_normed_kernel(const AddNormedParams<T> p) {
         ss += y[k][i] * y[k][i];
       }
     }
+  } else if (!p.first || p.scale != 1.f) {
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NI; ++k) {
+      const int e = threadIdx.x * V + k * step;
+      if (e >= p.W) continue;
+      if (p.first) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] *= p.scale;
+      } else {
+        float x[V];
+        load_vec<V>(p.x + t * p.ldx + e, x);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] += x[i];
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += y[k][i] * y[k][i];
+    }
+  }
+  if (p.step) {
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NI; ++k) {
+      const int e = threadIdx.x * V + k * step;
+      if (e >= p.W) continue;
+      float f[V];
+      load_vec<V>(p.step + e, f);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        y[k][i] += f[i];
+        ss += y[k][i] * y[k][i];
+      }
+    }
   }
   const float orstd = p.out_w ? 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps) : 1.f;
 #pragma unroll
@@ -399,12 +444,13 @@ add_normed_kernel(const AddNormedParams<T> p) {
 }
 
 template <typename T>
-static int add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const float* w,
-                      const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store, float eps, cudaStream_t st) {
-  AddNormedParams<T> p = {x, ldx, reinterpret_cast<const T*>(y), ldy, slot_of, pick_w, picks, w, out_w, reinterpret_cast<T*>(out), ldo, W, plus_one,
-                          store, eps};
+static int add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const void* extra,
+                      long long lde, const float* w, const float* out_w, const float* step, void* out, long long ldo, int rows, int W, int plus_one,
+                      int store, int first, float eps, float scale, cudaStream_t st) {
+  AddNormedParams<T> p = {x, ldx, reinterpret_cast<const T*>(y), ldy, slot_of, pick_w, picks, reinterpret_cast<const T*>(extra), lde, w, out_w, step,
+                          reinterpret_cast<T*>(out), ldo, W, plus_one, store, first, eps, scale};
   const bool vec = W % 8 == 0 && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(out, ldo) && vec_ok<float, 4>(x, ldx) && vec_ok<float, 4>(w, 0) &&
-                   vec_ok<float, 4>(out_w, 0);
+                   vec_ok<float, 4>(out_w, 0) && vec_ok<float, 4>(step, 0) && vec_ok<T, 8>(extra, lde);
   const int v = vec ? 8 : 1, pieces = (W + v - 1) / v;
   void (*k)(const AddNormedParams<T>) = nullptr;
   int ni = 1;
@@ -444,31 +490,35 @@ static int launch_head_gate(void* x, long long ldx, const float* g, long long ld
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
-// ----------------------------------------------------------------------------- clamped gated unit, tanh
-template <typename T, int V>
+// ----------------------------------------------------------------------------- gated units, tanh
+template <typename T, int V, bool kPaired>
 __global__ void __launch_bounds__(256)
-clamped_glu_kernel(const T* __restrict__ gu, long long ld, int I, T* y, long long ldy, float limit, float alpha) {
+gated_unit_kernel(const T* __restrict__ gu, long long ld, int I, T* y, long long ldy, GatedUnit unit) {
   chain_trigger();
   chain_wait();
   const long long t = blockIdx.x;
   const int e = (blockIdx.y * blockDim.x + threadIdx.x) * V;
   if (e >= I) return;
   float g[V], u[V], o[V];
-  load_vec<V>(gu + t * ld + e, g);
-  load_vec<V>(gu + t * ld + I + e, u);
+  if constexpr (kPaired) {
+    float f[2 * V];
+    load_vec<2 * V>(gu + t * ld + 2 * e, f);
 #pragma unroll
-  for (int i = 0; i < V; ++i) {
-    const float a = fminf(g[i], limit), b = fminf(fmaxf(u[i], -limit), limit);
-    o[i] = a / (1.f + expf(-alpha * a)) * (b + 1.f);
+    for (int i = 0; i < V; ++i) { g[i] = f[2 * i]; u[i] = f[2 * i + 1]; }
+  } else {
+    load_vec<V>(gu + t * ld + e, g);
+    load_vec<V>(gu + t * ld + I + e, u);
   }
+#pragma unroll
+  for (int i = 0; i < V; ++i) o[i] = gated_unit(g[i], u[i], unit);
   store_vec<V>(y + t * ldy + e, o);
 }
 
-template <typename T, int V>
-static int launch_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha, cudaStream_t st) {
+template <typename T, int V, bool kPaired = false>
+static int launch_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, GatedUnit unit, cudaStream_t st) {
   dim3 grid(rows, (I + 256 * V - 1) / (256 * V));
-  launch_chain_if(rows <= 256, clamped_glu_kernel<T, V>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(gu), ld, I,
-                  reinterpret_cast<T*>(y), ldy, limit, alpha);
+  launch_chain_if(rows <= 256, gated_unit_kernel<T, V, kPaired>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(gu), ld, I,
+                  reinterpret_cast<T*>(y), ldy, unit);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
@@ -517,17 +567,29 @@ extern "C" int atlas_token_shift_mix(const void* x, long long ldx, const float* 
              : launch_shift<B, 1>(x, ldx, mu, shift, seq_of_token, qsl, slots, has, out, rows, W, st);
 }
 
-extern "C" int atlas_clamped_glu(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha,
-                                 int f32, void* stream) {
+// gu: [gate | up], or alternating gate and up columns with `paired`
+extern "C" int atlas_gated_unit(const void* gu, long long ld, int rows, int I, void* y, long long ldy, float limit, float alpha,
+                                 float shift, int paired, int f32, void* stream) {
   if (rows <= 0 || I <= 0) return 0;
+  const GatedUnit unit = {limit, alpha, shift};
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (paired) {
+    if (f32) {
+      const bool vec = I % 4 == 0 && vec_ok<float, 4>(gu, ld) && vec_ok<float, 4>(y, ldy);
+      return vec ? launch_glu<float, 4, true>(gu, ld, rows, I, y, ldy, unit, st)
+                 : launch_glu<float, 1, true>(gu, ld, rows, I, y, ldy, unit, st);
+    }
+    using B = __nv_bfloat16;
+    const bool vec = I % 8 == 0 && vec_ok<B, 8>(gu, ld) && vec_ok<B, 8>(y, ldy);
+    return vec ? launch_glu<B, 8, true>(gu, ld, rows, I, y, ldy, unit, st) : launch_glu<B, 1, true>(gu, ld, rows, I, y, ldy, unit, st);
+  }
   if (f32) {
     const bool vec = I % 4 == 0 && vec_ok<float, 4>(gu, ld) && vec_ok<float, 4>(y, ldy);
-    return vec ? launch_glu<float, 4>(gu, ld, rows, I, y, ldy, limit, alpha, st) : launch_glu<float, 1>(gu, ld, rows, I, y, ldy, limit, alpha, st);
+    return vec ? launch_glu<float, 4>(gu, ld, rows, I, y, ldy, unit, st) : launch_glu<float, 1>(gu, ld, rows, I, y, ldy, unit, st);
   }
   using B = __nv_bfloat16;
   const bool vec = I % 8 == 0 && vec_ok<B, 8>(gu, ld) && vec_ok<B, 8>(y, ldy);
-  return vec ? launch_glu<B, 8>(gu, ld, rows, I, y, ldy, limit, alpha, st) : launch_glu<B, 1>(gu, ld, rows, I, y, ldy, limit, alpha, st);
+  return vec ? launch_glu<B, 8>(gu, ld, rows, I, y, ldy, unit, st) : launch_glu<B, 1>(gu, ld, rows, I, y, ldy, unit, st);
 }
 
 extern "C" int atlas_tanh(void* x, long long n, int f32, void* stream) {
@@ -551,16 +613,20 @@ extern "C" int atlas_group_norm_gate(const void* y, long long ldy, const void* z
              : gnorm<__nv_bfloat16>(y, ldy, z, ldz, w, out, ldo, rows, groups, gsize, eps, kind, den, st);
 }
 
-// fp32 residual x [rows, W]: x += rmsnorm(y) * w (w null: x = y), out = x or rmsnorm(x) * out_w.  picks > 0: y [*, W] holds expert rows,
-// slot_of / pick_w [rows, picks].  With plus_one the weights are stored around zero; store = 0 leaves x as it is.
+// fp32 residual x [rows, W]: x += rmsnorm(y) * w (w null: x += y; first: x = y * scale), then x += step (null: nothing), out = x or
+// rmsnorm(x) * out_w.  picks > 0: y [*, W] holds expert rows, slot_of / pick_w [rows, picks].  extra [rows, W] joins y.  With plus_one
+// the weights are stored around zero; store = 0 leaves x as it is.
 extern "C" int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks,
-                                const float* w, const float* out_w, void* out, long long ldo, int rows, int W, int plus_one, int store,
-                                float eps, int f32, void* stream) {
+                                const void* extra, long long lde, const float* w, const float* out_w, const float* step, void* out,
+                                long long ldo, int rows, int W, int plus_one, int store, int first, float eps, float scale, int f32,
+                                void* stream) {
   if (rows <= 0) return 0;
-  if (W < 1 || W > 32768 || picks < 0 || (picks > 0 && (!slot_of || !pick_w))) return -1;
+  if (W < 1 || W > 32768 || picks < 0 || (picks > 0 && (!slot_of || !pick_w)) || (first && w)) return -1;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  return f32 ? add_normed<float>(x, ldx, y, ldy, slot_of, pick_w, picks, w, out_w, out, ldo, rows, W, plus_one, store, eps, st)
-             : add_normed<__nv_bfloat16>(x, ldx, y, ldy, slot_of, pick_w, picks, w, out_w, out, ldo, rows, W, plus_one, store, eps, st);
+  return f32 ? add_normed<float>(x, ldx, y, ldy, slot_of, pick_w, picks, extra, lde, w, out_w, step, out, ldo, rows, W, plus_one, store, first, eps,
+                                 scale, st)
+             : add_normed<__nv_bfloat16>(x, ldx, y, ldy, slot_of, pick_w, picks, extra, lde, w, out_w, step, out, ldo, rows, W, plus_one, store,
+                                         first, eps, scale, st);
 }
 
 // x [rows, H, D] (row stride ldx) times sigmoid(g [rows, H]), in place

@@ -82,7 +82,7 @@ class LLMEngine:
             from .layers import Attention
             self.selector = BlockSelector(num_blocks, self.cfg.block_size, self.cfg.sparse_attention_blocks)
             for l in model.layers:
-                if l.kind == "attention" and type(l.mixer) is Attention and l.mixer.plain:
+                if l.kind == "attention" and type(l.mixer) is Attention and l.mixer.plain and len(model.weight_layers()) == len(model.layers):
                     l.mixer.selector = self.selector
         self.scheduler = Scheduler(self.cfg, self.pool, self.radix, self.state_pool, self.hybrid, host_tier=self.host_tier)
         self.sampler = Sampler(self.mcfg.vocab_size, self.mcfg.eos_ids())

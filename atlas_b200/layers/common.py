@@ -118,6 +118,12 @@ def shard_cols(w: torch.Tensor, rank: int, size: int) -> torch.Tensor:
     return w[:, rank * s:(rank + 1) * s]
 
 
+def paired_rows(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
+    """``[.., I, K]`` gate and up rows -> ``[.., 2I, K]`` in turn (gate 0, up 0, gate 1, ..): a gated unit then needs neighbouring
+    columns of the product only."""
+    return torch.stack([gate, up], -2).flatten(-3, -2)
+
+
 def randn_weight(gen: torch.Generator, n: int, k: int, std: float, dtype, device) -> torch.Tensor:
     """N(0, std) weight drawn on the generator's device, moved to ``device``."""
     w = torch.randn(n, k, generator=gen, dtype=torch.float32, device=gen.device) * std

@@ -14,15 +14,20 @@ from .. import ops
 from ..config import ModelConfig
 from ..ops import Act, LinearWeight
 from ..lora import add_delta
-from .common import ParallelCtx, make_weight, randn_weight, shard_cols, shard_rows
+from .common import ParallelCtx, make_weight, paired_rows, randn_weight, shard_cols, shard_rows
 
 
 class DenseMLP:
     def __init__(self, cfg: ModelConfig, pctx: ParallelCtx, quant_kind: str, intermediate: Optional[int] = None,
-                 shard: bool = True, activation: Optional[str] = None):
+                 shard: bool = True, activation: Optional[str] = None, glu_limit: Optional[float] = None, paired: bool = False):
+        """``paired``: gate and up rows alternate, so that the product's epilogue applies the gated unit (silu or clamped)."""
         self.cfg, self.pctx, self.quant_kind = cfg, pctx, quant_kind
+        self.paired = paired
         # "silu_glu": gate|up GEMM -> silu(gate) * up; "relu2": a single up GEMM -> relu(up)^2 (Nemotron-H)
         self.activation = activation or getattr(cfg, "mlp_activation", "silu_glu")
+        limit = cfg.glu_limit if glu_limit is None else glu_limit
+        self.unit = (limit, cfg.glu_alpha, 1.0) if self.activation == "clamped_glu" else ops.SILU_UNIT
+        assert not paired or self.activation in ("clamped_glu", "silu_glu")
         self.inter = intermediate or cfg.intermediate_size
         self.shard = shard and pctx.tp_size > 1 and self.inter % (pctx.tp_size * 128) == 0
         self.gate_up: Optional[LinearWeight] = None
@@ -34,6 +39,8 @@ class DenseMLP:
         tp, r = (self.pctx.tp_size, self.pctx.tp_rank) if self.shard else (1, 0)
         if self.activation == "relu2":
             gu = shard_rows(up, r, tp)
+        elif self.paired:
+            gu = paired_rows(shard_rows(gate, r, tp), shard_rows(up, r, tp)).contiguous()
         else:
             gu = torch.cat([shard_rows(gate, r, tp), shard_rows(up, r, tp)], 0)
         self.gate_up = make_weight(gu, self.quant_kind)
@@ -47,6 +54,8 @@ class DenseMLP:
 
     def hidden_act(self, act: Act) -> Act:
         """gate|up GEMM + SiLU * mul: the input of the down projection (no adapters)."""
+        if self.paired:
+            return ops.linear_gated_unit(act, self.gate_up, self.unit)
         if self.activation in ("gelu_tanh_glu", "clamped_glu"):
             return self._glu(ops.linear(act, self.gate_up), self.down.kind == "fp8_block")
         if self.down.kind == "fp8_block" and ops.swiglu_fusable(act, self.gate_up):
@@ -54,8 +63,8 @@ class DenseMLP:
         return ops.silu_mul_act(ops.linear(act, self.gate_up), want_fp8=self.down.kind == "fp8_block")
 
     def _glu(self, gate_up: torch.Tensor, want_fp8: bool) -> Act:
-        if self.activation == "clamped_glu":
-            return ops.clamped_glu_act(gate_up, self.cfg.glu_limit, self.cfg.glu_alpha)
+        if self.paired or self.activation == "clamped_glu":
+            return ops.gated_unit_act(gate_up, self.unit, self.paired)
         return ops.glu_act(gate_up, want_fp8, "gelu_tanh")
 
     def _relu2(self, act: Act, reduce: bool) -> torch.Tensor:
@@ -67,7 +76,7 @@ class DenseMLP:
         if self.activation == "relu2":
             return self._relu2(act, reduce)
         use_lora = self.lora is not None and batch is not None and batch.adapter_rows is not None and self.lora_prefix
-        if self.activation in ("gelu_tanh_glu", "clamped_glu") and not use_lora:
+        if (self.paired or self.activation in ("gelu_tanh_glu", "clamped_glu")) and not use_lora:
             a = self.hidden_act(act)
             return self.pctx.row_parallel_linear(a, self.down) if (self.shard and reduce) else ops.linear(a, self.down)
         if not use_lora and self.down.kind == "fp8_block" and ops.swiglu_fusable(act, self.gate_up):
@@ -76,9 +85,15 @@ class DenseMLP:
         gu = ops.linear(act, self.gate_up)
         if use_lora:
             xin, half = act.plain(), gu.shape[1] // 2
-            add_delta(gu, self.lora, self.lora_prefix + "gate_proj", xin, batch, 0, half)
-            add_delta(gu, self.lora, self.lora_prefix + "up_proj", xin, batch, half, half)
-        if self.activation in ("gelu_tanh_glu", "clamped_glu"):
+            if self.paired:
+                parts = torch.stack([gu[:, 0::2], gu[:, 1::2]]).contiguous()
+                add_delta(parts[0], self.lora, self.lora_prefix + "gate_proj", xin, batch, 0, half)
+                add_delta(parts[1], self.lora, self.lora_prefix + "up_proj", xin, batch, 0, half)
+                gu = torch.stack([parts[0], parts[1]], -1).flatten(1)
+            else:
+                add_delta(gu, self.lora, self.lora_prefix + "gate_proj", xin, batch, 0, half)
+                add_delta(gu, self.lora, self.lora_prefix + "up_proj", xin, batch, half, half)
+        if self.paired or self.activation in ("gelu_tanh_glu", "clamped_glu"):
             a = self._glu(gu, False)
         else:
             a = ops.silu_mul_act(gu, want_fp8=self.down.kind == "fp8_block" and not use_lora)

@@ -22,14 +22,15 @@ import torch.nn.functional as F
 from .. import ops, quant as Q
 from ..config import ModelConfig
 from ..ops import Act, LinearWeight, reference as ref
-from .common import ParallelCtx, make_weight, randn_weight
+from .common import ParallelCtx, make_weight, paired_rows, randn_weight
 from ..lora import add_delta
 from .mlp import DenseMLP
 
 
 @dataclass
 class ExpertWeights:
-    """Stacked local experts. ``w13 [E,2I,H]`` (gate rows then up rows; ``[E,I,H]`` for experts without a gate), ``w2 [E,H,I]``.
+    """Stacked local experts. ``w13 [E,2I,H]`` (gate rows then up rows, alternating ones for clamped units; ``[E,I,H]`` for
+    experts without a gate), ``w2 [E,H,I]``.
 
     kind ``dense`` keeps the model dtype; ``fp8_block`` adds ``*_scale [E, ceil(N/128), ceil(K/128)]``;
     ``nvfp4`` stores packed nibbles ``[E,N,K/2]``, e4m3 ``*_scale [E,N,K/16]`` and fp32 ``*_gscale [E]`` (or ``[E,N]``, one per output row).
@@ -97,7 +98,9 @@ class MoE:
         self.cfg, self.pctx = cfg, pctx
         self.expert_kind, self.dense_kind = expert_kind, dense_kind
         self.top_k = cfg.num_experts_per_tok
-        self.activation = "relu2" if cfg.mlp_activation == "relu2" else "silu_glu"      # silu(gate) * up, or relu(up)^2
+        # silu(gate) * up, relu(up)^2, or the clamped unit of alternating gate and up rows
+        self.activation = cfg.mlp_activation if cfg.mlp_activation in ("relu2", "clamped_glu") else "silu_glu"
+        self.unit = (cfg.glu_limit, cfg.glu_alpha, 1.0) if self.activation == "clamped_glu" else None
         self.router_f32 = cfg.router_f32
         self.e_lo, self.e_hi = cfg.local_expert_range(pctx.ep_rank, pctx.ep_size)
         self.ep_mode = ep_mode
@@ -110,7 +113,9 @@ class MoE:
         self.lora = None                    # lora.LoraSet shared by the model's layers
         self.lora_prefix = ""               # e.g. "layers.3.mlp."
         if cfg.shared_expert_intermediate_size:
-            self.shared = DenseMLP(cfg, pctx, dense_kind, cfg.shared_expert_intermediate_size, shard=False)
+            clamped = self.activation == "clamped_glu"
+            self.shared = DenseMLP(cfg, pctx, dense_kind, cfg.shared_expert_intermediate_size, shard=False, paired=clamped,
+                                   glu_limit=cfg.shared_glu_limit if clamped else None)
 
     # ------------------------------------------------------------------ weights
     def load(self, router: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor) -> None:
@@ -118,10 +123,12 @@ class MoE:
         self.router = LinearWeight("dense", router.contiguous())
         if w13.shape[0] == self.cfg.num_experts and self.pctx.ep_size > 1:
             w13, w2 = w13[self.e_lo:self.e_hi], w2[self.e_lo:self.e_hi]
-        if self.activation == "relu2" and w2.shape[2] % 64:
+        pad = -w2.shape[2] % 64
+        if self.activation == "clamped_glu":
+            w13 = paired_rows(*w13.chunk(2, 1))
+        if self.activation != "silu_glu" and pad:
             # whole GEMM tiles: hidden channels of zero weights stay zero through the activation
-            pad = 64 - w2.shape[2] % 64
-            w13, w2 = F.pad(w13, (0, 0, 0, pad)), F.pad(w2, (0, pad))
+            w13, w2 = F.pad(w13, (0, 0, 0, pad * w13.shape[1] // w2.shape[2])), F.pad(w2, (0, pad))
         self.experts = ExpertWeights.from_dense(w13, w2, self.expert_kind)
 
     def init_random(self, gen, std, dtype, device) -> None:
@@ -143,7 +150,8 @@ class MoE:
         self.load(router, torch.stack(w13_l), torch.stack(w2_l))
         if self.shared is not None:
             self.shared.init_random(gen, std, dtype, device)
-            self.shared_gate = randn_weight(gen, 1, h, std, dtype, device)
+            if self.activation != "clamped_glu":
+                self.shared_gate = randn_weight(gen, 1, h, std, dtype, device)
 
     # ------------------------------------------------------------------ forward
     def forward(self, act: Act, token_ids: Optional[torch.Tensor] = None, batch=None, rows_ok: bool = False):
@@ -158,10 +166,11 @@ class MoE:
                                          cfg.router_n_group, cfg.router_topk_group, cfg.routed_scaling_factor,
                                          self.hash_table, token_ids if self.hash_table is not None else None)
         if ops.on_gpu(x):
-            rows_ok = rows_ok and not adapters and self.shared is None and self.pctx.ep_size == 1
+            rows_ok = rows_ok and not adapters and self.shared_gate is None and self.pctx.ep_size == 1
             y = ops.cuda_ops().moe_forward(x, topk_w, topk_ids, self.experts, self.e_lo, self.pctx, self.ep_mode,
-                                           activation=self.activation, rows_ok=rows_ok)
+                                           activation=self.activation, rows_ok=rows_ok, unit=self.unit)
             if rows_ok:
+                y.extra = None if self.shared is None else self.shared.forward(act, reduce=False, batch=batch)
                 return y
         else:
             y = self._forward_ref(x, topk_w, topk_ids)
@@ -221,9 +230,13 @@ class MoE:
                 if self.activation == "relu2":
                     up = low_rank(xe, pair(ad, e, "up_proj"))
                     h = h + (F.pad(up, (0, inter - up.shape[1])) if torch.is_tensor(up) else up)
+                elif self.activation == "clamped_glu":
+                    wide = lambda d: F.pad(d, (0, inter - d.shape[1])) if torch.is_tensor(d) else d
+                    h = torch.stack([h[:, 0::2] + wide(low_rank(xe, pair(ad, e, "gate_proj"))),
+                                     h[:, 1::2] + wide(low_rank(xe, pair(ad, e, "up_proj")))], -1).flatten(1)
                 else:
                     h = torch.cat([h[:, :inter] + low_rank(xe, pair(ad, e, "gate_proj")), h[:, inter:] + low_rank(xe, pair(ad, e, "up_proj"))], 1)
-                a = ref.expert_act(h, self.activation).to(x.dtype).float()
+                a = ref.expert_act(h, self.activation, self.unit).to(x.dtype).float()
                 o = a @ w2.float().t() + low_rank(a[:, :self.cfg.moe_intermediate_size], pair(ad, e, "down_proj"))
                 part.index_add_(0, sel, o * (wts[sel] * hit[sel]).sum(-1, keepdim=True))
         p = self.pctx
@@ -241,9 +254,9 @@ class MoE:
         comm = p.ep_comm if p.ep_comm is not None else p.comm
         mode = self.ep_mode if self.ep_mode != "auto" else "allreduce"
         if p.ep_size == 1 or comm is None:
-            return ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation)
+            return ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation, self.unit)
         if mode == "allreduce":
-            return comm.all_reduce(ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation))
+            return comm.all_reduce(ref.moe_experts(x, w13, w2, topk_w, topk_ids, self.e_lo, self.activation, self.unit))
         return self._forward_alltoall_ref(x, topk_w, topk_ids, w13, w2, comm)
 
     def _forward_alltoall_ref(self, x, topk_w, topk_ids, w13, w2, comm) -> torch.Tensor:
@@ -270,7 +283,7 @@ class MoE:
                 continue
             ids = meta[:, 1:2].to(torch.int32)
             ones = torch.ones(rows.shape[0], 1, dtype=torch.float32, device=rows.device)
-            outs.append(ref.moe_experts(rows, w13, w2, ones, ids, self.e_lo, self.activation))
+            outs.append(ref.moe_experts(rows, w13, w2, ones, ids, self.e_lo, self.activation, self.unit))
         back = comm.all_to_all(outs)
         y = torch.zeros(T, H, dtype=torch.float32, device=x.device)
         for r in range(p.ep_size):

@@ -317,9 +317,47 @@ def _load_tomizen(model: DecoderLM, ck: Checkpoint) -> None:
     ck.close()
 
 
+def _load_kenovik(model: DecoderLM, ck: Checkpoint) -> None:
+    """Kenovik naming: ``embed``, ``loop.step``, ``l<i>.{norm1, norm2, mix.*, mlp.*}``, ``final.norm``; the embedding table is the
+    output projection."""
+    wt = lambda name: ck.get(name).to(device=model.device, dtype=model.dtype)
+    f32 = lambda name: ck.get(name).to(device=model.device, dtype=torch.float32).contiguous()
+    model.embed = wt("embed").contiguous()
+    if model.cfg.loop_steps:
+        model.loop_step = f32("loop.step")
+    for layer in model.weight_layers():
+        pre, mx = f"l{layer.number}.", layer.mixer
+        m = pre + "mix."
+        layer.input_norm = f32(pre + "norm1")
+        if layer.kind == "rglru":
+            mx.load(wt(m + "y"), f32(m + "y.b"), wt(m + "x"), f32(m + "x.b"), wt(m + "conv"), f32(m + "conv.b"), wt(m + "ra"), f32(m + "ra.b"),
+                    wt(m + "ri"), f32(m + "ri.b"), f32(m + "lam"), wt(m + "o"))
+        elif layer.cfg.qk_norm_rows:
+            mx.load(*(wt(m + n) for n in "qkvo"), f32(m + "q.norm"), f32(m + "k.norm"), rel=f32(m + "rel"))
+        else:
+            mx.load(*(wt(m + n) for n in "qkvo"), qkv_bias=tuple(f32(f"{m}{n}.b") for n in "qkv"), rope_interleaved=True)
+        if layer.ffn is None:
+            continue
+        layer.post_norm = f32(pre + "norm2")
+        part = lambda name: tuple(wt(f"{pre}mlp.{name}{n}") for n in ("gate", "up", "down"))
+        if not layer.is_moe:
+            layer.ffn.load(*part(""))
+            continue
+        stacks = [torch.stack(t) for t in zip(*(part(f"e{e}.") for e in range(layer.ffn.e_lo, layer.ffn.e_hi)))]
+        layer.ffn.router_bias = f32(pre + "mlp.correction")
+        layer.ffn.load(wt(pre + "mlp.router"), torch.cat(stacks[:2], 1), stacks[2])
+        if layer.ffn.shared is not None:
+            layer.ffn.shared.load(*part("shared."))
+    model.final_norm = f32("final.norm")
+    model.set_lm_head(model.embed)
+    ck.close()
+
+
 def load_weights(model: DecoderLM, ck: Checkpoint) -> None:
     cfg = model.cfg
     dense_kind, expert_kind = quant_kinds(cfg)
+    if cfg.model_type == "kenovik":
+        return _load_kenovik(model, ck)
     if cfg.model_type == "tomizen":
         return _load_tomizen(model, ck)
     if cfg.model_type == "papidra":

@@ -74,9 +74,9 @@ def localize(adapter: LoraAdapter, model) -> LoraAdapter:
     out = LoraAdapter(adapter.name, adapter.rank, adapter.alpha)
     for mod, (A, B) in adapter.weights.items():
         parts = mod.split(".")
-        known = len(parts) >= 4 and parts[0] == "layers" and parts[1].isdigit() and int(parts[1]) < len(model.layers)
+        known = len(parts) >= 4 and parts[0] == "layers" and parts[1].isdigit() and int(parts[1]) < len(model.weight_layers())
         if known:
-            layer, leaf = model.layers[int(parts[1])], parts[-1]
+            layer, leaf = model.weight_layers()[int(parts[1])], parts[-1]
             if parts[2] == "self_attn" and isinstance(layer.mixer, Attention):
                 at = layer.mixer
                 if leaf == "q_proj":

@@ -9,6 +9,7 @@ Reference parity: ``crates/spark-model/src/model/`` (``TransformerModel``), the 
 """
 from __future__ import annotations
 
+import copy
 import os
 from dataclasses import dataclass, field
 from typing import Dict, List, Optional, Tuple
@@ -346,6 +347,59 @@ class OutputNormLayer:
         return x, stream
 
 
+class InputNormLayer:
+    """A pre-norm layer of a model given by a list of layers: ``x += mixer(norm(x))``, then ``x += ffn(norm(x))`` where the layer has
+    a feed-forward, on an fp32 residual stream.  One object per run of the layer: later passes of a looped layer share the
+    weights of the first one and own a cache or state.  Same ``forward`` protocol as :class:`DecoderLayer`, with the pending
+    :class:`NormDelta` in place of the previous layer's output."""
+
+    def __init__(self, cfg: ModelConfig, idx: int, number: int, pctx: ParallelCtx, ep_mode: str = "auto"):
+        """``idx``: place in the order of execution (cache and state); ``number``: place in the checkpoint."""
+        spec = cfg.layer_specs[idx]
+        self.cfg, self.idx, self.number = cfg.for_layer(idx), idx, number
+        dense_kind, expert_kind = quant_kinds(cfg)
+        self.kind, self.is_moe, self.shared = spec.kind, cfg.is_moe_layer(idx), spec.weights_of >= 0
+        self.step_row = spec.step
+        self.step: Optional[torch.Tensor] = None               # fp32: added to the residual ahead of this run
+        self.mixer = MIXERS[spec.kind](self.cfg, number, pctx, dense_kind)
+        self.ffn = None
+        if spec.has_mlp:
+            self.ffn = MoE(self.cfg, pctx, expert_kind, dense_kind, ep_mode) if self.is_moe else DenseMLP(self.cfg, pctx, dense_kind, paired=dense_kind == "dense")
+        self.input_norm: Optional[torch.Tensor] = None         # fp32
+        self.post_norm: Optional[torch.Tensor] = None
+        self.rope_override: Optional[torch.Tensor] = None      # this layer's own rotary table
+
+    def init_random(self, gen, std, dtype, device):
+        fresh = lambda: torch.full((self.cfg.hidden_size,), 0.0 if self.cfg.norm_plus_one else 1.0, dtype=torch.float32, device=device)
+        self.mixer.init_random(gen, std, dtype, device)
+        self.input_norm = fresh()
+        if self.ffn is not None:
+            self.ffn.init_random(gen, std, dtype, device)
+            self.post_norm = fresh()
+
+    def share(self, first: "InputNormLayer") -> None:
+        """Take the weights of the layer's first run.  The mixer is an object of its own: it keeps rows between speculative
+        verification and commit."""
+        self.mixer, self.ffn = copy.copy(first.mixer), first.ffn
+        self.input_norm, self.post_norm = first.input_norm, first.post_norm
+
+    def accepts_prenormed(self) -> bool:
+        return False
+
+    def forward(self, x: NormDelta, stream: Optional[torch.Tensor], batch: ForwardBatch, cache: CacheStore, rope_cache, next_norm=None):
+        eps, p1 = self.cfg.rms_norm_eps, self.cfg.norm_plus_one
+        rope_cache = rope_cache if self.rope_override is None else self.rope_override
+        h, stream = ops.add_normed(stream, x, eps, p1, self.input_norm, step=self.step)
+        if attention_of(self) is not None:
+            x = NormDelta(self.mixer.forward(Act(x=h), batch, cache.layer_kv(self.idx), rope_cache))
+        else:
+            x = NormDelta(self.mixer.forward(Act(x=h), batch, cache.states[self.idx]))
+        if self.ffn is not None:
+            h, stream = ops.add_normed(stream, x, eps, p1, self.post_norm)
+            x = NormDelta(self.ffn.forward(Act(x=h), batch=batch, rows_ok=True) if self.is_moe else self.ffn.forward(Act(x=h), batch=batch))
+        return x, stream
+
+
 def attention_of(layer):
     """The attention block of a layer (None without one): the owner of the layer's KV cache."""
     if layer.kind == "parallel":
@@ -355,7 +409,7 @@ def attention_of(layer):
 
 def recurrent_of(layer):
     """The mixer of a layer that owns a recurrent state slot (None without one)."""
-    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel", "mlstm") else None
+    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel", "mlstm", "rglru") else None
 
 
 def kv_elements_of(attn) -> int:
@@ -372,10 +426,18 @@ class DecoderLM:
         self.device = torch.device(device)
         self.dtype = torch_dtype(cfg.dtype)
         if cfg.layer_specs:
-            if bool(cfg.residual_streams) == cfg.output_norms:
-                raise ValueError("a model given by a list of layers runs on hyper-connected residual streams or on normed outputs")
-            self.layers = [OutputNormLayer(cfg, i, self.pctx, ep_mode) if cfg.output_norms else StreamLayer(cfg, i, self.pctx)
-                           for i in range(cfg.num_hidden_layers)]
+            if bool(cfg.residual_streams) + cfg.output_norms + cfg.input_norms != 1:
+                raise ValueError("a model given by a list of layers runs on hyper-connected residual streams, on normed outputs or on "
+                                 "normed inputs")
+            if cfg.input_norms:
+                owners = [i for i, s in enumerate(cfg.layer_specs) if s.weights_of < 0]
+                number = lambda i, s: owners.index(i if s.weights_of < 0 else s.weights_of)
+                self.layers = [InputNormLayer(cfg, i, number(i, s), self.pctx, ep_mode) for i, s in enumerate(cfg.layer_specs)]
+            elif any(s.weights_of >= 0 or s.step >= 0 for s in cfg.layer_specs):
+                raise ValueError("layers run several times on normed inputs only")
+            else:
+                self.layers = [OutputNormLayer(cfg, i, self.pctx, ep_mode) if cfg.output_norms else StreamLayer(cfg, i, self.pctx)
+                               for i in range(cfg.num_hidden_layers)]
         elif cfg.block_types:
             self.layers = [SingleBlock(cfg, i, self.pctx) for i in range(cfg.num_hidden_layers)]
         else:
@@ -384,6 +446,7 @@ class DecoderLM:
         self.final_norm: Optional[torch.Tensor] = None
         self.lm_head: Optional[LinearWeight] = None          # vocab-parallel slice under TP
         self.rope_cache: Optional[torch.Tensor] = None
+        self.loop_step: Optional[torch.Tensor] = None        # fp32 [passes, hidden]: step vectors of looped layers
         self.mtp = None
         if (with_mtp if with_mtp is not None else cfg.mtp_num_layers > 0):
             from .mtp import MTPHead
@@ -406,8 +469,10 @@ class DecoderLM:
         gen = torch.Generator(device=gen_dev)
         gen.manual_seed(seed)
         self.embed = randn_weight(gen, cfg.vocab_size, cfg.hidden_size, std, dt, dev)
-        for layer in self.layers:
+        for layer in self.weight_layers():
             layer.init_random(gen, std, dt, dev)
+        if cfg.loop_steps:
+            self.loop_step = randn_weight(gen, cfg.loop_steps, cfg.hidden_size, std, torch.float32, dev)
         base = 0.0 if cfg.norm_plus_one else 1.0
         self.final_norm = torch.full((cfg.hidden_size,), base, dtype=torch.float32 if cfg.layer_specs else dt, device=dev)
         head = self.embed if cfg.tie_word_embeddings else randn_weight(gen, cfg.vocab_size, cfg.hidden_size, std, dt, dev)
@@ -416,6 +481,10 @@ class DecoderLM:
             self.mtp.init_random(gen, std, dt, dev)
         self.finalize(max_pos)
         return self
+
+    def weight_layers(self) -> list:
+        """The layers that own weights, in the checkpoint's order (one entry per layer, however often it runs)."""
+        return [l for l in self.layers if not getattr(l, "shared", False)]
 
     def enable_lora(self, max_slots: int = 7):
         """Attach one adapter set to the attention, dense-FFN and mixture-of-experts blocks of every layer."""
@@ -427,10 +496,11 @@ class DecoderLM:
                     attention_of(l).lora = self.lora
                 if l.ffn is None:
                     continue
-                l.ffn.lora, l.ffn.lora_prefix = self.lora, f"layers.{l.idx}.mlp."
+                prefix = f"layers.{getattr(l, 'number', l.idx)}.mlp."
+                l.ffn.lora, l.ffn.lora_prefix = self.lora, prefix
                 shared = getattr(l.ffn, "shared", None)
                 if shared is not None:
-                    shared.lora, shared.lora_prefix = self.lora, f"layers.{l.idx}.mlp.shared_expert."
+                    shared.lora, shared.lora_prefix = self.lora, prefix + "shared_expert."
         return self.lora
 
     def set_kv_rotation(self, on: bool = True) -> bool:
@@ -466,6 +536,10 @@ class DecoderLM:
     def finalize(self, max_pos: Optional[int] = None) -> None:
         cfg = self.cfg
         mp = max_pos or cfg.max_position_embeddings
+        for l, spec in zip(self.layers, cfg.layer_specs if cfg.input_norms else ()):
+            if spec.weights_of >= 0:
+                l.share(self.layers[spec.weights_of])
+            l.step = self.loop_step[spec.step] if spec.step >= 0 else None
         self.rope_cache = ref.build_rope_cache(cfg.rotary_dim, mp, cfg.rope_theta, cfg.rope_scaling, self.device)
         if cfg.rope_local_theta:
             local = ref.build_rope_cache(cfg.rotary_dim, mp, cfg.rope_local_theta, None, self.device)
@@ -535,7 +609,7 @@ class DecoderLM:
         if checked.ENABLED:
             checked.index_range("input_ids", ids, 0, self.cfg.vocab_size)
         e = self.embed[ids.long()]
-        if self.cfg.embed_scale != 1.0 and not self.cfg.residual_streams:
+        if self.cfg.embed_scale != 1.0 and not (self.cfg.residual_streams or self.cfg.input_norms):
             e = e * torch.tensor(self.cfg.embed_scale, dtype=e.dtype)      # the factor is rounded to the weight dtype first
         return e
 
@@ -609,8 +683,8 @@ class DecoderLM:
         residual = None
         if self.cfg.residual_streams:
             x = StreamDelta(x, scale=self.cfg.embed_scale)      # fp32 streams start from the scaled embedding
-        elif self.cfg.output_norms:
-            x = NormDelta(x)                  # so does the fp32 stream that takes normed outputs
+        elif self.cfg.output_norms or self.cfg.input_norms:
+            x = NormDelta(x, scale=self.cfg.embed_scale if self.cfg.input_norms else 1.0)      # so does a plain fp32 stream
         elif batch.inputs_embeds is not None:
             x = x.clone()                     # fused epilogues update the residual stream in place
         if layer_ids is not None:

@@ -139,28 +139,32 @@ def hyper_norm(streams: Optional[torch.Tensor], delta: StreamDelta, read: torch.
 @dataclass
 class ExpertRows:
     """Expert outputs before their weighted sum: ``y`` holds one row per (token, choice) pair, ``slot_of [T * k]`` the row of each
-    pair (-1: nothing to add), ``w [T, k]`` its weight."""
+    pair (-1: nothing to add), ``w [T, k]`` its weight; ``extra [T, W]`` joins the sum as it is (shared expert)."""
     y: torch.Tensor
     slot_of: torch.Tensor
     w: torch.Tensor
+    extra: Optional[torch.Tensor] = None
 
 
 @dataclass
 class NormDelta:
-    """What the last sublayer leaves for an fp32 residual stream that takes normed outputs: ``stream += rmsnorm(y) * norm``, with
-    ``y`` given as it is or as :class:`ExpertRows`.  Start of the model (``norm`` is None): the stream is ``y``."""
+    """What the last sublayer leaves for an fp32 residual stream: ``stream += rmsnorm(y) * norm``, or ``stream += y`` without
+    ``norm``, with ``y`` given as it is or as :class:`ExpertRows`.  Start of the model (no stream yet): the stream is
+    ``y * scale``."""
     y: object
     norm: Optional[torch.Tensor] = None
+    scale: float = 1.0
 
 
 def add_normed(stream: Optional[torch.Tensor], delta: NormDelta, eps: float, plus_one: bool, out_norm: Optional[torch.Tensor] = None,
-               write: bool = True) -> Tuple[torch.Tensor, torch.Tensor]:
-    """Apply ``delta`` to ``stream [T, W]`` (fp32, in place; None at the start) and return ``(h, stream)``: ``h`` is the stream in
-    the activations' dtype, normed with ``out_norm`` where one is given.  ``write=False`` leaves the stream as it is."""
+               write: bool = True, step: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Apply ``delta`` and then the vector ``step`` (fp32 ``[W]``) to ``stream [T, W]`` (fp32, in place; None at the start) and
+    return ``(h, stream)``: ``h`` is the stream in the activations' dtype, normed with ``out_norm`` where one is given.
+    ``write=False`` leaves the stream as it is."""
     y = delta.y.y if isinstance(delta.y, ExpertRows) else delta.y
     if on_gpu(y):
-        return cuda_ops().add_normed(stream, delta, eps, plus_one, out_norm, write)
-    return ref.add_normed(stream, delta, eps, plus_one, out_norm, write)
+        return cuda_ops().add_normed(stream, delta, eps, plus_one, out_norm, write, step)
+    return ref.add_normed(stream, delta, eps, plus_one, out_norm, write, step)
 
 
 # ----------------------------------------------------------------------------- elementwise / norm
@@ -210,11 +214,23 @@ def glu_act(gate_up: torch.Tensor, want_fp8=False, kind: str = "silu") -> Act:
     return Act(x=cuda_ops().gelu_tanh_mul(gate_up) if gpu else ref.gelu_tanh_mul(gate_up))
 
 
-def clamped_glu_act(gate_up: torch.Tensor, limit: float, alpha: float) -> Act:
-    """``g * sigmoid(alpha * g) * (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``."""
+SILU_UNIT = (float("inf"), 1.0, 0.0)        # silu(gate) * up as a gated unit
+
+
+def gated_unit_act(gate_up: torch.Tensor, unit: Tuple[float, float, float], paired: bool = False) -> Act:
+    """``g * sigmoid(alpha * g) * (u + shift)`` with ``unit = (limit, alpha, shift)``, ``g = min(gate, limit)`` and ``u = clamp(up,
+    -limit, limit)`` of ``[gate | up]``, or with ``paired`` of alternating gate and up columns."""
     if on_gpu(gate_up):
-        return Act(x=cuda_ops().clamped_glu(gate_up, limit, alpha))
-    return Act(x=ref.clamped_glu(gate_up, limit, alpha))
+        return Act(x=cuda_ops().gated_unit(gate_up, unit, paired))
+    return Act(x=ref.gated_unit(gate_up, unit, paired))
+
+
+def linear_gated_unit(a, w: LinearWeight, unit: Tuple[float, float, float]) -> Act:
+    """:func:`gated_unit_act` of a projection whose gate and up rows alternate; one kernel for unquantised bf16 weights."""
+    x = a.plain() if isinstance(a, Act) else a
+    if w.kind == "dense" and w.bias is None and on_gpu(x) and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
+        return Act(x=cuda_ops().gemm_bf16(x, w.weight, unit=unit))
+    return gated_unit_act(linear(a, w), unit, paired=True)
 
 
 def tanh_(x: torch.Tensor) -> torch.Tensor:
@@ -250,6 +266,8 @@ def silu_mul_act(gate_up: torch.Tensor, want_fp8=False) -> Act:
             q, s = ref.silu_mul_quant_fp8(gate_up)
         return Act(q=q, s=s, dtype=gate_up.dtype)
     if on_gpu(gate_up):
+        if gate_up.dtype == torch.float32 or inter % 8:
+            return gated_unit_act(gate_up, SILU_UNIT)
         return Act(x=cuda_ops().silu_mul(gate_up, quant=False))
     return Act(x=ref.silu_mul(gate_up))
 
@@ -284,9 +302,8 @@ def linear(a, w: LinearWeight, out: Optional[torch.Tensor] = None) -> torch.Tens
     else:
         x = act.plain()
         if dev_cuda and x.dtype == torch.bfloat16 and w.weight.dtype == torch.bfloat16:
-            y = cuda_ops().gemm_bf16(x, w.weight, out=out)
-        else:
-            y = torch.nn.functional.linear(x, w.weight)
+            return cuda_ops().gemm_bf16(x, w.weight, out=out, bias=w.bias)
+        return torch.nn.functional.linear(x, w.weight, w.bias)
     if w.bias is not None:
         y = y + w.bias
     return y
@@ -360,6 +377,18 @@ def qk_norm_rope_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v
                                      k_scale, v_scale, q_norm_w, k_norm_w, eps, norm_plus_one, rotate, norm_dim)
 
 
+def qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_norm_w, k_norm_w,
+                         eps: float, nq: int, nk: int, temp: float = 0.0, temp_every: int = 1, sums: Optional[torch.Tensor] = None):
+    """RMS norm of each row of ``q [T, Hq, D]`` and of ``k [T, Hkv, D]`` over all heads (``nq`` / ``nk`` channels, the rest is zero
+    padding) with fp32 weights, rotation, queries times ``1 + temp * ln(floor((seq_positions + 1) / temp_every) + 1)``, paged
+    cache write.  ``sums [T, 2]``: the rows' sums of squares where other ranks hold some of the heads."""
+    if on_gpu(q):
+        return cuda_ops().qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions,
+                                               q_norm_w, k_norm_w, eps, nq, nk, temp, temp_every, sums)
+    return ref.qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_norm_w,
+                                    k_norm_w, eps, nq, nk, temp, temp_every, sums)
+
+
 def head_rotate(x: torch.Tensor) -> torch.Tensor:
     """Orthonormal Walsh-Hadamard transform along the last (head) dimension of ``x [T, H, D]``; its own inverse."""
     if on_gpu(x) and x.shape[-1] == 128 and x.dtype == torch.bfloat16 and x.stride(2) == 1 and x.stride(1) == 128:
@@ -368,14 +397,15 @@ def head_rotate(x: torch.Tensor) -> torch.Tensor:
 
 
 def paged_attention(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None, chunk=0,
-                    sinks=None, softcap=0.0) -> torch.Tensor:
+                    sinks=None, softcap=0.0, distance=None) -> torch.Tensor:
     """Attention of the step's query rows over the paged cache. ``batch`` is a ``ForwardBatch``.  ``chunk`` > 0: a token sees
     only keys of its own ``chunk``-token block of the sequence; ``sinks [Hq]``: ``exp(sink)`` joins the softmax denominator;
-    ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)``."""
+    ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)``; ``distance [Hq, n]`` (fp32): column ``min(i - j, n - 1)``
+    joins the scaled score of query ``i`` and key ``j``."""
     if on_gpu(q):
-        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap)
+        return cuda_ops().paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap, distance)
     return ref.paged_attention(q, k_cache, v_cache, batch.block_tables, batch.seq_lens, batch.query_start_loc,
-                               scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap)
+                               scale, k_scale, v_scale, sliding_window, chunk, sinks, softcap, distance)
 
 
 def paged_attention_fp8_out(q, k_cache, v_cache, batch, scale, k_scale=1.0, v_scale=1.0, sliding_window=None) -> Optional[Act]:

@@ -444,14 +444,55 @@ def gemm_fp8_fused(xq, xs, wq, ws, mode: int = 0, out=None, residual=None, norm_
     return res
 
 
-def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None) -> torch.Tensor:
+def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.Tensor] = None, unit: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
+    """``x @ w^T (+ bias)``; with ``unit = (limit, alpha, shift)`` the gated unit of alternating gate and up columns, ``[M, N / 2]``."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     if x.shape[1] % 8:                 # rows that TMA cannot address (16-byte strides): a vendor product
-        y = torch.nn.functional.linear(x, w)
+        assert unit is None
+        y = torch.nn.functional.linear(x, w, None if bias is None else bias.to(x.dtype))
         return y if out is None else out.copy_(y)
     if x.stride(1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
-    return _gemm(0, x, w, None, None, out)
+    if bias is None and unit is None:
+        return _gemm(0, x, w, None, None, out)
+    M, K = x.shape
+    N = w.shape[0]
+    d = _dev(x)
+    assert w.stride(1) == 1
+    if out is None:
+        out = torch.empty(M, N if unit is None else N // 2, dtype=torch.bfloat16, device=x.device)
+    assert out.stride(1) == 1 and out.dtype == torch.bfloat16
+    if bias is not None:
+        assert bias.numel() == N
+        bias = _float_cached(bias)
+    L = lib()
+    if not getattr(L, "_bias_act_bound", False):
+        L.atlas_gemm_bias_act.argtypes = [_vp, _vp, _vp, _vp, _i, _f, _f, _f, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
+        L._bias_act_bound = True
+    sms = _num_sms[d]
+    bn, splits = gemm_plan(M, N, K, 0, sms)
+    ws = cnt = None
+    if splits > 1:
+        ws = scratch("gemm_ws", _GEMM_WS_BYTES, x.device)
+        cnt = scratch("gemm_counters", 1 << 18, x.device)
+    limit, alpha, shift = unit or (0.0, 0.0, 0.0)
+    _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(bias), 0 if unit is None else 2, float(limit), float(alpha), float(shift), M, N,
+                                 K, x.stride(0), w.stride(0), out.stride(0), bn, splits, _ptr(ws), _ptr(cnt), sms, _status_ptr[d], _stream()),
+           "gemm_bias_act")
+    return out
+
+
+_float_cache: dict = {}
+
+
+def _float_cached(t: torch.Tensor) -> torch.Tensor:
+    """fp32 copy of a (weight) vector, kept with the vector it was made from."""
+    if t.dtype == torch.float32 and t.is_contiguous():
+        return t
+    hit = _float_cache.get(t.data_ptr())
+    if hit is None or hit[0] is not t:
+        hit = _float_cache[t.data_ptr()] = (t, t.float().contiguous())
+    return hit[1]
 
 
 def linear_tail(x: torch.Tensor, w: torch.Tensor, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
@@ -586,7 +627,7 @@ def decode_splits(B: int, hkv: int, max_seq_len: int, sms: int) -> int:
     return int(max(1, min((2 * sms + ctas - 1) // ctas, (pages + 7) // 8, 64)))
 
 
-def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk=0, sinks=None, softcap=0.0):
+def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding_window, chunk=0, sinks=None, softcap=0.0, distance=None):
     T, Hq, D = q.shape
     nb, bs, Hkv, _ = k_cache.shape
     d = _dev(q)
@@ -600,13 +641,16 @@ def paged_attention(q, k_cache, v_cache, batch, scale, k_scale, v_scale, sliding
         checked.paged_read(batch.block_tables, batch.seq_lens, k_cache.shape[0], k_cache.shape[1])
     if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != Hq or not sinks.is_contiguous()):
         raise KernelError("attention sinks are one fp32 value per query head")
+    if distance is not None and (distance.dtype != torch.float32 or distance.shape[0] != Hq or not distance.is_contiguous()):
+        raise KernelError("a distance bias is one fp32 row per query head")
     if k_cache.dtype == torch.float32:
         from . import cuda_recurrent
-        return cuda_recurrent.attention_f32(q, k_cache, v_cache, batch, scale, window, int(chunk), sinks, float(softcap))
+        return cuda_recurrent.attention_f32(q, k_cache, v_cache, batch, scale, window, int(chunk), sinks, float(softcap), distance)
     if k_cache.dtype == torch.bfloat16:
-        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, chunk=int(chunk), sinks=sinks, softcap=float(softcap))
-    if chunk or sinks is not None or softcap:
-        raise KernelError("chunked attention, softmax sinks and bounded scores need a bf16 or fp32 KV cache")
+        return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, chunk=int(chunk), sinks=sinks, softcap=float(softcap),
+                                     distance=distance)
+    if chunk or sinks is not None or softcap or distance is not None:
+        raise KernelError("chunked attention, softmax sinks, bounded scores and distance biases need a bf16 or fp32 KV cache")
     if is_nvfp4_kv(k_cache):
         return _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=(float(k_scale), float(v_scale)))
     if nd > 0:
@@ -723,7 +767,8 @@ def _tc_tiles(q, batch, nd: int, tok: int):
     return tiles
 
 
-def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None, chunk=0, sinks=None, softcap=0.0):
+def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, scales=None, chunk=0, sinks=None, softcap=0.0,
+                          distance=None):
     """bf16 KV cache (or, with ``scales = (k_scale, v_scale)``, an NVFP4 one): the general mma.sync kernel serves decode
     rows (split-K + merge) and prefill tiles."""
     T, Hq, D = q.shape
@@ -740,9 +785,11 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
         raise KernelError("the NVFP4 KV cache is implemented for head_dim 128")
     if not getattr(L, "_kv16_bound", False):
         L.atlas_attn_decode_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i,
-                                             _vp, _vp, _vp, _i, _vp, _f]
-        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp, _i, _vp, _f]
+                                             _vp, _vp, _vp, _i, _vp, _f, _vp, _i]
+        L.atlas_attn_prefill_kv16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _f, _i, _i, _i, _i, _i, _vp, _i, _vp, _f,
+                                              _vp, _i]
         L._kv16_bound = True
+    bias = (_ptr(distance), distance.shape[1] - 1 if distance is not None else 0)
     bt, st, nd = batch.block_tables, _stream(), batch.num_decodes
     if nd > 0:
         visible = min(batch.max_seq_len, chunk or batch.max_seq_len, window or batch.max_seq_len)
@@ -760,18 +807,18 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
             _check(L.atlas_attn_decode_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                             bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                             0, nd, float(scale), Hq, Hkv, D, bs, window, splits, _ptr(po), _ptr(pml), st, chunk,
-                                            _ptr(sinks), softcap), "attn_decode_kv16")
+                                            _ptr(sinks), softcap, *bias), "attn_decode_kv16")
     if batch.num_seqs > nd and not fp4 and _TC_PREFILL and bs == 16 and D <= 128 and Hq // Hkv <= 128:
         # tcgen05 tiles of 128 // G query tokens; 1 = a shape the kernel does not take
         tdev, n_tiles, _ = _tc_tiles(q, batch, nd, 128 // (Hq // Hkv))
         if not getattr(L, "_tc16_bound", False):
             L.atlas_attn_prefill_tc16.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _f, _i, _i, _i, _i,
-                                                  _i, _i, _vp, _f, _vp, _vp]
+                                                  _i, _i, _vp, _f, _vp, _i, _vp, _vp]
             L._tc16_bound = True
         rc = L.atlas_attn_prefill_tc16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                        bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                        tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, T, float(scale), Hq, Hkv, D, bs, chunk,
-                                       window, _ptr(sinks), softcap, _status_ptr[d], st)
+                                       window, _ptr(sinks), softcap, *bias, _status_ptr[d], st)
         if rc != 1:
             _check(rc, "attn_prefill_tc16")
             return out
@@ -796,7 +843,7 @@ def _paged_attention_kv16(q, out, k_cache, v_cache, batch, scale, window, d, sca
             _check(L.atlas_attn_prefill_kv16(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                              bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                              tdev[0].data_ptr(), tdev[1].data_ptr(), n_tiles, float(scale), Hq, Hkv, D, bs, window, st, chunk,
-                                             _ptr(sinks), softcap), "attn_prefill_kv16")
+                                             _ptr(sinks), softcap, *bias), "attn_prefill_kv16")
     return out
 
 
@@ -894,9 +941,9 @@ def moe_route(logits, top_k, norm_topk, scoring, bias=None, n_group=0, topk_grou
     return cuda_ext.moe_route(logits, top_k, norm_topk, scoring, bias, n_group, topk_group, scale, hash_table, token_ids)
 
 
-def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation="silu_glu", rows_ok=False):
+def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation="silu_glu", rows_ok=False, unit=None):
     from . import cuda_ext
-    return cuda_ext.moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation=activation, rows_ok=rows_ok)
+    return cuda_ext.moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, activation=activation, rows_ok=rows_ok, unit=unit)
 
 
 def gdn_forward(layer, mixed, a, b, batch, state, commit):
@@ -939,6 +986,21 @@ def mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_
     return cuda_recurrent.mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_rows)
 
 
+def rglru_forward(layer, y, x, batch, state, commit):
+    from . import cuda_recurrent
+    return cuda_recurrent.rglru_forward(layer, y, x, batch, state, commit)
+
+
+def rglru_commit(layer, x, qlens, slots, has_state, state, num_accepted_rows):
+    from . import cuda_recurrent
+    return cuda_recurrent.rglru_commit(layer, x, qlens, slots, has_state, state, num_accepted_rows)
+
+
+def qk_row_norm_kv_write(*args):
+    from . import cuda_recurrent
+    return cuda_recurrent.qk_row_norm_kv_write(*args)
+
+
 def latent_attention(layer, q, ckv, batch, cache, rope_cache):
     from . import cuda_latent
     return cuda_latent.latent_attention(layer, q, ckv, batch, cache, rope_cache)
@@ -949,9 +1011,9 @@ def group_norm_gate(y, z, w, group, eps, gate_first, gate="silu", den=None):
     return cuda_recurrent.group_norm_gate(y, z, w, group, eps, gate_first, gate, den)
 
 
-def add_normed(stream, delta, eps, plus_one, out_norm, write):
+def add_normed(stream, delta, eps, plus_one, out_norm, write, step=None):
     from . import cuda_recurrent
-    return cuda_recurrent.add_normed(stream, delta, eps, plus_one, out_norm, write)
+    return cuda_recurrent.add_normed(stream, delta, eps, plus_one, out_norm, write, step)
 
 
 def head_gate(x, g):
@@ -969,9 +1031,9 @@ def token_shift_mix(x, mu, batch, shift):
     return cuda_recurrent.token_shift_mix(x, mu, batch, shift)
 
 
-def clamped_glu(gate_up, limit, alpha):
+def gated_unit(gate_up, unit, paired=False):
     from . import cuda_recurrent
-    return cuda_recurrent.clamped_glu(gate_up, limit, alpha)
+    return cuda_recurrent.gated_unit(gate_up, unit, paired)
 
 
 def tanh_(x):

@@ -18,8 +18,8 @@ def bind(lib) -> None:
     lib.atlas_moe_align.argtypes = [_vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i, _vp, _vp]
     lib.atlas_moe_gather.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _vp, _vp, _ll, _vp]
     lib.atlas_moe_combine.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _i, _vp, _ll, _vp, _ll, _vp]
-    lib.atlas_gemm_grouped.argtypes = [_i, _vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _ll, _ll, _ll, _i, _vp, _vp, _i, _vp, _vp, _i]
-    lib.atlas_moe_plain_gemm.argtypes = [_vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _ll, _i, _vp]
+    lib.atlas_gemm_grouped.argtypes = [_i, _vp, _vp, _vp, _vp, _ll, _vp, _i, _i, _i, _i, _ll, _ll, _ll, _i, _vp, _vp, _i, _vp, _vp, _i, _f, _f, _f]
+    lib.atlas_moe_plain_gemm.argtypes = [_vp, _ll, _vp, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _i, _i, _vp, _ll, _i, _vp]
     lib.atlas_moe_plain_combine.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _i, _vp, _ll, _i, _vp]
     lib.atlas_moe_dispatch_prep.argtypes = [_vp, _i, _i, _i, _vp, _vp, _vp]
     lib.atlas_moe_dispatch_pack.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _i, _vp, _i, _vp]
@@ -145,25 +145,25 @@ def _expert_stacks(experts):
 
 
 def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, addend: Optional[torch.Tensor] = None, activation: str = "silu_glu",
-                rows_ok: bool = False):
+                rows_ok: bool = False, unit=None):
     """Expert-sorted grouped FFN over this rank's experts.  Pairs routed to other ranks' experts contribute nothing
     here; with expert parallelism the partial outputs are summed across ranks (``allreduce`` mode, the default while
     activations are replicated across the group) or the rows travel to their experts and back (``alltoall`` mode)."""
     if ep_mode == "alltoall" and pctx is not None and pctx.ep_size > 1:
         comm = pctx.ep_comm if pctx.ep_comm is not None else pctx.comm
         if hasattr(comm, "all_to_all_rows"):
-            out = _moe_forward_alltoall(x, topk_w, topk_ids, experts, e_lo, pctx, comm, addend, activation)
+            out = _moe_forward_alltoall(x, topk_w, topk_ids, experts, e_lo, pctx, comm, addend, activation, unit)
             if out is not None:
                 return out
     comm = None
     if pctx is not None and pctx.ep_size > 1:
         comm = pctx.ep_comm if pctx.ep_comm is not None else pctx.comm
     if comm is None:
-        return _moe_local(x, topk_w, topk_ids, experts, e_lo, addend, activation=activation, rows_ok=rows_ok)
+        return _moe_local(x, topk_w, topk_ids, experts, e_lo, addend, activation=activation, rows_ok=rows_ok, unit=unit)
     # every rank runs its own experts on the replicated rows; the partial outputs are summed over the group.  With a
     # peer-memory backend and a decode-size step the weighted combine and that sum are ONE kernel.
     fused = comm if hasattr(comm, "moe_combine_all_reduce") else None
-    out, reduced = _moe_local(x, topk_w, topk_ids, experts, e_lo, addend, fused_comm=fused, grouped=True, activation=activation)
+    out, reduced = _moe_local(x, topk_w, topk_ids, experts, e_lo, addend, fused_comm=fused, grouped=True, activation=activation, unit=unit)
     if not reduced:
         out = comm.all_reduce(out)
         if addend is not None:
@@ -171,7 +171,7 @@ def moe_forward(x, topk_w, topk_ids, experts, e_lo, pctx, ep_mode, addend: Optio
     return out
 
 
-def _moe_forward_alltoall(x, topk_w, topk_ids, experts, e_lo, pctx, comm, addend, activation="silu_glu"):
+def _moe_forward_alltoall(x, topk_w, topk_ids, experts, e_lo, pctx, comm, addend, activation="silu_glu", unit=None):
     """Dispatch / combine over peer memory.  Activations are replicated across the group, so rank r dispatches only its
     slice of the tokens: every (token, expert) pair is computed exactly once, on the rank that owns the expert.
 
@@ -212,7 +212,7 @@ def _moe_forward_alltoall(x, topk_w, topk_ids, experts, e_lo, pctx, comm, addend
     K._check(lib.atlas_moe_recv_ids(recv.data_ptr(), row_bytes, H, recv_off.data_ptr(), W, cap, rid.data_ptr(), st),
              "moe_recv_ids")
     ones = _ones(cap, dev)
-    y_rows = _moe_local(recv[:, :H], ones, rid, experts, e_lo, None, activation=activation)          # [cap, H]; dead rows are zero
+    y_rows = _moe_local(recv[:, :H], ones, rid, experts, e_lo, None, activation=activation, unit=unit)          # [cap, H]; dead rows are zero
     back, _ = comm.all_to_all_rows(y_rows, recv_off, pairs_cap)
     out = torch.zeros(T, H, dtype=torch.bfloat16, device=dev)
     if Ts:
@@ -263,25 +263,33 @@ def _finish(lib, y, slot_of, topk_w, T, k, H, addend, fused_comm, grouped, dev, 
     return (out, False) if grouped else out
 
 
-def _moe_plain(lib, st, x, experts, row_token, tile_expert, num_tiles, max_rows, relu2: bool):
+_EXPERT_ACTS = {"relu2": 1, "clamped_glu": 2}        # activations that the expert products apply themselves
+
+
+def _unit(unit):
+    return (0.0, 0.0, 0.0) if unit is None else tuple(float(v) for v in unit)
+
+
+def _moe_plain(lib, st, x, experts, row_token, tile_expert, num_tiles, max_rows, activation: str, unit):
     """Expert rows in fp32 sums on the CUDA cores: fp32 models and sizes that the tensor-core tiles do not take."""
-    if experts.kind != "dense" or experts.w13.dtype != x.dtype or not relu2:
-        raise K.KernelError("the plain expert kernels take unquantised experts without a gate in the activations' dtype")
+    if experts.kind != "dense" or experts.w13.dtype != x.dtype or activation not in _EXPERT_ACTS:
+        raise K.KernelError("the plain expert kernels take unquantised experts in the activations' dtype whose activation they apply")
     f32 = 1 if x.dtype == torch.float32 else 0
     w13, w2 = experts.w13, experts.w2
     H, I = x.shape[1], w2.shape[2]
     assert x.stride(1) == 1 and w13.is_contiguous() and w2.is_contiguous()
     h = torch.empty(max_rows, I, dtype=x.dtype, device=x.device)
     K._check(lib.atlas_moe_plain_gemm(x.data_ptr(), x.stride(0), w13.data_ptr(), row_token.data_ptr(), tile_expert.data_ptr(), num_tiles.data_ptr(),
-                                      max_rows, 1, 1, I, H, h.data_ptr(), I, f32, st), "moe_plain_up")
+                                      max_rows, 1, _EXPERT_ACTS[activation], *_unit(unit), w13.shape[1], H, h.data_ptr(), I, f32,
+                                      st), "moe_plain_up")
     y = torch.empty(max_rows, H, dtype=x.dtype, device=x.device)
     K._check(lib.atlas_moe_plain_gemm(h.data_ptr(), I, w2.data_ptr(), row_token.data_ptr(), tile_expert.data_ptr(), num_tiles.data_ptr(), max_rows, 0,
-                                      0, H, I, y.data_ptr(), H, f32, st), "moe_plain_down")
+                                      0, 0.0, 0.0, 0.0, H, I, y.data_ptr(), H, f32, st), "moe_plain_down")
     return y
 
 
 def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor] = None, fused_comm=None, grouped=False,
-               activation: str = "silu_glu", rows_ok: bool = False):
+               activation: str = "silu_glu", rows_ok: bool = False, unit=None):
     if K.checked.ENABLED:
         K.checked.index_range("topk_ids", topk_ids, 0, 1 << 20)
         K.checked.finite("topk_w", topk_w)
@@ -290,9 +298,9 @@ def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor
     k = topk_ids.shape[1]
     d = K._dev(x)
     dev = x.device
-    relu2 = activation == "relu2"
+    own_act = activation in _EXPERT_ACTS               # not the SwiGLU of the other paths
     E = experts.num_local
-    plain = x.dtype == torch.float32 or (experts.kind == "dense" and relu2 and (H % 64 or experts.w2.shape[2] % 64))
+    plain = x.dtype == torch.float32 or (experts.kind == "dense" and own_act and (H % 64 or experts.w2.shape[2] % 64))
     if not plain:
         kind, w13, s13, w2, s2 = _expert_stacks(experts)
         I = w2.shape[2] * 2 if kind == 2 else w2.shape[2]
@@ -311,7 +319,7 @@ def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor
         return 128 if n % 128 == 0 else 64
 
     if plain:
-        y = _moe_plain(lib, st, x, experts, row_token, tile_expert, num_tiles, max_rows, relu2)
+        y = _moe_plain(lib, st, x, experts, row_token, tile_expert, num_tiles, max_rows, activation, unit)
         if rows_ok and addend is None:
             return ExpertRows(y, slot_of, topk_w)
         if grouped and fused_comm is not None and x.dtype == torch.bfloat16 and H % 8 == 0:
@@ -322,7 +330,7 @@ def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor
         if grouped:
             return out, False                          # the caller adds the addend after the group's sum
         return out if addend is None else out + addend
-    if kind == 2 and not relu2 and _small_moe_ok(T * k, E, H, I):
+    if kind == 2 and not own_act and _small_moe_ok(T * k, E, H, I):
         # decode-size batch on NVFP4 experts: a few rows per expert, so stream the weights through the register-level
         # dequant kernel (rows gathered by token inside it, SiLU fused) instead of 128-row tcgen05 tiles
         _bind_small(lib)
@@ -346,18 +354,19 @@ def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor
         K._check(lib.atlas_moe_gather(x.data_ptr(), x.stride(0), row_token.data_ptr(), num_tiles.data_ptr(), max_rows, H,
                                       xp.data_ptr(), None, None, 0, st), "moe_gather")
         a1, a1s = xp, None
-    h1 = torch.empty(max_rows, N1, dtype=torch.bfloat16, device=dev)
+    fused_act = _EXPERT_ACTS.get(activation, 0) if kind == 0 else 0       # bf16 experts: part of the product's epilogue
+    N1o = N1 // 2 if fused_act == 2 else N1
+    h1 = torch.empty(max_rows, N1o, dtype=torch.bfloat16, device=dev)
     if kind == 2:
         K._check(lib.atlas_gemm_w4a16_grouped(a1.data_ptr(), w13.data_ptr(), s13[0].data_ptr(), s13[1].data_ptr(), h1.data_ptr(),
                                               max_rows, N1, H, E, H, N1, bn_for(N1), tile_expert.data_ptr(),
                                               num_tiles.data_ptr(), sms, status, st), "moe_gemm1_w4")
     else:
         K._check(lib.atlas_gemm_grouped(kind, a1.data_ptr(), w13.data_ptr(), h1.data_ptr(), K._ptr(a1s), max_rows, K._ptr(s13),
-                                        max_rows, N1, H, E, H, H, N1, bn_for(N1), tile_expert.data_ptr(),
-                                        num_tiles.data_ptr(), sms, status, st, 1 if relu2 and kind == 0 else 0), "moe_gemm1")
-    if relu2:
-        # bf16 experts: the activation is part of the product's epilogue
-        act = h1 if kind == 0 else K.relu_squared(h1)
+                                        max_rows, N1, H, E, H, H, N1o, bn_for(N1), tile_expert.data_ptr(),
+                                        num_tiles.data_ptr(), sms, status, st, fused_act, *_unit(unit)), "moe_gemm1")
+    if own_act:
+        act = h1 if fused_act else (K.relu_squared(h1) if activation == "relu2" else K.gated_unit(h1, unit, paired=True))
         a2, a2s = K.quant_fp8(act) if kind == 1 else (act, None)
     elif kind == 1:
         aq = torch.empty(max_rows, I, dtype=FP8, device=dev)
@@ -378,7 +387,7 @@ def _moe_local(x, topk_w, topk_ids, experts, e_lo, addend: Optional[torch.Tensor
     else:
         K._check(lib.atlas_gemm_grouped(kind, a2.data_ptr(), w2.data_ptr(), y.data_ptr(), K._ptr(a2s), max_rows, K._ptr(s2),
                                         max_rows, H, I, E, I, I, H, bn_for(H), tile_expert.data_ptr(), num_tiles.data_ptr(),
-                                        sms, status, st, 0), "moe_gemm2")
+                                        sms, status, st, 0, 0.0, 0.0, 0.0), "moe_gemm2")
     if rows_ok and addend is None:
         return ExpertRows(y, slot_of, topk_w)
     return _finish(lib, y, slot_of, topk_w, T, k, H, addend, fused_comm, grouped, dev, st)

@@ -1,5 +1,5 @@
 """Binding of the residual-stream, recurrence and 32-bit attention kernels (``csrc/streams.cu``, ``csrc/recurrent.cu``,
-``csrc/mlstm.cu``, ``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
+``csrc/mlstm.cu``, ``csrc/rglru.cu``, ``csrc/row_norm_kv.cu``, ``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
 from __future__ import annotations
 
 import ctypes as C
@@ -14,27 +14,39 @@ _vp, _ll, _i, _f = C.c_void_p, C.c_longlong, C.c_int, C.c_float
 _bound = False
 
 
+class _Rglru(C.Structure):
+    """Mirror of ``AtlasRglru`` (csrc/host_api.h)."""
+    _fields_ = [("x", _vp), ("ldx", _ll), ("u", _vp), ("ldu", _ll), ("zr", _vp), ("zi", _vp), ("z_row", _ll), ("z_block", _ll), ("y", _vp),
+                ("ldy", _ll), ("conv_w", _vp), ("conv_b", _vp), ("conv_state", _vp), ("tiles", _vp), ("gate_bias", _vp), ("lam", _vp), ("h", _vp),
+                ("P", _vp), ("S", _vp), ("endP", _vp), ("endS", _vp), ("out", _vp), ("ldo", _ll), ("seq_of", _vp), ("qsl", _vp), ("slots", _vp),
+                ("has", _vp), ("limit", _vp), ("snap_rows", _vp), ("snap_slots", _vp), ("status", _vp), ("snaps", _i), ("rows", _i), ("C", _i),
+                ("n", _i), ("taps", _i), ("commit", _i), ("one_row", _i)]
+
+
 def _lib():
     global _bound
     lib = K.lib()
     if not _bound:
         lib.atlas_hyper_norm.argtypes = [_vp, _i, _i, _i, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _f, _f, _i, _vp]
         lib.atlas_token_shift_mix.argtypes = [_vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]
-        lib.atlas_clamped_glu.argtypes = [_vp, _ll, _i, _i, _vp, _ll, _f, _f, _i, _vp]
+        lib.atlas_gated_unit.argtypes = [_vp, _ll, _i, _i, _vp, _ll, _f, _f, _f, _i, _i, _vp]
+        lib.atlas_rglru_tc.argtypes = [C.POINTER(_Rglru), _vp]
+        lib.atlas_rglru_scan.argtypes = [C.POINTER(_Rglru), _i, _vp]
+        lib.atlas_row_norm_kv_write.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll] + [_vp] * 9 + [_i] * 8 + [_f, _f, _i, _i, _vp]
         lib.atlas_tanh.argtypes = [_vp, _ll, _i, _vp]
         lib.atlas_mamba2_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _vp] + [_i] * 9 + [_vp]
         lib.atlas_wkv_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _vp, _vp, _vp,
                                        _vp, _vp, _vp] + [_i] * 7 + [_vp]
         lib.atlas_group_norm_gate.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _i, _i, _vp, _i, _vp]
-        lib.atlas_add_normed.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _i, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _f, _i, _vp]
+        lib.atlas_add_normed.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _i, _vp, _ll, _vp, _vp, _vp, _vp, _ll] + [_i] * 5 + [_f, _f, _i, _vp]
         lib.atlas_head_gate.argtypes = [_vp, _ll, _vp, _ll, _i, _i, _i, _i, _vp]
         lib.atlas_mlstm_gates.argtypes = [_vp, _ll, _vp, _f] + [_vp] * 10 + [_i] * 4 + [_vp]
         lib.atlas_mlstm_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll] + [_vp] * 7 + [_i] * 8 + [_vp]
         lib.atlas_mlstm_chunk.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll] + [_vp] * 6 + [_i] * 6 + [_vp]
-        lib.atlas_conv1d_bias_silu.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _vp]
+        lib.atlas_conv1d_bias_silu.argtypes = [_vp, _ll, _vp, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp]
         lib.atlas_conv1d_state.argtypes = [_vp, _ll, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp]
         lib.atlas_rope_kv_write_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _f, _vp]
-        lib.atlas_attn_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp, _f, _vp]
+        lib.atlas_attn_f32.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _vp, _i, _vp, _vp, _i, _i, _f, _i, _i, _i, _i, _i, _i, _vp, _f, _vp, _i, _vp]
         _bound = True
     return lib
 
@@ -89,13 +101,13 @@ def token_shift_mix(x, mu, batch, shift):
     return out
 
 
-def clamped_glu(gate_up, limit: float, alpha: float):
+def gated_unit(gate_up, unit, paired: bool = False):
     T, I2 = gate_up.shape
     K._dev(gate_up)
     f32 = _f32(gate_up)
     y = torch.empty(T, I2 // 2, dtype=gate_up.dtype, device=gate_up.device)
-    K._check(_lib().atlas_clamped_glu(gate_up.data_ptr(), gate_up.stride(0), T, I2 // 2, y.data_ptr(), y.stride(0), float(limit),
-                                      float(alpha), f32, K._stream()), "clamped_glu")
+    K._check(_lib().atlas_gated_unit(gate_up.data_ptr(), gate_up.stride(0), T, I2 // 2, y.data_ptr(), y.stride(0),
+                                     *(float(v) for v in unit), 1 if paired else 0, f32, K._stream()), "gated_unit")
     return y
 
 
@@ -113,22 +125,12 @@ def group_norm_gate(y, z, w, group: int, eps: float, gate_first: bool, gate: str
     f32 = _f32(y)
     assert z.dtype == y.dtype and z.shape == y.shape and z.stride(1) == 1 and n % group == 0
     assert den is None or (den.dtype == torch.float32 and den.is_contiguous() and den.numel() == T * (n // group))
-    wf = w if w.dtype == torch.float32 else _float_cached(w)
+    wf = K._float_cached(w)
     out = torch.empty(T, n, dtype=y.dtype, device=y.device)
     K._check(_lib().atlas_group_norm_gate(y.data_ptr(), y.stride(0), z.data_ptr(), z.stride(0), wf.data_ptr(), out.data_ptr(), n, T,
                                           n // group, group, float(eps), 1 if gate_first else 0, 1 if gate == "sigmoid" else 0, K._ptr(den),
                                           f32, K._stream()), "group_norm_gate")
     return out
-
-
-_float_cache: dict = {}
-
-
-def _float_cached(t: torch.Tensor) -> torch.Tensor:
-    hit = _float_cache.get(t.data_ptr())
-    if hit is None or hit[0] is not t:
-        hit = _float_cache[t.data_ptr()] = (t, t.float().contiguous())
-    return hit[1]
 
 
 def _mamba2_run(layer, xbc, dt, meta: _Meta, state, commit: bool):
@@ -144,7 +146,7 @@ def _mamba2_run(layer, xbc, dt, meta: _Meta, state, commit: bool):
     out = torch.empty(T, layer.d_inner, dtype=xbc.dtype, device=xbc.device)
     K._check(lib.atlas_conv1d_bias_silu(xbc.data_ptr(), xbc.stride(0), layer.conv_w.data_ptr(), K._ptr(layer.conv_b), Cc, layer.W,
                                         conv.data_ptr(), meta.seq_of.data_ptr(), meta.qsl.data_ptr(), meta.slots.data_ptr(),
-                                        meta.has.data_ptr(), y.data_ptr(), Cc, T, f32, st), "conv1d")
+                                        meta.has.data_ptr(), y.data_ptr(), Cc, T, 1, f32, st), "conv1d")
     K._check(lib.atlas_mamba2_scan(y.data_ptr(), Cc, dt.data_ptr(), dt.stride(0), layer.A_log.data_ptr(), layer.D.data_ptr(),
                                    layer.dt_bias.data_ptr(), float(layer.cfg.mamba_dt_min), h.data_ptr(), out.data_ptr(),
                                    layer.d_inner, meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr(),
@@ -238,27 +240,95 @@ def mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_
     _mlstm_run(layer, None, k, v, raw, meta, state, True)
 
 
-# ----------------------------------------------------------------------------- normed outputs on an fp32 residual
-def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool, out_norm, write: bool):
+RGLRU_CHUNK = 64              # rows per chunk of the recurrence (kRgRows in csrc/rglru.cu)
+RGLRU_TENSOR_CORES = True     # tests switch this off to compare the two forms
+
+
+def _rglru_run(layer, y, x, meta: _Meta, state, commit: bool):
+    lib, st = _lib(), K._stream()
+    dev = K._dev(x)
+    f32 = _f32(x)
+    conv, h = state["conv"], state["h"]
+    T, Cc = x.shape
+    assert conv.dtype == x.dtype and h.dtype == torch.float32 and conv.is_contiguous() and h.is_contiguous() and Cc == layer.c
+    assert layer.conv_w.dtype == layer.conv_b.dtype == x.dtype and layer.gate_bias.dtype == layer.lam.dtype == torch.float32
+    out = torch.empty(T, Cc, dtype=x.dtype, device=x.device) if y is not None else None
+    a = _Rglru(x=x.data_ptr(), ldx=x.stride(0), conv_w=layer.conv_w.data_ptr(), conv_b=layer.conv_b.data_ptr(), conv_state=conv.data_ptr(),
+               gate_bias=layer.gate_bias.data_ptr(), lam=layer.lam.data_ptr(), h=h.data_ptr(), seq_of=meta.seq_of.data_ptr(),
+               qsl=meta.qsl.data_ptr(), slots=meta.slots.data_ptr(), has=meta.has.data_ptr(), limit=K._ptr(meta.limit),
+               snap_rows=meta.snap_rows.data_ptr(), snap_slots=meta.snap_slots.data_ptr(), status=K._status_ptr[dev], snaps=meta.snaps, rows=T,
+               C=Cc, n=layer.n, taps=layer.W, commit=1 if commit else 0)
+    if y is not None:
+        assert y.dtype == x.dtype and y.stride(1) == 1
+        a.y, a.ldy, a.out, a.ldo = y.data_ptr(), y.stride(0), out.data_ptr(), Cc
+    tc = RGLRU_TENSOR_CORES and layer.gate_tiles is not None
+    a.one_row = 1 if tc and meta.one_row and y is not None else 0
+    rc = 1
+    if a.one_row:
+        a.tiles = layer.gate_tiles.data_ptr()
+        rc = lib.atlas_rglru_tc(C.byref(a), st)
+        a.one_row = 1 if rc != 1 else 0
+        if rc != 1:
+            K._check(rc, "rglru_step")
+    if rc == 1:
+        rows, ends = torch.empty(2, T, Cc, dtype=torch.float32, device=x.device), torch.empty(2, -(-T // RGLRU_CHUNK), Cc, dtype=torch.float32, device=x.device)
+        a.P, a.S, a.endP, a.endS = rows[0].data_ptr(), rows[1].data_ptr(), ends[0].data_ptr(), ends[1].data_ptr()
+        if tc:
+            a.tiles = layer.gate_tiles.data_ptr()
+            rc = lib.atlas_rglru_tc(C.byref(a), st)
+            if rc != 1:
+                K._check(rc, "rglru_tc")
+    if rc == 1:
+        u = torch.empty(T, Cc, dtype=x.dtype, device=x.device)
+        K._check(lib.atlas_conv1d_bias_silu(x.data_ptr(), x.stride(0), layer.conv_w.data_ptr(), layer.conv_b.data_ptr(), Cc, layer.W, conv.data_ptr(),
+                                            meta.seq_of.data_ptr(), meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr(), u.data_ptr(),
+                                            Cc, T, 0, f32, st), "conv1d")
+        # gate sums [2, blocks, T, n] in fp32
+        z = torch.matmul(u.float().view(T, layer.blocks, layer.n).transpose(0, 1), layer.gates.float().transpose(2, 3))
+        a.u, a.ldu, a.zr, a.zi, a.z_row, a.z_block = u.data_ptr(), Cc, z[0].data_ptr(), z[1].data_ptr(), layer.n, T * layer.n
+        K._check(lib.atlas_rglru_scan(C.byref(a), f32, st), "rglru_scan")
+    if commit:
+        K._check(lib.atlas_conv1d_state(x.data_ptr(), x.stride(0), Cc, layer.W, conv.data_ptr(), meta.qsl.data_ptr(), meta.slots.data_ptr(),
+                                        meta.has.data_ptr(), K._ptr(meta.limit), meta.snap_rows.data_ptr(), meta.snap_slots.data_ptr(), meta.snaps,
+                                        meta.B, f32, st), "conv1d_state")
+    return out
+
+
+def rglru_forward(layer, y, x, batch, state, commit):
+    return _rglru_run(layer, y, x, step_meta(batch, x.device), state, commit)
+
+
+def rglru_commit(layer, x, qlens, slots, has_state, state, num_accepted_rows):
+    meta = _Meta(qlens, slots, has_state, x.device, None, limit=list(num_accepted_rows))
+    _rglru_run(layer, None, x, meta, state, True)
+
+
+# ----------------------------------------------------------------------------- sublayer outputs on an fp32 residual
+def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool, out_norm, write: bool, step=None):
     rows = delta.y if hasattr(delta.y, "slot_of") else None
     y = rows.y if rows is not None else delta.y
     W = y.shape[1]
     T = rows.w.shape[0] if rows is not None else y.shape[0]
     K._dev(y)
     f32 = _f32(y)
-    if stream is None:
+    first = stream is None
+    if first:
         assert delta.norm is None
         stream, write = torch.empty(T, W, dtype=torch.float32, device=y.device), True
     assert stream.dtype == torch.float32 and stream.shape == (T, W) and stream.is_contiguous()
-    for w in (delta.norm, out_norm):
+    for w in (delta.norm, out_norm, step):
         assert w is None or (w.dtype == torch.float32 and w.numel() == W and w.is_contiguous())
     if rows is not None:
         assert rows.slot_of.dtype == torch.int32 and rows.w.dtype == torch.float32 and rows.w.is_contiguous()
+    extra = rows.extra if rows is not None else None
+    if extra is not None:
+        assert extra.dtype == y.dtype and extra.shape == (T, W) and extra.stride(1) == 1
     out = torch.empty(T, W, dtype=y.dtype, device=y.device)
     K._check(_lib().atlas_add_normed(stream.data_ptr(), W, y.data_ptr(), y.stride(0), K._ptr(rows.slot_of) if rows is not None else None,
                                      K._ptr(rows.w) if rows is not None else None, rows.w.shape[1] if rows is not None else 0,
-                                     K._ptr(delta.norm), K._ptr(out_norm), out.data_ptr(), W, T, W, 1 if plus_one else 0, 1 if write else 0,
-                                     float(eps), f32, K._stream()), "add_normed")
+                                     K._ptr(extra), extra.stride(0) if extra is not None else 0, K._ptr(delta.norm), K._ptr(out_norm),
+                                     K._ptr(step), out.data_ptr(), W, T, W, 1 if plus_one else 0, 1 if write else 0, 1 if first else 0, float(eps),
+                                     float(delta.scale), f32, K._stream()), "add_normed")
     return out, stream
 
 
@@ -268,6 +338,28 @@ def head_gate(x, g):
     assert x.stride(2) == 1 and x.stride(1) == D and g.dtype == torch.float32 and g.shape == (T, H) and g.stride(1) == 1
     K._check(_lib().atlas_head_gate(x.data_ptr(), x.stride(0), g.data_ptr(), g.stride(0), T, H, D, _f32(x), K._stream()), "head_gate")
     return x
+
+
+# ----------------------------------------------------------------------------- norm over all heads
+def qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_w, k_w, eps, nq, nk, temp,
+                         temp_every, sums):
+    T, Hq, D = q.shape
+    Hkv = k.shape[1]
+    K._dev(q)
+    K._kv_layout_ok(k_cache, v_cache)
+    f32 = _f32(q)
+    assert k_cache.dtype == v_cache.dtype == q.dtype == k.dtype == v.dtype, "this cache holds the activations' dtype"
+    assert q.stride(1) == k.stride(1) == v.stride(1) == D and positions.dtype == seq_positions.dtype == slot_mapping.dtype == torch.int32
+    assert q_w.dtype == k_w.dtype == torch.float32 and q_w.numel() == Hq * D and k_w.numel() == Hkv * D and q_w.is_contiguous() and k_w.is_contiguous()
+    assert sums is None or (sums.dtype == torch.float32 and sums.shape == (T, 2) and sums.is_contiguous())
+    if K.checked.ENABLED:
+        K.checked.kv_write(slot_mapping, positions, k_cache.shape[0], k_cache.shape[1], rope_cache.shape[0] if rotary_dim else 0)
+    K._check(_lib().atlas_row_norm_kv_write(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), positions.data_ptr(),
+                                            rope_cache.data_ptr(), seq_positions.data_ptr(), q_w.data_ptr(), k_w.data_ptr(), K._ptr(sums),
+                                            k_cache.data_ptr(), v_cache.data_ptr(), slot_mapping.data_ptr(), T, Hq, Hkv, D, rotary_dim,
+                                            k_cache.shape[1], int(nq), int(nk), float(eps), float(temp), int(temp_every), f32, K._stream()),
+             "row_norm_kv_write")
+    return q
 
 
 # ----------------------------------------------------------------------------- 32-bit attention
@@ -285,7 +377,7 @@ def rope_kv_write_f32(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cac
     return q
 
 
-def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, sinks, softcap: float = 0.0):
+def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, sinks, softcap: float = 0.0, distance=None):
     T, Hq, D = q.shape
     K._dev(q)
     assert k_cache.dtype == torch.float32 and q.stride(2) == 1 and q.stride(1) == D
@@ -294,5 +386,5 @@ def attention_f32(q, k_cache, v_cache, batch, scale, window: int, chunk: int, si
     K._check(_lib().atlas_attn_f32(q.data_ptr(), q.stride(0), out.data_ptr(), Hq * D, k_cache.data_ptr(), v_cache.data_ptr(),
                                    bt.data_ptr(), bt.stride(0), batch.seq_lens.data_ptr(), batch.query_start_loc.data_ptr(),
                                    batch.num_seqs, T, float(scale), Hq, k_cache.shape[2], D, k_cache.shape[1], window, chunk,
-                                   K._ptr(sinks), softcap, K._stream()), "attn_f32")
+                                   K._ptr(sinks), softcap, K._ptr(distance), distance.shape[1] - 1 if distance is not None else 0, K._stream()), "attn_f32")
     return out

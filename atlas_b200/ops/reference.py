@@ -182,16 +182,36 @@ def qk_norm_rope_kv_write(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos
     return q
 
 
+def qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_norm_w, k_norm_w,
+                         eps: float, nq: int, nk: int, temp: float, temp_every: int, sums=None):
+    """See ``ops.qk_row_norm_kv_write``; everything up to the result in fp32."""
+    def unit(x, w, n, ss):
+        ss = x.float().square().sum((1, 2)) if ss is None else ss
+        return x.float() * torch.rsqrt(ss / n + eps)[:, None, None] * w.float().view(x.shape[1:])
+    qf = unit(q, q_norm_w, nq, None if sums is None else sums[:, 0])
+    kf = unit(k, k_norm_w, nk, None if sums is None else sums[:, 1])
+    qf, kf = (apply_rope(t, positions, rope_cache, rotary_dim) for t in (qf, kf))
+    steps = torch.div(seq_positions + 1, temp_every, rounding_mode="floor") + 1
+    qf = qf * (1.0 + temp * torch.log(steps.float()))[:, None, None]
+    ok = slot_mapping >= 0
+    slots, bs = slot_mapping[ok].long(), k_cache.shape[1]
+    k_cache[slots // bs, slots % bs] = kf[ok].to(k_cache.dtype)
+    v_cache[slots // bs, slots % bs] = v[ok].to(v_cache.dtype)
+    return qf.to(q.dtype)
+
+
 # ----------------------------------------------------------------------------- attention
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
                     block_tables: torch.Tensor, seq_lens: torch.Tensor, query_start_loc: torch.Tensor,
                     scale: float, k_scale: float = 1.0, v_scale: float = 1.0,
                     sliding_window: Optional[int] = None, chunk: int = 0,
-                    sinks: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+                    sinks: Optional[torch.Tensor] = None, softcap: float = 0.0,
+                    distance: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention of new query rows over the paged cache (prefill chunks and decode alike).
 
     ``chunk`` > 0 limits a row to keys of its own ``chunk``-token block (counted from the sequence's first token);
-    ``sinks [Hq]`` adds ``exp(sink)`` to every row's softmax denominator; ``softcap`` > 0 bounds the scores.
+    ``sinks [Hq]`` adds ``exp(sink)`` to every row's softmax denominator; ``softcap`` > 0 bounds the scores; ``distance
+    [Hq, n]`` is added to them by the key's distance, its last column from there on.
 
     Sequence ``b`` owns query rows ``query_start_loc[b]:query_start_loc[b+1]``; its last row sits
     at position ``seq_lens[b]-1``.  ``q [T,Hq,D]`` -> ``out [T,Hq,D]``.
@@ -217,6 +237,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             s = softcap * torch.tanh(s / softcap)
         qpos = torch.arange(L - ql, L, device=q.device)[:, None]
         kpos = torch.arange(L, device=q.device)[None, :]
+        if distance is not None:
+            back = (qpos - kpos).clamp(0, distance.shape[1] - 1)
+            s = s + distance.view(Hkv, G, -1)[:, :, back]
         mask = kpos <= qpos
         if sliding_window:
             mask &= kpos > qpos - sliding_window
@@ -338,7 +361,7 @@ def latent_attention(q, cache, rp: int, block_tables, seq_lens, query_start_loc,
     return out
 
 
-def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool):
+def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool, step=None):
     """See ``ops.add_normed``."""
     if hasattr(delta.y, "slot_of"):
         e = delta.y
@@ -346,10 +369,15 @@ def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool)
         slots = e.slot_of.view(T, k).long()
         picked = e.y.float()[slots.clamp_min(0)] * (slots >= 0)[..., None]
         y, dtype = (picked * e.w[..., None]).sum(1), e.y.dtype
+        y = y if e.extra is None else y + e.extra.float()
     else:
         y, dtype = delta.y.float(), delta.y.dtype
     unit = lambda t, w: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + 1.0 if plus_one else w.float())
-    x = y.clone() if delta.norm is None else stream + unit(y, delta.norm)
+    if stream is None:
+        x = y * delta.scale
+    else:
+        x = stream + (y if delta.norm is None else unit(y, delta.norm))
+    x = x if step is None else x + step
     if write and stream is not None:
         stream.copy_(x)
     h = x if out_norm is None else unit(x, out_norm)
@@ -357,10 +385,13 @@ def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool)
 
 
 # ----------------------------------------------------------------------------- activations
-def clamped_glu(gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+def gated_unit(gate_up: torch.Tensor, unit: Tuple[float, float, float], paired: bool = False) -> torch.Tensor:
+    """See ``ops.gated_unit_act``."""
+    limit, alpha, shift = unit
     i = gate_up.shape[-1] // 2
-    g, u = gate_up[..., :i].float().clamp(max=limit), gate_up[..., i:].float().clamp(-limit, limit)
-    return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(gate_up.dtype)
+    g, u = (gate_up[..., 0::2], gate_up[..., 1::2]) if paired else (gate_up[..., :i], gate_up[..., i:])
+    g, u = g.float().clamp(max=limit), u.float().clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + shift)).to(gate_up.dtype)
 
 
 def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
@@ -443,19 +474,23 @@ def _topk_low_ties(x: torch.Tensor, k: int) -> torch.Tensor:
     return torch.sort(x, dim=-1, descending=True, stable=True).indices[..., :k]
 
 
-def expert_act(h: torch.Tensor, activation: str) -> torch.Tensor:
-    """``silu_glu``: silu(gate) * up of ``[gate | up]``; ``relu2``: squared relu of a single up projection."""
+def expert_act(h: torch.Tensor, activation: str, unit: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
+    """``silu_glu``: silu(gate) * up of ``[gate | up]``; ``relu2``: squared relu of a single up projection; ``clamped_glu``: the
+    gated unit ``(limit, alpha, shift)`` of alternating gate and up columns."""
     if activation == "relu2":
         return torch.relu(h).square()
+    if activation == "clamped_glu":
+        return gated_unit(h, unit, paired=True)
     i = h.shape[-1] // 2
     return F.silu(h[..., :i]) * h[..., i:]
 
 
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
-                topk_ids: torch.Tensor, expert_lo: int = 0, activation: str = "silu_glu") -> torch.Tensor:
+                topk_ids: torch.Tensor, expert_lo: int = 0, activation: str = "silu_glu",
+                unit: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
     """Dense-math MoE over local experts ``[expert_lo, expert_lo+E_local)``.
 
-    ``w13 [E,2I,H]`` (gate rows then up rows; ``relu2``: ``[E,I,H]``), ``w2 [E,H,I]`` already dequantized.
+    ``w13 [E,2I,H]`` (gate rows then up rows; ``relu2``: ``[E,I,H]``; ``clamped_glu``: alternating), ``w2 [E,H,I]`` already dequantized.
     Tokens routed to non-local experts contribute zero (their owner rank adds them).
     """
     T, H = x.shape
@@ -469,7 +504,7 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
             continue
         wgt = (topk_w * sel).sum(-1)[tok]
         h = xf[tok] @ w13[e].float().t()
-        a = expert_act(h, activation).to(x.dtype).float()
+        a = expert_act(h, activation, unit).to(x.dtype).float()
         y = a @ w2[e].float().t()
         out.index_add_(0, tok, y * wgt[:, None])
     return out.to(x.dtype)
@@ -494,6 +529,22 @@ def causal_conv1d(x: torch.Tensor, conv_state: torch.Tensor, weight: torch.Tenso
         y = F.silu(y)
     new_state = full[full.shape[0] - (W - 1):].t().contiguous().to(conv_state.dtype)
     return y.to(x.dtype), new_state
+
+
+def rglru_gates(u, zr, zi, lam):
+    """RG-LRU: decay ``a`` and drive ``sqrt(1 - a^2) i u`` of every row and channel in fp32, from the raw gates ``zr`` / ``zi``
+    (biases included): ``log a = -8 sigmoid(zr) softplus(lam)``, ``i = sigmoid(zi)``."""
+    log_a = -8.0 * torch.sigmoid(zr.float()) * F.softplus(lam.float())
+    return torch.exp(log_a), torch.sqrt(-torch.expm1(2.0 * log_a)) * torch.sigmoid(zi.float()) * u.float()
+
+
+def linear_recurrence(a, drive, h):
+    """``h_t = a_t h_(t-1) + drive_t`` row by row: every state ``[T, C]`` (the last one carries on)."""
+    out = []
+    for t in range(a.shape[0]):
+        h = a[t] * h + drive[t]
+        out.append(h)
+    return torch.stack(out)
 
 
 def gdn_gates(a: torch.Tensor, b: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor):

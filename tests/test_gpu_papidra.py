@@ -84,7 +84,7 @@ def test_clamped_glu_meets_its_limits(dtype, n):
     from atlas_b200 import ops
     gu = rnd(6, 2 * n, std=3.0).to(dtype)
     for limit in (0.5, 1.0, 7.0):
-        close(ops.clamped_glu_act(gu.cuda(), limit, 1.702).x, O.clamped_glu(gu[:, :n].double(), gu[:, n:].double(), limit), dtype)
+        close(ops.gated_unit_act(gu.cuda(), (limit, 1.702, 1.0)).x, O.clamped_glu(gu[:, :n].double(), gu[:, n:].double(), limit), dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
