@@ -42,11 +42,11 @@ def distance_bucket(n: int, rows: int, reach: int) -> int:
 
 
 def distance_table(rel: torch.Tensor, reach: int) -> torch.Tensor:
-    """``rel [rows, heads]`` per bucket -> fp32 ``[heads, reach + 1]`` per distance; farther keys share the last column."""
+    """``rel [rows, heads]`` per bucket -> fp32 ``[heads, n]`` per distance; keys from ``n - 1`` tokens on share the last column."""
     rows = rel.shape[0]
-    if rows % 2 or rows < 2 or reach <= rows // 2:
+    if rows < 2 or reach < 1:
         raise ValueError(f"a distance table of {rows} rows does not reach {reach} tokens")
-    idx = torch.tensor([distance_bucket(n, rows, reach) for n in range(reach + 1)], device=rel.device)
+    idx = torch.tensor([distance_bucket(n, rows, reach) for n in range(max(reach, rows // 2) + 1)], device=rel.device)
     return rel.float()[idx].t().contiguous()
 
 
@@ -68,7 +68,7 @@ class Attention:
         self.sinks: Optional[torch.Tensor] = None       # [hq] fp32: extra term exp(sink) of the softmax denominator
         self.softcap = cfg.attn_softcap     # > 0: scores are bounded before the softmax
         self.norm_plus_one = cfg.norm_plus_one if cfg.qk_norm_plus_one is None else cfg.qk_norm_plus_one
-        self.distance: Optional[torch.Tensor] = None    # [hq, reach + 1] fp32: bias of a score by the distance of its key
+        self.distance: Optional[torch.Tensor] = None    # [hq, n] fp32: bias of a score by the distance of its key
         self.gated_qkv: Optional[TailLinear] = None     # head gates: q | k | v with one gate number per head as an fp32 tail
         # models with per-layer attention kinds (Gemma): only "sliding_attention" layers use the window
         kinds = cfg.layer_types if (cfg.family != "hybrid" and cfg.layer_types) else None
