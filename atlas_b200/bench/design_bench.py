@@ -1,13 +1,14 @@
 """Prefill and decode throughput of a design's layers beside the closest other model at equal size, and the rooflines of their
 kernels.
 
-    python bench.py --design papidra|tomizen    # or: python -m atlas_b200.bench.design_bench --design ...
+    python bench.py --design papidra|tomizen|kenovik    # or: python -m atlas_b200.bench.design_bench --design ...
 
 ``papidra`` beside Nemotron-H: the same width, feed-forward size, attention heads, Mamba-2 heads, vocabulary and cache dtype.  One
 period is, for Papidra, a WKV layer and a layer with attention beside Mamba-2 plus a feed-forward; for Nemotron-H the blocks with
 the same work: Mamba-2, attention, Mamba-2, MLP.
 
-``tomizen`` (tomizen_bench.py) beside Qwen3-Next, and its latent attention beside DeepSeek's.
+``tomizen`` (tomizen_bench.py) beside Qwen3-Next, and its latent attention beside DeepSeek's; ``kenovik`` (kenovik_bench.py) beside
+Qwen3-Next.
 
 All with random bf16 weights.  Steps are timed with CUDA events around a captured step (L2 flushed in between), kernels the same
 way one by one.
@@ -163,9 +164,10 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
 
 def designs() -> dict:
     """name -> (name of the model beside it, sizes, configuration of both by size, kernel table, layers)"""
-    from . import tomizen_bench as T
+    from . import kenovik_bench as V, tomizen_bench as T
     return {"papidra": ("nemotron_h", SIZES, papidra, nemotron, kernel_table, f"{PERIODS} periods"),
-            "tomizen": ("qwen3_next", T.SIZES, T.tomizen, T.beside, T.kernel_table, "4 layers")}
+            "tomizen": ("qwen3_next", T.SIZES, T.tomizen, T.beside, T.kernel_table, "4 layers"),
+            "kenovik": ("qwen3_next", V.SIZES, V.kenovik, V.beside, V.kernel_table, "4 layers")}
 
 
 def run(sizes: Optional[List[str]] = None, kernels: bool = True, design: str = "papidra") -> dict:
@@ -195,13 +197,13 @@ def report(res: dict) -> str:
             w = r[b][key]
             lines.append(f"  {key:<18} {a} {v['ms']:>9} ms {v['tok_s']:>9} tok/s    {b} {w['ms']:>9} ms {w['tok_s']:>9} tok/s")
         for k in r.get("kernels", ()):
-            lines.append(f"  {k['pair']:<11} {k['kernel']:<38} {k['shape']:<20} {k['us']:>9} us  {k['roofline']:.3f} of roofline")
+            lines.append(f"  {k['pair']:<12} {k['kernel']:<46} {k['shape']:<20} {k['us']:>9} us  {k['roofline']:.3f} of roofline")
     return "\n".join(lines)
 
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="papidra", choices=["papidra", "tomizen"])
+    ap.add_argument("--design", default="papidra", choices=["papidra", "tomizen", "kenovik"])
     ap.add_argument("--sizes", default="", help="widths (default: all of the design)")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--out")

@@ -619,6 +619,8 @@ def _kenovik_ff(mlp: Dict[str, Any]) -> Dict[str, Any]:
     groups = r.get("groups") or {"count": 1, "keep": 1}
     if int(r["experts"]) % int(groups["count"]):
         raise ValueError(f"{r['experts']} experts do not form {groups['count']} equal groups")
+    if int(r["top"]) > int(r["experts"]) // int(groups["count"]) * int(groups["keep"]):
+        raise ValueError(f"{r['top']} experts per token do not fit into {groups['keep']} of {groups['count']} groups")
     return {"num_experts": int(r["experts"]), "num_experts_per_tok": int(r["top"]), "moe_intermediate_size": int(mlp["expert"]["ff"]),
             "mlp_activation": "clamped_glu", "glu_limit": float(mlp["expert"]["limit"]), "norm_topk_prob": True,
             "router_scoring": "sigmoid", "router_selection_bias": True, "router_f32": True, "routed_scaling_factor": float(r["scale"]),

@@ -8,6 +8,8 @@
 //                       tensor-core tiles do not take
 // Reference ops replaced: kernels/gb10/common/{moe_topk,moe_topk_sigmoid,moe_permute}.cu
 // (moe_count_experts, moe_sort_by_expert, moe_permute_tokens, moe_build_tile_worklist, moe_unpermute_reduce).
+#include <type_traits>
+
 #include "common.cuh"
 #include "host_api.h"
 
@@ -39,15 +41,14 @@ __device__ __forceinline__ float route_score(float x, float mx, int mode, const 
   return route_exp(x - mx, kind);
 }
 
-// one warp per token; E <= 1024
-template <typename T>
+// one warp per token; E <= 32 * kMaxPer
+template <typename T, int kMaxPer>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int k, int norm, RouteOpts o,
                  float* __restrict__ w_out, int* __restrict__ id_out) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
   if (t >= T_) return;
-  constexpr int kMaxPer = 32;
   float v[kMaxPer];            // unbiased scores (weights)
   float sel[kMaxPer];          // selection keys
   const int per = (E + 31) / 32;
@@ -92,6 +93,9 @@ moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int 
 
   if (o.n_group > 1 && o.topk_group > 0 && o.topk_group < o.n_group) {
     const int gsz = E / o.n_group;
+    int grp[kMaxPer];
+#pragma unroll
+    for (int i = 0; i < kMaxPer; ++i) grp[i] = (i * 32 + lane) / gsz;
     float my_g = -INFINITY;                    // lane g holds the score of group g
 #pragma unroll 1
     for (int g = 0; g < o.n_group; ++g) {
@@ -99,7 +103,7 @@ moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int 
 #pragma unroll
       for (int i = 0; i < kMaxPer; ++i) {
         const int e = i * 32 + lane;
-        if (i < per && e < E && e / gsz == g) {
+        if (i < per && e < E && grp[i] == g) {
           const float x = sel[i];
           if (x > a) { b = a; a = x; } else if (x > b) { b = x; }
         }
@@ -128,7 +132,7 @@ moe_route_kernel(const T* __restrict__ logits, long long ld, int T_, int E, int 
 #pragma unroll
     for (int i = 0; i < kMaxPer; ++i) {
       const int e = i * 32 + lane;
-      if (i < per && e < E && !((keep >> (e / gsz)) & 1u)) sel[i] = -INFINITY;
+      if (i < per && e < E && !((keep >> grp[i]) & 1u)) sel[i] = -INFINITY;
     }
   }
 
@@ -420,8 +424,15 @@ static int route_launch(const void* logits, long long ld, int is_bf16, int T, in
   if (o.hash_table && !o.token_ids) return -1;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   const int grid = (T + 3) / 4;
-  if (is_bf16) moe_route_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(reinterpret_cast<const __nv_bfloat16*>(logits), ld, T, E, k, norm, o, w_out, id_out);
-  else moe_route_kernel<float><<<grid, 128, 0, st>>>(reinterpret_cast<const float*>(logits), ld, T, E, k, norm, o, w_out, id_out);
+  auto run = [&](auto kern, auto* lg) { kern<<<grid, 128, 0, st>>>(lg, ld, T, E, k, norm, o, w_out, id_out); };
+  auto pick = [&](auto* lg) {
+    using L = std::remove_cv_t<std::remove_pointer_t<decltype(lg)>>;
+    if (E <= 64) run(moe_route_kernel<L, 2>, lg);
+    else if (E <= 256) run(moe_route_kernel<L, 8>, lg);
+    else run(moe_route_kernel<L, 32>, lg);
+  };
+  if (is_bf16) pick(reinterpret_cast<const __nv_bfloat16*>(logits));
+  else pick(reinterpret_cast<const float*>(logits));
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }
 

@@ -119,6 +119,48 @@ conv1d_state_kernel(const T* __restrict__ x, long long ldx, int C, int W, T* sta
   if (n > 0) window_after(n, slot);
 }
 
+// the same for bf16 windows of three inputs, eight channels per thread
+__global__ void __launch_bounds__(128)
+conv1d_state4_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, int C, __nv_bfloat16* state, const int* __restrict__ query_start_loc,
+                     const int* __restrict__ state_slots, const unsigned char* __restrict__ has_state, const int* __restrict__ limit,
+                     const int* __restrict__ snap_rows, const int* __restrict__ snap_slots, int num_snaps_per_seq) {
+  chain_trigger();
+  chain_wait();
+  const int b = blockIdx.y, c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  if (c >= C) return;
+  const int q0 = query_start_loc[b], qlen = query_start_loc[b + 1] - q0;
+  const long long slot = state_slots[b];
+  union Window { uint4 v[3]; __nv_bfloat16 e[8][3]; };
+  union Row { uint4 v; __nv_bfloat16 e[8]; };
+  Window old;
+#pragma unroll
+  for (int i = 0; i < 3; ++i)
+    old.v[i] = has_state[b] ? reinterpret_cast<const uint4*>(state + (slot * C + c) * 3)[i] : make_uint4(0u, 0u, 0u, 0u);
+  auto window_after = [&](int n, long long dst) {
+    Row r[3];
+#pragma unroll
+    for (int i = 0; i < 3; ++i) {
+      const int src = n - 3 + i;
+      r[i].v = src >= 0 ? *reinterpret_cast<const uint4*>(x + (long long)(q0 + src) * ldx + c) : make_uint4(0u, 0u, 0u, 0u);
+    }
+    Window w;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      w.e[k][0] = n >= 3 ? r[0].e[k] : (n == 2 ? old.e[k][2] : old.e[k][1]);
+      w.e[k][1] = n >= 2 ? r[1].e[k] : old.e[k][2];
+      w.e[k][2] = r[2].e[k];
+    }
+#pragma unroll
+    for (int i = 0; i < 3; ++i) reinterpret_cast<uint4*>(state + (dst * C + c) * 3)[i] = w.v[i];
+  };
+  for (int s = 0; s < num_snaps_per_seq; ++s) {
+    const int n = snap_rows[b * num_snaps_per_seq + s];
+    if (n > 0 && n <= qlen) window_after(n, snap_slots[b * num_snaps_per_seq + s]);
+  }
+  const int n = limit ? limit[b] : qlen;
+  if (n > 0) window_after(n, slot);
+}
+
 template <typename T, int kTaps>
 static int launch_conv(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                        const int* seq, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
@@ -220,6 +262,11 @@ extern "C" int atlas_conv1d_state(const void* x, long long ldx, int C, int W, vo
   if (W < 1 || W > kMaxTaps) return -1;
   dim3 grid((C + 255) / 256, B);
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (!f32 && W == 4 && C % 8 == 0 && vec_ok<bf16, 8>(x, ldx) && vec_ok<bf16, 8>(state, 0)) {
+    launch_chain_if(true, conv1d_state4_kernel, dim3((C / 8 + 127) / 128, B), dim3(128), 0, st, reinterpret_cast<const bf16*>(x), ldx, C,
+                    reinterpret_cast<bf16*>(state), qsl, slots, has, limit, snap_rows, snap_slots, snaps);
+    return cudaGetLastError() == cudaSuccess ? 0 : -21;
+  }
   if (f32) launch_chain_if(true, conv1d_state_kernel<float>, grid, dim3(256), 0, st, reinterpret_cast<const float*>(x), ldx, C, W,
                            reinterpret_cast<float*>(state), qsl, slots, has, limit, snap_rows, snap_slots, snaps);
   else launch_chain_if(true, conv1d_state_kernel<bf16>, grid, dim3(256), 0, st, reinterpret_cast<const bf16*>(x), ldx, C, W,

@@ -240,7 +240,7 @@ def mlstm_commit(layer, k, v, raw, qlens, slots, has_state, state, num_accepted_
     _mlstm_run(layer, None, k, v, raw, meta, state, True)
 
 
-RGLRU_CHUNK = 64              # rows per chunk of the recurrence (kRgRows in csrc/rglru.cu)
+RGLRU_CHUNK = 32              # rows per chunk of the recurrence (kRgChunk in csrc/rglru.cu)
 RGLRU_TENSOR_CORES = True     # tests switch this off to compare the two forms
 
 

@@ -129,7 +129,7 @@ def test_experts_with_groups_and_a_shared_one(dtype, T, H, I, E, top, count, kee
 
 # ------------------------------------------------------------------------------------------------- RG-LRU
 LENS = [([1, 1, 1], [True, False, True]), ([37, 1, 2, 18], [False, True, True, False]), ([64, 65, 130], [True, True, False]),
-        ([2, 2], [True, False]), ([63, 1, 1, 300], [True, True, False, True])]
+        ([2, 2], [True, False]), ([63, 1, 1, 300], [True, True, False, True]), ([1] * 83, [i % 5 != 2 for i in range(83)])]
 
 
 def rglru_layer(C, blocks, taps, dtype, seed=0):
@@ -162,7 +162,7 @@ def rglru_plain(y, x, w, old, h):
 
 
 @pytest.mark.parametrize("form", ["tensor cores", "gate sums", "fp32"])
-@pytest.mark.parametrize("lens,live", LENS, ids=["decode", "mixed", "chunk edges", "two rows", "long"])
+@pytest.mark.parametrize("lens,live", LENS, ids=["decode", "mixed", "chunk edges", "two rows", "long", "wide decode"])
 @pytest.mark.parametrize("C,blocks,taps", [(8, 1, 4), (160, 2, 4), (128, 1, 1), (417, 3, 7), (45, 9, 2), (512, 2, 4), (300, 2, 3)])
 def test_rglru(form, lens, live, C, blocks, taps):
     """Windows and states carried in, unequal lengths across the kernel's chunks, decays from nearly one to nearly none."""
@@ -171,8 +171,9 @@ def test_rglru(form, lens, live, C, blocks, taps):
     m, w = rglru_layer(C, blocks, taps, dtype)
     T = sum(lens)
     yx = rnd(T, 2 * C, seed=11).to(dtype)
-    slots = [4, 1, 0, 2][:len(lens)]
-    c0, h0 = rnd(5, C, taps - 1, seed=12).to(dtype), rnd(5, C, seed=13)
+    slots = [4, 1, 0, 2][:len(lens)] if len(lens) < 5 else [(7 * i) % 97 for i in range(len(lens))]
+    n_slots = max(slots) + 1
+    c0, h0 = rnd(n_slots, C, taps - 1, seed=12).to(dtype), rnd(n_slots, C, seed=13)
     state = {"conv": c0.cuda(), "h": h0.cuda()}
     g = yx.cuda()
     y, x = g[:, :C], g[:, C:]
@@ -195,7 +196,7 @@ def test_rglru(form, lens, live, C, blocks, taps):
         if taps > 1:
             assert torch.equal(state["conv"][s].cpu(), torch.cat([old.T.to(dtype), yx[rows, C:].T], 1)[:, -(taps - 1):])
         t0 += n
-    for s in set(range(5)) - set(slots):
+    for s in set(range(n_slots)) - set(slots):
         assert torch.equal(state["h"][s].cpu(), h0[s]) and torch.equal(state["conv"][s].cpu(), c0[s])
 
 
