@@ -46,30 +46,33 @@ struct RgParams {
 ATLAS_DEVICE float rg_coef(float lam) {        // -8 softplus(lam)
   return -8.f * (fmaxf(lam, 0.f) + log1pf(expf(-fabsf(lam))));
 }
-// 1 - e^t for t <= 0: the Taylor sum near zero, where the difference would cancel
-ATLAS_DEVICE float one_minus_exp(float t, float e) {
-  const float s = -t * (1.f + t * 0.5f * (1.f + t * (1.f / 3.f) * (1.f + t * 0.25f * (1.f + t * 0.2f * (1.f + t * (1.f / 6.f))))));
-  return t > -0.25f ? s : 1.f - e;
-}
 ATLAS_DEVICE float approx_sqrt(float x) {
   float y;
   asm("sqrt.approx.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// The decay a as its distance m = 1 - a from one, and the drive d = sqrt(1 - a^2) i u with 1 - a^2 = m (2 - m).  Close to one, where
+// states live for thousands of rows, m keeps the digits that a rounded a loses (and would lose the same way in every row): near
+// zero it is the Taylor sum of 1 - e^t.
 template <bool kFast>
-ATLAS_DEVICE void rg_gates(float zr, float zi, float u, float coef, float& a, float& d) {
+ATLAS_DEVICE void rg_gates(float zr, float zi, float u, float coef, float& m, float& d) {
+  float t, i;
   if (kFast) {
     // both sigmoids from one reciprocal; below -60 a gate is shut
     const float er = 1.f + __expf(-fmaxf(zr, -60.f)), ei = 1.f + __expf(-fmaxf(zi, -60.f)), inv = __fdividef(1.f, er * ei);
-    const float la = coef * (ei * inv);
-    a = __expf(la);
-    d = approx_sqrt(one_minus_exp(2.f * la, a * a)) * (er * inv) * u;
+    t = coef * (ei * inv);
+    i = er * inv;
   } else {
-    const float la = coef / (1.f + expf(-zr));
-    a = expf(la);
-    d = sqrtf(one_minus_exp(2.f * la, a * a)) * u / (1.f + expf(-zi));
+    t = coef / (1.f + expf(-zr));
+    i = 1.f / (1.f + expf(-zi));
   }
+  const float near = -t * (1.f + t * 0.5f * (1.f + t * (1.f / 3.f) * (1.f + t * 0.25f * (1.f + t * 0.2f * (1.f + t * (1.f / 6.f))))));
+  m = t > -0.25f ? near : 1.f - (kFast ? __expf(t) : expf(t));
+  const float gain = m * (2.f - m);
+  d = (kFast ? approx_sqrt(gain) : sqrtf(gain)) * i * u;
 }
+// a x + d
+ATLAS_DEVICE float decayed(float m, float x, float d) { return fmaf(-m, x, x + d); }
 // z (1 + tanh k) / 2 = z sigmoid(2 k)
 template <bool kFast>
 ATLAS_DEVICE float gelu_tanh1(float z) {
@@ -363,17 +366,17 @@ rglru_tc_kernel(const RgParams<bf16> p) {
       tmem_ld_32x32b_x8(ta + g * kG, r);
       tmem_ld_32x32b_x8(ta + kRows + g * kG, q);
       tmem_ld_wait();
-      float a[kG], d[kG];
+      float dm[kG], d[kG];
 #pragma unroll
       for (int j = 0; j < kG; ++j)
-        rg_gates<true>(__uint_as_float(r[j]) + br, __uint_as_float(q[j]) + bi, input(row0 + g * kG + j), coef, a[j], d[j]);
+        rg_gates<true>(__uint_as_float(r[j]) + br, __uint_as_float(q[j]) + bi, input(row0 + g * kG + j), coef, dm[j], d[j]);
       const long long t = t0 + row0 + g * kG;
       if constexpr (kStep) {
 #pragma unroll
         for (int j = 0; j < kG; ++j) {
           const int row = row0 + g * kG + j;
           if (!mine || s_rel[row] < 0) continue;
-          const float s = fmaf(a[j], hv[j], d[j]);
+          const float s = decayed(dm[j], hv[j], d[j]);
           if (p.commit) p.h[(long long)s_slot[row] * p.C + c] = s;
           p.out[(t + j) * p.ldo + c] = from_f32<bf16>(s * gelu_tanh1<true>(to_f32(yv[j])));
         }
@@ -381,8 +384,8 @@ rglru_tc_kernel(const RgParams<bf16> p) {
       } else if (smooth) {
 #pragma unroll
         for (int j = 0; j < kG; ++j) {
-          S = fmaf(a[j], S, d[j]);
-          P *= a[j];
+          S = decayed(dm[j], S, d[j]);
+          P = decayed(dm[j], P, 0.f);
           if (mine) {
             p.P[(t + j) * p.C + c] = P;
             p.S[(t + j) * p.C + c] = S;
@@ -394,11 +397,11 @@ rglru_tc_kernel(const RgParams<bf16> p) {
           const int row = row0 + g * kG + j, rel = s_rel[row];
           if (rel < 0 || !mine) continue;
           if (rel == 0) {
-            S = s_live[row] ? fmaf(a[j], p.h[(long long)s_slot[row] * p.C + c], d[j]) : d[j];
+            S = s_live[row] ? decayed(dm[j], p.h[(long long)s_slot[row] * p.C + c], d[j]) : d[j];
             P = 0.f;
           } else {
-            S = fmaf(a[j], S, d[j]);
-            P *= a[j];
+            S = decayed(dm[j], S, d[j]);
+            P = decayed(dm[j], P, 0.f);
           }
           p.P[(t + j) * p.C + c] = P;
           p.S[(t + j) * p.C + c] = S;
@@ -433,14 +436,14 @@ rglru_local_kernel(const RgParams<T> p) {
   const int t1 = min(p.rows, (chunk + 1) * kRgChunk);
   for (int t = chunk * kRgChunk; t < t1; ++t) {
     const int b = p.seq_of[t];
-    float a, d;
-    rg_gates<false>(p.zr[zo + t * p.z_row] + br, p.zi[zo + t * p.z_row] + bi, to_f32(p.u[t * p.ldu + c]), coef, a, d);
+    float dm, d;
+    rg_gates<false>(p.zr[zo + t * p.z_row] + br, p.zi[zo + t * p.z_row] + bi, to_f32(p.u[t * p.ldu + c]), coef, dm, d);
     if (t == p.qsl[b]) {
-      S = p.has[b] ? fmaf(a, p.h[(long long)p.slots[b] * p.C + c], d) : d;
+      S = p.has[b] ? decayed(dm, p.h[(long long)p.slots[b] * p.C + c], d) : d;
       P = 0.f;
     } else {
-      S = fmaf(a, S, d);
-      P *= a;
+      S = decayed(dm, S, d);
+      P = decayed(dm, P, 0.f);
     }
     p.P[(long long)t * p.C + c] = P;
     p.S[(long long)t * p.C + c] = S;
