@@ -163,7 +163,7 @@ def rglru_plain(y, x, w, old, h):
 
 @pytest.mark.parametrize("form", ["tensor cores", "gate sums", "fp32"])
 @pytest.mark.parametrize("lens,live", LENS, ids=["decode", "mixed", "chunk edges", "two rows", "long", "wide decode"])
-@pytest.mark.parametrize("C,blocks,taps", [(8, 1, 4), (160, 2, 4), (128, 1, 1), (417, 3, 7), (45, 9, 2), (512, 2, 4), (300, 2, 3)])
+@pytest.mark.parametrize("C,blocks,taps", [(8, 1, 4), (160, 2, 4), (128, 1, 1), (417, 3, 7), (45, 9, 2), (512, 2, 4), (300, 2, 3), (1024, 1, 4), (1400, 1, 4)])
 def test_rglru(form, lens, live, C, blocks, taps):
     """Windows and states carried in, unequal lengths across the kernel's chunks, decays from nearly one to nearly none."""
     from atlas_b200.ops import cuda as K, cuda_recurrent as R
@@ -198,6 +198,26 @@ def test_rglru(form, lens, live, C, blocks, taps):
         t0 += n
     for s in set(range(n_slots)) - set(slots):
         assert torch.equal(state["h"][s].cpu(), h0[s]) and torch.equal(state["conv"][s].cpu(), c0[s])
+
+
+def test_rglru_long_memories():
+    """Decays so close to one that a state lives for thousands of rows: the error stays that of a few roundings instead of growing
+    with the rows, in one portion and row by row."""
+    from atlas_b200.ops import cuda as K
+    C, T = 32, 6000
+    m, w = rglru_layer(C, 1, 4, torch.float32)
+    w["lam"] = torch.linspace(-13.0, -7.0, C, dtype=torch.float64)
+    m.lam = w["lam"].float().cuda()
+    yx = rnd(T, 2 * C, seed=1)
+    yx[:, C:] += 1.0
+    _, states = rglru_plain(yx[:, :C].double(), yx[:, C:].double(), w, torch.zeros(3, C, dtype=torch.float64), torch.zeros(C, dtype=torch.float64))
+    g = yx.cuda()
+    for cuts in ([T], [100] * 59 + [1] * 100):
+        state, t = {"conv": torch.zeros(1, C, 3).cuda(), "h": torch.zeros(1, C).cuda()}, 0
+        for n in cuts:
+            K.rglru_forward(m, g[t:t + n, :C], g[t:t + n, C:], batch_of([n], [t > 0], [0]), state, True)
+            t += n
+        assert ((state["h"][0].cpu() - states[-1]).abs() / states[-1].abs().clamp_min(1.0)).max() < 4e-6
 
 
 @pytest.mark.parametrize("form", ["tensor cores", "gate sums", "fp32"])
