@@ -68,6 +68,7 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
     mlp_a, mlp_b = DenseMLP(ours.for_layer(0), p, "dense", paired=True), DenseMLP(qwen, p, "dense", activation="silu_glu")
     for m in (lru, gd, moe_a, moe_b, mlp_a, mlp_b):
         m.init_random(gen, 0.02, bf, dev)
+    moe_a.fuse_inputs()
     for T, nseq in ((8192, 8), (8192, 1), (128, 128), (1, 1)):
         decode = T == nseq
         shape, lens = f"{T} rows, {nseq} seq", [T // nseq] * nseq
@@ -119,8 +120,8 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
         add("router", "fp32 logits, sigmoid, groups", shape, lambda: route(moe_a, True), T * W * 2 + E * W * 2)
         add("router", "bf16 logits, softmax (existing)", shape, lambda: route(moe_b, False), T * W * 2 + E * W * 2)
         eb, ef = T * W * 4 + (used + 1) * 6 * I * W, 6.0 * T * (top + 1) * W * I
-        add("experts", "clamped experts + shared, rows", shape, lambda: moe_a.forward(act, rows_ok=True), eb + T * top * W * 2, ef)
-        add("experts", "swiglu experts + shared, combined (existing)", shape, lambda: moe_b.forward(act), eb, ef)
+        add("experts", "router, clamped experts + shared, rows", shape, lambda: moe_a.forward(act, rows_ok=True), eb + T * top * W * 2, ef)
+        add("experts", "router, swiglu experts + shared (existing)", shape, lambda: moe_b.forward(act), eb, ef)
         # ---- attention
         (hq, hkv, d), ctx = s["attn"], 2048 if decode else 0
         per = (ctx + lens[0] + 15) // 16

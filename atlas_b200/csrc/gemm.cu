@@ -1029,6 +1029,13 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 #pragma unroll
           for (int j = 0; j < HALF; j += 16) {
             const int n = n_base + j;
+            if (p.tail != nullptr && n >= p.tail_col) {          // tail_col is a multiple of 16 here
+              float* trow = p.tail + (size_t)m * p.tail_ld - p.tail_col;
+#pragma unroll
+              for (int i = 0; i < 16; ++i)
+                if (n + i < p.N) trow[n + i] = acc[j + i];
+              continue;
+            }
             float o[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) o[i] = gated_unit_fast(acc[j + 2 * i], acc[j + 2 * i + 1], p.unit);
@@ -1408,13 +1415,16 @@ extern "C" int atlas_gemm_tail(const void* A, const void* B, void* C, float* tai
 }
 
 // bf16 GEMM with a bias row (fp32 [N] or null) and / or an activation in its epilogue: act 0 none, 1 relu squared, 2 gated
-// unit (common.cuh) of alternating gate and up columns (C has N / 2 columns).
-extern "C" int atlas_gemm_bias_act(const void* A, const void* B, void* C, const float* bias, int act, float glu_limit, float glu_alpha, float glu_shift, int M,
+// unit (common.cuh) of alternating gate and up columns (C has N / 2 columns).  tail (null = off): columns from n_main on leave as the
+// fp32 sums (with the bias, without the activation); n_main is a multiple of 16 then.
+extern "C" int atlas_gemm_bias_act(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, const float* bias, int act,
+                                   float glu_limit, float glu_alpha, float glu_shift, int M,
                                    int N, int K, long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace,
                                    int* counters, int num_sms, unsigned long long* status, void* stream) {
-  if (act < 0 || act > 2 || (act == 2 && N % 2)) return -46;
+  if (act < 0 || act > 2 || (act == 2 && !tail && N % 2)) return -46;
+  if (tail && (act != 2 || n_main % 16 || n_main < 0 || n_main >= N || tail_ld < N - n_main)) return -47;
   return gemm_impl(0, A, B, C, nullptr, 0, 0, nullptr, 0, M, N, K, lda, ldb, ldc, block_n, splits, workspace, counters, num_sms, status,
-                   stream, nullptr, nullptr, 0, nullptr, nullptr, 0, 0, bias, act, glu_limit, glu_alpha, glu_shift);
+                   stream, nullptr, nullptr, 0, nullptr, tail, tail_ld, tail ? n_main : 0, bias, act, glu_limit, glu_alpha, glu_shift);
 }
 
 // All-gather -> GEMM: the rows of A (and their scales) are written into this rank's memory by the ranks that own them;

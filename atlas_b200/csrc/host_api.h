@@ -88,8 +88,8 @@ int atlas_gemm_grouped(int kind, const void* A, const void* B, void* C, const fl
                        const float* b_scale, int max_rows, int N, int K, int E, long long lda, long long ldb,
                        long long ldc, int block_n, const int* tile_expert, const int* num_m_tiles, int num_sms,
                        unsigned long long* status, void* stream, int act, float glu_limit, float glu_alpha, float glu_shift);
-int atlas_gemm_bias_act(const void* A, const void* B, void* C, const float* bias, int act, float glu_limit, float glu_alpha, float glu_shift, int M, int N, int K,
-                        long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,
+int atlas_gemm_bias_act(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, const float* bias, int act,
+                        float glu_limit, float glu_alpha, float glu_shift, int M, int N, int K, long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,
                         unsigned long long* status, void* stream);
 int atlas_gemm_tail(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, int M, int N, int K, long long lda,
                     long long ldb, long long ldc, int block_n, int splits, float* workspace, int* counters, int num_sms,

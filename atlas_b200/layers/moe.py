@@ -110,6 +110,7 @@ class MoE:
         self.shared_gate: Optional[torch.Tensor] = None
         self.router_bias: Optional[torch.Tensor] = None      # fp32 [E]: selection-only correction (e_score_correction_bias)
         self.hash_table: Optional[torch.Tensor] = None       # int32 [vocab, k]: static token-id -> expert ids
+        self.fused_in: Optional[LinearWeight] = None         # the shared expert's gate / up rows and the router's in one product
         self.lora = None                    # lora.LoraSet shared by the model's layers
         self.lora_prefix = ""               # e.g. "layers.3.mlp."
         if cfg.shared_expert_intermediate_size:
@@ -130,6 +131,18 @@ class MoE:
             # whole GEMM tiles: hidden channels of zero weights stay zero through the activation
             w13, w2 = F.pad(w13, (0, 0, 0, pad * w13.shape[1] // w2.shape[2])), F.pad(w2, (0, pad))
         self.experts = ExpertWeights.from_dense(w13, w2, self.expert_kind)
+
+    def fuse_inputs(self) -> None:
+        """One product for the shared expert's gated unit and the router's fp32 logits, where the kernels take both (bf16, rows in
+        whole 16s); the two weights become its halves."""
+        if self.fused_in is not None or self.shared is None or not (self.shared.paired and self.router_f32):
+            return
+        gu, r = self.shared.gate_up, self.router
+        if gu.kind != "dense" or not ops.on_gpu(gu.weight) or gu.weight.dtype != torch.bfloat16 or gu.weight.shape[0] % 16 or gu.weight.shape[1] % 8:
+            return
+        n = gu.weight.shape[0]
+        self.fused_in = LinearWeight("dense", torch.cat([gu.weight, r.weight], 0).contiguous())
+        gu.weight, r.weight = self.fused_in.weight[:n], self.fused_in.weight[n:]
 
     def init_random(self, gen, std, dtype, device) -> None:
         cfg = self.cfg
@@ -158,8 +171,13 @@ class MoE:
         """``rows_ok``: the caller takes the weighted sum itself, so the result may be an :class:`ops.ExpertRows`."""
         x = act.plain()
         cfg = self.cfg
-        logits = ops.linear_tail(x, self.router, 0)[1] if self.router_f32 else ops.linear(x, self.router)
         adapters = self.lora is not None and batch is not None and batch.adapter_rows is not None and bool(self.lora_prefix)
+        shared_rows = None
+        if self.fused_in is not None and not adapters and ops.on_gpu(x):
+            a, logits = ops.linear_gated_unit_tail(act, self.fused_in, self.shared.unit, self.shared.gate_up.weight.shape[0])
+            shared_rows = ops.linear(a, self.shared.down)
+        else:
+            logits = ops.linear_tail(x, self.router, 0)[1] if self.router_f32 else ops.linear(x, self.router)
         if adapters:
             add_delta(logits, self.lora, self.lora_prefix + "gate", x, batch)
         topk_w, topk_ids = ops.moe_route(logits, self.top_k, cfg.norm_topk_prob, cfg.router_scoring, self.router_bias,
@@ -170,14 +188,14 @@ class MoE:
             y = ops.cuda_ops().moe_forward(x, topk_w, topk_ids, self.experts, self.e_lo, self.pctx, self.ep_mode,
                                            activation=self.activation, rows_ok=rows_ok, unit=self.unit)
             if rows_ok:
-                y.extra = None if self.shared is None else self.shared.forward(act, reduce=False, batch=batch)
+                y.extra = shared_rows if shared_rows is not None or self.shared is None else self.shared.forward(act, reduce=False, batch=batch)
                 return y
         else:
             y = self._forward_ref(x, topk_w, topk_ids)
         if adapters:
             y = self._adapter_rows_forward(x, y, topk_w, topk_ids, batch.adapter_rows)
         if self.shared is not None:
-            s = self.shared.forward(act, reduce=False, batch=batch)
+            s = shared_rows if shared_rows is not None else self.shared.forward(act, reduce=False, batch=batch)
             if (self.shared_gate is not None and ops.on_gpu(x) and x.dtype == torch.bfloat16 and y.dtype == torch.bfloat16
                     and self.shared_gate.dtype == torch.bfloat16 and x.shape[1] % 8 == 0 and y.is_contiguous()):
                 return ops.cuda_ops().shared_expert_blend(y if y._base is None else y.clone(), s, x, self.shared_gate)

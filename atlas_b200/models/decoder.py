@@ -546,6 +546,9 @@ class DecoderLM:
             for l in self.layers:
                 if l.kind == "attention" and getattr(l.mixer, "local", False):
                     l.rope_override = local
+        for l in self.layers:
+            if l.is_moe:
+                l.ffn.fuse_inputs()
         tables: Dict[str, torch.Tensor] = {}
         for l in self.layers if cfg.layer_specs else ():
             if attention_of(l) is not None:

@@ -233,6 +233,13 @@ def linear_gated_unit(a, w: LinearWeight, unit: Tuple[float, float, float]) -> A
     return gated_unit_act(linear(a, w), unit, paired=True)
 
 
+def linear_gated_unit_tail(a, w: LinearWeight, unit: Tuple[float, float, float], n_main: int) -> Tuple[Act, torch.Tensor]:
+    """:func:`linear_gated_unit` of the first ``n_main`` rows and, from the same product, the others as fp32 sums (bf16 weights on a
+    GPU, ``n_main`` a multiple of 16)."""
+    y, tail = cuda_ops().gemm_bf16(a.plain() if isinstance(a, Act) else a, w.weight, unit=unit, n_main=n_main)
+    return Act(x=y), tail
+
+
 def tanh_(x: torch.Tensor) -> torch.Tensor:
     """``tanh`` in place."""
     if on_gpu(x):

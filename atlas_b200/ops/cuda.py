@@ -444,8 +444,11 @@ def gemm_fp8_fused(xq, xs, wq, ws, mode: int = 0, out=None, residual=None, norm_
     return res
 
 
-def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.Tensor] = None, unit: Optional[Tuple[float, float, float]] = None) -> torch.Tensor:
-    """``x @ w^T (+ bias)``; with ``unit = (limit, alpha, shift)`` the gated unit of alternating gate and up columns, ``[M, N / 2]``."""
+def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.Tensor] = None, unit: Optional[Tuple[float, float, float]] = None,
+              n_main: Optional[int] = None):
+    """``x @ w^T (+ bias)``; with ``unit = (limit, alpha, shift)`` the gated unit of alternating gate and up columns, ``[M, N / 2]``.
+    ``n_main`` (a multiple of 16, with ``unit``): columns from there on are no part of the unit and leave as fp32 sums; returns
+    ``(out [M, n_main / 2], tail [M, N - n_main])``."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
     if x.shape[1] % 8:                 # rows that TMA cannot address (16-byte strides): a vendor product
         assert unit is None
@@ -459,15 +462,17 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.T
     N = w.shape[0]
     d = _dev(x)
     assert w.stride(1) == 1
+    assert n_main is None or (unit is not None and out is None)
+    tail = None if n_main is None else torch.empty(M, N - n_main, dtype=torch.float32, device=x.device)
     if out is None:
-        out = torch.empty(M, N if unit is None else N // 2, dtype=torch.bfloat16, device=x.device)
+        out = torch.empty(M, N if unit is None else (N if n_main is None else n_main) // 2, dtype=torch.bfloat16, device=x.device)
     assert out.stride(1) == 1 and out.dtype == torch.bfloat16
     if bias is not None:
         assert bias.numel() == N
         bias = _float_cached(bias)
     L = lib()
     if not getattr(L, "_bias_act_bound", False):
-        L.atlas_gemm_bias_act.argtypes = [_vp, _vp, _vp, _vp, _i, _f, _f, _f, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
+        L.atlas_gemm_bias_act.argtypes = [_vp, _vp, _vp, _vp, _ll, _i, _vp, _i, _f, _f, _f, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
         L._bias_act_bound = True
     sms = _num_sms[d]
     bn, splits = gemm_plan(M, N, K, 0, sms)
@@ -476,10 +481,11 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.T
         ws = scratch("gemm_ws", _GEMM_WS_BYTES, x.device)
         cnt = scratch("gemm_counters", 1 << 18, x.device)
     limit, alpha, shift = unit or (0.0, 0.0, 0.0)
-    _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(bias), 0 if unit is None else 2, float(limit), float(alpha), float(shift), M, N,
+    _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(tail), N - n_main if n_main is not None else 0, n_main or 0,
+                                 _ptr(bias), 0 if unit is None else 2, float(limit), float(alpha), float(shift), M, N,
                                  K, x.stride(0), w.stride(0), out.stride(0), bn, splits, _ptr(ws), _ptr(cnt), sms, _status_ptr[d], _stream()),
            "gemm_bias_act")
-    return out
+    return out if tail is None else (out, tail)
 
 
 _float_cache: dict = {}

@@ -90,6 +90,19 @@ def test_gated_units(dtype, unit, T, K, I):
         close(ops.silu_mul_act(flat).x, c * O.sigmoid(c) * d, dtype)
 
 
+@pytest.mark.parametrize("T,K,I,E", [(1, 2048, 96, 64), (5, 4096, 1408, 8), (130, 256, 8, 3), (700, 128, 72, 40), (64, 8192, 64, 16)])
+def test_gated_unit_and_fp32_logits_in_one_product(T, K, I, E):
+    """Router rows behind the gate / up rows, with and without a split of the sum over K."""
+    from atlas_b200 import ops
+    x, w = rnd(T, K).to(torch.bfloat16), rnd(2 * I + E, K, seed=1, std=1.5 * K ** -0.5).to(torch.bfloat16)
+    a, z = ops.linear_gated_unit_tail(x.cuda(), ops.LinearWeight("dense", w.cuda()), (0.9, 1.702, 1.0), 2 * I)
+    full = x.double() @ w.double().T
+    g, u = full[:, 0:2 * I:2].clamp(max=0.9), full[:, 1:2 * I:2].clamp(-0.9, 0.9)
+    close(a.x, g * O.sigmoid(1.702 * g) * (u + 1.0), torch.bfloat16)
+    assert z.dtype == torch.float32 and z.shape == (T, E)
+    close(z, full[:, 2 * I:], torch.float32, factor=2)
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T,H,I,E,top,count,keep,shared", [(1, 64, 64, 1, 1, 1, 1, 8), (7, 128, 40, 6, 2, 3, 2, 0), (150, 256, 192, 16, 4, 4, 2, 72), (33, 100, 36, 5, 5, 1, 1, 50),
                                                            (700, 64, 128, 8, 1, 8, 3, 64), (40, 90, 45, 64, 6, 32, 8, 30), (300, 128, 96, 12, 3, 2, 2, 96)])
@@ -119,6 +132,9 @@ def test_experts_with_groups_and_a_shared_one(dtype, T, H, I, E, top, count, kee
     _, got_ids = ops.moe_route(ops.linear_tail(x.cuda(), m.router, 0)[1], top, True, "sigmoid", m.router_bias, count, keep, 1.3)
     same = torch.tensor([sorted(a) == sorted(b) for a, b in zip(ids, got_ids.cpu().tolist())])
     assert same.float().mean() > 0.995
+    close(m.forward(ops.Act(x=x.cuda()))[same.cuda()], want[same], dtype, factor=1.5)
+    m.fuse_inputs()
+    assert (m.fused_in is not None) == (dtype == torch.bfloat16 and shared > 0 and shared % 8 == 0 and H % 8 == 0)
     close(m.forward(ops.Act(x=x.cuda()))[same.cuda()], want[same], dtype, factor=1.5)
     rows = m.forward(ops.Act(x=x.cuda()), rows_ok=True)
     assert isinstance(rows, ops.ExpertRows) and (rows.extra is not None) == bool(shared)
