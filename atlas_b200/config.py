@@ -27,7 +27,7 @@ _FAMILY_ALIASES = {
     "holo3_1_moe": "hybrid",
     "nemotron_h": "hybrid", "nemotron_h_puzzle": "hybrid",
     "deepseek_v2": "moe", "deepseek_v3": "moe", "deepseek_v32": "moe", "kimi_k2": "moe",
-    "papidra": "hybrid", "tomizen": "hybrid", "kenovik": "hybrid",
+    "papidra": "hybrid", "tomizen": "hybrid", "kenovik": "hybrid", "bisudra": "hybrid",
 }
 
 # widths the attention kernels are instantiated for; heads of any other size are zero-padded to the next one
@@ -138,6 +138,7 @@ class ModelConfig:
     norm_topk_prob: bool = True
     router_scoring: str = "softmax"   # softmax | sigmoid | sqrtsoftplus
     router_f32: bool = False          # router logits leave their matrix product in fp32
+    router_logit_bias: bool = False   # a learned number per expert joins the logits (selection and weights)
     routed_scaling_factor: float = 1.0
     router_n_group: int = 0           # group-limited routing (DeepSeek-V3): experts split into n_group groups ...
     router_topk_group: int = 0        # ... of which the topk_group best stay eligible
@@ -164,6 +165,15 @@ class ModelConfig:
     # norms on the sublayers' inputs, on an fp32 residual stream (models given by a list of layers)
     input_norms: bool = False
     loop_steps: int = 0               # passes of the looped layers that have a step vector
+    # parts of a layer on normed outputs: layer norms (mean taken off, with a bias) in place of RMS norms, also ahead of the head;
+    # sigmoid gates on the sublayers' results, computed from what the sublayer reads; a short causal convolution added to the
+    # mixer's input (number of taps, 0 = off); a second embedding of the tokens that every layer takes its share of (numbers per
+    # layer, 0 = off); every layer hands on a weighted sum of all layers' results so far
+    layer_norms: bool = False
+    sublayer_gates: bool = False
+    input_conv_taps: int = 0
+    token_side_dim: int = 0
+    depth_average: bool = False
     mamba_num_heads: int = 0
     mamba_head_dim: int = 64
     ssm_state_size: int = 128
@@ -183,7 +193,10 @@ class ModelConfig:
     mlstm_head_dim: int = 0
     mlstm_value_dim: int = 0
     mlstm_gate_cap: float = 0.0       # bound on the raw gates (cap * tanh(. / cap))
-    mlp_activation: str = "silu_glu"  # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down) | clamped_glu
+    # silu_glu (gated SwiGLU) | relu2 (up -> relu^2 -> down) | clamped_glu | silu_unit (SwiGLU on alternating gate and up rows, the
+    # form that the products' epilogues apply)
+    mlp_activation: str = "silu_glu"
+    mlp_bias: bool = False            # the dense feed-forward's projections have biases
     glu_limit: float = 0.0            # clamped_glu: bound on the gate (above) and on the up branch (both sides)
     glu_alpha: float = 1.702          # clamped_glu: slope inside the gate's sigmoid
     shared_glu_limit: float = 0.0     # the same bound for the shared expert
@@ -199,6 +212,9 @@ class ModelConfig:
     attn_distance_rows: int = 0
     attn_distance_reach: int = 0
     qk_norm_rows: bool = False        # q and k are normed over all heads at once, before they are split
+    # differential attention: two maps per head over the same values, output of the first minus a learned multiple of the second,
+    # with this constant in the multiple and 1 minus it on the result
+    attn_diff: float = 0.0
     attn_query_temp: float = 0.0      # queries times 1 + c ln(floor((position + 1) / every) + 1) (0 = off)
     attn_query_temp_every: int = 1
     rotary_dims: Optional[int] = None
@@ -316,13 +332,19 @@ class ModelConfig:
     def _spec_layer_params(self, spec: LayerSpec) -> int:
         """Projection weights of one layer described by a :class:`LayerSpec` (``self`` is the layer's own view)."""
         h = self.hidden_size
-        n = 3 * h * self.intermediate_size if spec.has_mlp and not self.num_experts else 0
+        n = (2 if self.mlp_activation == "relu2" else 3) * h * self.intermediate_size if spec.has_mlp and not self.num_experts else 0
+        if self.sublayer_gates:
+            n += (2 if spec.has_mlp else 1) * h * h
+        n += self.token_side_dim * (2 * h + self.vocab_size)
         if spec.has_mlp and self.num_experts:
             n += self.num_experts * (h + (2 if self.mlp_activation == "relu2" else 3) * h * self.moe_intermediate_size)
             n += 3 * h * self.shared_expert_intermediate_size
         if spec.kind in ("attention", "parallel"):
             dv = self.v_head_dim or self.head_dim
             n += h * (self.q_size + self.kv_size + self.num_key_value_heads * dv) + self.num_attention_heads * dv * h
+        if spec.kind == "differential":
+            dv, H = self.v_head_dim or self.head_dim, self.num_attention_heads
+            n += h * (2 * self.q_size + 2 * self.kv_size + self.num_key_value_heads * dv) + (2 if self.attn_output_gate else 1) * H * dv * h
         if spec.kind in ("mamba2", "parallel"):
             di = self.mamba_num_heads * self.mamba_head_dim
             n += h * (2 * di + 2 * self.mamba_n_groups * self.ssm_state_size + self.mamba_num_heads) + di * h
@@ -681,8 +703,48 @@ def kenovik_config(cfg: Dict[str, Any]) -> ModelConfig:
     return _size_by_heads(c)
 
 
+def _bisudra_ff(mlp: Dict[str, Any]) -> Dict[str, Any]:
+    if mlp.get("kind", "dense") == "dense":
+        return {"intermediate_size": int(mlp["ff"]), "mlp_activation": "relu2", "mlp_bias": True}
+    if mlp["kind"] != "moe":
+        raise ValueError(f"unsupported Bisudra feed-forward '{mlp['kind']}'")
+    r = mlp["router"]
+    if not 1 <= int(r["top"]) <= int(r["experts"]):
+        raise ValueError(f"{r['top']} of {r['experts']} experts per token")
+    return {"num_experts": int(r["experts"]), "num_experts_per_tok": int(r["top"]), "moe_intermediate_size": int(mlp["expert"]["ff"]),
+            "mlp_activation": "silu_unit", "norm_topk_prob": True, "router_scoring": "softmax", "router_f32": True, "router_logit_bias": True}
+
+
+def _bisudra_layer(lc: Dict[str, Any]) -> LayerSpec:
+    if lc["type"] != "attention":
+        raise ValueError(f"unsupported Bisudra layer type '{lc['type']}'")
+    m, mlp = lc["mixer"], lc.get("mlp")
+    mask = m.get("mask")
+    over = {**_attention_overrides(m), "attn_diff": float(m["diff"]), "attn_output_gate": True, "qk_norm": True, "qk_norm_plus_one": False,
+            "sliding_window": int(mask["size"]) if mask else None}
+    over["attn_cache_width"] = padded_head_width(2 * over["head_dim"], over["v_head_dim"])      # a cached key holds both maps' keys
+    if mlp is not None:
+        over.update(_bisudra_ff(mlp))
+    return LayerSpec("differential", mlp is not None, over)
+
+
+def bisudra_config(cfg: Dict[str, Any]) -> ModelConfig:
+    """Bisudra: differential attention in a sliding window behind an input convolution, dense or expert feed-forwards, gated and
+    layer-normed sublayer outputs, a token input per layer, depth averages."""
+    specs = [_bisudra_layer(lc) for lc in cfg["layers"]]
+    widest = lambda k: max([s.overrides.get(k, 0) for s in specs] + [0])
+    c = ModelConfig(model_type="bisudra", family="hybrid", vocab_size=int(cfg["vocab"]), hidden_size=int(cfg["width"]),
+                    intermediate_size=max(1, widest("intermediate_size"), widest("moe_intermediate_size")), num_hidden_layers=len(specs),
+                    num_attention_heads=1, num_key_value_heads=1, head_dim=64, rms_norm_eps=float(cfg["norm"]["eps"]), output_norms=True,
+                    layer_norms=True, sublayer_gates=True, input_conv_taps=int(cfg["canon"]["taps"]), token_side_dim=int(cfg["token_side"]["dim"]),
+                    depth_average=True, tie_word_embeddings=True, layer_specs=specs, dtype=str(cfg.get("torch_dtype", cfg.get("dtype", "bfloat16"))),
+                    quant=QuantConfig(kv_cache_dtype="bf16"), bos_token_id=cfg.get("bos_token_id"), eos_token_id=cfg.get("eos_token_id"))
+    c.moe_intermediate_size = widest("moe_intermediate_size")
+    return _size_by_heads(c)
+
+
 # ``architecture`` of a config.json that lists its layers one by one -> its reader
-_NATIVE_ARCHITECTURES = {"papidra": papidra_config, "tomizen": tomizen_config, "kenovik": kenovik_config}
+_NATIVE_ARCHITECTURES = {"papidra": papidra_config, "tomizen": tomizen_config, "kenovik": kenovik_config, "bisudra": bisudra_config}
 
 
 # ---------------------------------------------------------------------------- presets
@@ -875,13 +937,40 @@ def kenovik_20b(quant: str = "none") -> ModelConfig:
     return c
 
 
+def _bisudra(vocab: int, width: int, pattern: str, attn: tuple, ff: int, experts: tuple, taps: int, side: int, dtype: str) -> ModelConfig:
+    """``pattern``: ``d`` = layer with a dense feed-forward, ``e`` = with experts, ``n`` = without one; ``attn`` (heads, kv heads, dim,
+    vdim, rotated, window), ``experts`` (count, top, ff)."""
+    h, g, d, dv, rot, window = attn
+    mlps = {"d": {"kind": "dense", "ff": ff}, "n": None,
+            "e": {"kind": "moe", "expert": {"ff": experts[2]}, "router": {"experts": experts[0], "top": experts[1]}}}
+    layers = [{"type": "attention", "mixer": {"heads": h, "kv_heads": g, "dim": d, "vdim": dv, "scale": d ** -0.5, "diff": min(0.8 - 0.6 * math.exp(-0.3 * i), 0.8),
+                                              "mask": {"size": window}, "rot": {"base": 5e5, "dims": rot}}, "mlp": mlps[ch]}
+              for i, ch in enumerate(pattern)]
+    return bisudra_config({"vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "canon": {"taps": taps}, "token_side": {"dim": side},
+                           "layers": layers, "dtype": dtype})
+
+
+def tiny_bisudra(dtype: str = "float32") -> ModelConfig:
+    c = _bisudra(1024, 192, "dedn", (6, 2, 24, 40, 16, 72), 256, (8, 3, 72), 4, 20, dtype)
+    c.max_position_embeddings = 4096
+    return c
+
+
+def bisudra_8b(quant: str = "none") -> ModelConfig:
+    """Layers of the size of an 8B mixture-of-experts decoder: width 2048, 16 heads of two maps of 64 and values of 128 (4 kv),
+    64 experts of 1408 (6 per token) in every second layer."""
+    c = _bisudra(131072, 2048, "de" * 12, (16, 4, 64, 128, 64, 4096), 8192, (64, 6, 1408), 4, 128, "bfloat16")
+    c.quant = QuantConfig(method=quant, kv_cache_dtype="bf16")
+    return c
+
+
 PRESETS = {
     "tiny-dense": tiny_dense, "tiny-moe": tiny_moe, "tiny-hybrid": tiny_hybrid,
     "llama3-8b": llama3_8b, "llama3-70b": llama3_70b,
     "qwen3-30b-a3b": qwen3_30b_a3b, "qwen3-next-80b": qwen3_next_80b,
     "tiny-nemotron-h": tiny_nemotron_h, "nemotron-h-8b": nemotron_h_8b, "tiny-deepseek": tiny_deepseek,
     "tiny-papidra": tiny_papidra, "papidra-8b": papidra_8b, "tiny-tomizen": tiny_tomizen, "tomizen-16b": tomizen_16b,
-    "tiny-kenovik": tiny_kenovik, "kenovik-20b": kenovik_20b,
+    "tiny-kenovik": tiny_kenovik, "kenovik-20b": kenovik_20b, "tiny-bisudra": tiny_bisudra, "bisudra-8b": bisudra_8b,
 }
 
 

@@ -165,6 +165,8 @@ class LLMEngine:
                      c.hidden_size)
         tp = max(1, self.model.pctx.tp_size)
         act = self.cfg.max_prefill_tokens * (widest // tp + 4 * c.hidden_size) * 2 * 3
+        if c.depth_average:
+            act += self.cfg.max_prefill_tokens * (c.num_hidden_layers + 1) * c.hidden_size * 4      # every layer's result, fp32
         logits = self.cfg.max_num_seqs * c.vocab_size * 6
         return int(act + logits + (2 << 30))
 

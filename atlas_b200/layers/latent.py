@@ -41,6 +41,7 @@ def _pad_to(n: int, m: int) -> int:
 
 class LatentAttention:
     lora = None
+    takes_adapters = False
     gated = False
     plain = False                # the cache keeps the model's own dtype
 

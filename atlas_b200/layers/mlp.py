@@ -23,7 +23,8 @@ class DenseMLP:
         """``paired``: gate and up rows alternate, so that the product's epilogue applies the gated unit (silu or clamped)."""
         self.cfg, self.pctx, self.quant_kind = cfg, pctx, quant_kind
         self.paired = paired
-        # "silu_glu": gate|up GEMM -> silu(gate) * up; "relu2": a single up GEMM -> relu(up)^2 (Nemotron-H)
+        # "silu_glu": gate|up GEMM -> silu(gate) * up; "relu2": a single up GEMM -> relu(up)^2 (Nemotron-H), with biases where the
+        # configuration has them
         self.activation = activation or getattr(cfg, "mlp_activation", "silu_glu")
         limit = cfg.glu_limit if glu_limit is None else glu_limit
         self.unit = (limit, cfg.glu_alpha, 1.0) if self.activation == "clamped_glu" else ops.SILU_UNIT
@@ -32,25 +33,33 @@ class DenseMLP:
         self.shard = shard and pctx.tp_size > 1 and self.inter % (pctx.tp_size * 128) == 0
         self.gate_up: Optional[LinearWeight] = None
         self.down: Optional[LinearWeight] = None
+        self.down_bias: Optional[torch.Tensor] = None       # of a sharded down projection: joins the group's sum
         self.lora = None                    # lora.LoraSet shared by the model's layers
         self.lora_prefix = ""               # e.g. "layers.3.mlp."
 
-    def load(self, gate: Optional[torch.Tensor], up: torch.Tensor, down: torch.Tensor) -> None:
+    def load(self, gate: Optional[torch.Tensor], up: torch.Tensor, down: torch.Tensor, up_bias: Optional[torch.Tensor] = None,
+             down_bias: Optional[torch.Tensor] = None) -> None:
         tp, r = (self.pctx.tp_size, self.pctx.tp_rank) if self.shard else (1, 0)
+        if up_bias is not None:
+            assert self.activation == "relu2", "gated units have no biases"
+            up_bias = shard_rows(up_bias.to(up.dtype).reshape(-1, 1), r, tp)[:, 0].contiguous()
+            down_bias = down_bias.to(down.dtype).contiguous()
         if self.activation == "relu2":
             gu = shard_rows(up, r, tp)
         elif self.paired:
             gu = paired_rows(shard_rows(gate, r, tp), shard_rows(up, r, tp)).contiguous()
         else:
             gu = torch.cat([shard_rows(gate, r, tp), shard_rows(up, r, tp)], 0)
-        self.gate_up = make_weight(gu, self.quant_kind)
-        self.down = make_weight(shard_cols(down, r, tp).contiguous(), self.quant_kind)
+        self.gate_up = make_weight(gu, self.quant_kind, up_bias)
+        self.down_bias = down_bias if self.shard else None
+        self.down = make_weight(shard_cols(down, r, tp).contiguous(), self.quant_kind, None if self.shard else down_bias)
 
     def init_random(self, gen, std, dtype, device) -> None:
         h = self.cfg.hidden_size
-        self.load(randn_weight(gen, self.inter, h, std, dtype, device),
-                  randn_weight(gen, self.inter, h, std, dtype, device),
-                  randn_weight(gen, h, self.inter, std, dtype, device))
+        gate, up = (randn_weight(gen, self.inter, h, std, dtype, device) for _ in range(2))
+        down = randn_weight(gen, h, self.inter, std, dtype, device)
+        biases = [randn_weight(gen, 1, n, std, dtype, device)[0] for n in (self.inter, h)] if self.cfg.mlp_bias else []
+        self.load(gate, up, down, *biases)
 
     def hidden_act(self, act: Act) -> Act:
         """gate|up GEMM + SiLU * mul: the input of the down projection (no adapters)."""
@@ -68,9 +77,12 @@ class DenseMLP:
         return ops.glu_act(gate_up, want_fp8, "gelu_tanh")
 
     def _relu2(self, act: Act, reduce: bool) -> torch.Tensor:
-        u = ops.linear(act, self.gate_up)
-        a = ops.relu_squared(u)
-        return self.pctx.row_parallel_linear(a, self.down) if (self.shard and reduce) else ops.linear(a, self.down)
+        return self.down_product(ops.linear_relu2(act, self.gate_up), reduce)
+
+    def down_product(self, a: torch.Tensor, reduce: bool = True) -> torch.Tensor:
+        """Down projection of the hidden activations, summed over the group that shards it."""
+        y = self.pctx.row_parallel_linear(a, self.down) if (self.shard and reduce) else ops.linear(a, self.down)
+        return y if self.down_bias is None else y + self.down_bias
 
     def forward(self, act: Act, reduce: bool = True, batch=None) -> torch.Tensor:
         if self.activation == "relu2":

@@ -98,9 +98,10 @@ class MoE:
         self.cfg, self.pctx = cfg, pctx
         self.expert_kind, self.dense_kind = expert_kind, dense_kind
         self.top_k = cfg.num_experts_per_tok
-        # silu(gate) * up, relu(up)^2, or the clamped unit of alternating gate and up rows
-        self.activation = cfg.mlp_activation if cfg.mlp_activation in ("relu2", "clamped_glu") else "silu_glu"
-        self.unit = (cfg.glu_limit, cfg.glu_alpha, 1.0) if self.activation == "clamped_glu" else None
+        # silu(gate) * up, relu(up)^2, or a gated unit (clamped or silu) of alternating gate and up rows
+        self.activation = {"relu2": "relu2", "clamped_glu": "clamped_glu", "silu_unit": "clamped_glu"}.get(cfg.mlp_activation, "silu_glu")
+        self.unit = None if self.activation != "clamped_glu" else (ops.SILU_UNIT if cfg.mlp_activation == "silu_unit" else
+                                                                   (cfg.glu_limit, cfg.glu_alpha, 1.0))
         self.router_f32 = cfg.router_f32
         self.e_lo, self.e_hi = cfg.local_expert_range(pctx.ep_rank, pctx.ep_size)
         self.ep_mode = ep_mode
@@ -114,14 +115,17 @@ class MoE:
         self.lora = None                    # lora.LoraSet shared by the model's layers
         self.lora_prefix = ""               # e.g. "layers.3.mlp."
         if cfg.shared_expert_intermediate_size:
-            clamped = self.activation == "clamped_glu"
-            self.shared = DenseMLP(cfg, pctx, dense_kind, cfg.shared_expert_intermediate_size, shard=False, paired=clamped,
-                                   glu_limit=cfg.shared_glu_limit if clamped else None)
+            paired = self.activation == "clamped_glu"
+            self.shared = DenseMLP(cfg, pctx, dense_kind, cfg.shared_expert_intermediate_size, shard=False, paired=paired,
+                                   activation="silu_glu" if cfg.mlp_activation == "silu_unit" else None,
+                                   glu_limit=cfg.shared_glu_limit if paired else None)
 
     # ------------------------------------------------------------------ weights
-    def load(self, router: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor) -> None:
-        """``w13 [E,2I,H]`` / ``w2 [E,H,I]`` are the *global* expert stacks (or already-local stacks)."""
-        self.router = LinearWeight("dense", router.contiguous())
+    def load(self, router: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, logit_bias: Optional[torch.Tensor] = None) -> None:
+        """``w13 [E,2I,H]`` / ``w2 [E,H,I]`` are the *global* expert stacks (or already-local stacks); ``logit_bias [E]`` joins the
+        router's logits."""
+        assert logit_bias is None or self.router_f32
+        self.router = LinearWeight("dense", router.contiguous(), bias=None if logit_bias is None else logit_bias.float().to(router.device).contiguous())
         if w13.shape[0] == self.cfg.num_experts and self.pctx.ep_size > 1:
             w13, w2 = w13[self.e_lo:self.e_hi], w2[self.e_lo:self.e_hi]
         pad = -w2.shape[2] % 64
@@ -160,20 +164,24 @@ class MoE:
         assert len(w13_l) == n_local
         if cfg.router_selection_bias:
             self.router_bias = (torch.rand(cfg.num_experts, generator=gen, device=gen.device) * 0.1).to(device)
-        self.load(router, torch.stack(w13_l), torch.stack(w2_l))
+        bias = torch.randn(cfg.num_experts, generator=gen, device=gen.device) * 0.1 if cfg.router_logit_bias else None
+        self.load(router, torch.stack(w13_l), torch.stack(w2_l), bias)
         if self.shared is not None:
             self.shared.init_random(gen, std, dtype, device)
             if self.activation != "clamped_glu":
                 self.shared_gate = randn_weight(gen, 1, h, std, dtype, device)
 
     # ------------------------------------------------------------------ forward
-    def forward(self, act: Act, token_ids: Optional[torch.Tensor] = None, batch=None, rows_ok: bool = False):
-        """``rows_ok``: the caller takes the weighted sum itself, so the result may be an :class:`ops.ExpertRows`."""
+    def forward(self, act: Act, token_ids: Optional[torch.Tensor] = None, batch=None, rows_ok: bool = False, logits: Optional[torch.Tensor] = None):
+        """``rows_ok``: the caller takes the weighted sum itself, so the result may be an :class:`ops.ExpertRows`.  ``logits``: the
+        router's, where the caller has formed them already."""
         x = act.plain()
         cfg = self.cfg
         adapters = self.lora is not None and batch is not None and batch.adapter_rows is not None and bool(self.lora_prefix)
         shared_rows = None
-        if self.fused_in is not None and not adapters and ops.on_gpu(x):
+        if logits is not None:
+            pass
+        elif self.fused_in is not None and not adapters and ops.on_gpu(x):
             a, logits = ops.linear_gated_unit_tail(act, self.fused_in, self.shared.unit, self.shared.gate_up.weight.shape[0])
             shared_rows = ops.linear(a, self.shared.down)
         else:

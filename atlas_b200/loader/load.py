@@ -353,9 +353,41 @@ def _load_kenovik(model: DecoderLM, ck: Checkpoint) -> None:
     ck.close()
 
 
+def _load_bisudra(model: DecoderLM, ck: Checkpoint) -> None:
+    """Bisudra naming: ``embed``, ``side.embed``, ``l<i>.{norm1, norm2, canon1, rg1, rg2, dwa, side.*, mix.*, mlp.*}`` (``.b`` behind a name:
+    its bias), ``final.norm``; the embedding table is the output projection."""
+    wt = lambda name: ck.get(name).to(device=model.device, dtype=model.dtype)
+    f32 = lambda name: ck.get(name).to(device=model.device, dtype=torch.float32).contiguous()
+    norm = lambda name: (f32(name), f32(name + ".b"))
+    model.embed, model.side_embed = wt("embed").contiguous(), wt("side.embed").contiguous()
+    for i, layer in enumerate(model.layers):
+        pre = f"l{i}."
+        m, ff = pre + "mix.", pre + "mlp."
+        layer.input_norm, layer.input_bias = norm(pre + "norm1")
+        layer.mixer.load(*(wt(m + n) for n in "qkvog"), f32(m + "q.norm"), f32(m + "k.norm"), [f32(m + n) for n in ("lq1", "lk1", "lq2", "lk2")])
+        layer.conv.load(wt(pre + "canon1"))
+        layer.gate1.load(wt(pre + "rg1"), f32(pre + "rg1.b"))
+        layer.side.load(wt(pre + "side.gate"), wt(pre + "side.proj"), f32(pre + "side.norm"))
+        layer.depth_factors = f32(pre + "dwa")
+        if layer.ffn is None:
+            continue
+        layer.post_norm, layer.post_bias = norm(pre + "norm2")
+        layer.gate2.load(wt(pre + "rg2"), f32(pre + "rg2.b"))
+        if not layer.is_moe:
+            layer.ffn.load(None, wt(ff + "up"), wt(ff + "down"), f32(ff + "up.b"), f32(ff + "down.b"))
+            continue
+        gate, up, down = (torch.stack([wt(f"{ff}e{e}.{n}") for e in range(layer.ffn.e_lo, layer.ffn.e_hi)]) for n in ("gate", "up", "down"))
+        layer.ffn.load(wt(ff + "router"), torch.cat([gate, up], 1), down, f32(ff + "router.b"))
+    model.final_norm, model.final_bias = norm("final.norm")
+    model.set_lm_head(model.embed)
+    ck.close()
+
+
 def load_weights(model: DecoderLM, ck: Checkpoint) -> None:
     cfg = model.cfg
     dense_kind, expert_kind = quant_kinds(cfg)
+    if cfg.model_type == "bisudra":
+        return _load_bisudra(model, ck)
     if cfg.model_type == "kenovik":
         return _load_kenovik(model, ck)
     if cfg.model_type == "tomizen":

@@ -18,10 +18,10 @@ import torch
 
 from .. import ops
 from ..config import ModelConfig
-from ..layers import (MIXERS, Attention, DenseMLP, GatedDeltaNet, HyperConnection, Mamba2Mixer, MLAttention, MoE, ParallelCtx,
-                      ParallelMixer)
+from ..layers import (MIXERS, Attention, DenseMLP, GatedDeltaNet, HyperConnection, InputConvolution, Mamba2Mixer, MLAttention, MoE,
+                      ParallelCtx, SublayerGate, TokenSide)
 from ..layers.common import make_weight, randn_weight, shard_rows
-from ..ops import Act, LinearWeight, NormDelta, StreamDelta, reference as ref
+from ..ops import Act, DepthSum, LinearWeight, NormDelta, StreamDelta, reference as ref
 from .batch import ForwardBatch
 
 # tensor-parallel steps with at least this many rows run sequence-parallel (reduce-scatter / all-gather fused into the
@@ -305,7 +305,11 @@ class StreamLayer:
 class OutputNormLayer:
     """A layer whose norms sit on the sublayers' outputs: ``x += norm(mixer(x))``, then ``x += norm(ffn(x))`` where the layer has a
     feed-forward, on an fp32 residual stream that the sublayers read itself.  Same ``forward`` protocol as
-    :class:`DecoderLayer`, with the pending :class:`NormDelta` in place of the previous layer's output."""
+    :class:`DecoderLayer`, with the pending :class:`NormDelta` in place of the previous layer's output.
+
+    Where the configuration has them: layer norms in place of RMS norms, gates on the sublayers' results (from the stream as the
+    sublayer gets it), a convolution on the mixer's input, a token input behind the feed-forward, and a weighted sum over all
+    layers' results as what goes on."""
 
     def __init__(self, cfg: ModelConfig, idx: int, pctx: ParallelCtx, ep_mode: str = "auto"):
         spec = cfg.layer_specs[idx]
@@ -318,32 +322,89 @@ class OutputNormLayer:
             self.ffn = MoE(self.cfg, pctx, expert_kind, dense_kind, ep_mode) if self.is_moe else DenseMLP(self.cfg, pctx, dense_kind)
         self.input_norm: Optional[torch.Tensor] = None         # fp32, on the mixer's output
         self.post_norm: Optional[torch.Tensor] = None          # fp32, on the feed-forward's output
+        self.input_bias: Optional[torch.Tensor] = None         # fp32: layer norms
+        self.post_bias: Optional[torch.Tensor] = None
+        self.conv = InputConvolution(cfg.hidden_size, cfg.input_conv_taps) if cfg.input_conv_taps else None
+        if self.conv is not None and recurrent_of(self) is not self.conv:
+            raise ValueError("a convolution on the input of a recurrent mixer needs a second state slot")
+        self.gate1 = SublayerGate(cfg.hidden_size, dense_kind) if cfg.sublayer_gates else None
+        self.gate2 = SublayerGate(cfg.hidden_size, dense_kind) if cfg.sublayer_gates and spec.has_mlp else None
+        self.ffn_in: Optional[LinearWeight] = None             # the feed-forward's first product and its gate's in one
+        self.side = TokenSide(cfg.hidden_size, cfg.token_side_dim, idx, dense_kind) if cfg.token_side_dim else None
+        self.depth_factors: Optional[torch.Tensor] = None      # fp32 [idx + 2]: this layer's share of every result so far
         self.rope_override: Optional[torch.Tensor] = None      # this layer's own rotary table
 
     def init_random(self, gen, std, dtype, device):
-        fresh = lambda: torch.full((self.cfg.hidden_size,), 0.0 if self.cfg.norm_plus_one else 1.0, dtype=torch.float32, device=device)
+        cfg = self.cfg
+        fresh = lambda: torch.full((cfg.hidden_size,), 0.0 if cfg.norm_plus_one else 1.0, dtype=torch.float32, device=device)
+        bias = lambda: torch.zeros(cfg.hidden_size, dtype=torch.float32, device=device) if cfg.layer_norms else None
         self.mixer.init_random(gen, std, dtype, device)
-        self.input_norm = fresh()
+        self.input_norm, self.input_bias = fresh(), bias()
         if self.ffn is not None:
             self.ffn.init_random(gen, std, dtype, device)
-            self.post_norm = fresh()
+            self.post_norm, self.post_bias = fresh(), bias()
+        if self.conv is not None:
+            self.conv.init_random(gen, dtype, device)
+        for part in (self.gate1, self.gate2, self.side):
+            if part is not None:
+                part.init_random(gen, std, dtype, device)
+        if cfg.depth_average:
+            share = torch.rand(self.idx + 2, generator=gen, device=gen.device) * 0.1
+            share[-1] = 1.0
+            self.depth_factors = share.to(device)
+
+    def fuse_inputs(self) -> None:
+        """One product for the feed-forward's first projection, or its router, and for its gate, where the kernels take both (bf16, rows
+        in whole 16-byte pieces, unquantised); the weights become its parts."""
+        if self.gate2 is None or self.ffn_in is not None:
+            return
+        own = self.ffn.router if self.is_moe else self.ffn.gate_up
+        g = self.gate2.w
+        if (any(w.kind != "dense" or w.weight.dtype != torch.bfloat16 or w.bias is None or not ops.on_gpu(w.weight) for w in (own, g))
+                or g.weight.shape[1] % 8 or not (self.is_moe or self.ffn.activation == "relu2")):
+            return
+        first, second = (g, own) if self.is_moe else (own, g)
+        self.ffn_in = LinearWeight("dense", torch.cat([first.weight, second.weight], 0).contiguous(),
+                                   bias=torch.cat([first.bias.float(), second.bias.float()]).contiguous())
+        n = first.weight.shape[0]
+        first.weight, second.weight = self.ffn_in.weight[:n], self.ffn_in.weight[n:]
 
     def accepts_prenormed(self) -> bool:
         return False
 
+    def _feed_forward(self, act: Act, batch: ForwardBatch):
+        """The feed-forward's output and the argument of its gate (None without one)."""
+        ffn = self.ffn
+        if self.ffn_in is not None and batch.adapter_rows is None and ops.on_gpu(act.x):
+            if self.is_moe:
+                z, logits = ops.linear_tail(act, self.ffn_in, self.cfg.hidden_size)
+                return ffn.forward(act, batch=batch, rows_ok=True, logits=logits), z
+            n = ffn.gate_up.weight.shape[0]
+            both = ops.linear_relu2(act, self.ffn_in, n)
+            return ffn.down_product(both[:, :n]), both[:, n:]
+        y = ffn.forward(act, batch=batch, rows_ok=True) if self.is_moe else ffn.forward(act, batch=batch)
+        return y, self.gate2.forward(act) if self.gate2 is not None else None
+
     def forward(self, x: NormDelta, stream: Optional[torch.Tensor], batch: ForwardBatch, cache: CacheStore, rope_cache, next_norm=None):
         eps, p1 = self.cfg.rms_norm_eps, self.cfg.norm_plus_one
         rope_cache = rope_cache if self.rope_override is None else self.rope_override
+        history = x.depth.history if x.depth is not None else None
         h, stream = ops.add_normed(stream, x, eps, p1)
+        u = h if self.conv is None else self.conv.forward(h, batch, cache.states[self.idx])
         if attention_of(self) is not None:
-            y = self.mixer.forward(Act(x=h), batch, cache.layer_kv(self.idx), rope_cache)
+            y = self.mixer.forward(Act(x=u), batch, cache.layer_kv(self.idx), rope_cache)
         else:
-            y = self.mixer.forward(Act(x=h), batch, cache.states[self.idx])
-        x = NormDelta(y, self.input_norm)
+            y = self.mixer.forward(Act(x=u), batch, cache.states[self.idx])
+        x = NormDelta(y, self.input_norm, bias=self.input_bias, gate=self.gate1.forward(Act(x=h)) if self.gate1 is not None else None)
         if self.ffn is not None:
             h, stream = ops.add_normed(stream, x, eps, p1)
-            y = self.ffn.forward(Act(x=h), batch=batch, rows_ok=True) if self.is_moe else self.ffn.forward(Act(x=h), batch=batch)
-            x = NormDelta(y, self.post_norm)
+            y, z = self._feed_forward(Act(x=h), batch)
+            x = NormDelta(y, self.post_norm, bias=self.post_bias, gate=z)
+        if self.side is not None:
+            h, stream = ops.add_normed(stream, x, eps, p1)
+            x = NormDelta(self.side.forward(Act(x=h), batch.input_ids), self.side.norm)
+        if history is not None:
+            x.depth = DepthSum(history, self.idx + 1, self.depth_factors)
         return x, stream
 
 
@@ -404,12 +465,14 @@ def attention_of(layer):
     """The attention block of a layer (None without one): the owner of the layer's KV cache."""
     if layer.kind == "parallel":
         return layer.mixer.left
-    return layer.mixer if layer.kind in ("attention", "latent_attention") else None
+    return layer.mixer if layer.kind in ("attention", "latent_attention", "differential") else None
 
 
 def recurrent_of(layer):
-    """The mixer of a layer that owns a recurrent state slot (None without one)."""
-    return layer.mixer if layer.kind in ("gdn", "mamba2", "wkv", "parallel", "mlstm", "rglru") else None
+    """The block of a layer that owns a recurrent state slot: its mixer or the convolution on its input (None without one)."""
+    if layer.kind in ("gdn", "mamba2", "wkv", "parallel", "mlstm", "rglru"):
+        return layer.mixer
+    return getattr(layer, "conv", None)
 
 
 def kv_elements_of(attn) -> int:
@@ -443,7 +506,9 @@ class DecoderLM:
         else:
             self.layers = [DecoderLayer(cfg, i, self.pctx, ep_mode) for i in range(cfg.num_hidden_layers)]
         self.embed: Optional[torch.Tensor] = None
+        self.side_embed: Optional[torch.Tensor] = None       # [vocab, layers * token_side_dim]
         self.final_norm: Optional[torch.Tensor] = None
+        self.final_bias: Optional[torch.Tensor] = None       # fp32: the final norm is a layer norm
         self.lm_head: Optional[LinearWeight] = None          # vocab-parallel slice under TP
         self.rope_cache: Optional[torch.Tensor] = None
         self.loop_step: Optional[torch.Tensor] = None        # fp32 [passes, hidden]: step vectors of looped layers
@@ -475,6 +540,10 @@ class DecoderLM:
             self.loop_step = randn_weight(gen, cfg.loop_steps, cfg.hidden_size, std, torch.float32, dev)
         base = 0.0 if cfg.norm_plus_one else 1.0
         self.final_norm = torch.full((cfg.hidden_size,), base, dtype=torch.float32 if cfg.layer_specs else dt, device=dev)
+        if cfg.layer_norms:
+            self.final_bias = torch.zeros(cfg.hidden_size, dtype=torch.float32, device=dev)
+        if cfg.token_side_dim:
+            self.side_embed = randn_weight(gen, cfg.vocab_size, len(self.layers) * cfg.token_side_dim, 1.0, dt, dev)
         head = self.embed if cfg.tie_word_embeddings else randn_weight(gen, cfg.vocab_size, cfg.hidden_size, std, dt, dev)
         self.set_lm_head(head)
         if self.mtp is not None:
@@ -492,7 +561,7 @@ class DecoderLM:
         if getattr(self, "lora", None) is None:
             self.lora = LoraSet(max_slots)
             for l in self.layers:
-                if attention_of(l) is not None and l.kind != "latent_attention":
+                if attention_of(l) is not None and getattr(attention_of(l), "takes_adapters", True):
                     attention_of(l).lora = self.lora
                 if l.ffn is None:
                     continue
@@ -549,6 +618,10 @@ class DecoderLM:
         for l in self.layers:
             if l.is_moe:
                 l.ffn.fuse_inputs()
+            if isinstance(l, OutputNormLayer):
+                l.fuse_inputs()
+                if l.side is not None:
+                    l.side.table = self.side_embed
         tables: Dict[str, torch.Tensor] = {}
         for l in self.layers if cfg.layer_specs else ():
             if attention_of(l) is not None:
@@ -601,7 +674,7 @@ class DecoderLM:
                                    else alloc_kv(num_blocks, block_size, a.hkv, a.d, dt, self.device))
                 store.kv_scales[l.idx] = (1.0, 1.0)
             if recurrent_of(l) is not None:
-                store.states[l.idx] = l.mixer.alloc_state(max(1, state_slots), self.device, self.dtype)
+                store.states[l.idx] = recurrent_of(l).alloc_state(max(1, state_slots), self.device, self.dtype)
         if self.mtp is not None:
             self.mtp.alloc_cache(store, num_blocks, block_size, kv_dtype, self.device)
         return store
@@ -688,6 +761,9 @@ class DecoderLM:
             x = StreamDelta(x, scale=self.cfg.embed_scale)      # fp32 streams start from the scaled embedding
         elif self.cfg.output_norms or self.cfg.input_norms:
             x = NormDelta(x, scale=self.cfg.embed_scale if self.cfg.input_norms else 1.0)      # so does a plain fp32 stream
+            if self.cfg.depth_average:
+                entries = torch.empty((len(self.layers) + 1,) + tuple(x.y.shape), dtype=torch.float32, device=x.y.device)
+                x.depth = DepthSum(entries, 0)
         elif batch.inputs_embeds is not None:
             x = x.clone()                     # fused epilogues update the residual stream in place
         if layer_ids is not None:
@@ -716,7 +792,7 @@ class DecoderLM:
             y, _ = ops.hyper_norm(residual, x, self._stream_ones, self.final_norm, self.cfg.rms_norm_eps, write=False)
             return y
         if isinstance(x, NormDelta):
-            return ops.add_normed(residual, x, self.cfg.rms_norm_eps, self.cfg.norm_plus_one, self.final_norm, write=False)[0]
+            return ops.add_normed(residual, x, self.cfg.rms_norm_eps, self.cfg.norm_plus_one, self.final_norm, write=False, out_bias=self.final_bias)[0]
         y, _ = ops.rmsnorm(x, self.final_norm, self.cfg.rms_norm_eps, residual, self.cfg.norm_plus_one)
         return y
 
@@ -819,7 +895,7 @@ class DecoderLM:
         """After speculative verification: fold the accepted rows into every GDN layer's state."""
         for l in self.layers:
             if recurrent_of(l) is not None:
-                l.mixer.commit(accepted_rows, cache.states[l.idx])
+                recurrent_of(l).commit(accepted_rows, cache.states[l.idx])
 
     # ------------------------------------------------------------------ oracle
     @torch.inference_mode()

@@ -147,24 +147,38 @@ class ExpertRows:
 
 
 @dataclass
+class DepthSum:
+    """Weighted sums over the results of all layers: the stream that a delta leaves becomes entry ``index`` of ``history
+    [entries, T, W]`` (fp32), and what goes on is ``sum_j factors[j] * history[j]``, ``j = 0 .. index``, or, without ``factors``, the
+    entry as it is."""
+    history: torch.Tensor
+    index: int
+    factors: Optional[torch.Tensor] = None   # fp32 [index + 1]
+
+
+@dataclass
 class NormDelta:
     """What the last sublayer leaves for an fp32 residual stream: ``stream += rmsnorm(y) * norm``, or ``stream += y`` without
     ``norm``, with ``y`` given as it is or as :class:`ExpertRows`.  Start of the model (no stream yet): the stream is
-    ``y * scale``."""
+    ``y * scale``.  With ``bias`` the norm is a layer norm (mean taken off, bias added); ``gate [T, W]`` multiplies ``y`` by its
+    sigmoid first; ``depth`` replaces the new stream by a sum over the layers' results."""
     y: object
     norm: Optional[torch.Tensor] = None
     scale: float = 1.0
+    bias: Optional[torch.Tensor] = None
+    gate: Optional[torch.Tensor] = None
+    depth: Optional[DepthSum] = None
 
 
 def add_normed(stream: Optional[torch.Tensor], delta: NormDelta, eps: float, plus_one: bool, out_norm: Optional[torch.Tensor] = None,
-               write: bool = True, step: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+               write: bool = True, step: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """Apply ``delta`` and then the vector ``step`` (fp32 ``[W]``) to ``stream [T, W]`` (fp32, in place; None at the start) and
-    return ``(h, stream)``: ``h`` is the stream in the activations' dtype, normed with ``out_norm`` where one is given.
-    ``write=False`` leaves the stream as it is."""
+    return ``(h, stream)``: ``h`` is the stream in the activations' dtype, normed with ``out_norm`` where one is given (a layer norm
+    with ``out_bias``).  ``write=False`` leaves the stream, and the history of a :class:`DepthSum`, as they are."""
     y = delta.y.y if isinstance(delta.y, ExpertRows) else delta.y
     if on_gpu(y):
-        return cuda_ops().add_normed(stream, delta, eps, plus_one, out_norm, write, step)
-    return ref.add_normed(stream, delta, eps, plus_one, out_norm, write, step)
+        return cuda_ops().add_normed(stream, delta, eps, plus_one, out_norm, write, step, out_bias)
+    return ref.add_normed(stream, delta, eps, plus_one, out_norm, write, step, out_bias)
 
 
 # ----------------------------------------------------------------------------- elementwise / norm
@@ -316,14 +330,27 @@ def linear(a, w: LinearWeight, out: Optional[torch.Tensor] = None) -> torch.Tens
     return y
 
 
-def linear_tail(a, w: LinearWeight, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """``a @ W^T`` of an unquantised weight in two parts: the first ``n_main`` columns in the activations' dtype, the others as the
-    fp32 sums that the product forms.  Returns ``(main, tail)``."""
+def linear_relu2(a, w: LinearWeight, n_act: Optional[int] = None) -> torch.Tensor:
+    """``a @ W^T (+ bias)`` with the first ``n_act`` columns (all of them by default) as ``relu(.) ** 2``; one kernel for unquantised bf16
+    weights with a bias."""
     x = a.plain() if isinstance(a, Act) else a
-    assert w.kind == "dense" and w.bias is None
+    n_act = w.weight.shape[0] if n_act is None else n_act
+    if w.kind == "dense" and w.bias is not None and on_gpu(x) and x.dtype == torch.bfloat16 and x.shape[1] % 8 == 0:
+        return cuda_ops().gemm_bf16(x, w.weight, bias=w.bias, relu2_cols=n_act)
+    y = linear(a, w)
+    if n_act == y.shape[1]:
+        return relu_squared(y)
+    return torch.cat([torch.relu(y[:, :n_act]).square(), y[:, n_act:]], 1)
+
+
+def linear_tail(a, w: LinearWeight, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``a @ W^T (+ bias)`` of an unquantised weight in two parts: the first ``n_main`` columns in the activations' dtype, the others as
+    the fp32 sums that the product forms.  Returns ``(main, tail)``."""
+    x = a.plain() if isinstance(a, Act) else a
+    assert w.kind == "dense"
     if on_gpu(x) and x.dtype == torch.bfloat16:
-        return cuda_ops().linear_tail(x, w.weight, n_main)
-    y = torch.nn.functional.linear(x.float(), w.weight.float())
+        return cuda_ops().linear_tail(x, w.weight, n_main, w.bias)
+    y = torch.nn.functional.linear(x.float(), w.weight.float(), None if w.bias is None else w.bias.float())
     return y[:, :n_main].to(x.dtype), y[:, n_main:]
 
 
@@ -394,6 +421,31 @@ def qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_
                                                q_norm_w, k_norm_w, eps, nq, nk, temp, temp_every, sums)
     return ref.qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_norm_w,
                                     k_norm_w, eps, nq, nk, temp, temp_every, sums)
+
+
+def map_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm_w, k_norm_w, eps: float):
+    """Two maps per head: RMS norm (fp32 weights) and rotation of every map of ``q [T, H, 2, dim]`` and ``k [T, G, 2, dim]``.  Both maps'
+    keys go side by side into one cache row, ``v [T, G, vdim]`` beside them; returns the query rows ``[T, 2 H, D]`` of the cache width
+    ``D``: map 1 of head ``h`` in row ``2 h`` ahead of zeros, map 2 in row ``2 h + 1`` behind zeros, so that a row's product with a cache
+    row is its own map's score."""
+    if on_gpu(q):
+        return cuda_ops().map_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm_w, k_norm_w, eps)
+    return ref.map_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm_w, k_norm_w, eps)
+
+
+def map_difference(a: torch.Tensor, dv: int, lam: float, rest: float, eps: float, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``a [T, 2 H, D]``, the outputs of two maps per head in their first ``dv`` columns -> ``[T, H * dv]``: ``o = a_1 - lam a_2``, RMS norm
+    without a weight over a head's ``dv`` numbers, times ``rest`` and, with ``gate [T, H * dv]``, its sigmoid."""
+    if on_gpu(a):
+        return cuda_ops().map_difference(a, dv, lam, rest, eps, gate)
+    return ref.map_difference(a, dv, lam, rest, eps, gate)
+
+
+def gelu_embedding(z: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, first: int, n: int) -> torch.Tensor:
+    """``gelu_tanh(z[:, :n]) * table[ids, first : first + n]``, zeros in the columns of ``z`` from ``n`` on."""
+    if on_gpu(z):
+        return cuda_ops().gelu_embedding(z, table, ids, first, n)
+    return ref.gelu_embedding(z, table, ids, first, n)
 
 
 def head_rotate(x: torch.Tensor) -> torch.Tensor:

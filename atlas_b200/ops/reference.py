@@ -182,6 +182,33 @@ def qk_norm_rope_kv_write(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, pos
     return q
 
 
+def map_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, q_norm_w, k_norm_w, eps: float):
+    """See ``ops.map_norm_kv_write``; everything up to the result in fp32."""
+    T, H, _, n = q.shape
+    G, dv, D = k.shape[1], v.shape[2], k_cache.shape[3]
+
+    def turned(x, w):
+        x = x.float() * torch.rsqrt(x.float().pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        return apply_rope(x.reshape(T, -1, n), positions, rope_cache, rotary_dim)
+    qf, kf = turned(q, q_norm_w).view(T, H, 2, n), turned(k, k_norm_w).reshape(T, G, 2 * n)
+    ok = slot_mapping >= 0
+    slots, bs = slot_mapping[ok].long(), k_cache.shape[1]
+    k_cache[slots // bs, slots % bs, :, :2 * n] = kf[ok].to(k_cache.dtype)
+    v_cache[slots // bs, slots % bs, :, :dv] = v[ok].to(v_cache.dtype)
+    rows = torch.zeros(T, H, 2, D, dtype=q.dtype, device=q.device)
+    rows[:, :, 0, :n], rows[:, :, 1, n:2 * n] = qf[:, :, 0].to(q.dtype), qf[:, :, 1].to(q.dtype)
+    return rows.view(T, 2 * H, D)
+
+
+def map_difference(a, dv: int, lam: float, rest: float, eps: float, gate=None):
+    """See ``ops.map_difference``."""
+    T = a.shape[0]
+    o = a.float().view(T, -1, 2, a.shape[2])[..., :dv]
+    o = o[:, :, 0] - lam * o[:, :, 1]
+    o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * rest).reshape(T, -1)
+    return (o if gate is None else o * torch.sigmoid(gate.float())).to(a.dtype)
+
+
 def qk_row_norm_kv_write(q, k, v, positions, rope_cache, rotary_dim, k_cache, v_cache, slot_mapping, seq_positions, q_norm_w, k_norm_w,
                          eps: float, nq: int, nk: int, temp: float, temp_every: int, sums=None):
     """See ``ops.qk_row_norm_kv_write``; everything up to the result in fp32."""
@@ -361,7 +388,7 @@ def latent_attention(q, cache, rp: int, block_tables, seq_lens, query_start_loc,
     return out
 
 
-def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool, step=None):
+def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool, step=None, out_bias=None):
     """See ``ops.add_normed``."""
     if hasattr(delta.y, "slot_of"):
         e = delta.y
@@ -372,16 +399,37 @@ def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool,
         y = y if e.extra is None else y + e.extra.float()
     else:
         y, dtype = delta.y.float(), delta.y.dtype
-    unit = lambda t, w: t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + 1.0 if plus_one else w.float())
+    if delta.gate is not None:
+        y = y * torch.sigmoid(delta.gate.float())
+
+    def unit(t, w, b):
+        t = t if b is None else t - t.mean(-1, keepdim=True)
+        t = t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * (w.float() + 1.0 if plus_one else w.float())
+        return t if b is None else t + b.float()
     if stream is None:
         x = y * delta.scale
     else:
-        x = stream + (y if delta.norm is None else unit(y, delta.norm))
+        x = stream + (y if delta.norm is None else unit(y, delta.norm, delta.bias))
     x = x if step is None else x + step
+    if delta.depth is not None:
+        d, entry = delta.depth, x
+        if d.factors is not None:
+            x = entry * d.factors[d.index]
+            for j in range(d.index):
+                x = x + d.history[j] * d.factors[j]
+        if write or stream is None:
+            d.history[d.index] = entry
     if write and stream is not None:
         stream.copy_(x)
-    h = x if out_norm is None else unit(x, out_norm)
+    h = x if out_norm is None else unit(x, out_norm, out_bias)
     return h.to(dtype), (x if stream is None else stream)
+
+
+def gelu_embedding(z, table, ids, first: int, n: int):
+    """See ``ops.gelu_embedding``."""
+    out = torch.zeros_like(z)
+    out[:, :n] = (F.gelu(z[:, :n].float(), approximate="tanh") * table[ids.long(), first:first + n].float()).to(z.dtype)
+    return out
 
 
 # ----------------------------------------------------------------------------- activations

@@ -46,7 +46,7 @@ class ModelRunner:
         self._pin_turn: Dict[str, int] = {}
         # decode graphs of recurrent models read state slots from a device buffer; the kernels that take everything they
         # need from there are those of recurrent.cu
-        self._states_graph_safe = all(l.kind in ("mamba2", "wkv", "parallel", "mlstm", "rglru") for l in model.layers if recurrent_of(l) is not None)
+        self._states_graph_safe = all(l.kind != "gdn" for l in model.layers if recurrent_of(l) is not None)
         # slot of padding rows: the last one, which the engine allocates beyond those it hands out
         self.pad_state_slot = next((t.shape[0] - 1 for st in cache.states.values() for t in st.values()), None)
         if self.on_gpu:
