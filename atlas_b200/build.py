@@ -50,8 +50,8 @@ _UNITS_BASE = ("runtime",)
 _UNITS_BF16 = ("gemm", "elementwise", "attention", "attention_tc16")
 _UNITS_F32 = ("attention_f32",)
 _UNITS_LISTED = ("streams",)                   # residual forms of models that list their layers
-_UNITS_OF_KIND = {"rglru": ("recurrent", "rglru"), "wkv": ("recurrent",), "parallel": ("recurrent",), "mamba2": ("recurrent",), "mlstm": ("mlstm",),
-                  "latent_attention": ("latent",)}
+_UNITS_OF_KIND = {"rglru": ("conv1d", "rglru"), "wkv": ("recurrent",), "parallel": ("recurrent", "conv1d"), "mamba2": ("recurrent", "conv1d"),
+                  "mlstm": ("mlstm",), "latent_attention": ("latent",), "differential": ("differential",)}
 
 
 def units_for(cfg) -> Optional[List[str]]:
@@ -66,6 +66,8 @@ def units_for(cfg) -> Optional[List[str]]:
             units.add("row_norm_kv")
         if cfg.is_moe_layer(i):
             units.add("moe")
+    if cfg.input_conv_taps:
+        units.add("conv1d")
     return sorted(units)
 
 

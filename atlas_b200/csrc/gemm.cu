@@ -70,10 +70,11 @@ struct GemmParams {
   int b_scale_ld;           // k-groups per row of b_scale
   int vec_ok;               // 16-byte stores into C are legal
   // bf16 kernels: columns from tail_col on are stored as fp32 in `tail` [M, N - tail_col] (null = off); `bias` [N] joins the
-  // sums; act 1 squares the positive part of every value before the store, act 2 takes neighbouring columns as gate and up of
-  // a gated unit (common.cuh) and stores N / 2 columns
+  // sums; act 1 squares the positive part of every value of the first relu_cols columns before the store, act 2 takes neighbouring
+  // columns as gate and up of a gated unit (common.cuh) and stores N / 2 columns
   float* tail; long long tail_ld; int tail_col, tail_vec;
   const float* bias; int act; GatedUnit unit;
+  int relu_cols;
   int cluster_splits;       // > 1: the K splits of a tile are the CTAs of one thread-block cluster (one item per CTA, a
                             // single m-tile): partials meet in distributed shared memory instead of the workspace and
                             // every CTA finishes 128 / cluster_splits rows of the tile (see cluster_tail)
@@ -1022,7 +1023,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 #pragma unroll
           for (int i = 0; i < HALF; ++i) {
             const float r = fmaxf(acc[i], 0.f);
-            acc[i] = r * r;
+            acc[i] = n_base + i < p.relu_cols ? r * r : acc[i];
           }
         }
         if (!FP8 && p.act == 2) {
@@ -1315,7 +1316,7 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
                      int num_sms, unsigned long long* status, void* stream, const uint32_t* a_ready,
                      const unsigned int* a_ready_epoch, long long max_cycles, const AtlasEpilogue* epi = nullptr,
                      float* tail = nullptr, long long tail_ld = 0, int tail_col = 0, const float* bias = nullptr, int act = 0,
-                     float glu_limit = 0.f, float glu_alpha = 0.f, float glu_shift = 0.f) {
+                     float glu_limit = 0.f, float glu_alpha = 0.f, float glu_shift = 0.f, int relu_cols = 0) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const uint32_t esize = kind == 1 ? 1 : 2;
   const int elems_per_row = 128 / esize;
@@ -1348,7 +1349,7 @@ static int gemm_impl(int kind, const void* A, const void* B, void* C, const floa
   p.status = status; p.ldc = ldc; p.sa_k = sa_k; p.M = M; p.N = N; p.K = K;
   p.epi_mode = epi_mode;
   p.tail = tail; p.tail_ld = tail_ld; p.tail_col = tail_col;
-  p.bias = bias; p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift};
+  p.bias = bias; p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift}; p.relu_cols = relu_cols;
   p.tail_vec = tail_col % 4 == 0 && tail_ld % 4 == 0 && (reinterpret_cast<uintptr_t>(tail) & 15) == 0 ? 1 : 0;
   if (epi) {
     p.act_cols = N / 2; p.q_out = reinterpret_cast<uint8_t*>(epi->q_out); p.ldq = epi->ldq; p.s_out = epi->s_out; p.s_ld = epi->s_ld;
@@ -1414,17 +1415,20 @@ extern "C" int atlas_gemm_tail(const void* A, const void* B, void* C, float* tai
                    stream, nullptr, nullptr, 0, nullptr, n_main < N ? tail : nullptr, tail_ld, n_main);
 }
 
-// bf16 GEMM with a bias row (fp32 [N] or null) and / or an activation in its epilogue: act 0 none, 1 relu squared, 2 gated
-// unit (common.cuh) of alternating gate and up columns (C has N / 2 columns).  tail (null = off): columns from n_main on leave as the
-// fp32 sums (with the bias, without the activation); n_main is a multiple of 16 then.
+// bf16 GEMM with a bias row (fp32 [N] or null) and / or an activation in its epilogue: act 0 none, 1 relu squared (of the first n_main
+// columns, or of all with n_main 0), 2 gated unit (common.cuh) of alternating gate and up columns (C has N / 2 columns).  tail (null =
+// off; act 0 or 2): columns from n_main on leave as the fp32 sums (with the bias, without the activation); with act 2 n_main is a
+// multiple of 16 then.
 extern "C" int atlas_gemm_bias_act(const void* A, const void* B, void* C, float* tail, long long tail_ld, int n_main, const float* bias, int act,
                                    float glu_limit, float glu_alpha, float glu_shift, int M,
                                    int N, int K, long long lda, long long ldb, long long ldc, int block_n, int splits, float* workspace,
                                    int* counters, int num_sms, unsigned long long* status, void* stream) {
   if (act < 0 || act > 2 || (act == 2 && !tail && N % 2)) return -46;
-  if (tail && (act != 2 || n_main % 16 || n_main < 0 || n_main >= N || tail_ld < N - n_main)) return -47;
+  if (tail && (act == 1 || (act == 2 && n_main % 16) || n_main < 0 || n_main >= N || tail_ld < N - n_main || (n_main > 0 && !C))) return -47;
+  if (act == 1 && (n_main < 0 || n_main > N)) return -48;
   return gemm_impl(0, A, B, C, nullptr, 0, 0, nullptr, 0, M, N, K, lda, ldb, ldc, block_n, splits, workspace, counters, num_sms, status,
-                   stream, nullptr, nullptr, 0, nullptr, tail, tail_ld, tail ? n_main : 0, bias, act, glu_limit, glu_alpha, glu_shift);
+                   stream, nullptr, nullptr, 0, nullptr, tail, tail_ld, tail ? n_main : 0, bias, act, glu_limit, glu_alpha, glu_shift,
+                   n_main > 0 ? n_main : N);
 }
 
 // All-gather -> GEMM: the rows of A (and their scales) are written into this rank's memory by the ranks that own them;
@@ -1488,7 +1492,7 @@ extern "C" int atlas_gemm_grouped(int kind, const void* A, const void* B, void* 
   p.n_tiles = N / block_n;
   p.b_scale_ld = p.k_blocks;
   p.vec_ok = ((ldc % 8) == 0 && (reinterpret_cast<uintptr_t>(C) & 15) == 0) ? 1 : 0;
-  p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift};
+  p.act = act; p.unit = GatedUnit{glu_limit, glu_alpha, glu_shift}; p.relu_cols = N;
   p.tile_expert = tile_expert; p.num_m_tiles_ptr = num_m_tiles; p.expert_n = N;
   p.ar_state = nullptr; p.ar_world = 1; p.ar_rank = 0; p.ar_mode = 0; p.ar_parity_stride = 0; p.prefetch_b = 0;
   p.rs_tiles_per_rank = 1; p.a_ready = nullptr; p.a_ready_epoch = nullptr; p.ar_max_cycles = kMbarMaxCycles;

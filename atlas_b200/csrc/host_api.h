@@ -188,9 +188,19 @@ int atlas_wkv_scan(const void* r, long long ldr, const void* k, long long ldk, c
                    const int* snap_slots, int snaps, int B, int H, int D, int commit, int one_row, int f32, void* stream);
 int atlas_group_norm_gate(const void* y, long long ldy, const void* z, long long ldz, const float* w, void* out, long long ldo, int rows,
                           int groups, int gsize, float eps, int gate_first, int sigmoid, const float* den, int f32, void* stream);
+// gate [rows, W] (activations' type): y times sigmoid(gate) ahead of its norm; b / out_b [W]: the norm with weight w / out_w is a layer norm;
+// hist [entries][rows, W], hist_ld numbers apart: the new x becomes entry hist_index and sum_j factors[j] * entry j (null: x) goes on
+typedef struct {
+  const void* gate; long long ldg;
+  const float* b; const float* out_b;
+  float* hist; long long hist_ld;
+  const float* factors; int hist_index;
+} AtlasNormedExtras;
 int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const void* extra,
                      long long lde, const float* w, const float* out_w, const float* step, void* out, long long ldo, int rows, int W, int plus_one,
-                     int store, int first, float eps, float scale, int f32, void* stream);
+                     int store, int first, float eps, float scale, int f32, const AtlasNormedExtras* extras, void* stream);
+int atlas_gelu_embedding(const void* z, long long ldz, const void* table, long long ldt, const long long* ids, int first, int n, int N, void* out,
+                         long long ldo, int rows, int f32, void* stream);
 int atlas_head_gate(void* x, long long ldx, const float* g, long long ldg, int rows, int H, int D, int f32, void* stream);
 
 // ---- RG-LRU (rglru.cu): arguments of both forms, see the entry points
@@ -247,10 +257,20 @@ int atlas_latent_pages(const void* kv, const void* cache, const int* block_table
                        void* v_pages, void* stream);
 int atlas_latent_unpad(const void* in, const int* rows, int n, int H, int vd, int dx, void* out, void* stream);
 
-// ---- recurrences (recurrent.cu), continued
+// ---- differential attention (differential.cu)
+int atlas_map_norm_kv_write(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, void* rows,
+                            const int* positions, const float* rope, const float* qw, const float* kw, void* k_cache, void* v_cache,
+                            const int* slot_mapping, int T, int H, int G, int dim, int dv, int D, int rotary, int block_size, float eps, int f32,
+                            void* stream);
+int atlas_map_difference(const void* a, const void* gate, long long ldg, void* out, int T, int H, int D, int dv, float lam, float rest, float eps,
+                         int f32, void* stream);
+
+// ---- short convolution (conv1d.cu)
 int atlas_conv1d_bias_silu(const void* x, long long ldx, const void* w, const void* bias, int C, int W, const void* state,
                            const int* seq_of_token, const int* qsl, const int* slots, const unsigned char* has, void* y, long long ldy,
                            int rows, int silu, int f32, void* stream);
+int atlas_conv1d_add(const void* x, long long ldx, const void* w, int C, int W, void* state, const int* seq_of_token, const int* qsl,
+                     const int* slots, const unsigned char* has, void* y, long long ldy, int rows, int advance, int f32, void* stream);
 int atlas_conv1d_state(const void* x, long long ldx, int C, int W, void* state, const int* qsl, const int* slots,
                        const unsigned char* has, const int* limit, const int* snap_rows, const int* snap_slots, int snaps, int B, int f32,
                        void* stream);

@@ -12,7 +12,9 @@
 //                           norm(y) * w * silu(z) (WKV) or norm(y / den) * w * sigmoid(z) (mLSTM)
 //   add_normed_kernel       one CTA per token: x += rmsnorm(y) * w or x += y on an fp32 residual, y being a sublayer's output or the
 //                           weighted sum of expert rows (and a shared expert's row); adds a step vector where one is given and hands
-//                           the new x on in the activations' dtype, normed again where asked
+//                           the new x on in the activations' dtype, normed again where asked; the rich form also gates y, takes
+//                           layer norms and sums over the results of all layers so far
+//   gelu_embedding_kernel   gelu_tanh(z) times a slice of a token's embedding row
 //   head_gate_kernel        x[t, h, :] *= sigmoid(g[t, h])
 //   gated_unit_kernel       g = min(gate, limit), u = clamp(up, +-limit):  g * sigmoid(alpha g) * (u + shift), of [gate | up] or of
 //                           alternating columns
@@ -333,10 +335,39 @@ struct AddNormedParams {
   T* out; long long ldo;
   int W, plus_one, store, first;               // first: x = y * scale (start of the model)
   float eps, scale;
+  // kRich only
+  const T* gate; long long ldg;                // y is multiplied by sigmoid(gate) first (null = off)
+  const float* b; const float* out_b;          // biases: the norm with that weight is a layer norm (null = RMS norm)
+  float* hist; long long hist_ld;              // results of the layers, [entries][T, W]: the new x becomes entry hist_index (null = off) ...
+  const float* factors; int hist_index;        // ... and sum_j factors[j] * entry j goes on in its place (null = x itself)
 };
 
+// subtracts the row's mean from y and returns the sum of squares of what is left
+template <int V, int NI>
+ATLAS_DEVICE float take_mean_off(float (&y)[NI][V], int W, int step, float* red) {
+  float s = 0.f;
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    if (threadIdx.x * V + k * step >= W) continue;
+#pragma unroll
+    for (int i = 0; i < V; ++i) s += y[k][i];
+  }
+  const float mean = block_sum(s, red) / (float)W;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NI; ++k) {
+    if (threadIdx.x * V + k * step >= W) continue;
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      y[k][i] -= mean;
+      ss += y[k][i] * y[k][i];
+    }
+  }
+  return ss;
+}
+
 // NI pieces of V elements per thread, the row stays in registers
-template <typename T, int V, int NI>
+template <typename T, int V, int NI, bool kRich>
 __global__ void __launch_bounds__(1024)
 add_normed_kernel(const AddNormedParams<T> p) {
   __shared__ float red[32];
@@ -373,11 +404,18 @@ add_normed_kernel(const AddNormedParams<T> p) {
         for (int i = 0; i < V; ++i) y[k][i] = fmaf(wj, f[i], y[k][i]);
       }
     }
+    if (kRich && p.gate) {
+      float g[V];
+      load_vec<V>(p.gate + t * p.ldg + e, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) y[k][i] /= 1.f + expf(-g[i]);
+    }
 #pragma unroll
     for (int i = 0; i < V; ++i) ss += y[k][i] * y[k][i];
   }
   const float plus = p.plus_one ? 1.f : 0.f;
   if (p.w) {
+    if (kRich && p.b) ss = take_mean_off<V, NI>(y, p.W, step, red);
     const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps);
     ss = 0.f;
 #pragma unroll
@@ -390,7 +428,16 @@ add_normed_kernel(const AddNormedParams<T> p) {
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         y[k][i] = fmaf(y[k][i] * rstd, w[i] + plus, x[i]);
-        ss += y[k][i] * y[k][i];
+        if (!(kRich && p.b)) ss += y[k][i] * y[k][i];
+      }
+      if (kRich && p.b) {
+        float b[V];
+        load_vec<V>(p.b + e, b);
+#pragma unroll
+        for (int i = 0; i < V; ++i) {
+          y[k][i] += b[i];
+          ss += y[k][i] * y[k][i];
+        }
       }
     }
   } else if (!p.first || p.scale != 1.f) {
@@ -427,17 +474,54 @@ add_normed_kernel(const AddNormedParams<T> p) {
       }
     }
   }
+  if (kRich && p.hist) {
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NI; ++k) {
+      const int e = threadIdx.x * V + k * step;
+      if (e >= p.W) continue;
+      const float* past = p.hist + t * p.W + e;
+      if (p.store) store_vec<V>(p.hist + p.hist_index * p.hist_ld + t * p.W + e, y[k]);
+      if (p.factors) {
+        const float own = __ldg(p.factors + p.hist_index);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] *= own;
+#pragma unroll 4
+        for (int j = 0; j < p.hist_index; ++j) {
+          const float fj = __ldg(p.factors + j);
+          float h[V];
+          load_vec<V>(past + j * p.hist_ld, h);
+#pragma unroll
+          for (int i = 0; i < V; ++i) y[k][i] = fmaf(fj, h[i], y[k][i]);
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += y[k][i] * y[k][i];
+    }
+  }
+  if (p.store) {
+#pragma unroll
+    for (int k = 0; k < NI; ++k) {
+      const int e = threadIdx.x * V + k * step;
+      if (e < p.W) store_vec<V>(p.x + t * p.ldx + e, y[k]);
+    }
+  }
+  if (kRich && p.out_b) ss = take_mean_off<V, NI>(y, p.W, step, red);
   const float orstd = p.out_w ? 1.f / sqrtf(block_sum(ss, red) / (float)p.W + p.eps) : 1.f;
 #pragma unroll
   for (int k = 0; k < NI; ++k) {
     const int e = threadIdx.x * V + k * step;
     if (e >= p.W) continue;
-    if (p.store) store_vec<V>(p.x + t * p.ldx + e, y[k]);
     if (p.out_w) {
       float w[V];
       load_vec<V>(p.out_w + e, w);
 #pragma unroll
       for (int i = 0; i < V; ++i) y[k][i] = y[k][i] * orstd * (w[i] + plus);
+      if (kRich && p.out_b) {
+        load_vec<V>(p.out_b + e, w);
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[k][i] += w[i];
+      }
     }
     store_vec<V>(p.out + t * p.ldo + e, y[k]);
   }
@@ -446,20 +530,25 @@ add_normed_kernel(const AddNormedParams<T> p) {
 template <typename T>
 static int add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks, const void* extra,
                       long long lde, const float* w, const float* out_w, const float* step, void* out, long long ldo, int rows, int W, int plus_one,
-                      int store, int first, float eps, float scale, cudaStream_t st) {
+                      int store, int first, float eps, float scale, const AtlasNormedExtras& o, cudaStream_t st) {
   AddNormedParams<T> p = {x, ldx, reinterpret_cast<const T*>(y), ldy, slot_of, pick_w, picks, reinterpret_cast<const T*>(extra), lde, w, out_w, step,
-                          reinterpret_cast<T*>(out), ldo, W, plus_one, store, first, eps, scale};
+                          reinterpret_cast<T*>(out), ldo, W, plus_one, store, first, eps, scale, reinterpret_cast<const T*>(o.gate), o.ldg, o.b,
+                          o.out_b, o.hist, o.hist_ld, o.factors, o.hist_index};
+  const bool rich = o.gate || o.b || o.out_b || o.hist;
   const bool vec = W % 8 == 0 && vec_ok<T, 8>(y, ldy) && vec_ok<T, 8>(out, ldo) && vec_ok<float, 4>(x, ldx) && vec_ok<float, 4>(w, 0) &&
-                   vec_ok<float, 4>(out_w, 0) && vec_ok<float, 4>(step, 0) && vec_ok<T, 8>(extra, lde);
+                   vec_ok<float, 4>(out_w, 0) && vec_ok<float, 4>(step, 0) && vec_ok<T, 8>(extra, lde) && vec_ok<T, 8>(o.gate, o.ldg) &&
+                   vec_ok<float, 4>(o.b, 0) && vec_ok<float, 4>(o.out_b, 0) && vec_ok<float, 4>(o.hist, o.hist_ld);
   const int v = vec ? 8 : 1, pieces = (W + v - 1) / v;
   void (*k)(const AddNormedParams<T>) = nullptr;
   int ni = 1;
   if (vec) {
     ni = pieces <= 1024 ? 1 : 4;
-    k = ni == 1 ? add_normed_kernel<T, 8, 1> : add_normed_kernel<T, 8, 4>;
+    k = ni == 1 ? (rich ? add_normed_kernel<T, 8, 1, true> : add_normed_kernel<T, 8, 1, false>)
+                : (rich ? add_normed_kernel<T, 8, 4, true> : add_normed_kernel<T, 8, 4, false>);
   } else {
     ni = pieces <= 1024 ? 1 : 32;
-    k = ni == 1 ? add_normed_kernel<T, 1, 1> : add_normed_kernel<T, 1, 32>;
+    k = ni == 1 ? (rich ? add_normed_kernel<T, 1, 1, true> : add_normed_kernel<T, 1, 1, false>)
+                : (rich ? add_normed_kernel<T, 1, 32, true> : add_normed_kernel<T, 1, 32, false>);
   }
   const int threads = ((pieces + ni - 1) / ni + 31) / 32 * 32;
   if (threads > 1024) return -2;
@@ -519,6 +608,41 @@ static int launch_glu(const void* gu, long long ld, int rows, int I, void* y, lo
   dim3 grid(rows, (I + 256 * V - 1) / (256 * V));
   launch_chain_if(rows <= 256, gated_unit_kernel<T, V, kPaired>, grid, dim3(256), 0, st, reinterpret_cast<const T*>(gu), ld, I,
                   reinterpret_cast<T*>(y), ldy, unit);
+  return cudaGetLastError() == cudaSuccess ? 0 : -21;
+}
+
+// one thread per piece of V columns of a row
+template <typename T, int V>
+__global__ void __launch_bounds__(256)
+gelu_embedding_kernel(const T* __restrict__ z, long long ldz, const T* __restrict__ table, long long ldt, const long long* __restrict__ ids, int first,
+                      int n, int N, T* out, long long ldo, int rows) {
+  chain_trigger();
+  chain_wait();
+  const int pieces = N / V;
+  const long long unit = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (unit >= (long long)rows * pieces) return;
+  const long long t = unit / pieces;
+  const int e = (int)(unit % pieces) * V;
+  float o[V] = {};
+  if (e < n) {
+    float f[V];
+    load_vec<V>(z + t * ldz + e, o);
+    load_vec<V>(table + ids[t] * ldt + first + e, f);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      const float u = 0.7978845608028654f * (o[i] + 0.044715f * o[i] * o[i] * o[i]);
+      o[i] = 0.5f * o[i] * (1.f + tanhf(u)) * f[i];
+    }
+  }
+  store_vec<V>(out + t * ldo + e, o);
+}
+
+template <typename T, int V>
+static int launch_gelu_embedding(const void* z, long long ldz, const void* table, long long ldt, const long long* ids, int first, int n, int N,
+                                 void* out, long long ldo, int rows, cudaStream_t st) {
+  const long long units = (long long)rows * (N / V);
+  launch_chain_if(rows <= 256, gelu_embedding_kernel<T, V>, dim3((unsigned)((units + 255) / 256)), dim3(256), 0, st, reinterpret_cast<const T*>(z), ldz,
+                  reinterpret_cast<const T*>(table), ldt, ids, first, n, N, reinterpret_cast<T*>(out), ldo, rows);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 
@@ -615,18 +739,37 @@ extern "C" int atlas_group_norm_gate(const void* y, long long ldy, const void* z
 
 // fp32 residual x [rows, W]: x += rmsnorm(y) * w (w null: x += y; first: x = y * scale), then x += step (null: nothing), out = x or
 // rmsnorm(x) * out_w.  picks > 0: y [*, W] holds expert rows, slot_of / pick_w [rows, picks].  extra [rows, W] joins y.  With plus_one
-// the weights are stored around zero; store = 0 leaves x as it is.
+// the weights are stored around zero; store = 0 leaves x (and the history) as it is.  extras (null = none): see host_api.h.
 extern "C" int atlas_add_normed(float* x, long long ldx, const void* y, long long ldy, const int* slot_of, const float* pick_w, int picks,
                                 const void* extra, long long lde, const float* w, const float* out_w, const float* step, void* out,
                                 long long ldo, int rows, int W, int plus_one, int store, int first, float eps, float scale, int f32,
-                                void* stream) {
+                                const AtlasNormedExtras* extras, void* stream) {
   if (rows <= 0) return 0;
   if (W < 1 || W > 32768 || picks < 0 || (picks > 0 && (!slot_of || !pick_w)) || (first && w)) return -1;
+  const AtlasNormedExtras o = extras ? *extras : AtlasNormedExtras{};
+  if (o.hist && (o.hist_ld < (long long)rows * W || o.hist_index < 0)) return -3;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   return f32 ? add_normed<float>(x, ldx, y, ldy, slot_of, pick_w, picks, extra, lde, w, out_w, step, out, ldo, rows, W, plus_one, store, first, eps,
-                                 scale, st)
+                                 scale, o, st)
              : add_normed<__nv_bfloat16>(x, ldx, y, ldy, slot_of, pick_w, picks, extra, lde, w, out_w, step, out, ldo, rows, W, plus_one, store,
-                                         first, eps, scale, st);
+                                         first, eps, scale, o, st);
+}
+
+// out [rows, N] = gelu_tanh(z) * table[ids[row], first + column] in the first n columns, 0 in the others
+extern "C" int atlas_gelu_embedding(const void* z, long long ldz, const void* table, long long ldt, const long long* ids, int first, int n, int N,
+                                    void* out, long long ldo, int rows, int f32, void* stream) {
+  if (rows <= 0 || N <= 0) return 0;
+  if (n < 0 || n > N || first < 0 || first + n > ldt) return -1;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (f32) {
+    const bool vec = n % 4 == 0 && N % 4 == 0 && first % 4 == 0 && vec_ok<float, 4>(z, ldz) && vec_ok<float, 4>(table, ldt) && vec_ok<float, 4>(out, ldo);
+    return vec ? launch_gelu_embedding<float, 4>(z, ldz, table, ldt, ids, first, n, N, out, ldo, rows, st)
+               : launch_gelu_embedding<float, 1>(z, ldz, table, ldt, ids, first, n, N, out, ldo, rows, st);
+  }
+  using B = __nv_bfloat16;
+  const bool vec = n % 8 == 0 && N % 8 == 0 && first % 8 == 0 && vec_ok<B, 8>(z, ldz) && vec_ok<B, 8>(table, ldt) && vec_ok<B, 8>(out, ldo);
+  return vec ? launch_gelu_embedding<B, 8>(z, ldz, table, ldt, ids, first, n, N, out, ldo, rows, st)
+             : launch_gelu_embedding<B, 1>(z, ldz, table, ldt, ids, first, n, N, out, ldo, rows, st);
 }
 
 // x [rows, H, D] (row stride ldx) times sigmoid(g [rows, H]), in place

@@ -445,18 +445,19 @@ def gemm_fp8_fused(xq, xs, wq, ws, mode: int = 0, out=None, residual=None, norm_
 
 
 def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.Tensor] = None, unit: Optional[Tuple[float, float, float]] = None,
-              n_main: Optional[int] = None):
+              n_main: Optional[int] = None, relu2_cols: int = 0):
     """``x @ w^T (+ bias)``; with ``unit = (limit, alpha, shift)`` the gated unit of alternating gate and up columns, ``[M, N / 2]``.
     ``n_main`` (a multiple of 16, with ``unit``): columns from there on are no part of the unit and leave as fp32 sums; returns
-    ``(out [M, n_main / 2], tail [M, N - n_main])``."""
+    ``(out [M, n_main / 2], tail [M, N - n_main])``.  ``relu2_cols``: the first so many columns leave as ``relu(.) ** 2``."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
+    assert not relu2_cols or (unit is None and relu2_cols <= w.shape[0])
     if x.shape[1] % 8:                 # rows that TMA cannot address (16-byte strides): a vendor product
-        assert unit is None
+        assert unit is None and not relu2_cols
         y = torch.nn.functional.linear(x, w, None if bias is None else bias.to(x.dtype))
         return y if out is None else out.copy_(y)
     if x.stride(1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
-    if bias is None and unit is None:
+    if bias is None and unit is None and not relu2_cols:
         return _gemm(0, x, w, None, None, out)
     M, K = x.shape
     N = w.shape[0]
@@ -471,9 +472,7 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.T
         assert bias.numel() == N
         bias = _float_cached(bias)
     L = lib()
-    if not getattr(L, "_bias_act_bound", False):
-        L.atlas_gemm_bias_act.argtypes = [_vp, _vp, _vp, _vp, _ll, _i, _vp, _i, _f, _f, _f, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
-        L._bias_act_bound = True
+    _bind_bias_act(L)
     sms = _num_sms[d]
     bn, splits = gemm_plan(M, N, K, 0, sms)
     ws = cnt = None
@@ -481,11 +480,17 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, out=None, bias: Optional[torch.T
         ws = scratch("gemm_ws", _GEMM_WS_BYTES, x.device)
         cnt = scratch("gemm_counters", 1 << 18, x.device)
     limit, alpha, shift = unit or (0.0, 0.0, 0.0)
-    _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(tail), N - n_main if n_main is not None else 0, n_main or 0,
-                                 _ptr(bias), 0 if unit is None else 2, float(limit), float(alpha), float(shift), M, N,
+    _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), out.data_ptr(), _ptr(tail), N - n_main if n_main is not None else 0,
+                                 relu2_cols or n_main or 0, _ptr(bias), 1 if relu2_cols else (0 if unit is None else 2), float(limit), float(alpha), float(shift), M, N,
                                  K, x.stride(0), w.stride(0), out.stride(0), bn, splits, _ptr(ws), _ptr(cnt), sms, _status_ptr[d], _stream()),
            "gemm_bias_act")
     return out if tail is None else (out, tail)
+
+
+def _bind_bias_act(L) -> None:
+    if not getattr(L, "_bias_act_bound", False):
+        L.atlas_gemm_bias_act.argtypes = [_vp, _vp, _vp, _vp, _ll, _i, _vp, _i, _f, _f, _f, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
+        L._bias_act_bound = True
 
 
 _float_cache: dict = {}
@@ -501,19 +506,24 @@ def _float_cached(t: torch.Tensor) -> torch.Tensor:
     return hit[1]
 
 
-def linear_tail(x: torch.Tensor, w: torch.Tensor, n_main: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """bf16 product whose columns from ``n_main`` on stay fp32: ``(main [M, n_main] bf16, tail [M, N - n_main] fp32)``."""
+def linear_tail(x: torch.Tensor, w: torch.Tensor, n_main: int, bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """bf16 product (plus ``bias``) whose columns from ``n_main`` on stay fp32: ``(main [M, n_main] bf16, tail [M, N - n_main] fp32)``."""
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.stride(1) == 1
     M, K = x.shape
     N = w.shape[0]
     d = _dev(x)
     if K % 8:                          # rows that TMA cannot address (16-byte strides): vendor products
-        return torch.nn.functional.linear(x, w[:n_main]), torch.nn.functional.linear(x.float(), w[n_main:].float())
+        b = (None, None) if bias is None else (bias[:n_main].to(x.dtype), bias[n_main:].float())
+        return torch.nn.functional.linear(x, w[:n_main], b[0]), torch.nn.functional.linear(x.float(), w[n_main:].float(), b[1])
     if x.stride(1) != 1 or (x.stride(0) * 2) % 16 or x.data_ptr() % 16:
         x = x.contiguous()
     main = torch.empty(M, n_main, dtype=torch.bfloat16, device=x.device)
     tail = torch.empty(M, N - n_main, dtype=torch.float32, device=x.device)
     L = lib()
+    if bias is not None:
+        assert bias.numel() == N
+        bias = _float_cached(bias)
+    _bind_bias_act(L)
     if not getattr(L, "_tail_bound", False):
         L.atlas_gemm_tail.argtypes = [_vp, _vp, _vp, _vp, _ll, _i, _i, _i, _i, _ll, _ll, _ll, _i, _i, _vp, _vp, _i, _vp, _vp]
         L._tail_bound = True
@@ -523,6 +533,12 @@ def linear_tail(x: torch.Tensor, w: torch.Tensor, n_main: int) -> Tuple[torch.Te
     if splits > 1:
         ws = scratch("gemm_ws", _GEMM_WS_BYTES, x.device)
         cnt = scratch("gemm_counters", 1 << 18, x.device)
+    if bias is not None and n_main < N:
+        _check(L.atlas_gemm_bias_act(x.data_ptr(), w.data_ptr(), main.data_ptr() if n_main else None, tail.data_ptr(), N - n_main, n_main,
+                                     bias.data_ptr(), 0, 0.0, 0.0, 0.0, M, N, K, x.stride(0), w.stride(0), n_main, bn, splits, _ptr(ws),
+                                     _ptr(cnt), sms, _status_ptr[d], _stream()), "gemm_tail")
+        return main, tail
+    assert bias is None
     _check(L.atlas_gemm_tail(x.data_ptr(), w.data_ptr(), main.data_ptr() if n_main else None, tail.data_ptr() if n_main < N else None, N - n_main,
                              n_main, M, N, K, x.stride(0), w.stride(0), n_main, bn, splits, _ptr(ws), _ptr(cnt), sms, _status_ptr[d], _stream()),
            "gemm_tail")
@@ -1017,9 +1033,34 @@ def group_norm_gate(y, z, w, group, eps, gate_first, gate="silu", den=None):
     return cuda_recurrent.group_norm_gate(y, z, w, group, eps, gate_first, gate, den)
 
 
-def add_normed(stream, delta, eps, plus_one, out_norm, write, step=None):
+def input_conv(layer, h, batch, state, commit):
     from . import cuda_recurrent
-    return cuda_recurrent.add_normed(stream, delta, eps, plus_one, out_norm, write, step)
+    return cuda_recurrent.input_conv(layer, h, batch, state, commit)
+
+
+def input_conv_commit(layer, h, qlens, slots, has_state, state, num_accepted_rows):
+    from . import cuda_recurrent
+    return cuda_recurrent.input_conv_commit(layer, h, qlens, slots, has_state, state, num_accepted_rows)
+
+
+def map_norm_kv_write(*args):
+    from . import cuda_differential
+    return cuda_differential.map_norm_kv_write(*args)
+
+
+def map_difference(a, dv, lam, rest, eps, gate):
+    from . import cuda_differential
+    return cuda_differential.map_difference(a, dv, lam, rest, eps, gate)
+
+
+def gelu_embedding(z, table, ids, first, n):
+    from . import cuda_recurrent
+    return cuda_recurrent.gelu_embedding(z, table, ids, first, n)
+
+
+def add_normed(stream, delta, eps, plus_one, out_norm, write, step=None, out_bias=None):
+    from . import cuda_recurrent
+    return cuda_recurrent.add_normed(stream, delta, eps, plus_one, out_norm, write, step, out_bias)
 
 
 def head_gate(x, g):

@@ -1,5 +1,5 @@
 """Binding of the residual-stream, recurrence and 32-bit attention kernels (``csrc/streams.cu``, ``csrc/recurrent.cu``,
-``csrc/mlstm.cu``, ``csrc/rglru.cu``, ``csrc/row_norm_kv.cu``, ``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
+``csrc/conv1d.cu``, ``csrc/mlstm.cu``, ``csrc/rglru.cu``, ``csrc/row_norm_kv.cu``, ``csrc/attention_f32.cu``).  Activations are bf16 or fp32; every entry point takes the choice as its ``f32`` flag."""
 from __future__ import annotations
 
 import ctypes as C
@@ -23,6 +23,11 @@ class _Rglru(C.Structure):
                 ("n", _i), ("taps", _i), ("commit", _i), ("one_row", _i)]
 
 
+class _NormedExtras(C.Structure):
+    """Mirror of ``AtlasNormedExtras`` (csrc/host_api.h)."""
+    _fields_ = [("gate", _vp), ("ldg", _ll), ("b", _vp), ("out_b", _vp), ("hist", _vp), ("hist_ld", _ll), ("factors", _vp), ("hist_index", _i)]
+
+
 def _lib():
     global _bound
     lib = K.lib()
@@ -38,7 +43,9 @@ def _lib():
         lib.atlas_wkv_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _vp, _ll, _vp, _ll, _vp, _i, _vp, _vp, _vp,
                                        _vp, _vp, _vp] + [_i] * 7 + [_vp]
         lib.atlas_group_norm_gate.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _ll, _i, _i, _i, _f, _i, _i, _vp, _i, _vp]
-        lib.atlas_add_normed.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _i, _vp, _ll, _vp, _vp, _vp, _vp, _ll] + [_i] * 5 + [_f, _f, _i, _vp]
+        lib.atlas_add_normed.argtypes = [_vp, _ll, _vp, _ll, _vp, _vp, _i, _vp, _ll, _vp, _vp, _vp, _vp, _ll] + [_i] * 5 + [_f, _f, _i, C.POINTER(_NormedExtras), _vp]
+        lib.atlas_gelu_embedding.argtypes = [_vp, _ll, _vp, _ll, _vp, _i, _i, _i, _vp, _ll, _i, _i, _vp]
+        lib.atlas_conv1d_add.argtypes = [_vp, _ll, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _ll, _i, _i, _i, _vp]
         lib.atlas_head_gate.argtypes = [_vp, _ll, _vp, _ll, _i, _i, _i, _i, _vp]
         lib.atlas_mlstm_gates.argtypes = [_vp, _ll, _vp, _f] + [_vp] * 10 + [_i] * 4 + [_vp]
         lib.atlas_mlstm_scan.argtypes = [_vp, _ll, _vp, _ll, _vp, _ll, _vp, _vp, _vp, _f, _vp, _vp, _ll] + [_vp] * 7 + [_i] * 8 + [_vp]
@@ -304,7 +311,7 @@ def rglru_commit(layer, x, qlens, slots, has_state, state, num_accepted_rows):
 
 
 # ----------------------------------------------------------------------------- sublayer outputs on an fp32 residual
-def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool, out_norm, write: bool, step=None):
+def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool, out_norm, write: bool, step=None, out_bias=None):
     rows = delta.y if hasattr(delta.y, "slot_of") else None
     y = rows.y if rows is not None else delta.y
     W = y.shape[1]
@@ -316,7 +323,20 @@ def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool
         assert delta.norm is None
         stream, write = torch.empty(T, W, dtype=torch.float32, device=y.device), True
     assert stream.dtype == torch.float32 and stream.shape == (T, W) and stream.is_contiguous()
-    for w in (delta.norm, out_norm, step):
+    gate, depth = delta.gate, delta.depth
+    extras = None
+    if gate is not None or delta.bias is not None or out_bias is not None or depth is not None:
+        extras = _NormedExtras(b=K._ptr(delta.bias), out_b=K._ptr(out_bias))
+        if gate is not None:
+            assert gate.dtype == y.dtype and gate.shape == (T, W) and gate.stride(1) == 1
+            extras.gate, extras.ldg = gate.data_ptr(), gate.stride(0)
+        if depth is not None:
+            hist, fac = depth.history, depth.factors
+            assert hist.dtype == torch.float32 and hist.is_contiguous() and hist.shape[1:] == (T, W) and 0 <= depth.index < hist.shape[0]
+            assert fac is None or (fac.dtype == torch.float32 and fac.is_contiguous() and fac.numel() == depth.index + 1)
+            extras.hist, extras.hist_ld, extras.factors, extras.hist_index = hist.data_ptr(), T * W, K._ptr(fac), depth.index
+    assert (delta.bias is None or delta.norm is not None) and (out_bias is None or out_norm is not None)
+    for w in (delta.norm, out_norm, step, delta.bias, out_bias):
         assert w is None or (w.dtype == torch.float32 and w.numel() == W and w.is_contiguous())
     if rows is not None:
         assert rows.slot_of.dtype == torch.int32 and rows.w.dtype == torch.float32 and rows.w.is_contiguous()
@@ -328,8 +348,46 @@ def add_normed(stream: Optional[torch.Tensor], delta, eps: float, plus_one: bool
                                      K._ptr(rows.w) if rows is not None else None, rows.w.shape[1] if rows is not None else 0,
                                      K._ptr(extra), extra.stride(0) if extra is not None else 0, K._ptr(delta.norm), K._ptr(out_norm),
                                      K._ptr(step), out.data_ptr(), W, T, W, 1 if plus_one else 0, 1 if write else 0, 1 if first else 0, float(eps),
-                                     float(delta.scale), f32, K._stream()), "add_normed")
+                                     float(delta.scale), f32, C.byref(extras) if extras is not None else None, K._stream()), "add_normed")
     return out, stream
+
+
+def gelu_embedding(z, table, ids, first: int, n: int):
+    T, N = z.shape
+    K._dev(z)
+    assert table.dtype == z.dtype and table.is_contiguous() and ids.dtype == torch.int64 and ids.is_contiguous() and ids.numel() == T
+    out = torch.empty(T, N, dtype=z.dtype, device=z.device)
+    K._check(_lib().atlas_gelu_embedding(z.data_ptr(), z.stride(0), table.data_ptr(), table.shape[1], ids.data_ptr(), int(first), int(n), N,
+                                         out.data_ptr(), N, T, _f32(z), K._stream()), "gelu_embedding")
+    return out
+
+
+# ----------------------------------------------------------------------------- convolution on a sublayer's input
+def _input_conv_state(layer, h, meta: _Meta, win) -> None:
+    K._check(_lib().atlas_conv1d_state(h.data_ptr(), h.stride(0), layer.width, layer.W, win.data_ptr(), meta.qsl.data_ptr(), meta.slots.data_ptr(),
+                                       meta.has.data_ptr(), K._ptr(meta.limit), meta.snap_rows.data_ptr(), meta.snap_slots.data_ptr(), meta.snaps,
+                                       meta.B, _f32(h), K._stream()), "conv1d_state")
+
+
+def input_conv(layer, h, batch, state, commit: bool):
+    meta, win = step_meta(batch, h.device), state["inputs"]
+    T, W = h.shape
+    K._dev(h)
+    f32 = _f32(h)
+    assert W == layer.width and win.dtype == h.dtype == layer.w.dtype and win.is_contiguous() and layer.w.is_contiguous()
+    out = torch.empty(T, W, dtype=h.dtype, device=h.device)
+    advance = commit and meta.one_row
+    K._check(_lib().atlas_conv1d_add(h.data_ptr(), h.stride(0), layer.w.data_ptr(), W, layer.W, win.data_ptr(), meta.seq_of.data_ptr(),
+                                     meta.qsl.data_ptr(), meta.slots.data_ptr(), meta.has.data_ptr(), out.data_ptr(), W, T, 1 if advance else 0, f32,
+                                     K._stream()), "conv1d_add")
+    if commit and not advance:
+        _input_conv_state(layer, h, meta, win)
+    return out
+
+
+def input_conv_commit(layer, h, qlens, slots, has_state, state, num_accepted_rows):
+    K._dev(h)
+    _input_conv_state(layer, h, _Meta(qlens, slots, has_state, h.device, None, limit=list(num_accepted_rows)), state["inputs"])
 
 
 def head_gate(x, g):
