@@ -422,7 +422,7 @@ def add_normed(stream, delta, eps: float, plus_one: bool, out_norm, write: bool,
     if write and stream is not None:
         stream.copy_(x)
     h = x if out_norm is None else unit(x, out_norm, out_bias)
-    return h.to(dtype), (x if stream is None else stream)
+    return h.to(dtype), (x.clone() if stream is None else stream)      # the stream changes in place, h does not
 
 
 def gelu_embedding(z, table, ids, first: int, n: int):
