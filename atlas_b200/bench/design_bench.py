@@ -1,14 +1,14 @@
 """Prefill and decode throughput of a design's layers beside the closest other model at equal size, and the rooflines of their
 kernels.
 
-    python bench.py --design papidra|tomizen|kenovik    # or: python -m atlas_b200.bench.design_bench --design ...
+    python bench.py --design papidra|tomizen|kenovik|bisudra    # or: python -m atlas_b200.bench.design_bench --design ...
 
 ``papidra`` beside Nemotron-H: the same width, feed-forward size, attention heads, Mamba-2 heads, vocabulary and cache dtype.  One
 period is, for Papidra, a WKV layer and a layer with attention beside Mamba-2 plus a feed-forward; for Nemotron-H the blocks with
 the same work: Mamba-2, attention, Mamba-2, MLP.
 
 ``tomizen`` (tomizen_bench.py) beside Qwen3-Next, and its latent attention beside DeepSeek's; ``kenovik`` (kenovik_bench.py) beside
-Qwen3-Next.
+Qwen3-Next; ``bisudra`` (bisudra_bench.py) beside Kenovik's attention layers.
 
 All with random bf16 weights.  Steps are timed with CUDA events around a captured step (L2 flushed in between), kernels the same
 way one by one.
@@ -164,10 +164,11 @@ def kernel_table(size: str, timer, peaks) -> List[dict]:
 
 def designs() -> dict:
     """name -> (name of the model beside it, sizes, configuration of both by size, kernel table, layers)"""
-    from . import kenovik_bench as V, tomizen_bench as T
+    from . import bisudra_bench as B, kenovik_bench as V, tomizen_bench as T
     return {"papidra": ("nemotron_h", SIZES, papidra, nemotron, kernel_table, f"{PERIODS} periods"),
             "tomizen": ("qwen3_next", T.SIZES, T.tomizen, T.beside, T.kernel_table, "4 layers"),
-            "kenovik": ("qwen3_next", V.SIZES, V.kenovik, V.beside, V.kernel_table, "4 layers")}
+            "kenovik": ("qwen3_next", V.SIZES, V.kenovik, V.beside, V.kernel_table, "4 layers"),
+            "bisudra": ("kenovik", B.SIZES, B.bisudra, B.beside, B.kernel_table, "4 layers")}
 
 
 def run(sizes: Optional[List[str]] = None, kernels: bool = True, design: str = "papidra") -> dict:
@@ -203,7 +204,7 @@ def report(res: dict) -> str:
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default="papidra", choices=["papidra", "tomizen", "kenovik"])
+    ap.add_argument("--design", default="papidra", choices=["papidra", "tomizen", "kenovik", "bisudra"])
     ap.add_argument("--sizes", default="", help="widths (default: all of the design)")
     ap.add_argument("--no-kernels", action="store_true")
     ap.add_argument("--out")

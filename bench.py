@@ -158,7 +158,7 @@ def main():
     ap.add_argument("--ssm-cache-slots", type=int, default=0, help="hybrid models: snapshot slots (0 = concurrency + 8)")
     ap.add_argument("--comm", default="p2p", choices=["p2p", "nccl"],
                     help="tensor-parallel collectives: this engine's peer-memory kernels (default) or the NCCL baseline")
-    ap.add_argument("--design", default=None, choices=["papidra", "tomizen", "kenovik"],
+    ap.add_argument("--design", default=None, choices=["papidra", "tomizen", "kenovik", "bisudra"],
                     help="instead of the headline workload: prefill / decode throughput of this design's layers at a few sizes beside "
                          "the closest other model (one GPU; prints one JSON line)")
     args = ap.parse_args()

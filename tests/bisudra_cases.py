@@ -73,8 +73,8 @@ def weights(cfg, seed=0):
         put(x + "q", H * 2 * D, W)
         put(x + "k", G * 2 * D, W)
         put(x + "v", G * V, W)
-        put(x + "q.norm", D, std=0.3, mean=2.0)
-        put(x + "k.norm", D, std=0.3, mean=1.5)
+        put(x + "q.norm", D, std=0.3, mean=1.4)
+        put(x + "k.norm", D, std=0.3, mean=1.3)
         for n in ("lq1", "lk1", "lq2", "lk2"):
             put(x + n, D, std=0.6 * D ** -0.25)
         put(x + "g", H * V, W, std=2 * W ** -0.5)
@@ -167,5 +167,6 @@ def standing_out(device, dtype, heads, kv, dim, vdim, size, rot, total, rows, ke
                                    kn.to(device), eps)
         got = ops.paged_attention(rq, kc, vc, fb, scale, sliding_window=size or None)
     got = got.view(rows, heads, 2, D)[..., :vdim].cpu().double()
-    want = O.map_outputs(unit(q, pos), unit(k, pos), v.double(), scale, O.window(total, size))[-rows:]
+    held = lambda x: unit(x, pos).to(dtype).double()                  # queries and cached keys are held in the activations' dtype
+    want = O.map_outputs(held(q), held(k), v.double(), scale, O.window(total, size))[-rows:]
     return got, want
