@@ -13,17 +13,17 @@
 namespace atlas {
 
 constexpr int kMaxTaps = 16;
-constexpr int kConvRows = 8;                   // consecutive rows of one thread (kTaps > 0: the window stays in registers)
+constexpr int kConvRows = 8;                   // consecutive rows of one thread in large steps (kTaps > 0: the window stays in registers)
 
 enum ConvAfter { kConvPlain = 0, kConvSilu = 1, kConvAddInput = 2 };
 
 // kTaps: number of taps known at compile time (0 = p.W, at most kMaxTaps, inputs re-read per row).  advance (one row per sequence):
-// every thread replaces the window of its channels by the one that ends with its row.
+// every thread replaces the window of its channels by the one that ends with its row.  span: rows of a block.
 template <typename T, int kTaps, int V>
 __global__ void __launch_bounds__(256)
 conv1d_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, const T* __restrict__ bias, int C, int W,
               T* state, const int* __restrict__ seq_of_token, const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
-              const unsigned char* __restrict__ has_state, T* y, long long ldy, int rows, int after, int advance) {
+              const unsigned char* __restrict__ has_state, T* y, long long ldy, int rows, int after, int advance, int span) {
   chain_trigger();
   chain_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -48,7 +48,29 @@ conv1d_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ w, c
         f[v] = live ? to_f32(state[(slot * C + c + v) * (taps - 1) + (taps - 1) - (back - rel)]) : 0.f;
     }
   };
-  const int t0 = blockIdx.x * kConvRows, t1 = min(rows, t0 + kConvRows);
+  const int t0 = blockIdx.x * span, t1 = min(rows, t0 + span);
+  if constexpr (kTaps > 0 && V > 1) {
+    // all rows inside one portion, the window too: every load in flight at once
+    const int b = seq_of_token[t0];
+    if (t1 - t0 == kConvRows && seq_of_token[t1 - 1] == b && t0 - query_start_loc[b] >= kN - 1) {
+      float in[kN - 1 + kConvRows][V];
+#pragma unroll
+      for (int r = 0; r < kN - 1 + kConvRows; ++r) load_vec<V>(x + (long long)(t0 - (kN - 1) + r) * ldx + c, in[r]);
+#pragma unroll
+      for (int r = 0; r < kConvRows; ++r) {
+        float acc[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+          acc[v] = bs[v];
+#pragma unroll
+          for (int i = 0; i < kN; ++i) acc[v] = fmaf(in[r + i][v], wt[i][v], acc[v]);
+          acc[v] = after == kConvSilu ? acc[v] * sigmoid_for<T>(acc[v]) : (after == kConvAddInput ? acc[v] + in[r + kN - 1][v] : acc[v]);
+        }
+        store_vec<V>(y + (long long)(t0 + r) * ldy + c, acc);
+      }
+      return;
+    }
+  }
   int seq = -1, q0 = 0;
   long long slot = 0;
   bool live = false;
@@ -188,13 +210,14 @@ static int launch_conv(const void* x, long long ldx, const void* w, const void* 
   const T *xp = reinterpret_cast<const T*>(x), *wp = reinterpret_cast<const T*>(w), *bp = reinterpret_cast<const T*>(bias);
   T* sp = reinterpret_cast<T*>(state);
   T* yp = reinterpret_cast<T*>(y);
-  const unsigned gx = (rows + kConvRows - 1) / kConvRows;
+  const int span = rows <= 256 ? 1 : kConvRows;
+  const unsigned gx = (rows + span - 1) / span;
   if (kTaps > 0 && rows > 256 && C % 4 == 0 && vec_ok<T, 4>(x, ldx) && vec_ok<T, 4>(y, ldy))
     launch_chain_if(false, conv1d_kernel<T, kTaps, (kTaps > 0 ? 4 : 1)>, dim3(gx, (C + 1023) / 1024), dim3(256), 0, st, xp, ldx, wp, bp, C, W,
-                    sp, seq, qsl, slots, has, yp, ldy, rows, after, advance);
+                    sp, seq, qsl, slots, has, yp, ldy, rows, after, advance, span);
   else
     launch_chain_if(rows <= 256, conv1d_kernel<T, kTaps, 1>, dim3(gx, (C + 255) / 256), dim3(256), 0, st, xp, ldx, wp, bp, C, W, sp, seq, qsl,
-                    slots, has, yp, ldy, rows, after, advance);
+                    slots, has, yp, ldy, rows, after, advance, span);
   return cudaGetLastError() == cudaSuccess ? 0 : -21;
 }
 

@@ -207,14 +207,14 @@ map_difference_kernel(const MapDifferenceParams<T> p) {
     float g[8];
     if (gate) load_vec<8>(gate + e, g);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) o[i] = gate ? o[i] * f / (1.f + expf(-g[i])) : o[i] * f;
+    for (int i = 0; i < 8; ++i) o[i] = gate ? o[i] * f * sigmoid_for<T>(g[i]) : o[i] * f;
     store_vec<8>(out + e, o);
   }
   if (!kVec) {
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
       const int d = i * 32 + lane;
-      if (live && d < p.dv) out[d] = from_f32<T>(gate ? o[i] * f / (1.f + expf(-to_f32(gate[d]))) : o[i] * f);
+      if (live && d < p.dv) out[d] = from_f32<T>(gate ? o[i] * f * sigmoid_for<T>(to_f32(gate[d])) : o[i] * f);
     }
   }
 }

@@ -634,12 +634,12 @@ shared_expert_blend_kernel(__nv_bfloat16* y, long long ldy, const __nv_bfloat16*
   }
 }
 
-// y = relu(x)^2, eight bf16 per thread
+// y = relu(x)^2, eight bf16 per thread (vec: rows start on 16-byte boundaries)
 __global__ void __launch_bounds__(256)
-relu2_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* y, long long ldy, int cols) {
+relu2_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* y, long long ldy, int cols, int vec) {
   const long long t = blockIdx.x;
   for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8; c < cols; c += gridDim.y * blockDim.x * 8) {
-    if (c + 8 <= cols) {
+    if (vec && c + 8 <= cols) {
       const uint4 v = *reinterpret_cast<const uint4*>(x + t * ldx + c);
       const __nv_bfloat162* hv = reinterpret_cast<const __nv_bfloat162*>(&v);
       uint4 o;
@@ -653,7 +653,7 @@ relu2_kernel(const __nv_bfloat16* __restrict__ x, long long ldx, __nv_bfloat16* 
       }
       *reinterpret_cast<uint4*>(y + t * ldy + c) = o;
     } else {
-      for (int i = c; i < cols; ++i) {
+      for (int i = c; i < min(c + 8, cols); ++i) {
         const float f = __bfloat162float(x[t * ldx + i]);
         y[t * ldy + i] = __float2bfloat16_rn(f > 0.f ? f * f : 0.f);
       }
@@ -823,9 +823,9 @@ extern "C" int atlas_shared_expert_blend(void* y, long long ldy, const void* s, 
 
 extern "C" int atlas_relu2(const void* x, long long ldx, void* y, long long ldy, int T, int cols, void* stream) {
   if (T <= 0 || cols <= 0) return 0;
-  if ((ldx % 8) || (ldy % 8) || (reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(y) & 15)) return -1;
+  const int vec = ldx % 8 == 0 && ldy % 8 == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y)) & 15) == 0;
   dim3 grid(T, min(8, (cols / 8 + 255) / 256 > 0 ? (cols / 8 + 255) / 256 : 1));
   relu2_kernel<<<grid, 256, 0, reinterpret_cast<cudaStream_t>(stream)>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx,
-                                                                          reinterpret_cast<__nv_bfloat16*>(y), ldy, cols);
+                                                                          reinterpret_cast<__nv_bfloat16*>(y), ldy, cols, vec);
   return cudaGetLastError() == cudaSuccess ? 0 : -20;
 }

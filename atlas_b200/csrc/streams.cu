@@ -408,7 +408,7 @@ add_normed_kernel(const AddNormedParams<T> p) {
       float g[V];
       load_vec<V>(p.gate + t * p.ldg + e, g);
 #pragma unroll
-      for (int i = 0; i < V; ++i) y[k][i] /= 1.f + expf(-g[i]);
+      for (int i = 0; i < V; ++i) y[k][i] *= sigmoid_for<T>(g[i]);
     }
 #pragma unroll
     for (int i = 0; i < V; ++i) ss += y[k][i] * y[k][i];

@@ -76,6 +76,10 @@ ATLAS_DEVICE void store_vec(__nv_bfloat16* p, const float (&f)[V]) {
   }
 }
 
+// sigmoid(v) for results that leave in T: the fast exponential and division where they are rounded to bf16
+template <typename T> ATLAS_DEVICE float sigmoid_for(float v) { return 1.f / (1.f + expf(-v)); }
+template <> ATLAS_DEVICE float sigmoid_for<__nv_bfloat16>(float v) { return __fdividef(1.f, 1.f + __expf(-v)); }
+
 // rows of stride `ld` at `p` can be read V elements at a time (a null pointer can)
 template <typename T, int V>
 inline bool vec_ok(const void* p, long long ld) {

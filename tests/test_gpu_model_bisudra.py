@@ -99,6 +99,13 @@ def test_gelu_times_a_slice_of_an_embedding(dtype, T, n, layers, i):
 
 
 # ------------------------------------------------------------------------------------------------- products
+@pytest.mark.parametrize("T,n", [(1, 33), (5, 64), (130, 50), (3, 1), (7, 2056)])
+def test_squared_relu_of_any_width(T, n):
+    from atlas_b200 import ops
+    x = rnd(T, n, std=3.0).to(torch.bfloat16)
+    close(ops.relu_squared(x.cuda()), x.double().clamp(min=0) ** 2, torch.bfloat16, factor=0.5)
+
+
 @pytest.mark.parametrize("T,K,N,act", [(1, 256, 100, 64), (5, 96, 77, 77), (130, 2048, 4100, 2048), (300, 136, 40, 1), (64, 1024, 130, 33), (9, 90, 21, 8), (40, 4096, 128, 64)])
 def test_squared_relu_of_some_columns_in_the_product(T, K, N, act):
     from atlas_b200 import ops
@@ -359,7 +366,7 @@ def test_far_keys_and_window_edges_in_whole_models(tmp_path):
     """Weights with sharp scores and a window that hundreds of keys fit into: prompts, decoding and portions agree with the statement
     where a far key counts and where it has just left."""
     from atlas_b200.replay import build_engine
-    layer = lambda size: BC.attention(4, 2, 32, 64, size, 16, BC.ff(64), 0.5, scale=1.0)
+    layer = lambda size: BC.attention(4, 2, 32, 64, size, 16, BC.ff(64), 0.5, scale=0.4)
     cfg, w = BC.write_model(str(tmp_path), BC.model(200, 64, 4, 16, [layer(260), layer(129), layer(64)]))
     toks = BC.tokens(cfg, 600, 5)
     want = O.forward(cfg, w, toks)
