@@ -274,3 +274,11 @@ def test_bounds_reject_plausible_mistakes(folder, monkeypatch, mistake):
     name, wrong = MISTAKES[mistake]
     monkeypatch.setattr(O, name, wrong(getattr(O, name)))
     assert BC.spread(O.forward(cfg, w, toks), want) > 10 * TOL
+
+
+def test_units_that_a_model_is_compiled_from():
+    from atlas_b200 import build
+    from atlas_b200.config import tiny_bisudra
+    for dtype in ("bfloat16", "float32"):
+        units = build.units_for(tiny_bisudra(dtype))
+        assert {"differential", "conv1d", "streams", "moe"} <= set(units) and not {"recurrent", "rglru", "mlstm", "latent", "gdn"} & set(units)

@@ -414,11 +414,3 @@ def test_sampled_serving_preset_runs_in_bf16_and_quantised():
         eng = LLMEngine(model, EngineConfig(num_kv_blocks=64, max_num_seqs=4, max_seq_len=256, kv_cache_dtype="fp8"))
         outs = eng.generate([[1, 2, 3] * 9, [4, 5]], SamplingParams(max_tokens=30, temperature=0.8, top_p=0.9, seed=1, ignore_eos=True))
         assert all(len(o.output_tokens) == 30 for o in outs) and K.check_status() == 0
-
-
-def test_units_that_a_model_is_compiled_from():
-    from atlas_b200 import build
-    from atlas_b200.config import tiny_bisudra
-    for dtype in ("bfloat16", "float32"):
-        units = build.units_for(tiny_bisudra(dtype))
-        assert {"differential", "conv1d", "streams", "moe"} <= set(units) and not {"recurrent", "rglru", "mlstm", "latent", "gdn"} & set(units)
